@@ -1,5 +1,6 @@
 /* tffn.h — C ABI of the B200 inference path of tensor-ffn (Qwen2.5 decode with the base FFN
- * plus the expert-FFN delta at every layer).
+ * plus the expert-FFN delta at every layer; and, on the same sessions, models whose config.json lists their
+ * layers, see tffn_model_family).
  *
  * The reference has no FFI layer: its boundary is a set of C++ free functions over plain
  * structs of device pointers, called only from its main() (inference/src/main.cpp:97-204).
@@ -57,6 +58,13 @@ int tffn_device_count(void);
 /* ---- host-only helpers (no GPU needed) ------------------------------------------------- */
 /* qwen_config_from_json (inference/src/model/qwen.cu:21-63) */
 int tffn_config_read(const char* model_dir, tffn_config* out);
+/* Name of the model family config.json belongs to: "Qwen2" (the reference's), or the value of its "architecture"
+ * key for the families that list their layers ("Rafilix": chunked attention and gated-delta-rule layers, mixtures
+ * of squared-ReLU experts, fp32 residual stream). Unknown names give TFFN_ERR_UNSUPPORTED. For such a family
+ * tffn_config_read reports the width, the layer count, the vocabulary and eps; its per-head fields are the first
+ * layer's, eos / bos are -1 when the file has none, and max_position_embeddings is unbounded. Returns the length
+ * of the name (at most cap - 1 characters and a NUL are written). */
+int tffn_config_family(const char* model_dir, char* name, int cap);
 /* Header of an expert .bin (inference/src/io/checkpoint.cpp:15-31); also checks the file length. */
 int tffn_expert_probe(const char* path, uint32_t* version, uint32_t* num_layers, uint32_t* hidden,
                       uint32_t* intermediate);
@@ -95,6 +103,8 @@ int tffn_tokenizer_special(const tffn_tokenizer* t, uint32_t* eos, uint32_t* bos
 int tffn_model_load(const char* model_dir, int device, int tp_rank, int tp_size, tffn_model** out);
 void tffn_model_free(tffn_model* m); /* qwen_free (qwen.cu:176-209) */
 int tffn_model_config(const tffn_model* m, tffn_config* out);
+/* tffn_config_family of a loaded model */
+const char* tffn_model_family(const tffn_model* m);
 /* bytes of weight a decode step streams from HBM (every matrix once), with/without an expert */
 uint64_t tffn_model_weight_bytes(const tffn_model* m, int with_expert);
 
@@ -119,6 +129,14 @@ void tffn_expert_free(tffn_expert* e); /* expert_free (expert.cu:33-42) */
  * cudaStream_t, or NULL for a stream the session creates. */
 int tffn_session_create(const tffn_model* m, const tffn_expert* expert, int max_batch, int max_seq, void* cuda_stream,
                         tffn_session** out);
+/* tffn_session_create_tp (tp may be NULL) with a choice of what the session computes in: TFFN_COMPUTE_BF16 is what
+ * the other two create (bf16 matrix products and activations, fp32 accumulation; what a family keeps in fp32 is in
+ * fp32 either way), TFFN_COMPUTE_F32 keeps every activation, the cache and every product in true fp32 (weights stay
+ * the bf16 of the file), for families that list their layers (TFFN_ERR_UNSUPPORTED for Qwen2). */
+enum { TFFN_COMPUTE_BF16 = 0, TFFN_COMPUTE_F32 = 1 };
+typedef struct tffn_tp tffn_tp;
+int tffn_session_create_ex(const tffn_model* m, const tffn_expert* expert, int max_batch, int max_seq, void* cuda_stream,
+                           tffn_tp* tp, int compute, tffn_session** out);
 void tffn_session_free(tffn_session* s);
 
 /* ---- tensor parallelism (the reference is single-GPU: no counterpart) -------------------- */
@@ -140,7 +158,6 @@ void tffn_session_free(tffn_session* s);
  * launches (prefill) use ncclAllReduce. Creating and freeing a tensor-parallel session are collective calls.
  * Sampling and tffn_expert_forward are not available on a tensor-parallel model. NCCL (libnccl.so.2) is
  * opened at run time. */
-typedef struct tffn_tp tffn_tp;
 int tffn_tp_unique_id(uint8_t* id128);
 int tffn_tp_create(const uint8_t* id128, int tp_rank, int tp_size, int device, tffn_tp** out);
 void tffn_tp_free(tffn_tp* tp); /* after every session created with it has been freed */
@@ -177,6 +194,8 @@ int tffn_session_set_bs1_path(tffn_session* s, int enable);
 int tffn_session_capture_hidden(tffn_session* s, int max_rows);
 /* dst: bf16 bits [rows, hidden] of layer `layer` from the last captured call; returns rows. */
 int tffn_session_get_hidden(tffn_session* s, int layer, uint16_t* dst, int max_rows);
+/* the same in fp32: exact also where the residual stream is kept in fp32 (layer-list families) */
+int tffn_session_get_hidden_f32(tffn_session* s, int layer, float* dst, int max_rows);
 
 /* qwen_forward for a prompt (inference/src/main.cpp:172-180): appends seq_lens[i] tokens to
  * slot i for i < n_seqs (tokens concatenated in slot order), returns the greedy pick after

@@ -76,11 +76,11 @@ struct AttnCfg {
     static_assert(NST >= 2 && KB >= 1, "");
 };
 
-// One block of 16 cached keys (rows row0 .. row0+15 of a stage buffer, the first n_valid >= 1 of them
-// inside the context) for the query-head group held in qh / ql: S = Q K^T, online softmax of head
+// One block of 16 cached keys (rows row0 .. row0+15 of a stage buffer, those from n_skip < 16 up to n_valid >= 1
+// visible to the query) for the query-head group held in qh / ql: S = Q K^T, online softmax of head
 // lane / 4 (this thread: keys nt * 8 + (lane % 4) * 2 + {0, 1}), O += P V. The whole warp calls it.
 template <int HD>
-__device__ __forceinline__ void attn_block16(uint32_t kbuf, uint32_t vbuf, int row0, int n_valid,
+__device__ __forceinline__ void attn_block16(uint32_t kbuf, uint32_t vbuf, int row0, int n_skip, int n_valid,
                                              const uint32_t (&qh)[HD / 16][2], const uint32_t (&ql)[HD / 16][2], float scale,
                                              float& m_run, float& l_run, float (&o)[HD / 8][4], int lane) {
     using C = AttnCfg<HD>;
@@ -106,14 +106,15 @@ __device__ __forceinline__ void attn_block16(uint32_t kbuf, uint32_t vbuf, int r
     for (int nt = 0; nt < C::NT; ++nt) {
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
-            const bool live = nt * 8 + quad * 2 + j < n_valid;
+            const int key = nt * 8 + quad * 2 + j;
+            const bool live = key < n_valid && key >= n_skip;
             s[nt][j] = live ? (s[nt][j] + s[nt][j + 2]) * scale : kNegBig;  // q_hi . k + q_lo . k
             mx = fmaxf(mx, s[nt][j]);
         }
     }
     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
     mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-    const float mn = fmaxf(m_run, mx);  // finite: the first key of the block is in range
+    const float mn = fmaxf(m_run, mx);  // finite once a visible key has been seen; until then the weights below are zero
     const float corr = __expf(m_run - mn);
     m_run = mn;
     l_run *= corr;
@@ -122,8 +123,9 @@ __device__ __forceinline__ void attn_block16(uint32_t kbuf, uint32_t vbuf, int r
     uint32_t ph[C::NT], pl[C::NT];
 #pragma unroll
     for (int nt = 0; nt < C::NT; ++nt) {
-        const float p0 = (nt * 8 + quad * 2 < n_valid) ? __expf(s[nt][0] - mn) : 0.f;
-        const float p1 = (nt * 8 + quad * 2 + 1 < n_valid) ? __expf(s[nt][1] - mn) : 0.f;
+        const int k0 = nt * 8 + quad * 2, k1 = k0 + 1;
+        const float p0 = (k0 < n_valid && k0 >= n_skip) ? __expf(s[nt][0] - mn) : 0.f;
+        const float p1 = (k1 < n_valid && k1 >= n_skip) ? __expf(s[nt][1] - mn) : 0.f;
         l_run += p0 + p1;
         split_bf16x2(p0, p1, ph[nt], pl[nt]);
     }
@@ -146,7 +148,7 @@ template <int HD>
 __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __restrict__ q, KvView kv, int layer,
                                                               const int* __restrict__ tok_seq,
                                                               const int* __restrict__ tok_pos, bf16* __restrict__ ctx,
-                                                              int nh, int G, int splits, int early,
+                                                              int nh, int G_all, int splits, int early, AttnOptions opt,
                                                               float* __restrict__ ws, int* __restrict__ counters,
                                                               int* status, unsigned long long* tl,
                                                               unsigned long long* trace) {
@@ -176,15 +178,23 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
     if (!early) pdl_wait();
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int unit = blockIdx.x;  // t * nkv + kvh
+    // unit = (t * nkv + kvh) * parts + part: the query heads of a kv head come in parts of at most 8
+    const int unit = blockIdx.x;
     const int nkv = kv.nkv;
-    const int t = unit / nkv, kvh = unit % nkv;
+    const int parts_per_kv = (G_all + 7) / 8;
+    const int part = unit % parts_per_kv;
+    const int t = unit / parts_per_kv / nkv, kvh = unit / parts_per_kv % nkv;
+    const int G = min(8, G_all - part * 8);
+    const int head0 = kvh * G_all + part * 8;
+    const int kd = kv.hd, vd = kv.vd;  // widths of the cached rows: multiples of 8, at most HD
     const int split = blockIdx.y;
     const int seq = __ldcg(tok_seq + t);
     const int ctx_len = __ldcg(tok_pos + t) + 1;
-    int chunk = (ctx_len + splits - 1) / splits;
+    const int lo = opt.chunk > 0 ? (ctx_len - 1) / opt.chunk * opt.chunk : 0;  // first visible key
+    const int lo16 = lo & ~15;  // a warp's 16 rows start at a multiple of 16, so that they lie in one page
+    int chunk = (ctx_len - lo16 + splits - 1) / splits;
     chunk = (chunk + kPageTokens - 1) / kPageTokens * kPageTokens;
-    const int c_begin = split * chunk;
+    const int c_begin = lo16 + split * chunk;
     const int c_end = min(ctx_len, c_begin + chunk);
     ATTN_TRACE(1);
     const int* bt = kv.block_table + (size_t)seq * kv.max_pages_per_seq;
@@ -220,18 +230,19 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
             }
             const uint32_t kbuf = smem_base + (uint32_t)((st % C::NST) * C::STAGE_BYTES);
             const uint32_t vbuf = kbuf + (uint32_t)(C::STAGE_ROWS * C::ROW_BYTES);
-            const size_t page_off = ((size_t)(pg >= 0 ? pg : 0) * nkv + kvh) * kPageTokens * HD;
+            const size_t page_row = ((size_t)(pg >= 0 ? pg : 0) * nkv + kvh) * kPageTokens;
 #pragma unroll
             for (int i = 0; i < C::WARP_ROWS * C::GRAN / 32; ++i) {
                 const int idx = i * 32 + lane;
                 const int r = idx / C::GRAN, g = idx % C::GRAN;
                 const int row = wrow0 + r, tok = s_begin + r;
                 const bool valid = tok < c_end && pg >= 0;
-                const size_t off = page_off + (size_t)(tok % kPageTokens) * HD + g * 8;
+                const size_t pr = page_row + (size_t)(tok % kPageTokens);
                 const uint32_t dst = (uint32_t)(row * C::ROW_BYTES + ((g ^ (row & 7)) << 4));
                 if (!(early && st < C::NST && tok == ctx_len - 1)) {  // the newest row is copied after the wait
-                    cp_async16_zfill(kbuf + dst, kpool + off, valid ? 16u : 0u);
-                    cp_async16_zfill(vbuf + dst, vpool + off, valid ? 16u : 0u);
+                    const bool kok = valid && g * 8 < kd, vok = valid && g * 8 < vd;  // zeros past the cached width
+                    cp_async16_zfill(kbuf + dst, kpool + (kok ? pr * kd + g * 8 : 0), kok ? 16u : 0u);
+                    cp_async16_zfill(vbuf + dst, vpool + (vok ? pr * vd + g * 8 : 0), vok ? 16u : 0u);
                 }
             }
         }
@@ -257,10 +268,11 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
             int pg = newest_pg;
             const bool valid = pg >= 0 && pg < kv.num_pages;
             if (!valid) { bad = true; pg = 0; }
-            const size_t off = (((size_t)pg * nkv + kvh) * kPageTokens + (ctx_len - 1) % kPageTokens) * HD + g * 8;
+            const size_t pr = ((size_t)pg * nkv + kvh) * kPageTokens + (ctx_len - 1) % kPageTokens;
             const uint32_t dst = (uint32_t)(row * C::ROW_BYTES + ((g ^ (row & 7)) << 4));
-            cp_async16_zfill(kbuf + dst, kpool + off, valid ? 16u : 0u);
-            cp_async16_zfill(vbuf + dst, vpool + off, valid ? 16u : 0u);
+            const bool kok = valid && g * 8 < kd, vok = valid && g * 8 < vd;
+            cp_async16_zfill(kbuf + dst, kpool + (kok ? pr * kd + g * 8 : 0), kok ? 16u : 0u);
+            cp_async16_zfill(vbuf + dst, vpool + (vok ? pr * vd + g * 8 : 0), vok ? 16u : 0u);
         }
         cp_async_commit();
     }
@@ -270,19 +282,19 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
     const int hrow = lane >> 2, quad = lane & 3;
     uint32_t qh[C::KS][2], ql[C::KS][2];
     {
-        const float* qp = q + (size_t)t * nh * HD + (size_t)(kvh * G + hrow) * HD + quad * 2;
+        const float* qp = q + ((size_t)t * nh + head0 + hrow) * kd + quad * 2;
 #pragma unroll
         for (int ks = 0; ks < C::KS; ++ks) {
             float2 a = make_float2(0.f, 0.f), b = make_float2(0.f, 0.f);
             if (hrow < G) {
-                a = __ldcg((const float2*)(qp + ks * 16));
-                b = __ldcg((const float2*)(qp + ks * 16 + 8));
+                if (ks * 16 < kd) a = __ldcg((const float2*)(qp + ks * 16));
+                if (ks * 16 + 8 < kd) b = __ldcg((const float2*)(qp + ks * 16 + 8));
             }
             split_bf16x2(a.x, a.y, qh[ks][0], ql[ks][0]);
             split_bf16x2(b.x, b.y, qh[ks][1], ql[ks][1]);
         }
     }
-    const float scale = rsqrtf((float)HD);
+    const float scale = opt.scale;
     float m_run = kNegBig, l_run = 0.f;  // of head hrow; l_run is this thread's share (summed over the quad at the end)
     float o[C::DT][4];
 #pragma unroll
@@ -300,7 +312,7 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
         if (w_begin < c_end) {
             const uint32_t kbuf = smem_base + (uint32_t)((st % C::NST) * C::STAGE_BYTES);
             const uint32_t vbuf = kbuf + (uint32_t)(C::STAGE_ROWS * C::ROW_BYTES);
-            attn_block16<HD>(kbuf, vbuf, warp * C::WARP_ROWS, c_end - w_begin, qh, ql, scale, m_run, l_run, o, lane);
+            attn_block16<HD>(kbuf, vbuf, warp * C::WARP_ROWS, lo - w_begin, c_end - w_begin, qh, ql, scale, m_run, l_run, o, lane);
         }
         __syncwarp();  // every lane is done with the warp's rows of this buffer
         issue_stage(st + C::NST);  // commits a group even when there is nothing left to copy
@@ -322,8 +334,9 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
         }
     }
     __syncthreads();
-    float* part = ws + ((size_t)unit * splits + split) * (size_t)(G * (HD + 2));
-    bf16* ctx_tok = ctx + (size_t)t * nh * HD;
+    const int G_part = min(8, G_all);  // heads of a full part: the stride of the partial results
+    float* partial = ws + ((size_t)unit * splits + split) * (size_t)(G_part * (HD + 2));
+    bf16* ctx_tok = ctx + (size_t)t * opt.ctx_ld + (size_t)head0 * opt.vdim;
     for (int idx = tid; idx < G * HD; idx += kAttnCtaThreads) {
         const int g = idx / HD, d = idx % HD;
         float M = kNegBig;
@@ -338,10 +351,10 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
             A += mw[2 + d] * wgt;
         }
         if (splits == 1) {
-            ctx_tok[(size_t)(kvh * G + g) * HD + d] = __float2bfloat16_rn(A / L);
+            if (d < opt.vdim) ctx_tok[(size_t)g * opt.vdim + d] = __float2bfloat16_rn(A / L);
         } else {
-            part[g * (HD + 2) + 2 + d] = A;
-            if (d == 0) { part[g * (HD + 2)] = M; part[g * (HD + 2) + 1] = L; }
+            partial[g * (HD + 2) + 2 + d] = A;
+            if (d == 0) { partial[g * (HD + 2)] = M; partial[g * (HD + 2) + 1] = L; }
         }
     }
     if (bad) dev_fail(status, DEV_ERR_BOUNDS);
@@ -365,7 +378,7 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
         return;
     }
     __threadfence();
-    const float* parts = ws + (size_t)unit * splits * (size_t)(G * (HD + 2));
+    const float* parts = ws + (size_t)unit * splits * (size_t)(G_part * (HD + 2));
     constexpr int kMergeSplits = 16;  // up to here: one pass with every load in flight
     if (splits <= kMergeSplits) {
         // weight of split z for head g: exp(m_z - M) / sum_z l_z exp(m_z - M), kept in the (idle) merge buffer
@@ -375,7 +388,7 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
 #pragma unroll
             for (int z = 0; z < kMergeSplits; ++z) {
                 const bool live = z < splits;
-                const float* pz = parts + (size_t)(live ? z : 0) * G * (HD + 2) + tid * (HD + 2);
+                const float* pz = parts + (size_t)(live ? z : 0) * G_part * (HD + 2) + tid * (HD + 2);
                 mz[z] = live ? __ldcg(pz) : kNegBig;
                 lz[z] = live ? __ldcg(pz + 1) : 0.f;
             }
@@ -403,7 +416,7 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
                 float az[4];
 #pragma unroll
                 for (int j = 0; j < 4; ++j)
-                    az[j] = (on && z0 + j < splits) ? __ldcg(parts + (size_t)(z0 + j) * G * (HD + 2) + g * (HD + 2) + 2 + d) : 0.f;
+                    az[j] = (on && z0 + j < splits) ? __ldcg(parts + (size_t)(z0 + j) * G_part * (HD + 2) + g * (HD + 2) + 2 + d) : 0.f;
 #pragma unroll
                 for (int j = 0; j < 4; ++j)
                     if (z0 + j < splits) A += az[j] * wgt[g * kMergeSplits + z0 + j];
@@ -413,12 +426,12 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
 #pragma unroll
         for (int it = 0; it < ITERS; ++it) {
             const int idx = tid + it * kAttnCtaThreads;
-            if (idx < G * HD) ctx_tok[(size_t)(kvh * G + idx / HD) * HD + idx % HD] = __float2bfloat16_rn(res[it]);
+            if (idx < G * HD && idx % HD < opt.vdim) ctx_tok[(size_t)(idx / HD) * opt.vdim + idx % HD] = __float2bfloat16_rn(res[it]);
         }
     } else {
         for (int idx = tid; idx < G * HD; idx += kAttnCtaThreads) {
             const int g = idx / HD, d = idx % HD;
-            ctx_tok[(size_t)(kvh * G + g) * HD + d] = __float2bfloat16_rn(attn_merge_splits(parts, splits, G, HD, g, d));
+            if (d < opt.vdim) ctx_tok[(size_t)g * opt.vdim + d] = __float2bfloat16_rn(attn_merge_splits(parts, splits, G_part, HD, g, d));
         }
     }
     ATTN_TRACE(8);
@@ -437,7 +450,8 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_prefill(const float* _
                                                                const int* __restrict__ tok_pos,
                                                                const int* __restrict__ grp_first,
                                                                const int* __restrict__ grp_count, bf16* __restrict__ ctx,
-                                                               int nh, int G, int* status, unsigned long long* tl) {
+                                                               int nh, int G_all, AttnOptions opt, int* status,
+                                                               unsigned long long* tl) {
     using C = AttnCfg<HD>;
     extern __shared__ __align__(128) uint8_t smem[];
     if (threadIdx.x == 0) tl_mark(tl, 0);
@@ -445,13 +459,19 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_prefill(const float* _
     pdl_wait();  // the previous kernel wrote q and the K/V rows of these very tokens
     if (threadIdx.x == 0) tl_mark(tl, 1);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int kvh = blockIdx.y, nkv = kv.nkv;
+    const int nkv = kv.nkv, parts_per_kv = (G_all + 7) / 8;  // query heads of a kv head in parts of at most 8
+    const int kvh = blockIdx.y / parts_per_kv, part = blockIdx.y % parts_per_kv;
+    const int G = min(8, G_all - part * 8), head0 = kvh * G_all + part * 8;
+    const int kd = kv.hd, vd = kv.vd;
     const int first = __ldcg(grp_first + blockIdx.x), count = __ldcg(grp_count + blockIdx.x);
     const int seq = __ldcg(tok_seq + first);
     const int last_len = __ldcg(tok_pos + first + count - 1) + 1;  // positions ascend within a group
     const bool active = warp < count;
     const int t = first + (active ? warp : 0);
     const int my_len = active ? __ldcg(tok_pos + t) + 1 : 0;
+    // first key visible to this warp's token, and the group's first key (page-aligned): a group may cross a chunk's edge
+    const int my_lo = (opt.chunk > 0 && active) ? (my_len - 1) / opt.chunk * opt.chunk : 0;
+    const int grp_lo = opt.chunk > 0 ? (__ldcg(tok_pos + first) / opt.chunk * opt.chunk) / kPageTokens * kPageTokens : 0;
     const int* bt = kv.block_table + (size_t)seq * kv.max_pages_per_seq;
     const bf16* kpool = kv.k_pool + (size_t)layer * kv.layer_stride;
     const bf16* vpool = kv.v_pool + (size_t)layer * kv.layer_stride;
@@ -459,7 +479,7 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_prefill(const float* _
     bool bad = false;
 
     auto issue_stage = [&](int st) {  // all 256 threads
-        const int s_begin = st * C::STAGE_ROWS;
+        const int s_begin = grp_lo + st * C::STAGE_ROWS;
         if (s_begin < last_len) {
             constexpr int PPS = C::STAGE_ROWS / kPageTokens;
             int pgs[PPS];
@@ -479,34 +499,35 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_prefill(const float* _
                 const int row = i * ROWS_PER_IT + row0;
                 const int pg = pgs[(i * ROWS_PER_IT) / kPageTokens];
                 const bool valid = s_begin + row < last_len && pg >= 0;
-                const size_t off = (((size_t)(valid ? pg : 0) * nkv + kvh) * kPageTokens + row % kPageTokens) * HD + g * 8;
+                const size_t pr = ((size_t)(valid ? pg : 0) * nkv + kvh) * kPageTokens + row % kPageTokens;
                 const uint32_t dst = (uint32_t)(row * C::ROW_BYTES + ((g ^ (row & 7)) << 4));
-                cp_async16_zfill(kbuf + dst, kpool + off, valid ? 16u : 0u);
-                cp_async16_zfill(vbuf + dst, vpool + off, valid ? 16u : 0u);
+                const bool kok = valid && g * 8 < kd, vok = valid && g * 8 < vd;  // zeros past the cached width
+                cp_async16_zfill(kbuf + dst, kpool + (kok ? pr * kd + g * 8 : 0), kok ? 16u : 0u);
+                cp_async16_zfill(vbuf + dst, vpool + (vok ? pr * vd + g * 8 : 0), vok ? 16u : 0u);
             }
         }
         cp_async_commit();
     };
-    const int n_stages = (last_len + C::STAGE_ROWS - 1) / C::STAGE_ROWS;
+    const int n_stages = (last_len - grp_lo + C::STAGE_ROWS - 1) / C::STAGE_ROWS;
 #pragma unroll
     for (int st = 0; st < C::NST; ++st) issue_stage(st);
 
     const int hrow = lane >> 2, quad = lane & 3;
     uint32_t qh[C::KS][2], ql[C::KS][2];
     {
-        const float* qp = q + (size_t)t * nh * HD + (size_t)(kvh * G + hrow) * HD + quad * 2;
+        const float* qp = q + ((size_t)t * nh + head0 + hrow) * kd + quad * 2;
 #pragma unroll
         for (int ks = 0; ks < C::KS; ++ks) {
             float2 a = make_float2(0.f, 0.f), b = make_float2(0.f, 0.f);
             if (active && hrow < G) {
-                a = __ldcg((const float2*)(qp + ks * 16));
-                b = __ldcg((const float2*)(qp + ks * 16 + 8));
+                if (ks * 16 < kd) a = __ldcg((const float2*)(qp + ks * 16));
+                if (ks * 16 + 8 < kd) b = __ldcg((const float2*)(qp + ks * 16 + 8));
             }
             split_bf16x2(a.x, a.y, qh[ks][0], ql[ks][0]);
             split_bf16x2(b.x, b.y, qh[ks][1], ql[ks][1]);
         }
     }
-    const float scale = rsqrtf((float)HD);
+    const float scale = opt.scale;
     float m_run = kNegBig, l_run = 0.f;
     float o[C::DT][4];
 #pragma unroll
@@ -519,9 +540,10 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_prefill(const float* _
         const uint32_t vbuf = kbuf + (uint32_t)(C::STAGE_ROWS * C::ROW_BYTES);
 #pragma unroll 1
         for (int blk = 0; blk < C::STAGE_ROWS / 16; ++blk) {
-            const int k0 = st * C::STAGE_ROWS + blk * 16;
+            const int k0 = grp_lo + st * C::STAGE_ROWS + blk * 16;
             if (k0 >= my_len) break;  // warp-uniform: causal end of this token
-            attn_block16<HD>(kbuf, vbuf, blk * 16, my_len - k0, qh, ql, scale, m_run, l_run, o, lane);
+            if (k0 + 16 <= my_lo) continue;  // before its chunk
+            attn_block16<HD>(kbuf, vbuf, blk * 16, my_lo - k0, my_len - k0, qh, ql, scale, m_run, l_run, o, lane);
         }
         __syncthreads();  // every warp is done with this buffer
         issue_stage(st + C::NST);
@@ -531,31 +553,115 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_prefill(const float* _
     l_run += __shfl_xor_sync(0xffffffffu, l_run, 2);
     if (active && hrow < G) {
         const float inv = 1.f / l_run;  // my_len >= 1: at least one key
-        bf16* dst = ctx + (size_t)t * nh * HD + (size_t)(kvh * G + hrow) * HD + quad * 2;
+        const int vdim = opt.vdim;
+        bf16* dst = ctx + (size_t)t * opt.ctx_ld + (size_t)(head0 + hrow) * vdim + quad * 2;
 #pragma unroll
         for (int d = 0; d < C::DT; ++d) {
             const float a = (o[d][0] + o[d][2]) * inv, b = (o[d][1] + o[d][3]) * inv;  // P_hi V + P_lo V
-            *(uint32_t*)(dst + d * 8) = (uint32_t)bf16_bits(a) | ((uint32_t)bf16_bits(b) << 16);
+            const int col = d * 8 + quad * 2;
+            if ((vdim & 1) == 0) {
+                if (col < vdim) *(uint32_t*)(dst + d * 8) = (uint32_t)bf16_bits(a) | ((uint32_t)bf16_bits(b) << 16);
+            } else {
+                if (col < vdim) dst[d * 8] = __float2bfloat16_rn(a);
+                if (col + 1 < vdim) dst[d * 8 + 1] = __float2bfloat16_rn(b);
+            }
         }
     }
     if (bad) dev_fail(status, DEV_ERR_BOUNDS);
     if (tid == 0) tl_mark(tl, 2);
 }
 
+// Attention of one (query head, token) per block without tensor cores, for what the kernels above do not take: fp32
+// caches (a session that computes in fp32) and heads wider than 128. Every warp walks the visible keys with a stride
+// of kSimtWarps; the lanes share the dimensions of a key; exact exponentials; the warps merge at the end.
+constexpr int kSimtWarps = 8;
+constexpr int kSimtMaxLanes = 16;  // value columns per lane: heads of up to 512 columns
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void store_as(float* p, float v) { *p = v; }
+__device__ __forceinline__ void store_as(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+template <typename C>
+__global__ void __launch_bounds__(kSimtWarps * 32) k_attn_simt(const float* __restrict__ q, KvView kv, const int* __restrict__ tok_seq,
+                                                               const int* __restrict__ tok_pos, C* __restrict__ ctx, int nh,
+                                                               AttnOptions opt, int* status, unsigned long long* tl) {
+    extern __shared__ float simt_smem[];
+    if (threadIdx.x == 0) tl_mark(tl, 0);
+    pdl_launch_dependents();
+    pdl_wait();
+    if (threadIdx.x == 0) tl_mark(tl, 1);
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int head = blockIdx.x, t = blockIdx.y;
+    const int kvh = head / (nh / kv.nkv), kd = kv.hd, vd = kv.vd, vdim = opt.vdim;
+    float* sq = simt_smem;                 // [kd]
+    float* merge = simt_smem + kd;         // [warp][vdim + 2]
+    for (int i = tid; i < kd; i += kSimtWarps * 32) sq[i] = __ldcg(q + ((size_t)t * nh + head) * kd + i);
+    __syncthreads();
+    const int seq = __ldcg(tok_seq + t), last = __ldcg(tok_pos + t);
+    const int lo = opt.chunk > 0 ? last / opt.chunk * opt.chunk : 0;
+    const int* bt = kv.block_table + (size_t)seq * kv.max_pages_per_seq;
+    const C* kpool = (const C*)kv.k_pool;
+    const C* vpool = (const C*)kv.v_pool;
+    float m = kNegBig, l = 0.f, acc[kSimtMaxLanes];
+#pragma unroll
+    for (int j = 0; j < kSimtMaxLanes; ++j) acc[j] = 0.f;
+    bool bad = false;
+    for (int key = lo + warp; key <= last; key += kSimtWarps) {
+        const int pg = __ldcg(bt + key / kPageTokens);
+        if (pg < 0 || pg >= kv.num_pages) { bad = true; continue; }
+        const size_t row = ((size_t)pg * kv.nkv + kvh) * kPageTokens + key % kPageTokens;
+        float s = 0.f;
+        for (int i = lane; i < kd; i += 32) s += sq[i] * to_f32(kpool[row * kd + i]);
+        s = warp_sum(s) * opt.scale;
+        const float mn = fmaxf(m, s), corr = expf(m - mn), p = expf(s - mn);
+        m = mn;
+        l = l * corr + p;
+#pragma unroll
+        for (int j = 0; j < kSimtMaxLanes; ++j) {
+            const int d = j * 32 + lane;
+            if (d < vdim) acc[j] = acc[j] * corr + p * to_f32(vpool[row * vd + d]);
+        }
+    }
+    float* mw = merge + warp * (vdim + 2);
+    if (lane == 0) { mw[0] = m; mw[1] = l; }
+#pragma unroll
+    for (int j = 0; j < kSimtMaxLanes; ++j)
+        if (j * 32 + lane < vdim) mw[2 + j * 32 + lane] = acc[j];
+    __syncthreads();
+    float M = kNegBig, L = 0.f;
+    for (int w = 0; w < kSimtWarps; ++w) M = fmaxf(M, merge[w * (vdim + 2)]);
+    for (int w = 0; w < kSimtWarps; ++w) L += merge[w * (vdim + 2) + 1] * expf(merge[w * (vdim + 2)] - M);
+    for (int d = tid; d < vdim; d += kSimtWarps * 32) {
+        float A = 0.f;
+        for (int w = 0; w < kSimtWarps; ++w) A += merge[w * (vdim + 2) + 2 + d] * expf(merge[w * (vdim + 2)] - M);
+        store_as(ctx + (size_t)t * opt.ctx_ld + (size_t)head * vdim + d, A / L);
+    }
+    if (bad && lane == 0) dev_fail(status, DEV_ERR_BOUNDS);
+    if (tid == 0) tl_mark(tl, 2);
+}
+
 template <int HD>
 void launch_hd(dim3 grid, cudaStream_t s, bool pdl, const float* q, const KvView& kv, int layer, const int* tok_seq,
-               const int* tok_pos, bf16* ctx, int nh, int G, int splits, int early, float* ws, int* counters, int* status,
-               unsigned long long* tl, unsigned long long* trace) {
+               const int* tok_pos, bf16* ctx, int nh, int G, int splits, int early, const AttnOptions& opt, float* ws,
+               int* counters, int* status, unsigned long long* tl, unsigned long long* trace) {
     launch_k(k_attn_decode<HD>, grid, dim3(kAttnCtaThreads), (size_t)AttnCfg<HD>::SMEM, s, pdl, q, kv, layer, tok_seq, tok_pos, ctx,
-             nh, G, splits, early, ws, counters, status, tl, trace);
+             nh, G, splits, early, opt, ws, counters, status, tl, trace);
 }
 
 template <int HD>
 void launch_prefill_hd(dim3 grid, cudaStream_t s, bool pdl, const float* q, const KvView& kv, int layer, const int* tok_seq,
-                       const int* tok_pos, const int* grp_first, const int* grp_count, bf16* ctx, int nh, int G, int* status,
-                       unsigned long long* tl) {
+                       const int* tok_pos, const int* grp_first, const int* grp_count, bf16* ctx, int nh, int G,
+                       const AttnOptions& opt, int* status, unsigned long long* tl) {
     launch_k(k_attn_prefill<HD>, grid, dim3(kAttnCtaThreads), (size_t)AttnCfg<HD>::SMEM, s, pdl, q, kv, layer, tok_seq, tok_pos,
-             grp_first, grp_count, ctx, nh, G, status, tl);
+             grp_first, grp_count, ctx, nh, G, opt, status, tl);
+}
+
+// options with their defaults filled in
+AttnOptions resolve(AttnOptions o, const KvView& kv, int nh) {
+    if (o.scale == 0.f) o.scale = 1.f / sqrtf((float)kv.hd);
+    if (o.vdim == 0) o.vdim = kv.vd;
+    if (o.ctx_ld == 0) o.ctx_ld = (int64_t)nh * o.vdim;
+    return o;
 }
 
 }  // namespace
@@ -571,6 +677,8 @@ int attn_prepare() {
     if (e == cudaSuccess) e = prefer_max_shared(k_attn_decode<128>);
     if (e == cudaSuccess) e = prefer_max_shared(k_attn_prefill<64>);
     if (e == cudaSuccess) e = prefer_max_shared(k_attn_prefill<128>);
+    if (e == cudaSuccess) e = prefer_max_shared(k_attn_simt<float>);
+    if (e == cudaSuccess) e = prefer_max_shared(k_attn_simt<bf16>);
     return (int)e;
 }
 
@@ -585,8 +693,9 @@ int attention_splits(int T, int nh, int nkv, int hd, int max_ctx, const AttnWork
     // gets at least 1024 keys (batch 1 at a few hundred keys of context: 0.94 -> 0.82 ms per token
     // without splits; halving the minimum for 128-wide heads gained 1.4 us per launch for 32 sequences on a
     // quarter of the 7B shape's heads and cost batch 1 on the 1.5B shape 16 %: 576 -> 483 tok/s).
-    const int G = nh / nkv;
-    const int units = T * nkv;
+    const int G = nh / nkv < 8 ? nh / nkv : 8;
+    const int units = T * nkv * ((nh / nkv + 7) / 8);
+    hd = hd <= 64 ? 64 : 128;  // columns of a partial result
     int splits = 1;
     if (units * 2 <= num_sms) {
         splits = num_sms / units;
@@ -601,24 +710,38 @@ int attention_splits(int T, int nh, int nkv, int hd, int max_ctx, const AttnWork
 
 void launch_attention(const float* q, KvView kv, int layer, const int* tok_seq, const int* tok_pos, bf16* ctx, int T,
                       int nh, int max_ctx, AttnWorkspace ws, int num_sms, int* status, cudaStream_t s, bool pdl,
-                      bool only_newest_row_fresh, unsigned long long* tl, unsigned long long* trace, int trace_ctas) {
+                      bool only_newest_row_fresh, unsigned long long* tl, unsigned long long* trace, int trace_ctas,
+                      const AttnOptions& options) {
     const int early = (pdl && only_newest_row_fresh) ? 1 : 0;
-    const int G = nh / kv.nkv;  // at most 8 (checked when the model is loaded)
-    const int units = T * kv.nkv;
-    const int splits = attention_splits(T, nh, kv.nkv, kv.hd, max_ctx, ws, num_sms);
+    const AttnOptions opt = resolve(options, kv, nh);
+    const int G = nh / kv.nkv;
+    const int units = T * kv.nkv * ((G + 7) / 8);
+    const int wide = kv.hd > kv.vd ? kv.hd : kv.vd;
+    const int splits = attention_splits(T, nh, kv.nkv, wide, max_ctx, ws, num_sms);
     dim3 grid(units, splits);
     if ((long long)units * splits > trace_ctas) trace = nullptr;
-    if (kv.hd == 64) launch_hd<64>(grid, s, pdl, q, kv, layer, tok_seq, tok_pos, ctx, nh, G, splits, early, ws.partials, ws.counters, status, tl, trace);
-    else if (kv.hd == 128) launch_hd<128>(grid, s, pdl, q, kv, layer, tok_seq, tok_pos, ctx, nh, G, splits, early, ws.partials, ws.counters, status, tl, trace);
+    if (wide <= 64) launch_hd<64>(grid, s, pdl, q, kv, layer, tok_seq, tok_pos, ctx, nh, G, splits, early, opt, ws.partials, ws.counters, status, tl, trace);
+    else if (wide <= 128) launch_hd<128>(grid, s, pdl, q, kv, layer, tok_seq, tok_pos, ctx, nh, G, splits, early, opt, ws.partials, ws.counters, status, tl, trace);
 }
 
 void launch_attention_prefill(const float* q, KvView kv, int layer, const int* tok_seq, const int* tok_pos, const int* grp_first,
                               const int* grp_count, int n_groups, bf16* ctx, int nh, int* status, cudaStream_t s, bool pdl,
-                              unsigned long long* tl) {
+                              unsigned long long* tl, const AttnOptions& options) {
+    const AttnOptions opt = resolve(options, kv, nh);
     const int G = nh / kv.nkv;
-    dim3 grid(n_groups, kv.nkv);
-    if (kv.hd == 64) launch_prefill_hd<64>(grid, s, pdl, q, kv, layer, tok_seq, tok_pos, grp_first, grp_count, ctx, nh, G, status, tl);
-    else if (kv.hd == 128) launch_prefill_hd<128>(grid, s, pdl, q, kv, layer, tok_seq, tok_pos, grp_first, grp_count, ctx, nh, G, status, tl);
+    const int wide = kv.hd > kv.vd ? kv.hd : kv.vd;
+    dim3 grid(n_groups, kv.nkv * ((G + 7) / 8));
+    if (wide <= 64) launch_prefill_hd<64>(grid, s, pdl, q, kv, layer, tok_seq, tok_pos, grp_first, grp_count, ctx, nh, G, opt, status, tl);
+    else if (wide <= 128) launch_prefill_hd<128>(grid, s, pdl, q, kv, layer, tok_seq, tok_pos, grp_first, grp_count, ctx, nh, G, opt, status, tl);
+}
+
+void launch_attention_simt(const float* q, KvView kv, bool f32, const int* tok_seq, const int* tok_pos, void* ctx, int T, int nh,
+                           const AttnOptions& options, int* status, cudaStream_t s, bool pdl, unsigned long long* tl) {
+    const AttnOptions opt = resolve(options, kv, nh);
+    const dim3 grid(nh, T), block(kSimtWarps * 32);
+    const size_t smem = (size_t)(kv.hd + kSimtWarps * (opt.vdim + 2)) * 4;
+    if (f32) launch_k(k_attn_simt<float>, grid, block, smem, s, pdl, q, kv, tok_seq, tok_pos, (float*)ctx, nh, opt, status, tl);
+    else launch_k(k_attn_simt<bf16>, grid, block, smem, s, pdl, q, kv, tok_seq, tok_pos, (bf16*)ctx, nh, opt, status, tl);
 }
 
 }  // namespace tffn

@@ -65,6 +65,21 @@ int tffn_config_read(const char* model_dir, tffn_config* out) {
     });
 }
 
+int tffn_config_family(const char* model_dir, char* name, int cap) {
+    int len = 0;
+    int rc = guard([&] {
+        need(model_dir, "NULL argument");
+        const std::string f = read_config(model_dir).family;
+        len = (int)f.size();
+        if (name && cap > 0) {
+            const int n = len < cap - 1 ? len : cap - 1;
+            memcpy(name, f.data(), n);
+            name[n] = 0;
+        }
+    });
+    return rc < 0 ? rc : len;
+}
+
 int tffn_expert_probe(const char* path, uint32_t* version, uint32_t* num_layers, uint32_t* hidden, uint32_t* intermediate) {
     return guard([&] {
         need(path, "NULL path");
@@ -196,6 +211,7 @@ int tffn_model_config(const tffn_model* m, tffn_config* out) {
         out->eos_token_id = c.eos_token_id; out->bos_token_id = c.bos_token_id; out->tie_embeddings = c.tie_embeddings;
     });
 }
+const char* tffn_model_family(const tffn_model* m) { return m ? m->m->cfg.family.c_str() : ""; }
 uint64_t tffn_model_weight_bytes(const tffn_model* m, int with_expert) {
     if (!m) return 0;
     const Config& c = m->m->cfg;
@@ -236,10 +252,15 @@ int tffn_session_create(const tffn_model* m, const tffn_expert* expert, int max_
 }
 int tffn_session_create_tp(const tffn_model* m, const tffn_expert* expert, int max_batch, int max_seq, void* cuda_stream,
                            tffn_tp* tp, tffn_session** out) {
+    return tffn_session_create_ex(m, expert, max_batch, max_seq, cuda_stream, tp, TFFN_COMPUTE_BF16, out);
+}
+int tffn_session_create_ex(const tffn_model* m, const tffn_expert* expert, int max_batch, int max_seq, void* cuda_stream,
+                           tffn_tp* tp, int compute, tffn_session** out) {
     return guard([&] {
         need(m && out, "NULL argument");
+        need(compute == TFFN_COMPUTE_BF16 || compute == TFFN_COMPUTE_F32, "unknown compute type");
         std::unique_ptr<Session> s(new Session(m->m, expert ? expert->e : nullptr, max_batch, max_seq, (cudaStream_t)cuda_stream,
-                                               tp ? tp->c : nullptr));
+                                               tp ? tp->c : nullptr, compute == TFFN_COMPUTE_F32));
         *out = new tffn_session{s.release()};
     });
 }
@@ -330,6 +351,14 @@ int tffn_session_get_hidden(tffn_session* s, int layer, uint16_t* dst, int max_r
     int rc = guard([&] {
         need(s, "NULL session");
         rows = s->s->get_hidden(layer, dst, max_rows);
+    });
+    return rc < 0 ? rc : rows;
+}
+int tffn_session_get_hidden_f32(tffn_session* s, int layer, float* dst, int max_rows) {
+    int rows = 0;
+    int rc = guard([&] {
+        need(s, "NULL session");
+        rows = s->s->get_hidden_f32(layer, dst, max_rows);
     });
     return rc < 0 ? rc : rows;
 }

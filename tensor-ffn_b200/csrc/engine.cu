@@ -1,5 +1,6 @@
 #include "engine.h"
 #include "launch.h"
+#include "upload.h"
 #include <algorithm>
 #include <cmath>
 #include <cstring>
@@ -40,91 +41,6 @@ void DeviceBuffer::release() {
 }
 
 namespace {
-
-void upload(DeviceBuffer& dst, const void* src, size_t bytes) {
-    dst.alloc(bytes);
-    TFFN_CUDA(cudaMemcpy(dst.p, src, bytes, cudaMemcpyHostToDevice));
-    // from pageable memory the call may return once the data is staged: wait for it to reach the device,
-    // the streams that will read it are not ordered after the default stream
-    TFFN_CUDA(cudaStreamSynchronize(0));
-}
-
-// Host-to-device staging for the loaders: the weight files are memory-mapped (pageable), so a plain
-// cudaMemcpy would page each tensor in, stage it inside the driver and block. Here the host thread copies the
-// next chunk out of the mapping into one of two pinned buffers while the copy engine still moves the previous
-// one; everything (copies, the re-layout kernels that follow them) is ordered on one stream and the loader
-// waits once at the end.
-class Stager {
-public:
-    explicit Stager(size_t chunk_bytes = (size_t)32 << 20) : chunk_(chunk_bytes) {
-        TFFN_CUDA(cudaStreamCreateWithFlags(&s_, cudaStreamNonBlocking));
-        for (int i = 0; i < 2; ++i) {
-            TFFN_CUDA(cudaMallocHost((void**)&buf_[i], chunk_));
-            TFFN_CUDA(cudaEventCreateWithFlags(&ev_[i], cudaEventDisableTiming));
-        }
-    }
-    ~Stager() {
-        cudaStreamSynchronize(s_);
-        for (int i = 0; i < 2; ++i) {
-            if (buf_[i]) cudaFreeHost(buf_[i]);
-            if (ev_[i]) cudaEventDestroy(ev_[i]);
-        }
-        cudaStreamDestroy(s_);
-    }
-    Stager(const Stager&) = delete;
-    Stager& operator=(const Stager&) = delete;
-    cudaStream_t stream() const { return s_; }
-    void copy(void* dst, const void* src, size_t bytes) {
-        for (size_t o = 0; o < bytes; o += chunk_) put((char*)dst + o, (const char*)src + o, std::min(chunk_, bytes - o), 0, 0, 0);
-    }
-    // `rows` rows of `width` bytes, `src_pitch` bytes apart in the mapping -> dense on the device
-    void copy2d(void* dst, const void* src, size_t src_pitch, size_t width, size_t rows) {
-        if (width == 0 || rows == 0) return;
-        if (src_pitch == width) return copy(dst, src, width * rows);
-        if (width > chunk_) throw Error(kErrUnsupported, "a matrix row is longer than the staging buffer");
-        const size_t rows_per = chunk_ / width;
-        for (size_t r = 0; r < rows; r += rows_per) {
-            const size_t nr = std::min(rows_per, rows - r);
-            put((char*)dst + r * width, (const char*)src + r * src_pitch, nr * width, src_pitch, width, nr);
-        }
-    }
-    void finish() { TFFN_CUDA(cudaStreamSynchronize(s_)); }
-
-private:
-    // one chunk: wait until the pinned buffer's previous transfer has left it, fill it, send it
-    void put(void* dst, const char* src, size_t bytes, size_t pitch, size_t width, size_t rows) {
-        uint8_t* b = buf_[cur_];
-        if (used_[cur_]) TFFN_CUDA(cudaEventSynchronize(ev_[cur_]));
-        if (rows == 0) {
-            memcpy(b, src, bytes);
-        } else {
-            for (size_t r = 0; r < rows; ++r) memcpy(b + r * width, src + r * pitch, width);
-        }
-        TFFN_CUDA(cudaMemcpyAsync(dst, b, bytes, cudaMemcpyHostToDevice, s_));
-        TFFN_CUDA(cudaEventRecord(ev_[cur_], s_));
-        used_[cur_] = true;
-        cur_ ^= 1;
-    }
-    size_t chunk_;
-    cudaStream_t s_ = nullptr;
-    uint8_t* buf_[2] = {nullptr, nullptr};
-    cudaEvent_t ev_[2] = {nullptr, nullptr};
-    bool used_[2] = {false, false};
-    int cur_ = 0;
-};
-
-// carves 256-byte aligned views out of one allocation
-struct Slab {
-    DeviceBuffer* mem;
-    size_t off = 0;
-    void take(DeviceBuffer& dst, size_t bytes) {
-        const size_t a = (off + 255) & ~(size_t)255;
-        if (a + bytes > mem->bytes) throw Error(kErrInvalid, "weight slab too small (internal size computation)");
-        dst.view((char*)mem->p + a, bytes);
-        off = a + bytes;
-    }
-    static size_t padded(size_t bytes) { return (bytes + 255) & ~(size_t)255; }
-};
 
 // one block: publish the picks as the next step's inputs, advance the sequence lengths
 __global__ void k_decode_advance(const int* __restrict__ picks, int n, int* __restrict__ dec_tokens, int* __restrict__ seq_len,
@@ -210,9 +126,25 @@ Model* Model::load(const std::string& dir, int device, int tp_rank, int tp_size)
     if (prop.major < 10) throw Error(kErrUnsupported, "this library is built for sm_100a (B200) only");
     m->num_sms = prop.multiProcessorCount;
     m->cfg = read_config(dir);
+    m->tp = tp_partition(m->cfg, tp_rank, tp_size);
+    // the weight loaders of the families in model_families()
+    static const struct {
+        const char* family;
+        void (Model::*load)(const std::string&);
+    } loaders[] = {{"Qwen2", &Model::load_qwen2}, {"Rafilix", &Model::load_stack}};
+    for (const auto& l : loaders)
+        if (m->cfg.family == l.family) {
+            (m.get()->*l.load)(dir);
+            return m.release();
+        }
+    throw Error(kErrUnsupported, "no weight loader for the " + m->cfg.family + " family");
+}
+
+void Model::load_qwen2(const std::string& dir) {
+    Model* const m = this;
     const Config& c = m->cfg;
-    m->tp = tp_partition(c, tp_rank, tp_size);
     const TpPartition& tp = m->tp;
+    const int tp_size = tp.tp_size;
     m->nh = tp.n_q_heads;
     m->nkv = tp.n_kv_heads;
     m->I = tp.n_i;
@@ -292,7 +224,7 @@ Model* Model::load(const std::string& dir, int device, int tp_rank, int tp_size)
     m->bs1_ok = tp_size == 1 && bs1_supported((int)H, (int)I, (int)hd, (int)nh, (int)nkv);
     const uint64_t per_layer = (nqkv * H + H * nq + 3 * I * H) * 2 + 2 * H * 2 + (uint64_t)(m->layers[0].has_bias ? nqkv * 2 : 0);
     m->weight_bytes_base = per_layer * c.num_layers + (uint64_t)m->V * H * 2 + H * 2;
-    return m.release();
+    m->embed_ld = (int64_t)H;
 }
 
 // ------------------------------------------------------------------------------------------ Expert
@@ -348,7 +280,7 @@ Expert* Expert::load(const Model* m, const std::string& path, float scale) {
 }
 
 // ------------------------------------------------------------------------------------------ Session
-Session::Session(const Model* m, const Expert* e, int max_batch, int max_seq, cudaStream_t stream, TpComm* tp)
+Session::Session(const Model* m, const Expert* e, int max_batch, int max_seq, cudaStream_t stream, TpComm* tp, bool f32)
     : m_(m), e_(e), tp_(tp), max_batch_(max_batch), max_seq_(max_seq), stream_(stream) {
     if (!m) throw Error(kErrInvalid, "model is NULL");
     if (m->tp.tp_size > 1) {
@@ -366,16 +298,10 @@ Session::Session(const Model* m, const Expert* e, int max_batch, int max_seq, cu
         TFFN_CUDA(cudaStreamCreateWithFlags(&stream_, cudaStreamNonBlocking));
         own_stream_ = true;
     }
-    const Config& c = m->cfg;
-    // this rank's sizes (the whole model without tensor parallelism)
-    const size_t H = c.hidden_size, I = m->I, V = c.vocab_size;
-    const size_t nh = m->nh, nkv = m->nkv, hd = c.head_dim, L = c.num_layers;
+    if (f32 && m->stack.empty()) throw Error(kErrUnsupported, "sessions of the " + m->cfg.family + " family compute in bf16 only");
 
     max_pages_per_seq_ = (max_seq + kPageTokens - 1) / kPageTokens;
     num_pages_ = max_batch * max_pages_per_seq_;
-    const size_t layer_stride = (size_t)num_pages_ * nkv * kPageTokens * hd;
-    k_pool_.alloc(L * layer_stride * 2);
-    v_pool_.alloc(L * layer_stride * 2);
     h_block_table_.assign((size_t)max_batch * max_pages_per_seq_, -1);
     block_table_.alloc(h_block_table_.size() * 4);
     TFFN_CUDA(cudaMemcpy(block_table_.p, h_block_table_.data(), h_block_table_.size() * 4, cudaMemcpyHostToDevice));
@@ -385,29 +311,7 @@ Session::Session(const Model* m, const Expert* e, int max_batch, int max_seq, cu
     seq_len_dev_.alloc((size_t)max_batch * 4);
     free_pages_.resize(num_pages_);
     for (int i = 0; i < num_pages_; ++i) free_pages_[i] = num_pages_ - 1 - i;  // pop_back hands out 0,1,2,...
-    kv_.k_pool = k_pool_.as<bf16>();
-    kv_.v_pool = v_pool_.as<bf16>();
-    kv_.block_table = block_table_.as<int>();
-    kv_.max_pages_per_seq = max_pages_per_seq_;
-    kv_.num_pages = num_pages_;
-    kv_.layer_stride = layer_stride;
-    kv_.nkv = (int)nkv;
-    kv_.hd = (int)hd;
-
-    // RoPE tables in float, as the reference builds them on the host (inference/src/model/qwen.cu:120-132)
-    {
-        const int half = (int)hd / 2;
-        std::vector<float> cs((size_t)max_seq * half), sn((size_t)max_seq * half);
-        for (int pos = 0; pos < max_seq; ++pos)
-            for (int i = 0; i < half; ++i) {
-                float freq = 1.f / powf(c.rope_theta, (float)(2 * i) / (float)hd);
-                cs[(size_t)pos * half + i] = cosf(pos * freq);
-                sn[(size_t)pos * half + i] = sinf(pos * freq);
-            }
-        upload(rope_cos_, cs.data(), cs.size() * 4);
-        upload(rope_sin_, sn.data(), sn.size() * 4);
-    }
-
+    const size_t H = m->cfg.hidden_size;
     cap_tokens_ = H <= 2048 ? 4096 : 2048;
     if (cap_tokens_ < ((max_batch + 255) / 256) * 256) cap_tokens_ = ((max_batch + 255) / 256) * 256;
     const size_t T = cap_tokens_;
@@ -423,6 +327,55 @@ Session::Session(const Model* m, const Expert* e, int max_batch, int max_seq, cu
         std::vector<int> id(T);
         for (size_t i = 0; i < T; ++i) id[i] = (int)i;
         upload(identity_, id.data(), T * 4);
+    }
+    if (m->stack.empty()) alloc_uniform();
+    else alloc_stack(f32);
+    ensure_logits(std::max<size_t>(256, max_batch));
+    attn_partials_.alloc((size_t)32 << 20);
+    attn_counters_.alloc(16384 * 4);
+    status_.alloc(4);
+    step_counter_.alloc(4);
+    TFFN_CUDA(cudaMallocHost(&h_status_, 4));
+    *h_status_ = 0;
+
+    cuda_check((cudaError_t)gemm_prepare(), "gemm_prepare", __FILE__, __LINE__);
+    cuda_check((cudaError_t)attn_prepare(), "attn_prepare", __FILE__, __LINE__);
+    cuda_check((cudaError_t)rows_prepare(), "rows_prepare", __FILE__, __LINE__);
+    cuda_check(prefer_max_shared(k_decode_advance), "carveout", __FILE__, __LINE__);
+}
+
+// cache, activations and exchange buffers of the uniform Qwen2 stack
+void Session::alloc_uniform() {
+    const Model* m = m_;
+    const Config& c = m->cfg;
+    // this rank's sizes (the whole model without tensor parallelism)
+    const size_t H = c.hidden_size, I = m->I, T = cap_tokens_;
+    const size_t nh = m->nh, nkv = m->nkv, hd = c.head_dim, L = c.num_layers;
+    const int max_seq = max_seq_;
+    const size_t layer_stride = (size_t)num_pages_ * nkv * kPageTokens * hd;
+    k_pool_.alloc(L * layer_stride * 2);
+    v_pool_.alloc(L * layer_stride * 2);
+    kv_.k_pool = k_pool_.as<bf16>();
+    kv_.v_pool = v_pool_.as<bf16>();
+    kv_.block_table = block_table_.as<int>();
+    kv_.max_pages_per_seq = max_pages_per_seq_;
+    kv_.num_pages = num_pages_;
+    kv_.layer_stride = layer_stride;
+    kv_.nkv = (int)nkv;
+    kv_.hd = kv_.vd = (int)hd;
+
+    // RoPE tables in float, as the reference builds them on the host (inference/src/model/qwen.cu:120-132)
+    {
+        const int half = (int)hd / 2;
+        std::vector<float> cs((size_t)max_seq * half), sn((size_t)max_seq * half);
+        for (int pos = 0; pos < max_seq; ++pos)
+            for (int i = 0; i < half; ++i) {
+                float freq = 1.f / powf(c.rope_theta, (float)(2 * i) / (float)hd);
+                cs[(size_t)pos * half + i] = cosf(pos * freq);
+                sn[(size_t)pos * half + i] = sinf(pos * freq);
+            }
+        upload(rope_cos_, cs.data(), cs.size() * 4);
+        upload(rope_sin_, sn.data(), sn.size() * 4);
     }
     h_.alloc(T * H * 2);
     xn_.alloc(T * H * 2);
@@ -465,18 +418,6 @@ Session::Session(const Model* m, const Expert* e, int max_batch, int max_seq, cu
         tp_pick_sync_.calls += kTpFlagBlocks;
         for (int p = 0; p < kTpMaxRanks; ++p) tp_pick_parts_.part[p] = p < R ? (const float2*)((const char*)tp_peers_[p] + tp_pick_off_) : nullptr;
     }
-    ensure_logits(std::max<size_t>(256, max_batch));
-    attn_partials_.alloc((size_t)32 << 20);
-    attn_counters_.alloc(16384 * 4);
-    status_.alloc(4);
-    step_counter_.alloc(4);
-    TFFN_CUDA(cudaMallocHost(&h_status_, 4));
-    *h_status_ = 0;
-
-    cuda_check((cudaError_t)gemm_prepare(), "gemm_prepare", __FILE__, __LINE__);
-    cuda_check((cudaError_t)attn_prepare(), "attn_prepare", __FILE__, __LINE__);
-    cuda_check((cudaError_t)rows_prepare(), "rows_prepare", __FILE__, __LINE__);
-    cuda_check(prefer_max_shared(k_decode_advance), "carveout", __FILE__, __LINE__);
     if (m->bs1_ok) cuda_check((cudaError_t)bs1_prepare((int)H, true), "bs1_prepare", __FILE__, __LINE__);
     bs1_h_.alloc(2 * H * 2);  // the residual stream alternates between two buffers from layer to layer
     bs1_acc_.alloc(2 * bs1_acc_words((int)H) * 8);
@@ -485,7 +426,6 @@ Session::Session(const Model* m, const Expert* e, int max_batch, int max_seq, cu
     bs1_tickets_.alloc(256 * 4);
     bs1_lm_val_.alloc((size_t)m->num_sms * 2 * 4);
     bs1_lm_idx_.alloc((size_t)m->num_sms * 2 * 4);
-    (void)V;
 }
 
 Session::~Session() {
@@ -504,6 +444,21 @@ Session::~Session() {
     if (h_pinned_i32_) cudaFreeHost(h_pinned_i32_);
     if (h_sample_u_) cudaFreeHost(h_sample_u_);
     if (own_stream_) cudaStreamDestroy(stream_);
+}
+
+int32_t* PinnedI32::get(size_t n) {
+    if (n > cap) {
+        release();
+        const size_t c = std::max<size_t>(n, 4096);
+        TFFN_CUDA(cudaMallocHost(&p, c * 4));
+        cap = c;
+    }
+    return p;
+}
+void PinnedI32::release() {
+    if (p) cudaFreeHost(p);
+    p = nullptr;
+    cap = 0;
 }
 
 int32_t* Session::pinned_i32(size_t n) {
@@ -662,16 +617,30 @@ void Session::capture_hidden(int max_rows) {
     TFFN_CUDA(cudaStreamSynchronize(stream_));
     hidden_rows_cap_ = max_rows;
     hidden_rows_ = 0;
-    if (max_rows > 0) hidden_.alloc((size_t)m_->cfg.num_layers * max_rows * m_->cfg.hidden_size * 2);
+    const size_t elem = st_ ? 4 : 2;  // the residual stream's own type
+    if (max_rows > 0) hidden_.alloc((size_t)m_->cfg.num_layers * max_rows * m_->cfg.hidden_size * elem);
     else hidden_.release();
 }
-int Session::get_hidden(int layer, uint16_t* dst, int max_rows) {
+int Session::get_hidden_f32(int layer, float* dst, int max_rows) {
     if (layer < 0 || layer >= m_->cfg.num_layers || !dst) throw Error(kErrInvalid, "bad layer or destination");
     const int rows = std::min(hidden_rows_, max_rows);
     if (rows <= 0) return 0;
-    const size_t H = m_->cfg.hidden_size;
+    const size_t H = m_->cfg.hidden_size, first = (size_t)layer * hidden_rows_cap_ * H;
     TFFN_CUDA(cudaStreamSynchronize(stream_));
-    TFFN_CUDA(cudaMemcpy(dst, hidden_.as<bf16>() + (size_t)layer * hidden_rows_cap_ * H, (size_t)rows * H * 2, cudaMemcpyDeviceToHost));
+    if (st_) {
+        TFFN_CUDA(cudaMemcpy(dst, hidden_.as<float>() + first, (size_t)rows * H * 4, cudaMemcpyDeviceToHost));
+        return rows;
+    }
+    std::vector<uint16_t> half((size_t)rows * H);
+    TFFN_CUDA(cudaMemcpy(half.data(), hidden_.as<bf16>() + first, half.size() * 2, cudaMemcpyDeviceToHost));
+    for (size_t i = 0; i < half.size(); ++i) dst[i] = bf16_to_f32(half[i]);
+    return rows;
+}
+int Session::get_hidden(int layer, uint16_t* dst, int max_rows) {
+    if (!dst || max_rows < 0) throw Error(kErrInvalid, "bad layer or destination");
+    std::vector<float> wide((size_t)std::min(hidden_rows_, max_rows) * m_->cfg.hidden_size + 1);
+    const int rows = get_hidden_f32(layer, wide.data(), max_rows);
+    for (size_t i = 0; i < (size_t)rows * m_->cfg.hidden_size; ++i) dst[i] = f32_to_bf16(wide[i]);
     return rows;
 }
 
@@ -694,7 +663,9 @@ void Session::check_status() {
 const char* kclass_name(int c) {
     static const char* names[KC_COUNT] = {"embed_rows", "rmsnorm_rows", "gemm_tc:qkv", "attn_decode",
                                           "gemm_tc:o_proj", "gemm_tc:gate_up_swiglu", "gemm_tc:down", "gemm_tc:lm_head",
-                                          "argmax_rows", "decode_advance", "bs1_qkv", "bs1_oproj", "bs1_ffn", "bs1_lmhead", "tp_all_reduce"};
+                                          "argmax_rows", "decode_advance", "bs1_qkv", "bs1_oproj", "bs1_ffn", "bs1_lmhead", "tp_all_reduce",
+                                          "residual_rows", "gemm:mixer_in", "qk_norm_rope", "gemm:low_rank", "delta_prep", "delta_scan",
+                                          "gemm:router", "moe_route", "moe_gather", "gemm:expert_up", "gemm:expert_down"};
     return (c >= 0 && c < KC_COUNT) ? names[c] : "?";
 }
 void Session::set_profile(bool on) {
@@ -752,10 +723,10 @@ int Session::read_profile(float* ms, int* counts, int cap) {
 }
 
 // ---------------------------------------------------------------- batched path (tensor-core GEMMs)
-int Session::build_groups(const int* seq, const int* pos, int T, int32_t* first, int32_t* count) {
+int Session::build_groups(const int* seq, const int* pos, int T, int limit, int32_t* first, int32_t* count) {
     int n = 0;
     for (int i = 0; i < T; ++i) {
-        const bool extend = n > 0 && count[n - 1] < 8 && seq[i] == seq[i - 1] && pos[i] == pos[i - 1] + 1;
+        const bool extend = n > 0 && count[n - 1] < limit && seq[i] == seq[i - 1] && pos[i] == pos[i - 1] + 1;
         if (extend) {
             ++count[n - 1];
         } else {
@@ -767,11 +738,108 @@ int Session::build_groups(const int* seq, const int* pos, int T, int32_t* first,
     return n;
 }
 
-void Session::run_batched(int T, int n_logit_rows, bool logit_rows_are_all, bool decode, int max_ctx, int n_groups) {
+// one GEMM of a step: tensor cores, or true fp32 in a session that computes in fp32
+void Session::gemm(GemmCall& call, int cls, bool pdl) {
+    if ((ablate_mask_ >> cls) & 1u) return;  // timing-only ablation: results are then meaningless
+    call.pdl = pdl;
+    call.tl = tl_next(cls);
+    call.trace = (tl_on_ && (int)tl_cls_.size() - 1 == tl_trace_launch_) ? tl_trace_buf_.as<unsigned long long>() : nullptr;
+    call.trace_ctas = (int)(tl_trace_buf_.bytes / (64 * 8));
+    prof_begin(cls);
+    const int rc = st_ && st_->f32 ? launch_gemm_f32(call, stream_) : launch_gemm(call, gemm_ws(), stream_);
+    prof_end();
+    if (rc == -1000) throw Error(kErrCuda, "cuTensorMapEncodeTiled failed or is unavailable");
+    if (rc != 0) cuda_check((cudaError_t)rc, "GEMM launch", __FILE__, __LINE__);
+    launches_++;
+}
+
+Session::Staged Session::stage_rows(const int32_t* tsp, int T) {
+    const int32_t *seq = tsp + T, *pos = tsp + 2 * T;
+    TFFN_CUDA(cudaMemcpyAsync(tokens_.p, tsp, (size_t)T * 4, cudaMemcpyHostToDevice, stream_));
+    TFFN_CUDA(cudaMemcpyAsync(tok_seq_.p, seq, (size_t)T * 4, cudaMemcpyHostToDevice, stream_));
+    TFFN_CUDA(cudaMemcpyAsync(tok_pos_.p, pos, (size_t)T * 4, cudaMemcpyHostToDevice, stream_));
+    int32_t* runs = h_pinned_runs_.get((size_t)T * 4);
+    Staged r;
+    r.n_groups = build_groups(seq, pos, T, 8, runs, runs + T);
+    TFFN_CUDA(cudaMemcpyAsync(grp_first_.p, runs, (size_t)r.n_groups * 4, cudaMemcpyHostToDevice, stream_));
+    TFFN_CUDA(cudaMemcpyAsync(grp_count_.p, runs + T, (size_t)r.n_groups * 4, cudaMemcpyHostToDevice, stream_));
+    r.n_segs = 0;
+    if (st_) {
+        r.n_segs = build_groups(seq, pos, T, T, runs + 2 * T, runs + 3 * T);
+        TFFN_CUDA(cudaMemcpyAsync(st_->seg_first.p, runs + 2 * T, (size_t)r.n_segs * 4, cudaMemcpyHostToDevice, stream_));
+        TFFN_CUDA(cudaMemcpyAsync(st_->seg_count.p, runs + 3 * T, (size_t)r.n_segs * 4, cudaMemcpyHostToDevice, stream_));
+    }
+    return r;
+}
+
+// logits (and picks) of n_rows normalised rows
+void Session::lm_head(const void* x, int64_t ldx, int n_rows, bool decode, bool pdl) {
+    const int V = m_->cfg.vocab_size, Vl = m_->V;
+    const bool tp = tp_ != nullptr;
+    auto live = [&](int cls) { return ((ablate_mask_ >> cls) & 1u) == 0; };
+    GemmCall g;
+    memset(&g, 0, sizeof g);
+    g.x_rows_alloc = cap_tokens_;
+    g.T = n_rows;
+    g.alpha = 1.f;
+    g.op[0] = {m_->lm_head, m_->embed_ld, (const bf16*)x, ldx, m_->cfg.hidden_size};
+    g.N = Vl;  // this rank's rows of the vocabulary
+    g.mode = GEMM_STORE_F32;
+    g.ldo = Vl;
+    // The greedy pick rides in the LM head's epilogue (per-tile maxima, combined by a tiny kernel); the
+    // fp32 logits themselves are written only when the caller asked for them. The attention workspace is
+    // idle by now and serves as scratch.
+    const AttnWorkspace aw = attn_ws();
+    const int v_tiles = (Vl + 127) / 128;
+    const bool fused_pick = !sampling() && !(st_ && st_->f32) && (size_t)n_rows * v_tiles * 2 <= aw.partial_floats;
+    if (tp && !fused_pick) throw Error(kErrUnsupported, "tensor parallel: sampling and very large logit batches are not split across ranks");
+    if (fused_pick) {
+        g.amax_val = aw.partials;
+        g.amax_idx = (int*)(aw.partials + (size_t)n_rows * v_tiles);
+    }
+    g.out = (store_logits_ || !fused_pick) ? logits_.p : nullptr;
+    gemm(g, KC_GEMM_LMHEAD, pdl);
+    prof_begin(KC_ARGMAX);
+    if (live(KC_ARGMAX)) {
+        if (fused_pick && tp) {
+            // every rank's best of its vocabulary slice, exchanged (8 bytes per row and rank), then the same
+            // pick on every rank: largest value, lowest global index among equals (main.cpp:45-51)
+            const size_t bytes = (size_t)n_rows * 8;
+            if (tp_pick_send_.bytes < bytes) throw Error(kErrCapacity, "tensor parallel: more logits rows than the session was sized for");
+            if (tp_fused_ && n_rows <= tp_small_rows_) {
+                // candidates left in this rank's window, the pick kernel hand-shakes and loads every rank's: no NCCL call
+                // in a decode step
+                launch_argmax_tiles(g.amax_val, g.amax_idx, n_rows, v_tiles, picks_.as<int>(), stream_, pdl, tl_next(KC_ARGMAX),
+                                    (char*)tp_win_.p + tp_pick_off_, m_->tp.v0);
+                launch_tp_pick_peer(tp_pick_parts_, tp_pick_sync_, n_rows, picks_.as<int>(), status_.as<int>(), stream_, pdl);
+                launches_ += 1;
+            } else {
+                launch_argmax_tiles(g.amax_val, g.amax_idx, n_rows, v_tiles, picks_.as<int>(), stream_, pdl, tl_next(KC_ARGMAX),
+                                    tp_pick_send_.p, m_->tp.v0);
+                tp_all_gather_bytes(tp_, tp_pick_send_.p, tp_pick_recv_.p, bytes, stream_);
+                launch_tp_pick(tp_pick_recv_.p, m_->tp.tp_size, n_rows, picks_.as<int>(), stream_, pdl);
+                launches_ += 2;
+            }
+        } else if (fused_pick)
+            launch_argmax_tiles(g.amax_val, g.amax_idx, n_rows, v_tiles, picks_.as<int>(), stream_, pdl, tl_next(KC_ARGMAX));
+        else if (sampling())
+            launch_sample(logits_.as<float>(), n_rows, V, sample_temp_, sample_u_.as<double>(),
+                          decode ? step_counter_.as<int>() : nullptr, picks_.as<int>(), stream_, pdl, tl_next(KC_ARGMAX));
+        else
+            launch_argmax(logits_.as<float>(), n_rows, V, picks_.as<int>(), aw.partials, aw.partial_floats, aw.counters,
+                          aw.num_counters, m_->num_sms, stream_, pdl, tl_next(KC_ARGMAX));
+    }
+    prof_end();
+    launches_ += 2;
+}
+
+void Session::run_batched(int T, int n_logit_rows, bool logit_rows_are_all, bool decode, int max_ctx, Staged runs) {
+    if (st_) return run_stack(T, n_logit_rows, logit_rows_are_all, decode, max_ctx, runs.n_groups, runs.n_segs);
+    const int n_groups = runs.n_groups;
     const Config& c = m_->cfg;
     // this rank's slice of the heads, of the intermediate dimension and of the LM head (everything without
     // tensor parallelism); the vocabulary of the embedding is always the whole one
-    const int H = c.hidden_size, I = m_->I, V = c.vocab_size, Vl = m_->V;
+    const int H = c.hidden_size, I = m_->I, V = c.vocab_size;
     const int nh = m_->nh, nkv = m_->nkv, hd = c.head_dim;
     const int nqkv = (nh + 2 * nkv) * hd;
     const bool tp = tp_ != nullptr;
@@ -800,22 +868,8 @@ void Session::run_batched(int T, int n_logit_rows, bool logit_rows_are_all, bool
     const int* tok_seq = decode ? identity_.as<int>() : tok_seq_.as<int>();
     const int* tok_pos = decode ? seq_len_dev_.as<int>() : tok_pos_.as<int>();
     int* status = status_.as<int>();
-    const GemmWorkspace gws = gemm_ws();
     // timing-only ablation: a class in the mask is not launched (results are then meaningless)
     auto live = [&](int cls) { return ((ablate_mask_ >> cls) & 1u) == 0; };
-    auto gemm = [&](GemmCall& call, int cls) {
-        if (!live(cls)) return;
-        call.pdl = pdl;
-        call.tl = tl_next(cls);
-        call.trace = (tl_on_ && (int)tl_cls_.size() - 1 == tl_trace_launch_) ? tl_trace_buf_.as<unsigned long long>() : nullptr;
-        call.trace_ctas = (int)(tl_trace_buf_.bytes / (64 * 8));
-        prof_begin(cls);
-        int rc = launch_gemm(call, gws, stream_);
-        prof_end();
-        if (rc == -1000) throw Error(kErrCuda, "cuTensorMapEncodeTiled failed or is unavailable");
-        if (rc != 0) cuda_check((cudaError_t)rc, "tensor-core GEMM launch", __FILE__, __LINE__);
-        launches_++;
-    };
     prof_begin(KC_EMBED);
     launch_embed(tokens, m_->embed.as<bf16>(), h_.as<bf16>(), T, H, V, status, stream_, false, tl_next(KC_EMBED));
     prof_end();
@@ -854,7 +908,7 @@ void Session::run_batched(int T, int n_logit_rows, bool logit_rows_are_all, bool
         g.qkv = &qe;
         g.out = nullptr;
         g.ldo = nqkv;
-        gemm(g, KC_GEMM_QKV);
+        gemm(g, KC_GEMM_QKV, pdl);
         g.qkv = nullptr;
         prof_begin(KC_ATTENTION);
         if (live(KC_ATTENTION) && n_groups > 0) {
@@ -875,7 +929,7 @@ void Session::run_batched(int T, int n_logit_rows, bool logit_rows_are_all, bool
         g.mode = tp ? GEMM_STORE_F32 : GEMM_RESIDUAL;
         g.out = fused ? (void*)((float*)tp_win_.p + tp_part_off_[0]) : tp ? delta_.p : h_.p;
         g.ldo = H;
-        gemm(g, KC_GEMM_OPROJ);
+        gemm(g, KC_GEMM_OPROJ, pdl);
         prof_begin(KC_RMSNORM);
         if (fused) {
             prof_end();
@@ -909,7 +963,7 @@ void Session::run_batched(int T, int n_logit_rows, bool logit_rows_are_all, bool
                 g.op2[1] = {erec + H, (int64_t)3 * H, xn_.as<bf16>(), H, H};
                 g.out2 = act_e_.p;
             }
-            gemm(g, KC_GEMM_GATEUP);
+            gemm(g, KC_GEMM_GATEUP, pdl);
             g.out2 = nullptr;
         }
         // down projections of base and expert into two accumulators, summed in fp32, + residual
@@ -924,7 +978,7 @@ void Session::run_batched(int T, int n_logit_rows, bool logit_rows_are_all, bool
         g.mode = tp ? GEMM_STORE_F32 : GEMM_RESIDUAL;
         g.out = fused ? (void*)((float*)tp_win_.p + tp_part_off_[1]) : tp ? delta_.p : h_.p;
         g.ldo = H;
-        gemm(g, KC_GEMM_DOWN);
+        gemm(g, KC_GEMM_DOWN, pdl);
         g.alpha = 1.f;
         if (fused) {
             reduce_fused(1, l + 1 < c.num_layers ? m_->layers[l + 1].attn_norm.as<bf16>() : nullptr);
@@ -951,60 +1005,7 @@ void Session::run_batched(int T, int n_logit_rows, bool logit_rows_are_all, bool
         launch_rmsnorm(h_.as<bf16>(), m_->final_norm.as<bf16>(), xn_last_.as<bf16>(), n_logit_rows, H, c.rms_norm_eps, rows, stream_, pdl,
                        tl_next(KC_RMSNORM));
         prof_end();
-        GemmCall g;
-        memset(&g, 0, sizeof g);
-        g.x_rows_alloc = cap_tokens_;
-        g.T = n_logit_rows;
-        g.alpha = 1.f;
-        g.op[0] = {m_->lm_head, H, xn_last_.as<bf16>(), H, H};
-        g.N = Vl;  // this rank's rows of the vocabulary
-        g.mode = GEMM_STORE_F32;
-        g.ldo = Vl;
-        // The greedy pick rides in the LM head's epilogue (per-tile maxima, combined by a tiny kernel); the
-        // fp32 logits themselves are written only when the caller asked for them. The attention workspace is
-        // idle by now and serves as scratch.
-        const AttnWorkspace aw = attn_ws();
-        const int v_tiles = (Vl + 127) / 128;
-        const bool fused_pick = !sampling() && (size_t)n_logit_rows * v_tiles * 2 <= aw.partial_floats;
-        if (tp && !fused_pick) throw Error(kErrUnsupported, "tensor parallel: sampling and very large logit batches are not split across ranks");
-        if (fused_pick) {
-            g.amax_val = aw.partials;
-            g.amax_idx = (int*)(aw.partials + (size_t)n_logit_rows * v_tiles);
-        }
-        g.out = (store_logits_ || !fused_pick) ? logits_.p : nullptr;
-        gemm(g, KC_GEMM_LMHEAD);
-        prof_begin(KC_ARGMAX);
-        if (live(KC_ARGMAX)) {
-            if (fused_pick && tp) {
-                // every rank's best of its vocabulary slice, exchanged (8 bytes per row and rank), then the same
-                // pick on every rank: largest value, lowest global index among equals (main.cpp:45-51)
-                const size_t bytes = (size_t)n_logit_rows * 8;
-                if (tp_pick_send_.bytes < bytes) throw Error(kErrCapacity, "tensor parallel: more logits rows than the session was sized for");
-                if (tp_fused_ && n_logit_rows <= tp_small_rows_) {
-                    // candidates left in this rank's window, the pick kernel hand-shakes and loads every rank's: no NCCL call
-                    // in a decode step
-                    launch_argmax_tiles(g.amax_val, g.amax_idx, n_logit_rows, v_tiles, picks_.as<int>(), stream_, pdl, tl_next(KC_ARGMAX),
-                                        (char*)tp_win_.p + tp_pick_off_, m_->tp.v0);
-                    launch_tp_pick_peer(tp_pick_parts_, tp_pick_sync_, n_logit_rows, picks_.as<int>(), status_.as<int>(), stream_, pdl);
-                    launches_ += 1;
-                } else {
-                    launch_argmax_tiles(g.amax_val, g.amax_idx, n_logit_rows, v_tiles, picks_.as<int>(), stream_, pdl, tl_next(KC_ARGMAX),
-                                        tp_pick_send_.p, m_->tp.v0);
-                    tp_all_gather_bytes(tp_, tp_pick_send_.p, tp_pick_recv_.p, bytes, stream_);
-                    launch_tp_pick(tp_pick_recv_.p, m_->tp.tp_size, n_logit_rows, picks_.as<int>(), stream_, pdl);
-                    launches_ += 2;
-                }
-            } else if (fused_pick)
-                launch_argmax_tiles(g.amax_val, g.amax_idx, n_logit_rows, v_tiles, picks_.as<int>(), stream_, pdl, tl_next(KC_ARGMAX));
-            else if (sampling())
-                launch_sample(logits_.as<float>(), n_logit_rows, V, sample_temp_, sample_u_.as<double>(),
-                              decode ? step_counter_.as<int>() : nullptr, picks_.as<int>(), stream_, pdl, tl_next(KC_ARGMAX));
-            else
-                launch_argmax(logits_.as<float>(), n_logit_rows, V, picks_.as<int>(), aw.partials, aw.partial_floats, aw.counters,
-                              aw.num_counters, m_->num_sms, stream_, pdl, tl_next(KC_ARGMAX));
-        }
-        prof_end();
-        launches_ += 2;
+        lm_head(xn_last_.p, H, n_logit_rows, decode, pdl);
     }
     TFFN_CUDA(cudaGetLastError());
 }
@@ -1190,9 +1191,7 @@ void Session::run_decode_batched(int n_seqs, int max_ctx) {
         body();
         return;
     }
-    const Config& c = m_->cfg;
-    const int splits = attention_splits(n_seqs, c.num_heads, c.num_kv_heads, c.head_dim, max_ctx, attn_ws(), m_->num_sms);
-    const auto key = std::make_pair(n_seqs, splits * 2 + (store_logits_ ? 1 : 0));
+    const auto key = std::make_pair(n_seqs, decode_graph_key(n_seqs, max_ctx) * 2 + (store_logits_ ? 1 : 0));
     auto it = dec_graphs_.find(key);
     if (it == dec_graphs_.end()) {
         cudaGraph_t graph = nullptr;
@@ -1247,7 +1246,7 @@ void Session::prefill(const int32_t* tokens, const int32_t* seq_lens, int n_seqs
     }
     for (size_t c0 = 0; c0 < total; c0 += cap_tokens_) {
         const int T = (int)std::min<size_t>(cap_tokens_, total - c0);
-        int32_t* pin = pinned_i32((size_t)T * 6);
+        int32_t* pin = pinned_i32((size_t)T * 4);
         std::vector<int> last_rows, last_slots;
         int max_ctx = 1;
         for (int i = 0; i < T; ++i) {
@@ -1261,17 +1260,12 @@ void Session::prefill(const int32_t* tokens, const int32_t* seq_lens, int n_seqs
             }
         }
         for (size_t i = 0; i < last_rows.size(); ++i) pin[3 * T + i] = last_rows[i];
-        TFFN_CUDA(cudaMemcpyAsync(tokens_.p, pin, (size_t)T * 4, cudaMemcpyHostToDevice, stream_));
-        TFFN_CUDA(cudaMemcpyAsync(tok_seq_.p, pin + T, (size_t)T * 4, cudaMemcpyHostToDevice, stream_));
-        TFFN_CUDA(cudaMemcpyAsync(tok_pos_.p, pin + 2 * T, (size_t)T * 4, cudaMemcpyHostToDevice, stream_));
         if (!last_rows.empty())
             TFFN_CUDA(cudaMemcpyAsync(row_idx_.p, pin + 3 * T, last_rows.size() * 4, cudaMemcpyHostToDevice, stream_));
-        const int n_groups = build_groups(pin + T, pin + 2 * T, T, pin + 4 * T, pin + 5 * T);
-        TFFN_CUDA(cudaMemcpyAsync(grp_first_.p, pin + 4 * T, (size_t)n_groups * 4, cudaMemcpyHostToDevice, stream_));
-        TFFN_CUDA(cudaMemcpyAsync(grp_count_.p, pin + 5 * T, (size_t)n_groups * 4, cudaMemcpyHostToDevice, stream_));
+        const Staged runs = stage_rows(pin, T);
         store_logits_ = logits_last != nullptr || sampling();
         if (sampling() && !last_rows.empty()) upload_draws(last_rows.size());  // one draw per sequence, slot order
-        run_batched(T, (int)last_rows.size(), false, false, max_ctx, n_groups);
+        run_batched(T, (int)last_rows.size(), false, false, max_ctx, runs);
         if (!last_rows.empty()) {
             std::vector<int> picks(last_rows.size());
             std::vector<float> rows_host;
@@ -1319,37 +1313,32 @@ void Session::forward(int slot, const int32_t* tokens, int T, float* logits) {
     int last_pick = 0;
     for (int c0 = 0; c0 < T; c0 += chunk_cap) {
         const int n = std::min(chunk_cap, T - c0);
-        int32_t* pin = pinned_i32((size_t)n * 5 + 2);  // the last two: row index in, pick out
+        int32_t* pin = pinned_i32((size_t)n * 3 + 2);  // the last two: row index in, pick out
         for (int i = 0; i < n; ++i) {
             pin[i] = tokens[c0 + i];
             pin[n + i] = slot;
             pin[2 * n + i] = h_seq_len_[slot] + c0 + i;
         }
-        const int n_groups = build_groups(pin + n, pin + 2 * n, n, pin + 3 * n, pin + 4 * n);
-        TFFN_CUDA(cudaMemcpyAsync(grp_first_.p, pin + 3 * n, (size_t)n_groups * 4, cudaMemcpyHostToDevice, stream_));
-        TFFN_CUDA(cudaMemcpyAsync(grp_count_.p, pin + 4 * n, (size_t)n_groups * 4, cudaMemcpyHostToDevice, stream_));
-        TFFN_CUDA(cudaMemcpyAsync(tokens_.p, pin, (size_t)n * 4, cudaMemcpyHostToDevice, stream_));
-        TFFN_CUDA(cudaMemcpyAsync(tok_seq_.p, pin + n, (size_t)n * 4, cudaMemcpyHostToDevice, stream_));
-        TFFN_CUDA(cudaMemcpyAsync(tok_pos_.p, pin + 2 * n, (size_t)n * 4, cudaMemcpyHostToDevice, stream_));
+        const Staged runs = stage_rows(pin, n);
         store_logits_ = logits != nullptr;
         if (logits) {
-            run_batched(n, n, true, false, h_seq_len_[slot] + c0 + n, n_groups);
+            run_batched(n, n, true, false, h_seq_len_[slot] + c0 + n, runs);
             copy_logits_to_host(logits + (size_t)c0 * V, (size_t)n);
             TFFN_CUDA(cudaMemcpyAsync(pin, picks_.as<int>() + (n - 1), 4, cudaMemcpyDeviceToHost, stream_));
             TFFN_CUDA(cudaStreamSynchronize(stream_));
             last_pick = pin[0];
         } else if (c0 + n < T) {
-            run_batched(n, 0, true, false, h_seq_len_[slot] + c0 + n, n_groups);
+            run_batched(n, 0, true, false, h_seq_len_[slot] + c0 + n, runs);
             TFFN_CUDA(cudaStreamSynchronize(stream_));
         } else {
             // no logits wanted: the LM head still runs for the last row, whose greedy pick feeds a
             // following decode step that passes no tokens
-            pin[5 * n] = n - 1;
-            TFFN_CUDA(cudaMemcpyAsync(row_idx_.p, pin + 5 * n, 4, cudaMemcpyHostToDevice, stream_));
-            run_batched(n, 1, false, false, h_seq_len_[slot] + c0 + n, n_groups);
-            TFFN_CUDA(cudaMemcpyAsync(pin + 5 * n + 1, picks_.p, 4, cudaMemcpyDeviceToHost, stream_));
+            pin[3 * n] = n - 1;
+            TFFN_CUDA(cudaMemcpyAsync(row_idx_.p, pin + 3 * n, 4, cudaMemcpyHostToDevice, stream_));
+            run_batched(n, 1, false, false, h_seq_len_[slot] + c0 + n, runs);
+            TFFN_CUDA(cudaMemcpyAsync(pin + 3 * n + 1, picks_.p, 4, cudaMemcpyDeviceToHost, stream_));
             TFFN_CUDA(cudaStreamSynchronize(stream_));
-            last_pick = pin[5 * n + 1];
+            last_pick = pin[3 * n + 1];
         }
     }
     h_seq_len_[slot] += T;

@@ -6,6 +6,7 @@
 #include "kernels.h"
 #include <cstdint>
 #include <map>
+#include <memory>
 #include <string>
 #include <random>
 #include <vector>
@@ -32,6 +33,18 @@ struct DeviceBuffer {
     T* as() const { return (T*)p; }
 };
 
+// growing page-locked staging for small integer lists
+struct PinnedI32 {
+    int32_t* p = nullptr;
+    size_t cap = 0;
+    PinnedI32() = default;
+    PinnedI32(const PinnedI32&) = delete;
+    PinnedI32& operator=(const PinnedI32&) = delete;
+    ~PinnedI32() { release(); }
+    int32_t* get(size_t n);
+    void release();
+};
+
 // One FFN (base or expert) of one layer: records [I][3][H] (gate row, up row, down column) for
 // the batch-1 kernel and, as strided views of the same records, for the tensor-core GEMM;
 // plus down as [H, I] for the GEMM's K-major operand.
@@ -45,6 +58,21 @@ struct LayerWeights {
     bool has_bias = false;
     FfnWeights ffn;
 };
+
+// One entry of a layer list (Config::layers): weights as the kernels read them. Matrices bf16 with rows padded to 8
+// elements, vectors widened to fp32. w_in stacks every projection of the mixer's input (each block of rows padded to
+// 8), so that one GEMM makes them all: q | k | v (attention) or q | k | v | b | a1 | g1 (delta rule).
+struct StackLayer {
+    LayerSpec spec;
+    int in_rows = 0, k_off = 0, v_off = 0, b_off = 0, a1_off = 0, g1_off = 0;
+    int a_rank = 0, g_rank = 0;
+    DeviceBuffer w_in, wo, a2, g2;
+    DeviceBuffer norm1, norm1b, norm2, norm2b;  // in front of and behind the mixer and the feed-forward
+    DeviceBuffer q_norm, k_norm;
+    DeviceBuffer conv, a_log, dt_bias, out_norm;  // conv: [taps][channels]
+    DeviceBuffer router, correction, up, down;    // up [experts * ff][width], down [experts * width][ff]
+};
+inline int64_t pad8(int64_t n) { return (n + 7) & ~(int64_t)7; }
 
 // NCCL communicator of a tensor-parallel group (the library is opened at run time; see tp_comm.cpp)
 struct TpComm;
@@ -69,9 +97,16 @@ struct Model {
     DeviceBuffer embed, final_norm, lm_head_own;
     const bf16* lm_head = nullptr;
     std::vector<LayerWeights> layers;
+    std::vector<StackLayer> stack;  // instead of `layers` when the configuration lists its layers
+    int64_t embed_ld = 0;           // row stride of embed (and of the LM head)
+    DeviceBuffer final_norm_f32;
     bool bs1_ok = false;
     uint64_t weight_bytes_base = 0;  // bytes one decode step streams (every matrix once, LM head included)
     static Model* load(const std::string& dir, int device, int tp_rank, int tp_size);
+
+private:
+    void load_qwen2(const std::string& dir);
+    void load_stack(const std::string& dir);
 };
 
 struct Expert {
@@ -90,9 +125,36 @@ struct Expert {
 // kernel classes of the per-launch profile (tffn_session_profile_*)
 enum KClass : int {
     KC_EMBED = 0, KC_RMSNORM, KC_GEMM_QKV, KC_ATTENTION, KC_GEMM_OPROJ, KC_GEMM_GATEUP, KC_GEMM_DOWN,
-    KC_GEMM_LMHEAD, KC_ARGMAX, KC_ADVANCE, KC_BS1_QKV, KC_BS1_OPROJ, KC_BS1_FFN, KC_BS1_LMHEAD, KC_ALLREDUCE, KC_COUNT
+    KC_GEMM_LMHEAD, KC_ARGMAX, KC_ADVANCE, KC_BS1_QKV, KC_BS1_OPROJ, KC_BS1_FFN, KC_BS1_LMHEAD, KC_ALLREDUCE,
+    KC_ROWS, KC_GEMM_IN, KC_QK_ROPE, KC_GEMM_LOWRANK, KC_DELTA_PREP, KC_DELTA_SCAN, KC_GEMM_ROUTER, KC_ROUTE, KC_GATHER,
+    KC_GEMM_UP, KC_GEMM_EXPERT_DOWN, KC_COUNT
 };
 const char* kclass_name(int c);
+
+// What a session keeps and computes in when the model lists its layers: per attention layer a view of the paged
+// cache (one block table and one page allocator for all layers), per recurrent layer the state of every slot, and
+// the step's buffers. Activations are bf16, or fp32 throughout in a session that computes in fp32.
+struct StackState {
+    bool f32 = false;
+    size_t act = 2;  // bytes of an activation
+    struct LayerCache {
+        DeviceBuffer k, v;         // attention: pages of this layer
+        KvView kv;
+        int rope = -1;             // index into rope
+        DeviceBuffer state, ring;  // delta rule: see DeltaRule
+        size_t state_stride = 0, ring_stride = 0;
+        int dimP = 0, vdimP = 0;
+        int moe = -1;              // index of the layer among those with experts
+    };
+    std::vector<LayerCache> layers;
+    std::vector<DeviceBuffer> rope;  // one table per distinct rotation: [max_seq][dims / 2] (cos, sin)
+    std::vector<RopeSpec> rope_specs;
+    int64_t h_ld = 0, proj_ld = 0, ctx_ld = 0, decay_ld = 0, gate_ld = 0, delta_ld = 0, router_ld = 0, act_ld = 0;
+    int max_top = 0, max_experts = 0, moe_layers = 0, max_tiles = 0;
+    DeviceBuffer proj, delta, qn, kn, v, g, bk, decay, gate;
+    DeviceBuffer router, counts, pair, pair_w, pair_row, xg, act_e, y, tiles;
+    DeviceBuffer seg_first, seg_count, ones;
+};
 
 class Session {
 public:
@@ -106,7 +168,7 @@ public:
     void set_profile(bool on);
     // accumulated device time (ms) and launches per class since set_profile(true); returns KC_COUNT
     int read_profile(float* ms, int* counts, int cap);
-    Session(const Model* m, const Expert* e, int max_batch, int max_seq, cudaStream_t stream, TpComm* tp = nullptr);
+    Session(const Model* m, const Expert* e, int max_batch, int max_seq, cudaStream_t stream, TpComm* tp = nullptr, bool f32 = false);
     ~Session();
     void reset(int slot);
     int seq_len(int slot) const { return h_seq_len_[slot]; }
@@ -125,12 +187,14 @@ public:
     void set_sampling(float temperature, uint32_t seed);
     void capture_hidden(int max_rows);
     int get_hidden(int layer, uint16_t* dst, int max_rows);
+    int get_hidden_f32(int layer, float* dst, int max_rows);
     int status();
     uint64_t launch_count() const { return launches_; }
     cudaStream_t stream() const { return stream_; }
     const Model* model() const { return m_; }
 
 private:
+    struct Staged { int n_groups, n_segs; };  // runs of rows: at most 8 positions of a sequence; all of a sequence
     const Model* m_;
     const Expert* e_;
     TpComm* tp_ = nullptr;  // not owned
@@ -194,6 +258,7 @@ private:
     int* h_status_ = nullptr;  // pinned
     int32_t* h_pinned_i32_ = nullptr;
     size_t h_pinned_cap_ = 0;
+    PinnedI32 h_pinned_runs_;
 
     // batch-1 path
     DeviceBuffer bs1_h_, bs1_acc_, bs1_q_, bs1_ctx_, bs1_tickets_, bs1_lm_val_, bs1_lm_idx_;
@@ -220,6 +285,21 @@ private:
     DeviceBuffer hidden_;
     int hidden_rows_cap_ = 0, hidden_rows_ = 0;
 
+    // layer lists (engine_stack.cu)
+    std::unique_ptr<StackState> st_;
+    void alloc_uniform();
+    void alloc_stack(bool f32);
+    void run_stack(int T, int n_logit_rows, bool logit_rows_are_all, bool decode, int max_ctx, int n_groups, int n_segs);
+    int attn_ctx(const LayerSpec& l, int max_ctx) const { return l.chunk > 0 && l.chunk < max_ctx ? l.chunk : max_ctx; }
+    AttnOptions attn_options(const LayerSpec& l) const;
+    // everything in a captured decode step's grids that depends on the context
+    int decode_graph_key(int n_seqs, int max_ctx) const;
+
+    void gemm(GemmCall& call, int cls, bool pdl);
+    void lm_head(const void* x, int64_t ldx, int n_rows, bool decode, bool pdl);
+    // tokens, slots and positions of T rows (three consecutive lists) to the device, with the runs the kernels need
+    Staged stage_rows(const int32_t* tok_seq_pos, int T);
+
     GemmWorkspace gemm_ws() const;
     TmapCache* tmaps_ = tmap_cache_create();  // encoded tensor maps of this session's GEMM launches
     AttnWorkspace attn_ws() const;
@@ -228,9 +308,10 @@ private:
     void ensure_logits(size_t rows);
     void ensure_ring(int entries);
     // runs T tokens already staged in tokens_/tok_seq_/tok_pos_ (or decode state when decode=true)
-    void run_batched(int T, int n_logit_rows, bool logit_rows_are_all, bool decode, int max_ctx, int n_groups = 0);
+    void run_batched(int T, int n_logit_rows, bool logit_rows_are_all, bool decode, int max_ctx, Staged runs = {0, 0});
     // groups for launch_attention_prefill from the rows' (slot, position) lists; fills pin[0..2*n) and returns n
-    static int build_groups(const int* seq, const int* pos, int T, int32_t* first, int32_t* count);
+    // (runs of consecutive positions of one sequence, at most `limit` rows each)
+    static int build_groups(const int* seq, const int* pos, int T, int limit, int32_t* first, int32_t* count);
     void run_bs1(bool want_logits);
     void launch_bs1_step(bool want_logits, bool pdl);
     Bs1Ctx bs1_ctx(bool want_logits) const;

@@ -1,0 +1,557 @@
+// Models that list their layers (Config::layers): weight loading, what a session keeps for them, and the step. The step
+// runs under the same prefill / forward / decode calls, page allocator, slots, graphs and pick as the uniform stack
+// (engine.cu); every layer is described by its LayerSpec, so a family that combines the same mechanisms differently
+// needs a reader in host_io.cpp and nothing here.
+#include "engine.h"
+#include "launch.h"
+#include "upload.h"
+#include <cmath>
+
+namespace tffn {
+
+namespace {
+
+int64_t pad4(int64_t n) { return (n + 3) & ~(int64_t)3; }
+
+// bf16 matrix of the file -> device rows of `ld` elements (the padding was zeroed when the slab was made)
+void put_matrix(Stager& up, bf16* dst, const uint16_t* src, size_t rows, size_t cols, size_t ld) {
+    if (ld == cols) return up.copy(dst, src, rows * cols * 2);
+    std::vector<uint16_t> wide(rows * ld, 0);
+    for (size_t r = 0; r < rows; ++r) memcpy(wide.data() + r * ld, src + r * cols, cols * 2);
+    up.copy(dst, wide.data(), wide.size() * 2);
+}
+void put_vector(Stager& up, const DeviceBuffer& dst, const uint16_t* src, size_t n) {
+    std::vector<float> wide(n);
+    for (size_t i = 0; i < n; ++i) wide[i] = bf16_to_f32(src[i]);
+    up.copy(dst.p, wide.data(), n * 4);
+}
+
+// every weight buffer of a layer with its size, in slab order
+template <typename Take>
+void layout_layer(StackLayer& l, size_t H, Take take) {
+    const LayerSpec& s = l.spec;
+    const size_t ld = pad8(H), nv = (size_t)s.heads * s.vdim;
+    take(l.w_in, (size_t)l.in_rows * ld * 2);
+    take(l.wo, H * pad8(nv) * 2);
+    take(l.norm1, H * 4);
+    take(l.norm1b, H * 4);
+    if (s.mixer == Mixer::Attention) {
+        take(l.q_norm, (size_t)s.dim * 4);
+        take(l.k_norm, (size_t)s.dim * 4);
+    } else {
+        take(l.conv, (2 * (size_t)s.kv_heads * s.dim + nv) * s.conv * 4);
+        take(l.a_log, (size_t)s.heads * 4);
+        take(l.dt_bias, (size_t)s.heads * s.dim * 4);
+        take(l.out_norm, (size_t)s.vdim * 4);
+        take(l.a2, (size_t)s.heads * s.dim * pad8(l.a_rank) * 2);
+        take(l.g2, nv * pad8(l.g_rank) * 2);
+    }
+    if (s.experts > 0) {
+        take(l.norm2, H * 4);
+        take(l.norm2b, H * 4);
+        take(l.router, (size_t)(s.experts + s.identity) * ld * 2);
+        take(l.correction, (size_t)(s.experts + s.identity) * 4);
+        take(l.up, (size_t)s.experts * s.ff * ld * 2);
+        take(l.down, (size_t)s.experts * H * pad8(s.ff) * 2);
+    }
+}
+
+__global__ void k_copy_rows_f32(const float* __restrict__ src, float* __restrict__ dst, size_t n) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) dst[i] = src[i];
+}
+
+}  // namespace
+
+void Model::load_stack(const std::string& dir) {
+    const Config& c = cfg;
+    const size_t H = c.hidden_size, vocab = c.vocab_size, ld = pad8(H);
+    V = c.vocab_size;
+    if (H > 16384) throw Error(kErrUnsupported, "the residual stream is wider than 16384");
+    SafeTensorsDir st(dir);
+    stack.resize(c.layers.size());
+    size_t total = Slab::padded(vocab * ld * 2) + Slab::padded(H * 4);
+    auto name = [](size_t i) { return "l" + std::to_string(i) + "."; };
+    for (size_t i = 0; i < stack.size(); ++i) {
+        StackLayer& l = stack[i];
+        const LayerSpec& s = l.spec = c.layers[i];
+        const std::string p = name(i) + "mix.";
+        const int nq = s.kv_heads * s.dim, nv = s.heads * s.vdim;
+        if (s.dim > 512 || s.vdim > 512) throw Error(kErrUnsupported, "heads wider than 512 are not supported");
+        if (s.mixer == Mixer::Attention) {
+            l.k_off = (int)pad8((int64_t)s.heads * s.dim);
+            l.v_off = l.k_off + (int)pad8(nq);
+            l.in_rows = l.v_off + (int)pad8((int64_t)s.kv_heads * s.vdim);
+        } else {
+            if (!delta_supported(s.dim, s.vdim)) throw Error(kErrUnsupported, "delta-rule heads wider than 256 are not supported");
+            auto rank = [&](const char* t) {  // rows of a [rank, width] tensor
+                const TensorInfo& ti = st.get(p + t);
+                if (ti.shape.size() != 2 || ti.shape[0] < 1) throw Error(kErrShape, "Tensor " + p + t + " is not a matrix");
+                return (int)ti.shape[0];
+            };
+            l.a_rank = rank("a1");
+            l.g_rank = rank("g1");
+            l.k_off = (int)pad8(nq);
+            l.v_off = 2 * l.k_off;
+            l.b_off = l.v_off + (int)pad8(nv);
+            l.a1_off = l.b_off + (int)pad8(s.heads);
+            l.g1_off = l.a1_off + (int)pad8(l.a_rank);
+            l.in_rows = l.g1_off + (int)pad8(l.g_rank);
+        }
+        if (s.experts + s.identity > 1024) throw Error(kErrUnsupported, "more than 1024 experts in a layer");
+        layout_layer(l, H, [&](DeviceBuffer&, size_t bytes) { total += Slab::padded(bytes); });
+    }
+    slab.alloc(total + 256);  // zero-filled: the padding of rows is never written again
+    Slab carve{&slab};
+    Stager up;
+    carve.take(embed, vocab * ld * 2);
+    put_matrix(up, embed.as<bf16>(), st.bf16("embed", {(int64_t)vocab, (int64_t)H}), vocab, H, ld);
+    embed_ld = (int64_t)ld;
+    lm_head = embed.as<bf16>();
+    carve.take(final_norm_f32, H * 4);
+    put_vector(up, final_norm_f32, st.bf16("final.norm", {(int64_t)H}), H);
+    uint64_t weights = vocab * H * 2;
+    for (size_t i = 0; i < stack.size(); ++i) {
+        StackLayer& l = stack[i];
+        const LayerSpec& s = l.spec;
+        layout_layer(l, H, [&](DeviceBuffer& b, size_t bytes) { carve.take(b, bytes); });
+        const std::string n = name(i), p = n + "mix.", f = n + "mlp.";
+        const int64_t W = (int64_t)H, nq = (int64_t)s.kv_heads * s.dim, nv = (int64_t)s.heads * s.vdim;
+        auto in_block = [&](const char* t, int row, int64_t rows) {  // rows of the stacked input projection
+            put_matrix(up, l.w_in.as<bf16>() + (size_t)row * ld, st.bf16(p + t, {rows, W}), rows, H, ld);
+            weights += (uint64_t)rows * H * 2;
+        };
+        auto vec = [&](const DeviceBuffer& b, const std::string& t, int64_t len) { put_vector(up, b, st.bf16(t, {len}), len); };
+        auto mat = [&](bf16* dst, const std::string& t, int64_t rows, int64_t cols) {
+            put_matrix(up, dst, st.bf16(t, {rows, cols}), rows, cols, pad8(cols));
+            weights += (uint64_t)rows * cols * 2;
+        };
+        if (s.mixer == Mixer::Attention) {
+            in_block("q", 0, (int64_t)s.heads * s.dim);
+            in_block("k", l.k_off, nq);
+            in_block("v", l.v_off, (int64_t)s.kv_heads * s.vdim);
+            vec(l.q_norm, p + "q.norm", s.dim);
+            vec(l.k_norm, p + "k.norm", s.dim);
+        } else {
+            in_block("q", 0, nq);
+            in_block("k", l.k_off, nq);
+            in_block("v", l.v_off, nv);
+            in_block("b", l.b_off, s.heads);
+            in_block("a1", l.a1_off, l.a_rank);
+            in_block("g1", l.g1_off, l.g_rank);
+            mat(l.a2.as<bf16>(), p + "a2", (int64_t)s.heads * s.dim, l.a_rank);
+            mat(l.g2.as<bf16>(), p + "g2", nv, l.g_rank);
+            vec(l.a_log, p + "A_log", s.heads);
+            vec(l.dt_bias, p + "dt_bias", (int64_t)s.heads * s.dim);
+            vec(l.out_norm, p + "norm", s.vdim);
+            const size_t C = 2 * nq + nv;
+            std::vector<float> taps(C * s.conv);
+            size_t ch = 0;
+            for (const char* t : {"q.conv", "k.conv", "v.conv"}) {
+                const size_t rows = t[0] == 'v' ? nv : nq;
+                const uint16_t* w = st.bf16(p + t, {(int64_t)rows, (int64_t)s.conv});
+                for (size_t r = 0; r < rows; ++r, ++ch)
+                    for (int j = 0; j < s.conv; ++j) taps[(size_t)j * C + ch] = bf16_to_f32(w[r * s.conv + j]);
+            }
+            up.copy(l.conv.p, taps.data(), taps.size() * 4);
+        }
+        mat(l.wo.as<bf16>(), p + "o", W, nv);
+        vec(l.norm1, n + "norm1", W);
+        vec(l.norm1b, n + "norm1b", W);
+        if (s.experts > 0) {
+            vec(l.norm2, n + "norm2", W);
+            vec(l.norm2b, n + "norm2b", W);
+            mat(l.router.as<bf16>(), f + "router", s.experts + s.identity, W);
+            vec(l.correction, f + "correction", s.experts + s.identity);
+            for (int e = 0; e < s.experts; ++e) {
+                const std::string en = f + "e" + std::to_string(e) + ".";
+                mat(l.up.as<bf16>() + (size_t)e * s.ff * ld, en + "up", s.ff, W);
+                mat(l.down.as<bf16>() + (size_t)e * H * pad8(s.ff), en + "down", W, s.ff);
+            }
+        }
+    }
+    up.finish();
+    weight_bytes_base = weights;
+}
+
+void Session::alloc_stack(bool f32) {
+    if (e_) throw Error(kErrUnsupported, "expert deltas belong to the Qwen2 family");
+    const Model* m = m_;
+    const size_t T = cap_tokens_, H = m->cfg.hidden_size;
+    st_.reset(new StackState());
+    StackState& s = *st_;
+    s.f32 = f32;
+    s.act = f32 ? 4 : 2;
+    s.h_ld = pad8((int64_t)H);
+    s.delta_ld = pad4((int64_t)H);
+    s.layers.resize(m->stack.size());
+    size_t q_cols = 0, qn = 0, vn = 0, gn = 0, heads = 0, pairs = 0;
+    for (size_t i = 0; i < m->stack.size(); ++i) {
+        const StackLayer& l = m->stack[i];
+        const LayerSpec& sp = l.spec;
+        StackState::LayerCache& c = s.layers[i];
+        s.proj_ld = std::max<int64_t>(s.proj_ld, l.in_rows);
+        s.ctx_ld = std::max<int64_t>(s.ctx_ld, pad8((int64_t)sp.heads * sp.vdim));
+        if (sp.mixer == Mixer::Attention) {
+            KvView& kv = c.kv;
+            kv.nkv = sp.kv_heads;
+            kv.hd = (int)pad8(sp.dim);
+            kv.vd = (int)pad8(sp.vdim);
+            kv.num_pages = num_pages_;
+            kv.max_pages_per_seq = max_pages_per_seq_;
+            kv.block_table = block_table_.as<int>();
+            kv.layer_stride = 0;
+            c.k.alloc((size_t)num_pages_ * kv.nkv * kPageTokens * kv.hd * s.act);  // zeros: padding columns stay zero
+            c.v.alloc((size_t)num_pages_ * kv.nkv * kPageTokens * kv.vd * s.act);
+            kv.k_pool = c.k.as<bf16>();
+            kv.v_pool = c.v.as<bf16>();
+            q_cols = std::max<size_t>(q_cols, (size_t)sp.heads * kv.hd);
+            for (size_t r = 0; r < s.rope_specs.size(); ++r)
+                if (s.rope_specs[r] == sp.rope) c.rope = (int)r;
+            if (c.rope < 0) {
+                c.rope = (int)s.rope_specs.size();
+                s.rope_specs.push_back(sp.rope);
+                const int half = sp.rope.dims / 2;
+                std::vector<float> cs((size_t)max_seq_ * half * 2 + 2);
+                for (int j = 0; j < half; ++j) {
+                    const double f = rope_frequency(sp.rope, j);
+                    for (int pos = 0; pos < max_seq_; ++pos) {
+                        cs[((size_t)pos * half + j) * 2] = (float)std::cos(pos * f);
+                        cs[((size_t)pos * half + j) * 2 + 1] = (float)std::sin(pos * f);
+                    }
+                }
+                s.rope.emplace_back();
+                upload(s.rope.back(), cs.data(), cs.size() * 4);
+            }
+        } else {
+            c.dimP = delta_padded_dim(sp.dim);
+            c.vdimP = (int)pad4(sp.vdim);
+            c.state_stride = (size_t)sp.heads * c.dimP * c.vdimP;
+            c.ring_stride = (size_t)(sp.conv - 1) * (2 * sp.kv_heads * sp.dim + sp.heads * sp.vdim);
+            c.state.alloc((size_t)max_batch_ * c.state_stride * 4);
+            c.ring.alloc(std::max<size_t>(4, (size_t)max_batch_ * c.ring_stride * 4));
+            s.decay_ld = std::max<int64_t>(s.decay_ld, pad4((int64_t)sp.heads * sp.dim));
+            s.gate_ld = std::max<int64_t>(s.gate_ld, pad4((int64_t)sp.heads * sp.vdim));
+            qn = std::max<size_t>(qn, (size_t)sp.kv_heads * c.dimP);
+            gn = std::max<size_t>(gn, (size_t)sp.heads * c.dimP);
+            vn = std::max<size_t>(vn, (size_t)sp.heads * c.vdimP);
+            heads = std::max<size_t>(heads, sp.heads);
+        }
+        if (sp.experts > 0) {
+            c.moe = s.moe_layers++;
+            s.max_top = std::max(s.max_top, sp.top);
+            s.max_experts = std::max(s.max_experts, sp.experts);
+            s.router_ld = std::max<int64_t>(s.router_ld, pad4(sp.experts + sp.identity));
+            s.act_ld = std::max<int64_t>(s.act_ld, pad8(sp.ff));
+            // tiles of the finest kind: one partly filled tile per expert and the full ones
+            s.max_tiles = std::max<int>(s.max_tiles, sp.experts + (int)(T * sp.top / 16) + 1);
+        }
+    }
+    pairs = T * s.max_top;
+    h_.alloc(T * H * 4);
+    xn_.alloc(T * s.h_ld * s.act);
+    xn_last_.alloc(T * s.h_ld * s.act);
+    s.proj.alloc(T * s.proj_ld * s.act);
+    ctx_.alloc(T * s.ctx_ld * s.act);
+    s.delta.alloc(T * s.delta_ld * 4);
+    if (q_cols) q_.alloc(T * q_cols * 4);
+    if (heads) {
+        s.qn.alloc(T * qn * 4);
+        s.kn.alloc(T * qn * 4);
+        s.g.alloc(T * gn * 4);
+        s.v.alloc(T * vn * 4);
+        s.bk.alloc(T * heads * 8);
+        s.decay.alloc(T * s.decay_ld * 4);
+        s.gate.alloc(T * s.gate_ld * 4);
+    }
+    if (pairs) {
+        s.router.alloc(T * s.router_ld * 4);
+        s.counts.alloc((size_t)s.moe_layers * s.max_experts * 4);
+        s.pair.alloc(pairs * 8);
+        s.pair_w.alloc(pairs * 4);
+        s.pair_row.alloc(pairs * 4);
+        s.xg.alloc(pairs * s.h_ld * s.act);
+        s.act_e.alloc(pairs * s.act_ld * s.act);
+        s.y.alloc(pairs * s.h_ld * s.act);
+        s.tiles.alloc((size_t)s.max_tiles * sizeof(GroupTile));
+    }
+    s.seg_first.alloc(T * 4);
+    s.seg_count.alloc(T * 4);
+    std::vector<int> ones(T, 1);
+    upload(s.ones, ones.data(), T * 4);
+    cuda_check((cudaError_t)stack_rows_prepare(), "stack_rows_prepare", __FILE__, __LINE__);
+    cuda_check((cudaError_t)delta_prepare(), "delta_prepare", __FILE__, __LINE__);
+    cuda_check((cudaError_t)moe_prepare(), "moe_prepare", __FILE__, __LINE__);
+}
+
+AttnOptions Session::attn_options(const LayerSpec& l) const {
+    AttnOptions o;
+    o.scale = l.scale;
+    o.chunk = l.chunk;
+    o.vdim = l.vdim;
+    o.ctx_ld = pad8((int64_t)l.heads * l.vdim);
+    return o;
+}
+
+int Session::decode_graph_key(int n_seqs, int max_ctx) const {
+    if (!st_) {
+        const Config& c = m_->cfg;
+        return attention_splits(n_seqs, c.num_heads, c.num_kv_heads, c.head_dim, max_ctx, attn_ws(), m_->num_sms);
+    }
+    int key = 0;  // at most 64 splits per layer; layers that see the same context agree, so one digit per distinct choice
+    std::vector<int> seen;
+    for (const StackLayer& l : m_->stack) {
+        if (l.spec.mixer != Mixer::Attention) continue;
+        const int wide = (int)pad8(std::max(l.spec.dim, l.spec.vdim));
+        const int sp = attention_splits(n_seqs, l.spec.heads, l.spec.kv_heads, wide, attn_ctx(l.spec, max_ctx), attn_ws(), m_->num_sms);
+        seen.push_back(sp);
+    }
+    for (int sp : seen) key = (int)(((uint32_t)key * 257u + (uint32_t)sp) & 0x3fffffffu);
+    return key;
+}
+
+void Session::run_stack(int T, int n_logit_rows, bool logit_rows_are_all, bool decode, int max_ctx, int n_groups, int n_segs) {
+    StackState& s = *st_;
+    const Config& c = m_->cfg;
+    const int H = c.hidden_size;
+    const bool f32 = s.f32, pdl = launch_mode_ >= 1 && !profile_;
+    const int* tok_seq = decode ? identity_.as<int>() : tok_seq_.as<int>();
+    const int* tok_pos = decode ? seq_len_dev_.as<int>() : tok_pos_.as<int>();
+    const int* seg_first = decode ? identity_.as<int>() : s.seg_first.as<int>();
+    const int* seg_count = decode ? s.ones.as<int>() : s.seg_count.as<int>();
+    if (decode) n_segs = T;
+    int* status = status_.as<int>();
+    auto live = [&](int cls) { return ((ablate_mask_ >> cls) & 1u) == 0; };
+    auto step = [&](int cls, auto&& launch) {  // one kernel that is not a GEMM
+        prof_begin(cls);
+        if (live(cls)) launch(tl_next(cls));
+        prof_end();
+        launches_++;
+    };
+    const bf16* xn = xn_.as<bf16>();
+    // out[., n] = rows of X . W, activations out of and into the step's buffers
+    auto product = [&](const bf16* W, int64_t ldw, const void* X, int64_t ldx, int K, int N, int mode, void* out, int64_t ldo) {
+        GemmCall g;
+        memset(&g, 0, sizeof g);
+        g.x_rows_alloc = cap_tokens_;
+        g.T = T;
+        g.alpha = 1.f;
+        g.op[0] = {W, ldw, (const bf16*)X, ldx, K};
+        g.N = N;
+        g.mode = mode;
+        g.out = out;
+        g.ldo = ldo;
+        return g;
+    };
+    auto run_product = [&](int cls, const bf16* W, int64_t ldw, const void* X, int64_t ldx, int K, int N, int mode, void* out, int64_t ldo) {
+        GemmCall g = product(W, ldw, X, ldx, K, N, mode, out, ldo);
+        gemm(g, cls, pdl);
+    };
+    auto act_at = [&](const DeviceBuffer& b, int64_t col) { return (const void*)((const char*)b.p + col * s.act); };
+
+    ResidualRows rows;
+    memset(&rows, 0, sizeof rows);
+    rows.x = h_.as<float>();
+    rows.H = H;
+    rows.eps = c.rms_norm_eps;
+    rows.status = status;
+    rows.out = xn_.p;
+    rows.out_ld = s.h_ld;
+
+    if (s.moe_layers) TFFN_CUDA(cudaMemsetAsync(s.counts.p, 0, s.counts.bytes, stream_));
+    // the step's first kernel is a full dependency: all that earlier steps wrote is complete for every kernel of this one
+    rows.source = ROWS_EMBED;
+    rows.tokens = decode ? dec_tokens_.as<int>() : tokens_.as<int>();
+    rows.table = m_->embed.as<bf16>();
+    rows.table_ld = m_->embed_ld;
+    rows.V = c.vocab_size;
+    rows.next_w = m_->stack[0].norm1.as<float>();
+    step(KC_EMBED, [&](unsigned long long* tl) { launch_residual_rows(rows, f32, T, stream_, false, tl); });
+
+    for (size_t li = 0; li < m_->stack.size(); ++li) {
+        const StackLayer& l = m_->stack[li];
+        const LayerSpec& sp = l.spec;
+        StackState::LayerCache& cache = s.layers[li];
+        const bool last = li + 1 == m_->stack.size();
+        // the norm behind this layer: the next layer's, or the model's own when every row gets logits
+        const float* after = !last ? m_->stack[li + 1].norm1.as<float>()
+                                   : (n_logit_rows == T && logit_rows_are_all ? m_->final_norm_f32.as<float>() : nullptr);
+        const int64_t nv = (int64_t)sp.heads * sp.vdim, ctx_ld = pad8(nv);
+
+        run_product(KC_GEMM_IN, l.w_in.as<bf16>(), s.h_ld, xn, s.h_ld, H, l.in_rows, GEMM_STORE_BF16, s.proj.p, l.in_rows);
+        if (sp.mixer == Mixer::Attention) {
+            QkNormRope q;
+            memset(&q, 0, sizeof q);
+            q.qkv = s.proj.p;
+            q.ld = l.in_rows;
+            q.k_off = l.k_off;
+            q.v_off = l.v_off;
+            q.q_norm = l.q_norm.as<float>();
+            q.k_norm = l.k_norm.as<float>();
+            q.eps = c.rms_norm_eps;
+            q.nh = sp.heads;
+            q.dim = sp.dim;
+            q.vdim = sp.vdim;
+            q.rope_dims = sp.rope.dims;
+            q.rope = s.rope[cache.rope].as<float2>();
+            q.max_pos = max_seq_;
+            q.tok_seq = tok_seq;
+            q.tok_pos = tok_pos;
+            q.q_out = q_.as<float>();
+            q.kv = cache.kv;
+            q.status = status;
+            step(KC_QK_ROPE, [&](unsigned long long* tl) { launch_qk_norm_rope(q, f32, T, stream_, pdl, tl); });
+            const AttnOptions opt = attn_options(sp);
+            step(KC_ATTENTION, [&](unsigned long long* tl) {
+                if (f32 || !attention_tc_supported(cache.kv.hd, cache.kv.vd))
+                    launch_attention_simt(q_.as<float>(), cache.kv, f32, tok_seq, tok_pos, ctx_.p, T, sp.heads, opt, status, stream_, pdl, tl);
+                else if (n_groups > 0)
+                    launch_attention_prefill(q_.as<float>(), cache.kv, 0, tok_seq, tok_pos, grp_first_.as<int>(), grp_count_.as<int>(),
+                                             n_groups, ctx_.as<bf16>(), sp.heads, status, stream_, pdl, tl, opt);
+                else
+                    launch_attention(q_.as<float>(), cache.kv, 0, tok_seq, tok_pos, ctx_.as<bf16>(), T, sp.heads, attn_ctx(sp, max_ctx),
+                                     attn_ws(), m_->num_sms, status, stream_, pdl, decode, tl, nullptr, 0, opt);
+            });
+        } else {
+            // the second halves of the two low-rank projections; one launch when they have the same shape
+            const int na = sp.heads * sp.dim;
+            GemmCall a = product(l.a2.as<bf16>(), pad8(l.a_rank), act_at(s.proj, l.a1_off), l.in_rows, l.a_rank, na,
+                                 GEMM_STORE_F32, s.decay.p, s.decay_ld);
+            if (na == nv && l.a_rank == l.g_rank && s.decay_ld == s.gate_ld) {
+                a.op2[0] = {l.g2.as<bf16>(), pad8(l.g_rank), (const bf16*)act_at(s.proj, l.g1_off), l.in_rows, l.g_rank};
+                a.out2 = s.gate.p;
+                gemm(a, KC_GEMM_LOWRANK, pdl);
+            } else {
+                gemm(a, KC_GEMM_LOWRANK, pdl);
+                run_product(KC_GEMM_LOWRANK, l.g2.as<bf16>(), pad8(l.g_rank), act_at(s.proj, l.g1_off), l.in_rows, l.g_rank, (int)nv,
+                            GEMM_STORE_F32, s.gate.p, s.gate_ld);
+            }
+            DeltaRule d;
+            memset(&d, 0, sizeof d);
+            d.heads = sp.heads;
+            d.kv_heads = sp.kv_heads;
+            d.dim = sp.dim;
+            d.vdim = sp.vdim;
+            d.dimP = cache.dimP;
+            d.vdimP = cache.vdimP;
+            d.taps = sp.conv;
+            d.eps = c.rms_norm_eps;
+            d.proj = s.proj.p;
+            d.proj_ld = l.in_rows;
+            d.k_off = l.k_off;
+            d.v_off = l.v_off;
+            d.b_off = l.b_off;
+            d.conv = l.conv.as<float>();
+            d.a_log = l.a_log.as<float>();
+            d.dt_bias = l.dt_bias.as<float>();
+            d.decay_in = s.decay.as<float>();
+            d.decay_ld = s.decay_ld;
+            d.gate_in = s.gate.as<float>();
+            d.gate_ld = s.gate_ld;
+            d.out_norm = l.out_norm.as<float>();
+            d.state = cache.state.as<float>();
+            d.ring = cache.ring.as<float>();
+            d.state_stride = cache.state_stride;
+            d.ring_stride = cache.ring_stride;
+            d.qn = s.qn.as<float>();
+            d.kn = s.kn.as<float>();
+            d.v = s.v.as<float>();
+            d.g = s.g.as<float>();
+            d.bk = s.bk.as<float>();
+            d.out = ctx_.p;
+            d.out_ld = ctx_ld;
+            d.tok_seq = tok_seq;
+            d.tok_pos = tok_pos;
+            d.seg_first = seg_first;
+            d.seg_count = seg_count;
+            d.max_slots = max_batch_;
+            d.status = status;
+            step(KC_DELTA_PREP, [&](unsigned long long* tl) { launch_delta_prep(d, f32, T, stream_, pdl, tl); });
+            step(KC_DELTA_SCAN, [&](unsigned long long* tl) { launch_delta_scan(d, f32, n_segs, stream_, pdl, tl); });
+        }
+        run_product(KC_GEMM_OPROJ, l.wo.as<bf16>(), ctx_ld, ctx_.p, ctx_ld, (int)nv, H, GEMM_STORE_F32, s.delta.p, s.delta_ld);
+        rows.source = ROWS_DELTA;
+        rows.delta = s.delta.as<float>();
+        rows.delta_ld = s.delta_ld;
+        rows.post_w = l.norm1b.as<float>();
+        rows.next_w = sp.experts > 0 ? l.norm2.as<float>() : after;
+        step(KC_ROWS, [&](unsigned long long* tl) { launch_residual_rows(rows, f32, T, stream_, pdl, tl); });
+
+        if (sp.experts > 0) {
+            const int outs = sp.experts + sp.identity, pairs = T * sp.top;
+            const int tile = f32 ? kGemmF32Tile : gemm_group_tile((pairs + outs - 1) / outs);
+            const int tiles = std::min(sp.experts, pairs) + pairs / tile;
+            run_product(KC_GEMM_ROUTER, l.router.as<bf16>(), s.h_ld, xn, s.h_ld, H, outs, GEMM_STORE_F32, s.router.p, s.router_ld);
+            MoeRoute r;
+            r.logits = s.router.as<float>();
+            r.ld = s.router_ld;
+            r.correction = l.correction.as<float>();
+            r.experts = sp.experts;
+            r.identity = sp.identity;
+            r.top = sp.top;
+            r.counts = s.counts.as<int>() + (size_t)cache.moe * s.max_experts;
+            r.pair = s.pair.as<int2>();
+            r.pair_w = s.pair_w.as<float>();
+            step(KC_ROUTE, [&](unsigned long long* tl) { launch_moe_route(r, T, stream_, pdl, tl); });
+            MoeGather g;
+            g.x = xn_.p;
+            g.x_ld = s.h_ld;
+            g.H = H;
+            g.experts = sp.experts;
+            g.top = sp.top;
+            g.counts = r.counts;
+            g.pair = r.pair;
+            g.xg = s.xg.p;
+            g.pair_row = s.pair_row.as<int>();
+            g.tiles = s.tiles.as<GroupTile>();
+            g.max_tiles = tiles;
+            g.tile_rows = tile;
+            step(KC_GATHER, [&](unsigned long long* tl) { launch_moe_gather(g, f32, T, stream_, pdl, tl); });
+            auto grouped = [&](int cls, const bf16* W, int64_t ldw, const void* X, int64_t ldx, int K, int N, int mode, void* out, int64_t ldo) {
+                GemmCall e = product(W, ldw, X, ldx, K, N, mode, out, ldo);
+                e.x_rows_alloc = cap_tokens_ * s.max_top;
+                e.T = pairs;
+                e.grp = g.tiles;
+                e.grp_tiles = tiles;
+                e.grp_bn = tile;
+                e.grp_count = sp.experts;
+                gemm(e, cls, pdl);
+            };
+            const int64_t ffp = pad8(sp.ff);
+            grouped(KC_GEMM_UP, l.up.as<bf16>(), s.h_ld, s.xg.p, s.h_ld, H, sp.ff, GEMM_RELU2, s.act_e.p, ffp);
+            grouped(KC_GEMM_EXPERT_DOWN, l.down.as<bf16>(), ffp, s.act_e.p, ffp, sp.ff, H, GEMM_STORE_BF16, s.y.p, s.h_ld);
+            rows.source = ROWS_MOE;
+            rows.y = s.y.p;
+            rows.y_ld = s.h_ld;
+            rows.pair_row = s.pair_row.as<int>();
+            rows.pair_w = s.pair_w.as<float>();
+            rows.top = sp.top;
+            rows.post_w = l.norm2b.as<float>();
+            rows.next_w = after;
+            step(KC_ROWS, [&](unsigned long long* tl) { launch_residual_rows(rows, f32, T, stream_, pdl, tl); });
+        }
+        if (hidden_rows_cap_ > 0) {
+            const int n = std::min(T, hidden_rows_cap_);
+            const size_t elems = (size_t)n * H;
+            k_copy_rows_f32<<<(unsigned)((elems + 255) / 256), 256, 0, stream_>>>(
+                h_.as<float>(), hidden_.as<float>() + li * (size_t)hidden_rows_cap_ * H, elems);
+            hidden_rows_ = n;
+            launches_++;
+        }
+    }
+    if (n_logit_rows > 0) {
+        const void* x = xn_.p;
+        if (!(n_logit_rows == T && logit_rows_are_all)) {
+            rows.source = ROWS_KEEP;
+            rows.next_w = m_->final_norm_f32.as<float>();
+            rows.row_idx = logit_rows_are_all ? nullptr : row_idx_.as<int>();
+            rows.out = xn_last_.p;
+            step(KC_RMSNORM, [&](unsigned long long* tl) { launch_residual_rows(rows, f32, n_logit_rows, stream_, pdl, tl); });
+            x = xn_last_.p;
+        }
+        lm_head(x, s.h_ld, n_logit_rows, decode, pdl);
+    }
+    TFFN_CUDA(cudaGetLastError());
+}
+
+}  // namespace tffn

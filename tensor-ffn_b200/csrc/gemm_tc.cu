@@ -49,6 +49,7 @@ struct GemmDev {
     GemmQkvEpilogue qkv;  // GEMM_QKV only
     unsigned long long* trace;  // optional: 64 timestamps (ns) per CTA, see GemmCall::trace
     unsigned long long* tl;     // optional: step timeline of this launch
+    const GroupTile* grp;       // grouped launch: one entry per token tile (blockIdx.y), see GemmCall::grp
     float* amax_val;            // GEMM_STORE_F32: per (token, tile) maximum and its index, or nullptr
     int* amax_idx;
 };
@@ -205,7 +206,21 @@ __device__ __forceinline__ void finalize_plain(const GemmDev& p, void* out, int 
             }
             break;
         }
-        default:  // GEMM_STORE_BF16, GEMM_SWIGLU
+        default:  // GEMM_STORE_BF16, GEMM_SWIGLU, GEMM_RELU2
+            if (p.mode == GEMM_RELU2) {
+                float r[4];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const float a = fmaxf(f[j], 0.f);
+                    r[j] = a * a;
+                }
+                if (vec) {
+                    *(uint2*)((bf16*)out + o) = pack_bf16x4(r[0], r[1], r[2], r[3]);
+                } else {
+                    for (int j = 0; j < 4 && n + j < p.N; ++j) ((bf16*)out)[o + j] = __float2bfloat16_rn(r[j]);
+                }
+                break;
+            }
             if (vec) {
                 *(uint2*)((bf16*)out + o) = pack_bf16x4(f[0], f[1], f[2], f[3]);
             } else {
@@ -267,7 +282,19 @@ __global__ void __launch_bounds__(kGemmThreads, (BN <= 64) ? 2 : 1) k_gemm_tc(co
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int prob = blockIdx.y / p.t_tiles;  // independent problems (base / expert gate-up) share a launch
-    const int n0 = blockIdx.x * p.tile_n, t0 = (blockIdx.y % p.t_tiles) * BN;
+    const int n0 = blockIdx.x * p.tile_n;
+    int t0 = (blockIdx.y % p.t_tiles) * BN, t_end = p.T, w_row0 = n0;
+    if (p.grp) {
+        // grouped launch: which group's weights and which rows this tile covers was written by an earlier kernel, so
+        // nothing can be requested ahead of the wait; unused tiles (the grid is sized for the worst case) leave
+        // together, all CTAs of a cluster alike
+        pdl_wait();
+        const int4 g = __ldcg((const int4*)(p.grp + blockIdx.y));
+        if (g.x < 0) return;
+        t0 = g.y;
+        t_end = min(g.z, g.y + BN);
+        w_row0 = g.x * p.N + n0;
+    }
     const bool halves = p.mode == GEMM_SWIGLU;  // A tile = 64 gate rows over 64 up rows, one accumulator
     void* const out = p.out[prob];
     const int total_kb = p.kblocks[0] + p.kblocks[1];
@@ -313,10 +340,10 @@ __global__ void __launch_bounds__(kGemmThreads, (BN <= 64) ? 2 : 1) k_gemm_tc(co
                 const int kb = seg ? i - p.kblocks[0] : i;
                 mbar_arrive_expect_tx(&full[it], Cfg::STAGE_BYTES);
                 if (halves) {
-                    tma_load_2d(smem + it * Cfg::STAGE_BYTES, &p.tmW[prob * 2], kb * BK, n0, &full[it]);
-                    tma_load_2d(smem + it * Cfg::STAGE_BYTES + Cfg::A_BYTES / 2, &p.tmW[prob * 2 + 1], kb * BK, n0, &full[it]);
+                    tma_load_2d(smem + it * Cfg::STAGE_BYTES, &p.tmW[prob * 2], kb * BK, w_row0, &full[it]);
+                    tma_load_2d(smem + it * Cfg::STAGE_BYTES + Cfg::A_BYTES / 2, &p.tmW[prob * 2 + 1], kb * BK, w_row0, &full[it]);
                 } else {
-                    tma_load_2d(smem + it * Cfg::STAGE_BYTES, &p.tmW[prob * 2 + seg], kb * BK, n0, &full[it]);
+                    tma_load_2d(smem + it * Cfg::STAGE_BYTES, &p.tmW[prob * 2 + seg], kb * BK, w_row0, &full[it]);
                 }
             }
             TFFN_TRACE(1);
@@ -340,10 +367,10 @@ __global__ void __launch_bounds__(kGemmThreads, (BN <= 64) ? 2 : 1) k_gemm_tc(co
                 uint8_t* b = a + Cfg::A_BYTES;
                 mbar_arrive_expect_tx(&full[s], Cfg::STAGE_BYTES);
                 if (halves) {
-                    tma_load_2d(a, &p.tmW[prob * 2], kb * BK, n0, &full[s]);
-                    tma_load_2d(a + Cfg::A_BYTES / 2, &p.tmW[prob * 2 + 1], kb * BK, n0, &full[s]);
+                    tma_load_2d(a, &p.tmW[prob * 2], kb * BK, w_row0, &full[s]);
+                    tma_load_2d(a + Cfg::A_BYTES / 2, &p.tmW[prob * 2 + 1], kb * BK, w_row0, &full[s]);
                 } else {
-                    tma_load_2d(a, &p.tmW[prob * 2 + seg], kb * BK, n0, &full[s]);
+                    tma_load_2d(a, &p.tmW[prob * 2 + seg], kb * BK, w_row0, &full[s]);
                 }
                 tma_load_2d(b, &p.tmX[prob * 2 + seg], kb * BK, t0, &full[s]);
             }
@@ -388,7 +415,7 @@ __global__ void __launch_bounds__(kGemmThreads, (BN <= 64) ? 2 : 1) k_gemm_tc(co
 #pragma unroll
             for (int u = 0; u < 2; ++u) {
                 const int jj = (warp - 2) + 4 * u, t = t0 + jj * S + rank;
-                if (cps <= 8 && jj < cps && t < p.T) {
+                if (cps <= 8 && jj < cps && t < t_end) {
                     if (p.mode == GEMM_QKV) prefetch_qkv(p, n0 + lane * 4, t, pre[u]);
                     else if (p.mode == GEMM_RESIDUAL) prefetch_residual(p, out, n0 + lane * 4, t, pre[u]);
                 }
@@ -405,7 +432,7 @@ __global__ void __launch_bounds__(kGemmThreads, (BN <= 64) ? 2 : 1) k_gemm_tc(co
         float* plane = (float*)smem;
 #pragma unroll 1
         for (int c0 = 0; c0 < BN; c0 += 16) {
-            if (t0 + c0 >= p.T) break;
+            if (t0 + c0 >= t_end) break;
             uint32_t v0[16], v1[16];
             if (live && has0) tmem_ld16(lane_addr + (uint32_t)c0, v0);
             if (live && has1) tmem_ld16(lane_addr + (uint32_t)(BN + c0), v1);
@@ -442,7 +469,7 @@ __global__ void __launch_bounds__(kGemmThreads, (BN <= 64) ? 2 : 1) k_gemm_tc(co
         // Unsplit tile: every column comes from this CTA's own plane, nothing to wait for, so all six
         // warps (the copy and MMA warps are idle by now) take columns, four in flight per warp.
         const int w = warp;
-        const int ncols = min(BN, p.T - t0);
+        const int ncols = min(BN, t_end - t0);
         const float* plane = (const float*)smem;
         if (threadIdx.x == 64) TFFN_TRACE(9);
         if (halves) {
@@ -539,7 +566,7 @@ __global__ void __launch_bounds__(kGemmThreads, (BN <= 64) ? 2 : 1) k_gemm_tc(co
 #pragma unroll
             for (int u = 0; u < 2; ++u) {
                 const int jj = w + 4 * u, c = jj * S + (int)rank;
-                have[u] = n_iters > 0 && jj < cps && t0 + c < p.T;  // warp-uniform
+                have[u] = n_iters > 0 && jj < cps && t0 + c < t_end;  // warp-uniform
                 acc[u] = have[u] ? column_sum(c, r4) : zero4;
                 up[u] = (have[u] && halves && lane < 16) ? column_sum(c, r4 + 64) : zero4;
             }
@@ -553,7 +580,7 @@ __global__ void __launch_bounds__(kGemmThreads, (BN <= 64) ? 2 : 1) k_gemm_tc(co
             none.valid = false;
             for (int jj = w; jj < cps && n_iters > 0; jj += 4) {
                 const int c = jj * S + (int)rank;
-                if (t0 + c >= p.T) break;  // warp-uniform
+                if (t0 + c >= t_end) break;  // warp-uniform
                 const float4 acc = column_sum(c, r4);
                 const float4 up = (halves && lane < 16) ? column_sum(c, r4 + 64) : zero4;
                 finish(t0 + c, acc, up, none);
@@ -681,7 +708,8 @@ int launch_bn(const GemmCall& c, const GemmWorkspace& ws, cudaStream_t stream, i
             if (pr == 0) p.kblocks[i] = o.K > 0 ? (o.K + BK - 1) / BK : 0;
             if (o.K <= 0) continue;
             if (pr == 1 && (o.K + BK - 1) / BK != p.kblocks[i]) return (int)cudaErrorInvalidValue;
-            if (!make_tmap(ws.tmaps, &p.tmW[pr * 2 + i], o.W, (uint64_t)c.N, (uint64_t)o.K, (uint64_t)o.ldw, halves ? BM / 2 : BM)) return -1000;
+            const uint64_t w_rows = (uint64_t)c.N * (c.grp ? c.grp_count : 1);
+            if (!make_tmap(ws.tmaps, &p.tmW[pr * 2 + i], o.W, w_rows, (uint64_t)o.K, (uint64_t)o.ldw, halves ? BM / 2 : BM)) return -1000;
             if (!make_tmap(ws.tmaps, &p.tmX[pr * 2 + i], o.X, (uint64_t)(c.x_rows_alloc > c.T ? c.x_rows_alloc : c.T), (uint64_t)o.K,
                            (uint64_t)o.ldx, BN))
                 return -1000;
@@ -710,7 +738,10 @@ int launch_bn(const GemmCall& c, const GemmWorkspace& ws, cudaStream_t stream, i
         if (!c.qkv || c.op[1].K > 0 || c.out2 || (c.qkv->kv.hd != 64 && c.qkv->kv.hd != 128)) return (int)cudaErrorInvalidValue;
         p.qkv = *c.qkv;
     }
-    const int n_tiles = (c.N + p.tile_n - 1) / p.tile_n, t_tiles = (c.T + BN - 1) / BN;
+    const int n_tiles = (c.N + p.tile_n - 1) / p.tile_n, t_tiles = c.grp ? c.grp_tiles : (c.T + BN - 1) / BN;
+    if (c.grp && (c.grp_bn != BN || c.op[1].K > 0 || c.out2 || halves || c.mode == GEMM_QKV || c.grp_tiles < 1 || c.grp_count < 1))
+        return (int)cudaErrorInvalidValue;
+    p.grp = c.grp;
     const int total_kb = p.kblocks[0] + p.kblocks[1];
     const int tiles = n_tiles * t_tiles * nprob;
     p.t_tiles = t_tiles;
@@ -807,8 +838,26 @@ int gemm_prepare() {
     return 0;
 }
 
+// Groups differ in size: a tile of the average size would leave the larger half of the groups a second, nearly
+// empty tile and their weights would be streamed twice, so the tile has room for twice the average.
+int gemm_group_tile(int rows) {
+    int bn = 16;
+    while (bn < 256 && bn < 2 * rows) bn *= 2;
+    return bn;
+}
+
 int launch_gemm(const GemmCall& c, const GemmWorkspace& ws, cudaStream_t stream, int force_splits) {
     if (c.T <= 0 || c.N <= 0 || c.op[0].K <= 0) return (int)cudaErrorInvalidValue;
+    if (c.grp) {
+        switch (c.grp_bn) {
+            case 16: return launch_bn<16>(c, ws, stream, force_splits);
+            case 32: return launch_bn<32>(c, ws, stream, force_splits);
+            case 64: return launch_bn<64>(c, ws, stream, force_splits);
+            case 128: return launch_bn<128>(c, ws, stream, force_splits);
+            case 256: return launch_bn<256>(c, ws, stream, force_splits);
+            default: return (int)cudaErrorInvalidValue;
+        }
+    }
     // A short K extent with few output tiles (the attention projections of a small model): the grid is
     // filled by splitting K, and the cost of such a launch is the exchange of the partial tiles (measured:
     // 28 KB per CTA over distributed shared memory take 2 to 3.6 us). Halving the token tile (two token

@@ -1,6 +1,7 @@
 #include "host_io.h"
 #include "json_lite.h"
 #include <algorithm>
+#include <cmath>
 #include <cstring>
 #include <dirent.h>
 #include <fcntl.h>
@@ -32,16 +33,7 @@ static int first_int(const JsonValue& j, const char* key, int def) {
     return def;
 }
 
-Config read_config(const std::string& dir) {
-    bool ok;
-    std::string text = read_text_file(dir + "/config.json", &ok);
-    if (!ok) throw Error(kErrIO, "Cannot open " + dir + "/config.json");
-    JsonValue j;
-    try {
-        j = json_parse(text);
-    } catch (const std::exception& e) {
-        throw Error(kErrFormat, dir + "/config.json: " + e.what());
-    }
+static Config read_qwen2(const JsonValue& j) {
     Config c;
     c.hidden_size = (int)j.value_int("hidden_size", 896);
     c.intermediate_size = (int)j.value_int("intermediate_size", 4864);
@@ -64,7 +56,158 @@ Config read_config(const std::string& dir) {
     return c;
 }
 
+// ---------------------------------------------------------------- layer lists (Rafilix)
+// Every size and constant is stated by the file; nothing has a default.
+static const JsonValue& need_key(const JsonValue& j, const char* key, const std::string& where) {
+    const JsonValue* v = j.find(key);
+    if (!v || v->is_null()) throw Error(kErrFormat, "config.json: " + where + " has no '" + key + "'");
+    return *v;
+}
+static double need_number(const JsonValue& j, const char* key, const std::string& where) {
+    const JsonValue& v = need_key(j, key, where);
+    if (!v.is_number()) throw Error(kErrFormat, "config.json: " + where + "." + key + " is not a number");
+    return v.as_double();
+}
+static int need_size(const JsonValue& j, const char* key, const std::string& where, int at_least = 1) {
+    const double d = need_number(j, key, where);
+    if (d != (double)(int)d || (int)d < at_least) throw Error(kErrFormat, "config.json: " + where + "." + key + " is out of range");
+    return (int)d;
+}
+static bool has_value(const JsonValue& j, const char* key) {
+    const JsonValue* v = j.find(key);
+    return v && !v->is_null();
+}
+
+static RopeSpec read_rope(const JsonValue& j, int dim, const std::string& where) {
+    RopeSpec r;
+    r.dims = need_size(j, "dims", where, 0);
+    r.base = need_number(j, "base", where);
+    if (r.dims % 2 != 0 || r.dims > dim || !(r.base > 0)) throw Error(kErrFormat, "config.json: " + where + " is not a rotation of this head");
+    if (has_value(j, "scaling")) {
+        const JsonValue& s = need_key(j, "scaling", where);
+        r.scaled = true;
+        r.factor = need_number(s, "factor", where + ".scaling");
+        r.low = need_number(s, "low", where + ".scaling");
+        r.high = need_number(s, "high", where + ".scaling");
+        r.original = need_number(s, "original", where + ".scaling");
+        if (!(r.factor > 0) || !(r.low > 0) || !(r.high > 0) || !(r.original > 0))
+            throw Error(kErrFormat, "config.json: " + where + ".scaling has a non-positive constant");
+    }
+    return r;
+}
+
+double rope_frequency(const RopeSpec& r, int i) {
+    const double f = std::pow(r.base, -2.0 * i / r.dims);
+    if (!r.scaled) return f;
+    const double wave = 2.0 * 3.14159265358979323846 / f;
+    if (wave < r.original / r.high) return f;
+    if (wave > r.original / r.low) return f / r.factor;
+    const double s = (r.original / wave - r.low) / (r.high - r.low);
+    return (1.0 - s) * f / r.factor + s * f;
+}
+
+static LayerSpec read_layer(const JsonValue& j, const std::string& where) {
+    LayerSpec l;
+    const JsonValue& type = need_key(j, "type", where);
+    const JsonValue& m = need_key(j, "mixer", where);
+    const std::string mw = where + ".mixer";
+    l.heads = need_size(m, "heads", mw);
+    l.kv_heads = need_size(m, "kv_heads", mw);
+    l.dim = need_size(m, "dim", mw);
+    l.vdim = need_size(m, "vdim", mw);
+    if (l.heads % l.kv_heads != 0) throw Error(kErrFormat, "config.json: " + mw + ": kv_heads do not divide heads");
+    if (type.is_string() && type.str == "attention") {
+        l.mixer = Mixer::Attention;
+        l.scale = (float)need_number(m, "scale", mw);
+        if (has_value(m, "rot")) l.rope = read_rope(need_key(m, "rot", mw), l.dim, mw + ".rot");
+        if (has_value(m, "mask")) l.chunk = need_size(need_key(m, "mask", mw), "size", mw + ".mask");
+    } else if (type.is_string() && type.str == "channel_delta") {
+        l.mixer = Mixer::ChannelDelta;
+        l.conv = need_size(m, "conv", mw);
+    } else {
+        throw Error(kErrUnsupported, "config.json: " + where + ": unknown layer type '" + type.str + "'");
+    }
+    if (has_value(j, "mlp")) {
+        const std::string fw = where + ".mlp";
+        const JsonValue& f = need_key(j, "mlp", where);
+        const JsonValue& kind = need_key(f, "kind", fw);
+        if (kind.str != "moe") throw Error(kErrUnsupported, "config.json: " + fw + ": unknown kind '" + kind.str + "'");
+        l.ff = need_size(need_key(f, "expert", fw), "ff", fw + ".expert");
+        const JsonValue& r = need_key(f, "router", fw);
+        l.experts = need_size(r, "experts", fw + ".router");
+        l.identity = has_value(r, "identity") ? need_size(r, "identity", fw + ".router", 0) : 0;
+        l.top = need_size(r, "top", fw + ".router");
+        if (l.top > l.experts + l.identity) throw Error(kErrFormat, "config.json: " + fw + ".router: top exceeds the number of experts");
+    }
+    return l;
+}
+
+static Config read_rafilix(const JsonValue& j) {
+    Config c;
+    c.hidden_size = need_size(j, "width", "the model");
+    c.vocab_size = need_size(j, "vocab", "the model");
+    c.rms_norm_eps = (float)need_number(need_key(j, "norm", "the model"), "eps", "norm");
+    const JsonValue& ls = need_key(j, "layers", "the model");
+    if (!ls.is_array() || ls.arr.empty()) throw Error(kErrFormat, "config.json: 'layers' is not a list of layers");
+    for (size_t i = 0; i < ls.arr.size(); ++i) c.layers.push_back(read_layer(ls.arr[i], "layer " + std::to_string(i)));
+    c.num_layers = (int)c.layers.size();
+    const LayerSpec& l0 = c.layers[0];
+    c.num_heads = l0.heads;
+    c.num_kv_heads = l0.kv_heads;
+    c.head_dim = l0.dim;
+    c.intermediate_size = 0;
+    c.rope_theta = 0.f;
+    for (const LayerSpec& l : c.layers) {
+        c.intermediate_size = std::max(c.intermediate_size, l.ff);
+        if (l.mixer == Mixer::Attention && c.rope_theta == 0.f) c.rope_theta = (float)l.rope.base;
+    }
+    c.max_seq_len = 1 << 30;  // no table of positions is stored
+    c.eos_token_id = first_int(j, "eos_token_id", -1);
+    c.bos_token_id = first_int(j, "bos_token_id", -1);
+    c.tie_embeddings = true;
+    return c;
+}
+
+// Families that list their layers name themselves under "architecture"; a file without that key is the
+// HF-style Qwen2 configuration the reference reads.
+static bool names_itself(const JsonValue& j, const char* name) {
+    const JsonValue* a = j.find("architecture");
+    return a && a->is_string() && a->str == name;
+}
+const std::vector<ModelFamily>& model_families() {
+    static const std::vector<ModelFamily> families = {
+        {"Rafilix", [](const JsonValue& j) { return names_itself(j, "Rafilix"); }, read_rafilix},
+        {"Qwen2", [](const JsonValue& j) { return j.find("architecture") == nullptr; }, read_qwen2},
+    };
+    return families;
+}
+
+Config read_config(const std::string& dir) {
+    bool ok;
+    std::string text = read_text_file(dir + "/config.json", &ok);
+    if (!ok) throw Error(kErrIO, "Cannot open " + dir + "/config.json");
+    JsonValue j;
+    try {
+        j = json_parse(text);
+    } catch (const std::exception& e) {
+        throw Error(kErrFormat, dir + "/config.json: " + e.what());
+    }
+    for (const ModelFamily& f : model_families())
+        if (f.claims(j)) {
+            Config c = f.read(j);
+            c.family = f.name;
+            return c;
+        }
+    throw Error(kErrUnsupported, "config.json: no model family of this library is named '" + j.find("architecture")->str + "'");
+}
+
 TpPartition tp_partition(const Config& c, int rank, int size) {
+    if (!c.layers.empty()) {
+        if (size != 1 || rank != 0) throw Error(kErrUnsupported, "tensor parallel: the " + c.family + " family is not split across ranks");
+        TpPartition whole;
+        whole.n_v = c.vocab_size;
+        return whole;
+    }
     if (size < 1 || rank < 0 || rank >= size) throw Error(kErrInvalid, "tensor-parallel rank / size out of range");
     TpPartition p;
     p.tp_rank = rank;
@@ -223,6 +366,12 @@ const uint16_t* SafeTensorsDir::bf16(const std::string& name, size_t elems) cons
     const TensorInfo& ti = get(name);
     if (ti.dtype != "BF16") throw Error(kErrFormat, "Tensor " + name + " is " + ti.dtype + ", expected BF16");
     if (ti.nbytes != elems * 2) throw Error(kErrShape, "Size mismatch for " + name);
+    return (const uint16_t*)ti.data;
+}
+const uint16_t* SafeTensorsDir::bf16(const std::string& name, std::initializer_list<int64_t> shape) const {
+    const TensorInfo& ti = get(name);
+    if (ti.dtype != "BF16") throw Error(kErrFormat, "Tensor " + name + " is " + ti.dtype + ", expected BF16");
+    if (ti.shape != std::vector<int64_t>(shape)) throw Error(kErrShape, "Tensor " + name + " does not have the shape its layer needs");
     return (const uint16_t*)ti.data;
 }
 size_t SafeTensorsDir::num_tensors() const {

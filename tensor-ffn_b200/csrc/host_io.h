@@ -3,12 +3,15 @@
 #pragma once
 #include <cstdint>
 #include <cstdio>
+#include <initializer_list>
 #include <stdexcept>
 #include <string>
 #include <unordered_map>
 #include <vector>
 
 namespace tffn {
+
+struct JsonValue;
 
 struct Error : std::runtime_error {
     int code;
@@ -21,7 +24,40 @@ enum { kOk = 0, kErrInvalid = -1, kErrIO = -2, kErrFormat = -3, kErrShape = -4, 
 // Mirrors QwenConfig (inference/include/model/qwen.h:9-23) and qwen_config_from_json
 // (inference/src/model/qwen.cu:21-63): same keys, same defaults, head_dim = hidden / heads,
 // eos/bos given as a number or as an array whose first element counts.
+// A model whose layers are listed one by one (`layers` not empty) is described by LayerSpec entries instead of
+// the uniform Qwen2 fields; the uniform fields then hold what is common (width, vocabulary, layer count, eps) or
+// the first layer's value.
+struct RopeSpec {
+    int dims = 0;         // rotated leading dimensions of a head (0: none), neighbours (2i, 2i + 1) form a pair
+    double base = 10000.0;
+    bool scaled = false;  // wavelength-dependent frequency scaling: long waves / factor, short ones kept, a ramp between
+    double factor = 1.0, low = 1.0, high = 1.0, original = 1.0;
+    bool operator==(const RopeSpec& o) const {
+        return dims == o.dims && base == o.base && scaled == o.scaled && factor == o.factor && low == o.low && high == o.high &&
+               original == o.original;
+    }
+};
+// frequency of pair i (radians per position)
+double rope_frequency(const RopeSpec& r, int i);
+
+enum class Mixer { Attention, ChannelDelta };
+struct LayerSpec {
+    Mixer mixer = Mixer::Attention;
+    int heads = 0, kv_heads = 0;  // query (value) heads; key/value (query/key) heads they share
+    int dim = 0, vdim = 0;        // query/key size and value size of a head
+    // attention
+    int chunk = 0;                // a position sees the keys of its own chunk of this many positions (0: every earlier key)
+    float scale = 0.f;            // factor of the scores
+    RopeSpec rope;
+    // gated delta rule with one decay per key channel
+    int conv = 0;                 // taps of the short causal convolution
+    // feed-forward: a mixture of squared-ReLU experts (experts == 0: none)
+    int experts = 0, identity = 0, top = 0, ff = 0;
+};
+
 struct Config {
+    std::string family = "Qwen2";   // name in the model registry (model_families)
+    std::vector<LayerSpec> layers;  // empty: the uniform Qwen2 stack
     int hidden_size = 896, intermediate_size = 4864, num_layers = 24, num_heads = 14, num_kv_heads = 2;
     int head_dim = 64, vocab_size = 151936, max_seq_len = 131072;
     float rms_norm_eps = 1e-6f, rope_theta = 1e6f;
@@ -29,6 +65,15 @@ struct Config {
     bool tie_embeddings = true;
 };
 Config read_config(const std::string& model_dir);
+
+// The model registry: which families exist, how a config.json is recognised and read. Loading the weights is
+// Model::load's table of the same names (engine.cu).
+struct ModelFamily {
+    const char* name;
+    bool (*claims)(const JsonValue& config);
+    Config (*read)(const JsonValue& config);
+};
+const std::vector<ModelFamily>& model_families();
 
 // What one tensor-parallel rank owns. The reference is single-GPU; these are the slices of its matrices
 // (q/k/v rows by head: inference/src/model/qwen.cu:317-319; o_proj columns: :413-415; gate/up rows and down
@@ -79,6 +124,8 @@ public:
     // BF16 tensor with exactly `elems` elements, else throws (the reference checks the byte
     // size only: inference/src/model/qwen.cu:69-78)
     const uint16_t* bf16(const std::string& name, size_t elems) const;
+    // the same with every dimension checked
+    const uint16_t* bf16(const std::string& name, std::initializer_list<int64_t> shape) const;
     size_t num_shards() const { return shards_.size(); }
     size_t num_tensors() const;
 

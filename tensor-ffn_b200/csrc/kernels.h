@@ -12,14 +12,17 @@ typedef __nv_bfloat16 bf16;
 constexpr int kPageTokens = 32;  // tokens per KV page
 
 // ------------------------------------------------------------------ paged KV cache view
+// K rows may differ from V rows in width (kv.vd); with uniform layers one pool holds all of them (layer_stride),
+// with listed layers every attention layer has a view of its own (layer 0 of it).
 struct KvView {
-    bf16* k_pool;            // [L][pages][nkv][kPageTokens][hd]
-    bf16* v_pool;
+    bf16* k_pool;            // [L][pages][nkv][kPageTokens][hd]; fp32 rows instead in a session that computes in fp32
+    bf16* v_pool;            // [L][pages][nkv][kPageTokens][vd]
     const int* block_table;  // [max_batch][max_pages_per_seq]
     int max_pages_per_seq;
     int num_pages;           // pages per layer
     size_t layer_stride;     // elements between layers of a pool
     int nkv, hd;
+    int vd;                  // width of a V row (= hd for the uniform layers); hd and vd are multiples of 8
 };
 
 // ------------------------------------------------------------------ tensor-core GEMM (batched path)
@@ -29,6 +32,7 @@ enum GemmMode : int {
     GEMM_STORE_BF16 = 1,  // out bf16  = bf16(a0 (+ alpha * a1))
     GEMM_RESIDUAL = 2,    // out bf16 += a0 (+ alpha * a1), i.e. out = bf16(float(out) + sum)
     GEMM_SWIGLU = 3,      // out bf16  = bf16(silu(bf16(a0)) * bf16(a1))   (a0 gate rows, a1 up rows)
+    GEMM_RELU2 = 5,       // out bf16  = bf16(max(a0, 0)^2)
     GEMM_QKV = 4,         // q|k|v rows: bias + RoPE + page writes in the epilogue (GemmCall::qkv), no `out`
 };
 struct GemmQkvEpilogue {
@@ -75,7 +79,24 @@ struct GemmCall {
     int trace_ctas;          // CTAs the trace buffer holds; a larger grid is not traced
     unsigned long long* tl;  // optional 6 u64 of the step timeline (see tl_mark)
     bool pdl;          // launch with programmatic dependent launch (the kernel waits before touching X / out)
+    // Grouped launch (the experts of a mixture): the rows of X are sorted by group, W holds the groups' matrices back
+    // to back (N rows each) and grp[0 .. grp_tiles) says which group and rows each token tile of grp_bn rows covers
+    // (written by an earlier kernel, see GroupTile). op[1], op2 and GEMM_QKV are not available with it.
+    const struct GroupTile* grp;
+    int grp_tiles, grp_bn, grp_count;  // grp_count: groups in W
 };
+struct GroupTile {
+    int group;           // -1: this tile and all later ones are unused
+    int row0, row_end;   // rows [row0, min(row0 + grp_bn, row_end)) of X and out belong to it
+    int pad;
+};
+// token tile (16 .. 256) of a grouped launch whose groups hold `rows` rows on average
+int gemm_group_tile(int rows);
+// The same products in true fp32 (fp32 X and out, fp32 FMA, weights still bf16): modes STORE_F32, STORE_BF16 and
+// RELU2 (which then store fp32), one operand pair per problem, grouped launches included. The operands' X pointers
+// are fp32 arrays behind the bf16 type.
+int launch_gemm_f32(const GemmCall& c, cudaStream_t stream);
+constexpr int kGemmF32Tile = 64;  // its token tile (grp_bn)
 // Encoded tensor maps of the (buffer, shape, box) combinations a caller keeps launching with: encoding one costs
 // microseconds of host time and a decode step needs about 200. Owned by whoever owns the buffers (a session keeps
 // one for its lifetime), so entries die with the buffers they describe.
@@ -155,10 +176,24 @@ struct AttnWorkspace {
     int* counters;    // [T*nkv]
     int num_counters;
 };
+// Which keys a query sees and how the scores are scaled, when it differs from the uniform layers' causal attention
+// over 1 / sqrt(hd).
+struct AttnOptions {
+    float scale = 0.f;  // 0: 1 / sqrt(hd)
+    int chunk = 0;      // > 0: only the keys of the query's own chunk of `chunk` positions, counted from position 0
+    int vdim = 0;       // > 0: columns of an output head (kv.vd is the padded row); 0: kv.vd
+    int64_t ctx_ld = 0; // row stride of ctx (0: nh * vdim)
+};
 // opt the attention kernels into their dynamic shared memory (once per device, outside stream capture)
 int attn_prepare();
 // context splits launch_attention will use (a CUDA-graph key: the grid depends on it)
 int attention_splits(int T, int nh, int nkv, int hd, int max_ctx, const AttnWorkspace& ws, int num_sms);
+// whether the tensor-core kernels take this head geometry (else launch_attention_simt)
+inline bool attention_tc_supported(int hd, int vd) { return hd <= 128 && vd <= 128; }
+// One warp-per-key-group attention without tensor cores: any head size up to 512, bf16 or (f32) fp32 cache and
+// output, prompt and decode rows alike.
+void launch_attention_simt(const float* q, KvView kv, bool f32, const int* tok_seq, const int* tok_pos, void* ctx, int T, int nh,
+                           const AttnOptions& opt, int* status, cudaStream_t s, bool pdl = false, unsigned long long* tl = nullptr);
 // one query token per (t): context = tok_pos[t] + 1 cached tokens of sequence tok_seq[t].
 // only_newest_row_fresh (decode): of everything the kernel reads, only q and the cached row at
 // tok_pos[t] were written since the last kernel of the stream that was launched WITHOUT programmatic
@@ -166,13 +201,127 @@ int attention_splits(int T, int nh, int nkv, int hd, int max_ctx, const AttnWork
 void launch_attention(const float* q, KvView kv, int layer, const int* tok_seq, const int* tok_pos, bf16* ctx, int T,
                       int nh, int max_ctx, AttnWorkspace ws, int num_sms, int* status, cudaStream_t s, bool pdl = false,
                       bool only_newest_row_fresh = false, unsigned long long* tl = nullptr,
-                      unsigned long long* trace = nullptr, int trace_ctas = 0);  // trace: 16 u64 per CTA, see attn.cu
+                      unsigned long long* trace = nullptr, int trace_ctas = 0,  // trace: 16 u64 per CTA, see attn.cu
+                      const AttnOptions& opt = AttnOptions());
 
 // Prompt tokens: rows grp_first[g] .. grp_first[g] + grp_count[g] - 1 (at most 8, consecutive positions of
 // one sequence) share one pass over that sequence's cache; n_groups groups cover the T rows of the call.
 void launch_attention_prefill(const float* q, KvView kv, int layer, const int* tok_seq, const int* tok_pos, const int* grp_first,
                               const int* grp_count, int n_groups, bf16* ctx, int nh, int* status, cudaStream_t s,
-                              bool pdl = false, unsigned long long* tl = nullptr);
+                              bool pdl = false, unsigned long long* tl = nullptr, const AttnOptions& opt = AttnOptions());
+
+// ------------------------------------------------------------------ layers with an fp32 residual stream
+// "f32" below selects the storage type of activations and cache: fp32 in a session that computes in fp32, else bf16.
+enum RowSource : int { ROWS_KEEP = 0, ROWS_EMBED, ROWS_DELTA, ROWS_MOE };
+// One pass over the residual stream per sublayer: x = table[token] | x + norm(delta) * post_w | x + norm(sum of the
+// chosen experts' outputs) * post_w, then out = norm(x) * next_w. Norm: v / sqrt(mean(v^2) + eps). All in fp32.
+struct ResidualRows {
+    float* x;                 // [T][H]
+    int H;
+    float eps;
+    int source;               // RowSource
+    const int* tokens;        // ROWS_EMBED
+    const bf16* table;
+    int64_t table_ld;
+    int V;
+    int* status;
+    const float* delta;       // ROWS_DELTA: [T][delta_ld]
+    int64_t delta_ld;
+    const void* y;            // ROWS_MOE: expert outputs, rows in expert order [.][y_ld]
+    int64_t y_ld;
+    const int* pair_row;      // [T][top] row of y, or -1: the pair's output is the sublayer's input itself (`out` before this call)
+    const float* pair_w;      // [T][top]
+    int top;
+    const float* post_w;      // norm of the sublayer's output
+    const float* next_w;      // nullptr: no `out`
+    void* out;                // [.][out_ld]
+    int64_t out_ld;
+    const int* row_idx;       // with ROWS_KEEP: out row r = norm of x row row_idx[r]
+};
+int stack_rows_prepare();
+void launch_residual_rows(const ResidualRows& a, bool f32, int rows, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
+
+// q|k|v rows of one projection -> per-head norm of q and k (weights shared by the heads), rotation of neighbouring
+// pairs, q in fp32 for the attention kernels, k and v into the sequence's page.
+struct QkNormRope {
+    const void* qkv;          // [T][ld]: q at 0, k at k_off, v at v_off
+    int64_t ld;
+    int k_off, v_off;
+    const float *q_norm, *k_norm;
+    float eps;
+    int nh, dim, vdim, rope_dims;
+    const float2* rope;       // [max_pos][rope_dims / 2] (cos, sin)
+    int max_pos;
+    const int *tok_seq, *tok_pos;
+    float* q_out;             // [T][nh][kv.hd], zeros past dim
+    KvView kv;
+    int* status;
+};
+void launch_qk_norm_rope(const QkNormRope& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
+
+// ------------------------------------------------------------------ gated delta rule, one decay per key channel
+// Recurrent state of a slot: S [heads][vdimP][dimP] fp32 (transposed: a value column's keys are contiguous; dimP a
+// multiple of 32, vdimP of 4, the padding stays zero) and the last taps - 1 inputs of the convolution as a ring
+// [taps - 1][channels] fp32 addressed by position. A sequence that starts at position 0 starts from zeros whatever
+// the slot held before.
+struct DeltaRule {
+    int heads, kv_heads, dim, vdim, dimP, vdimP, taps;
+    float eps;
+    const void* proj;         // [T][proj_ld]: q at q_off, k at k_off, v at v_off, beta logits at b_off
+    int64_t proj_ld;
+    int q_off, k_off, v_off, b_off;
+    const float* conv;        // [taps][channels], channels = q | k | v
+    const float* a_log;       // [heads]
+    const float* dt_bias;     // [heads * dim]
+    const float* decay_in;    // [T][decay_ld]: W_a2 (W_a1 h)
+    int64_t decay_ld;
+    const float* gate_in;     // [T][gate_ld]: W_g2 (W_g1 h)
+    int64_t gate_ld;
+    const float* out_norm;    // [vdim]
+    float *state, *ring;      // of slot 0
+    size_t state_stride, ring_stride;  // floats between slots
+    // per token, from the preparation to the scan
+    float *qn, *kn;           // [T][kv_heads][dimP] unit vectors, q scaled
+    float *v;                 // [T][heads][vdimP]
+    float *g;                 // [T][heads][dimP] decays
+    float *bk;                // [T][heads][2]: beta, k . q
+    void* out;                // [T][out_ld]
+    int64_t out_ld;
+    const int *tok_seq, *tok_pos;
+    const int *seg_first, *seg_count;  // runs of consecutive positions of one sequence among the T rows
+    int max_slots;
+    int* status;
+};
+void launch_delta_prep(const DeltaRule& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
+void launch_delta_scan(const DeltaRule& a, bool f32, int n_segs, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
+int delta_prepare();
+int delta_padded_dim(int dim);  // dimP
+inline bool delta_supported(int dim, int vdim) { return dim <= 256 && vdim <= 256; }
+
+// ------------------------------------------------------------------ mixture of experts
+int moe_prepare();
+struct MoeRoute {
+    const float* logits;      // [T][ld], experts + identity columns
+    int64_t ld;
+    const float* correction;  // [experts + identity]
+    int experts, identity, top;
+    int* counts;              // [experts], zero before the launch
+    int2* pair;               // [T][top]: expert (-1: identity) and the pair's place within it
+    float* pair_w;            // [T][top] softmax score (without the correction)
+};
+void launch_moe_route(const MoeRoute& a, int T, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
+struct MoeGather {
+    const void* x;            // [T][x_ld]
+    int64_t x_ld;
+    int H, experts, top;
+    const int* counts;
+    const int2* pair;
+    void* xg;                 // [T * top][x_ld] rows sorted by expert
+    int* pair_row;            // [T][top] row of xg, -1 for identity
+    GroupTile* tiles;         // [max_tiles]
+    int max_tiles, tile_rows;
+};
+void launch_moe_gather(const MoeGather& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
 
 // ------------------------------------------------------------------ batch-1 fused decode kernels
 struct Bs1Layer {

@@ -50,6 +50,7 @@ _SIGS = {
     "tffn_version": (_i, []),
     "tffn_device_count": (_i, []),
     "tffn_config_read": (_i, [_cp, ctypes.POINTER(Config)]),
+    "tffn_config_family": (_i, [_cp, _vp, _i]),
     "tffn_expert_probe": (_i, [_cp] + [ctypes.POINTER(ctypes.c_uint32)] * 4),
     "tffn_expert_write": (_i, [_cp, ctypes.c_uint32, ctypes.c_uint32, ctypes.c_uint32, ctypes.POINTER(_vp)]),
     "tffn_safetensors_probe": (_i, [_cp, _cp, ctypes.POINTER(ctypes.c_int32), ctypes.POINTER(ctypes.c_int32), _vp,
@@ -65,6 +66,7 @@ _SIGS = {
     "tffn_model_load": (_i, [_cp, _i, _i, _i, _pp]),
     "tffn_model_free": (None, [_vp]),
     "tffn_model_config": (_i, [_vp, ctypes.POINTER(Config)]),
+    "tffn_model_family": (_cp, [_vp]),
     "tffn_model_weight_bytes": (ctypes.c_uint64, [_vp, _i]),
     "tffn_expert_load": (_i, [_vp, _cp, _f, _pp]),
     "tffn_expert_set_scale": (_i, [_vp, _f]),
@@ -73,6 +75,7 @@ _SIGS = {
     "tffn_session_create": (_i, [_vp, _vp, _i, _i, _vp, _pp]),
     "tffn_session_free": (None, [_vp]),
     "tffn_session_create_tp": (_i, [_vp, _vp, _i, _i, _vp, _vp, _pp]),
+    "tffn_session_create_ex": (_i, [_vp, _vp, _i, _i, _vp, _vp, _i, _pp]),
     "tffn_tp_unique_id": (_i, [_vp]),
     "tffn_tp_create": (_i, [_vp, _i, _i, _i, _pp]),
     "tffn_tp_free": (None, [_vp]),
@@ -87,6 +90,7 @@ _SIGS = {
     "tffn_session_set_bs1_path": (_i, [_vp, _i]),
     "tffn_session_capture_hidden": (_i, [_vp, _i]),
     "tffn_session_get_hidden": (_i, [_vp, _i, _vp, _i]),
+    "tffn_session_get_hidden_f32": (_i, [_vp, _i, _vp, _i]),
     "tffn_prefill": (_i, [_vp, _vp, _vp, _i, _vp, _vp]),
     "tffn_forward": (_i, [_vp, _i, _vp, _i, _vp]),
     "tffn_decode_step": (_i, [_vp, _vp, _i, _vp, _vp]),
@@ -132,6 +136,13 @@ def qwen_config_from_json(model_dir: str) -> Config:
     c = Config()
     _check(_L.tffn_config_read(model_dir.encode(), ctypes.byref(c)))
     return c
+
+
+def model_family(model_dir: str) -> str:
+    """name of the model family a config.json belongs to ("Qwen2", "Rafilix")"""
+    buf = ctypes.create_string_buffer(64)
+    _check(_L.tffn_config_family(model_dir.encode(), buf, 64))
+    return buf.value.decode()
 
 
 def expert_probe(path: str):
@@ -246,6 +257,10 @@ class QwenModel:
         self.cfg = Config()
         _check(_L.tffn_model_config(self._h, ctypes.byref(self.cfg)))
 
+    @property
+    def family(self) -> str:
+        return _L.tffn_model_family(self._h).decode()
+
     def weight_bytes(self, with_expert: bool) -> int:
         return int(_L.tffn_model_weight_bytes(self._h, int(with_expert)))
 
@@ -265,6 +280,9 @@ def qwen_load(model_dir: str, device: int = 0, tp_rank: int = 0, tp_size: int = 
     h = _vp()
     _check(_L.tffn_model_load(model_dir.encode(), device, tp_rank, tp_size, ctypes.byref(h)))
     return QwenModel(h)
+
+
+load_model = qwen_load  # every family: config.json says which
 
 
 def tp_unique_id() -> bytes:
@@ -338,13 +356,14 @@ class Session:
     """KV cache + scratch (the second half of qwen_load, inference/src/model/qwen.cu:134-171), paged."""
 
     def __init__(self, model: QwenModel, expert: ExpertModel | None = None, max_batch: int = 1, max_seq: int = 2048,
-                 stream: int | None = None, tp: "TpGroup | None" = None):
+                 stream: int | None = None, tp: "TpGroup | None" = None, compute: str = "bfloat16"):
+        """compute: "bfloat16", or "float32" for everything in true fp32 (families that list their layers)"""
         self.model, self.expert, self.tp = model, expert, tp
         self.max_batch, self.max_seq = max_batch, max_seq
         self.V = model.cfg.vocab_size
         self._h = _vp()
-        _check(_L.tffn_session_create_tp(model._h, expert._h if expert else None, max_batch, max_seq, stream,
-                                         tp._h if tp else None, ctypes.byref(self._h)))
+        _check(_L.tffn_session_create_ex(model._h, expert._h if expert else None, max_batch, max_seq, stream,
+                                         tp._h if tp else None, {"bfloat16": 0, "float32": 1}[compute], ctypes.byref(self._h)))
 
     def free(self):
         if getattr(self, "_h", None):
@@ -386,6 +405,11 @@ class Session:
     def get_hidden(self, layer: int, rows: int) -> np.ndarray:
         out = np.zeros((rows, self.model.cfg.hidden_size), dtype=np.uint16)
         n = _check(_L.tffn_session_get_hidden(self._h, layer, out.ctypes.data, rows))
+        return out[:n]
+
+    def get_hidden_f32(self, layer: int, rows: int) -> np.ndarray:
+        out = np.zeros((rows, self.model.cfg.hidden_size), dtype=np.float32)
+        n = _check(_L.tffn_session_get_hidden_f32(self._h, layer, out.ctypes.data, rows))
         return out[:n]
 
     def qwen_forward(self, tokens, slot: int = 0, want_logits: bool = True):

@@ -5,7 +5,8 @@
 // int32 ids instead of --prompt), --ignore-eos, --device <N>, --host-sampling (with --temperature: sample
 // on the host from downloaded logits as the reference does, instead of on the device), --bpe (tokenise the
 // prompt and print the output with the byte-level BPE that tokenizer.json specifies, instead of the
-// reference's encoder, which drops spaces and newlines).
+// reference's encoder, which drops spaces and newlines), --dtype float32 (compute in fp32, for the families that
+// can). With --prompt-ids a model folder needs no tokenizer.json: without one the generated ids are printed.
 // The usage text, the flag scanning, the ChatML sequence, the stdout protocol and the host sampler
 // are the reference's own (inference/src/main.cpp:17-63, 127-144, 157-198), reproduced on purpose:
 // they ARE the command-line contract. What differs is what runs underneath: the six calls into the
@@ -99,14 +100,21 @@ int main(int argc, char** argv) {
     bool use_chat = has_switch(argc, argv, "--chat");
     bool ignore_eos = has_switch(argc, argv, "--ignore-eos");
     bool bpe = has_switch(argc, argv, "--bpe");
+    std::string dtype = get_flag(argc, argv, "--dtype", "bfloat16");
 
     if (model_dir.empty() || (prompt.empty() && ids_path.empty())) {
         fprintf(stderr, "--model and --prompt are required\n");
         usage();
     }
 
+    if (dtype != "bfloat16" && dtype != "float32") {
+        fprintf(stderr, "--dtype is bfloat16 or float32\n");
+        usage();
+    }
     tffn_tokenizer* tok = nullptr;
-    CHECK(tffn_tokenizer_load(model_dir.c_str(), &tok));
+    FILE* tok_file = fopen((model_dir + "/tokenizer.json").c_str(), "rb");
+    if (tok_file) fclose(tok_file);
+    if (tok_file || ids_path.empty()) CHECK(tffn_tokenizer_load(model_dir.c_str(), &tok));
     tffn_model* mdl = nullptr;
     CHECK(tffn_model_load(model_dir.c_str(), device, 0, 1, &mdl));
     tffn_config cfg;
@@ -166,9 +174,11 @@ int main(int argc, char** argv) {
     printf("\nPrompt (%d tokens): %s\n", prompt_len, prompt.c_str());
 
     tffn_session* sess = nullptr;
-    CHECK(tffn_session_create(mdl, expert, 1, max_seq, nullptr, &sess));
+    CHECK(tffn_session_create_ex(mdl, expert, 1, max_seq, nullptr, nullptr, dtype == "float32" ? TFFN_COMPUTE_F32 : TFFN_COMPUTE_BF16,
+                                 &sess));
     uint32_t eos = 151645;
-    tffn_tokenizer_special(tok, &eos, nullptr, nullptr);
+    if (tok) tffn_tokenizer_special(tok, &eos, nullptr, nullptr);
+    else eos = (uint32_t)cfg.eos_token_id;  // -1 (never generated) where the configuration names none
 
     std::vector<int32_t> h_tokens(prompt_ids.begin(), prompt_ids.end());
     const int V = cfg.vocab_size;
@@ -194,7 +204,8 @@ int main(int argc, char** argv) {
         }
         char text[512];
         uint32_t id = (uint32_t)next;
-        (bpe ? tffn_tokenizer_decode_bpe : tffn_tokenizer_decode)(tok, &id, 1, text, sizeof text);
+        if (tok) (bpe ? tffn_tokenizer_decode_bpe : tffn_tokenizer_decode)(tok, &id, 1, text, sizeof text);
+        else snprintf(text, sizeof text, "%s%u", step ? " " : "", id);
         printf("%s", text);
         fflush(stdout);
         int32_t fed = next;

@@ -236,6 +236,88 @@ def write_model(dirpath: str, shape: str | dict = "tiny", seed: int = 1234, qkv_
     return cfg
 
 
+# ------------------------------------------------------------------------------------------- layer-list models (Rafilix)
+def attention_layer(heads, kv_heads, dim, vdim, chunk=None, rot_dims=None, base=10000.0, scaling=None, scale=None, mlp=None) -> dict:
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale if scale is not None else dim ** -0.5,
+         "rot": {"base": base, "dims": dim if rot_dims is None else rot_dims}}
+    if scaling:
+        m["rot"]["scaling"] = scaling
+    if chunk:
+        m["mask"] = {"size": chunk}
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def channel_delta_layer(heads, kv_heads, dim, vdim, conv=4, mlp=None) -> dict:
+    return {"type": "channel_delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}, "mlp": mlp}
+
+
+def moe_mlp(experts, top, ff, identity=0) -> dict:
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "identity": identity, "top": top}}
+
+
+def rafilix_config(width, vocab, layers, eps=1e-5) -> dict:
+    return {"architecture": "Rafilix", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": layers}
+
+
+def rafilix_specs(cfg: dict, rank: int = 16, qk_norm: float = 1.0):
+    """(name, shape, kind, parameter) of every tensor. kind: 'w' normal with that standard deviation, 'n' norm weight
+    around that value, 'u' uniform in that interval. rank: of the two low-rank projections of a delta-rule layer."""
+    H = cfg["width"]
+    specs = [("embed", (cfg["vocab"], H), "w", 0.5)]
+    for i, layer in enumerate(cfg["layers"]):
+        m, n = layer["mixer"], f"l{i}."
+        p, f = n + "mix.", n + "mlp."
+        h, g, d, v = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        lin = lambda name, out, inp, gain=1.0: (name, (out, inp), "w", gain * inp ** -0.5)
+        specs += [(n + t, (H,), "n", 1.0) for t in ("norm1", "norm1b")]
+        if layer["type"] == "attention":
+            specs += [lin(p + "q", h * d, H), lin(p + "k", g * d, H), lin(p + "v", g * v, H),
+                      (p + "q.norm", (d,), "n", qk_norm), (p + "k.norm", (d,), "n", qk_norm)]
+        else:
+            specs += [lin(p + "q", g * d, H), lin(p + "k", g * d, H), lin(p + "v", h * v, H)]
+            specs += [(p + t + ".conv", (c, m["conv"]), "w", 0.6) for t, c in (("q", g * d), ("k", g * d), ("v", h * v))]
+            specs += [lin(p + "b", h, H), (p + "A_log", (h,), "u", (-3.0, 1.0)), (p + "norm", (v,), "n", 1.0), lin(p + "a1", rank, H),
+                      lin(p + "a2", h * d, rank), (p + "dt_bias", (h * d,), "u", (-4.0, 1.0)), lin(p + "g1", rank, H), lin(p + "g2", h * v, rank)]
+        specs.append(lin(p + "o", H, h * v))
+        if layer.get("mlp"):
+            r, ff = layer["mlp"]["router"], layer["mlp"]["expert"]["ff"]
+            specs += [(n + t, (H,), "n", 1.0) for t in ("norm2", "norm2b")]
+            for e in range(r["experts"]):
+                specs += [lin(f"{f}e{e}.up", ff, H), lin(f"{f}e{e}.down", H, ff)]
+            outs = r["experts"] + r["identity"]
+            specs += [lin(f + "router", outs, H, 2.0), (f + "correction", (outs,), "w", 0.05)]
+    specs.append(("final.norm", (H,), "n", 1.0))
+    return specs
+
+
+def write_rafilix(dirpath: str, cfg: dict, seed: int = 1, rank: int = 16, qk_norm: float = 1.0, fast: bool = False, edit=None) -> dict:
+    """config.json and model.safetensors with seeded random weights. edit(name, float array) -> array or None may replace
+    a tensor before it is rounded to bf16. fast: matrices cut out of one random block (throughput runs)."""
+    os.makedirs(dirpath, exist_ok=True)
+    with open(os.path.join(dirpath, "config.json"), "w") as f:
+        json.dump(cfg, f, indent=1)
+    out = []
+    for i, (name, shape, kind, par) in enumerate(rafilix_specs(cfg, rank, qk_norm)):
+        n = int(np.prod(shape))
+        if fast and kind == "w" and n > 1 << 16:
+            out.append((name, shape, _tiled_bf16([seed, i], n, float(np.float16(par)))))
+            continue
+        rng = np.random.default_rng([seed, i])
+        if kind == "w":
+            x = rng.standard_normal(n, dtype=np.float32) * np.float32(par)
+        elif kind == "n":
+            x = np.float32(par) * (1.0 + 0.1 * rng.standard_normal(n, dtype=np.float32))
+        else:
+            x = rng.uniform(par[0], par[1], n).astype(np.float32)
+        x = x.reshape(shape)
+        if edit is not None:
+            y = edit(name, x)
+            x = x if y is None else y
+        out.append((name, shape, f32_to_bf16(np.ascontiguousarray(x, dtype=np.float32).reshape(-1))))
+    write_safetensors(os.path.join(dirpath, "model.safetensors"), out)
+    return cfg
+
+
 def write_expert(path: str, cfg: dict, seed: int = 4321, std: float = 0.02, threads: int = 0,
                  num_layers: int | None = None, hidden: int | None = None, inter: int | None = None,
                  magic: int = EXPERT_MAGIC, truncate_bytes: int = 0, fast: bool = False):

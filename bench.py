@@ -657,6 +657,218 @@ def run_expert_forward_case(a):
                       "frac": tf / peak if peak else None, "finite": bool(torch.isfinite(out).all().item())}))
 
 
+# ------------------------------------------------------------------------------------------- layer-list models
+# Sizes that resemble a real model's layers, beside a Qwen2 stack of the same width, depth, head geometry and vocabulary
+# whose FFN is as large as the experts a token uses.
+STACK_SIZES = {
+    "w896": dict(width=896, vocab=32768, depth=8, heads=14, kv=2, dim=64, d_heads=14, d_kv=14, d_dim=64, experts=16, top=4, ff=1792,
+                 identity=2, chunk=1024, rank=64, qwen_ff=4864),
+    "w2048": dict(width=2048, vocab=32768, depth=8, heads=16, kv=2, dim=128, d_heads=16, d_kv=8, d_dim=128, experts=32, top=4, ff=1536,
+                  identity=2, chunk=2048, rank=128, qwen_ff=4096),
+}
+
+
+def stack_models(name: str) -> tuple[str, dict, str, dict]:
+    """(folder, config) of the layer-list model and of the Qwen2 stack beside it, written once per machine"""
+    import synth
+    z = STACK_SIZES[name]
+    mlp = synth.moe_mlp(z["experts"], z["top"], z["ff"], identity=z["identity"])
+    att = synth.attention_layer(z["heads"], z["kv"], z["dim"], z["dim"], chunk=z["chunk"], mlp=mlp)
+    rec = synth.channel_delta_layer(z["d_heads"], z["d_kv"], z["d_dim"], z["d_dim"], mlp=mlp)
+    cfg = synth.rafilix_config(z["width"], z["vocab"], [att if i % 2 == 0 else rec for i in range(z["depth"])])
+    d = model_dir("rafilix_" + name)
+    if not os.path.exists(os.path.join(d, ".complete")):
+        shutil.rmtree(d, ignore_errors=True)
+        synth.write_rafilix(d, cfg, seed=5, rank=z["rank"], fast=True)
+        open(os.path.join(d, ".complete"), "w").close()
+    q = model_dir("qwen2_" + name)
+    shape = dict(hidden_size=z["width"], num_hidden_layers=z["depth"], num_attention_heads=z["width"] // z["dim"], num_key_value_heads=z["kv"],
+                 intermediate_size=z["qwen_ff"], vocab_size=z["vocab"], tie_word_embeddings=True, eos_token_id=1, bos_token_id=1)
+    if not os.path.exists(os.path.join(q, ".complete")):
+        shutil.rmtree(q, ignore_errors=True)
+        shape = synth.write_model(q, shape, seed=6, fast=True)
+        open(os.path.join(q, ".complete"), "w").close()
+    return d, cfg, q, shape
+
+
+def stack_work(cfg: dict, rows: int, ctx: float, rank: int, seqs: int) -> dict:
+    """per kernel class of one launch over `rows` tokens (`seqs` sequences): (HBM bytes, FLOPs), every weight a launch needs
+    once, activations once in and once out; summed over the layers"""
+    H, out = cfg["width"], {}
+
+    def add(k, b, f=0.0):
+        x = out.setdefault(k, [0.0, 0.0])
+        x[0] += b
+        x[1] += f
+    rows_b = rows * H * 4
+    for l in cfg["layers"]:
+        m = l["mixer"]
+        h, g, d, v = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        if l["type"] == "attention":
+            n_in = h * d + g * (d + v)
+            c = min(ctx, m.get("mask", {}).get("size", ctx))
+            add("qk_norm_rope", rows * (2 * n_in + 4 * h * d + 2 * g * (d + v)))
+            add("attn_decode", seqs * c * g * (d + v) * 2 + rows * h * (4 * d + 2 * v), 2.0 * rows * (c if rows == seqs else c / 2) * h * (d + v))
+        else:
+            n_in = g * 2 * d + h * v + h + 2 * rank
+            add("gemm:low_rank", h * (d + v) * rank * 2 + rows * (2 * rank * 2 + h * (d + v) * 4), 2.0 * rows * h * (d + v) * rank)
+            tok = 4 * (2 * g * d + h * v + h * d + 2 * h)
+            add("delta_prep", rows * (2 * (2 * g * d + h * v) + 4 * h * d + tok))
+            add("delta_scan", seqs * 2 * 4 * h * d * v + rows * (tok + 4 * h * v + 2 * h * v), 8.0 * rows * h * d * v)
+        add("gemm:mixer_in", n_in * H * 2 + rows * (H + n_in) * 2, 2.0 * rows * n_in * H)
+        add("gemm_tc:o_proj", h * v * H * 2 + rows * (h * v * 2 + H * 4), 2.0 * rows * h * v * H)
+        add("residual_rows", 2 * rows_b + rows * H * (4 + 2))
+        r, ff = l["mlp"]["router"], l["mlp"]["expert"]["ff"]
+        outs, top = r["experts"] + r["identity"], r["top"]
+        pairs = rows * top * r["experts"] / outs
+        used = r["experts"] * (1 - (1 - top / outs) ** rows)  # experts a launch touches when choices are even
+        add("gemm:router", outs * H * 2 + rows * (H * 2 + outs * 4), 2.0 * rows * outs * H)
+        add("moe_route", rows * (outs * 4 + top * 12))
+        add("moe_gather", 2 * pairs * H * 2)
+        add("gemm:expert_up", used * ff * H * 2 + pairs * (H + ff) * 2, 2.0 * pairs * ff * H)
+        add("gemm:expert_down", used * ff * H * 2 + pairs * (H + ff) * 2, 2.0 * pairs * ff * H)
+        add("residual_rows", 2 * rows_b + pairs * H * 2 + rows * H * 2)
+    add("embed_rows", rows * H * (2 + 4 + 2))
+    n = seqs  # rows that get logits
+    add("gemm_tc:lm_head", cfg["vocab"] * H * 2 + n * H * 2, 2.0 * n * cfg["vocab"] * H)
+    return out
+
+
+def qwen_work(cfg: dict, rows: int, ctx: float, seqs: int) -> dict:
+    H, I, L, V = cfg["hidden_size"], cfg["intermediate_size"], cfg["num_hidden_layers"], cfg["vocab_size"]
+    nh, nkv = cfg["num_attention_heads"], cfg["num_key_value_heads"]
+    hd = H // nh
+    n_in = (nh + 2 * nkv) * hd
+    b = {"gemm_tc:qkv": (L * (n_in * H * 2 + rows * (H * 2 + nh * hd * 4 + 2 * nkv * hd * 2)), 2.0 * L * rows * n_in * H),
+         "attn_decode": (L * (seqs * ctx * 2 * nkv * hd * 2 + rows * nh * hd * 6), 4.0 * L * rows * (ctx if rows == seqs else ctx / 2) * nh * hd),
+         "gemm_tc:o_proj": (L * (H * H * 2 + rows * H * 6), 2.0 * L * rows * H * H),
+         "gemm_tc:gate_up_swiglu": (L * (2 * I * H * 2 + rows * (H + I) * 2), 4.0 * L * rows * I * H),
+         "gemm_tc:down": (L * (I * H * 2 + rows * (I * 2 + H * 4)), 2.0 * L * rows * I * H),
+         "rmsnorm_rows": ((2 * L + 1) * rows * H * 4, 0.0), "embed_rows": (rows * H * 4, 0.0),
+         "gemm_tc:lm_head": (V * H * 2 + seqs * H * 2, 2.0 * seqs * V * H)}
+    for a, k in (("bs1_qkv", "gemm_tc:qkv"), ("bs1_oproj", "gemm_tc:o_proj"), ("bs1_lmhead", "gemm_tc:lm_head")):
+        b[a] = b[k]
+    b["bs1_ffn"] = (L * 3 * I * H * 2, 6.0 * L * rows * I * H)
+    return {k: list(v) for k, v in b.items()}
+
+
+def run_stack(a):
+    """--stack SIZE: prefill and decode throughput of a layer-list (Rafilix) model and of the Qwen2 stack beside it, with
+    the time every kernel class adds to a decode step (in-kernel stamps) and to a prefill launch (CUDA events), against
+    the measured roofline (the larger of bytes / HBM peak and FLOPs / bf16 GEMM peak; the recurrence's FLOPs are fp32
+    work of the CUDA cores and are listed, not converted). One JSON line. L2 is not flushed: weights of a decode step
+    and activations of a prefill launch exceed it."""
+    import torch
+    import tffn
+    torch.cuda.set_device(0)
+    stream = torch.cuda.Stream()
+    hbm, kind = peaks()
+    tflops = 1590.0
+    pk = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    if os.path.exists(pk):
+        with open(pk) as f:
+            tflops = float(json.load(f)["bf16_tflops"])
+    d, cfg, q, qcfg = stack_models(a.stack)
+    rank = STACK_SIZES[a.stack]["rank"]
+    sampler = ClockSampler(None)
+    line = {"metric": f"layer-list model {a.stack}: decode tok/s and prefill tok/s beside a Qwen2 stack of equal size", "unit": "tok/s",
+            "data": "synthetic", "dtype": "bf16", "steps": a.steps, "warmup": a.warmup, "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "kind": kind},
+            "sizes": STACK_SIZES[a.stack]}
+    K = min(a.steps, 64)
+    for which, path in (("rafilix", d), ("qwen2", q)):
+        model = tffn.load_model(path)
+        work = (lambda rows, ctx, seqs: stack_work(cfg, rows, ctx, rank, seqs)) if which == "rafilix" else \
+            (lambda rows, ctx, seqs: qwen_work(qcfg, rows, ctx, seqs))
+        res = {"weight_bytes": model.weight_bytes(False)}
+
+        def table(times, w):  # times: class -> (us per step, launches per step)
+            rows = []
+            for k, (us, cnt) in sorted(times.items(), key=lambda kv: -kv[1][0]):
+                r = {"kernel": k, "us": round(us, 2), "launches": round(cnt, 2)}
+                if k in w and us > 0:
+                    ideal = max(w[k][0] / hbm / 1e3, 0.0 if k == "delta_scan" else w[k][1] / tflops / 1e6)
+                    r["roofline_frac"] = round(ideal / us, 3)
+                    if k == "delta_scan":
+                        r["fp32_tflops"] = round(w[k][1] / us / 1e6, 1)
+                rows.append(r)
+            return rows
+
+        def decode(sess, n, ctx):
+            sess.decode_run(n, max(a.warmup, 3), want_tokens=False)
+            ms, reps, _, _ = timed_decode(sess, stream, n, K, 5, torch.cuda.synchronize, lambda x: x)
+            names, tl = sess.timeline(n)
+            tl, times = tl.astype(np.int64), {}
+            prev = int(tl[:, 0].min())
+            for nm, r in zip(names, tl):
+                e = times.setdefault(nm, [0.0, 0])
+                e[0] += (int(r[5]) - prev) / 1e3
+                e[1] += 1
+                prev = int(r[5])
+            return {"tok_s": n * K / (ms / 1e3), "ms_per_step": ms / K, "rep_ms": reps, "kernels": table(times, work(n, ctx, n))}
+
+        n, P = a.seqs, a.prompt
+        sess = tffn.Session(model, max_batch=n, max_seq=P + K * 5 + a.warmup + 64, stream=stream.cuda_stream)
+        sess.set_launch_mode(a.launch_mode)
+        prompts = np.random.default_rng(3).integers(2, STACK_SIZES[a.stack]["vocab"], (n, P)).astype(np.int32)
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        times = []
+        for rep in range(max(a.warmup, 3) + 5):
+            sess.qwen_reset()
+            torch.cuda.synchronize()
+            e0.record(stream)
+            sess.prefill(list(prompts))
+            e1.record(stream)
+            torch.cuda.synchronize()
+            if rep >= max(a.warmup, 3):
+                times.append(e0.elapsed_time(e1))
+        ms = float(np.median(times))
+        sess.qwen_reset()
+        sess.profile(True)
+        sess.prefill(list(prompts))
+        prof = sess.profile_read()
+        sess.profile(False)
+        launches = prof["embed_rows"][1]
+        rows = n * P // launches
+        res["prefill"] = {"tok_s": n * P / (ms / 1e3), "ms": ms, "rows_per_launch": rows, "launches": launches, "rep_ms": times,
+                          "kernels_per_launch": table({k: (v[0] * 1e3 / launches, v[1] / launches) for k, v in prof.items()},
+                                                      work(rows, P, rows // P))}
+        res["decode"] = decode(sess, n, P + K * 2.5)
+        sess.free()
+        s1 = tffn.Session(model, max_batch=1, max_seq=P + K * 5 + a.warmup + 64, stream=stream.cuda_stream)
+        s1.set_launch_mode(a.launch_mode)
+        s1.prefill([prompts[0]])
+        res["decode_bs1"] = decode(s1, 1, P + K * 2.5)
+        s1.free()
+        long_p = np.random.default_rng(4).integers(2, STACK_SIZES[a.stack]["vocab"], 4096).astype(np.int32)
+        s2 = tffn.Session(model, max_batch=1, max_seq=4200, stream=stream.cuda_stream)
+        s2.set_launch_mode(a.launch_mode)
+        times = []
+        for rep in range(max(a.warmup, 3) + 3):
+            s2.qwen_reset()
+            torch.cuda.synchronize()
+            e0.record(stream)
+            s2.prefill([long_p])
+            e1.record(stream)
+            torch.cuda.synchronize()
+            if rep >= max(a.warmup, 3):
+                times.append(e0.elapsed_time(e1))
+        ms = float(np.median(times))
+        s2.qwen_reset()
+        s2.profile(True)
+        s2.prefill([long_p])
+        prof = s2.profile_read()
+        launches = prof["embed_rows"][1]
+        res["prefill_one_4096"] = {"tok_s": 4096 / (ms / 1e3), "ms": ms,
+                                   "kernels_per_launch": table({k: (v[0] * 1e3 / launches, v[1] / launches) for k, v in prof.items()},
+                                                               work(4096 // launches, 2048 if which == "rafilix" else 4096, 1))}
+        s2.free()
+        model.free()
+        line[which] = res
+    line["value"] = line["rafilix"]["decode"]["tok_s"]
+    line["clocks"] = sampler.stop()
+    print(json.dumps(line), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -680,10 +892,15 @@ def main():
     ap.add_argument("--kernel-case", default="", choices=["", "gemm", "expert_forward"],
                     help="run only the tensor-core GEMM on the decode step's two largest shapes (gate|up rows, LM head) "
                          "through the op-level entry point and exit: the small program that ncu captures are taken from")
+    ap.add_argument("--stack", default="", choices=[""] + sorted(STACK_SIZES),
+                    help="measure a layer-list (Rafilix) model of this size beside a Qwen2 stack of equal size and exit")
     ap.add_argument("--traffic", type=float, default=None,
                     help="DRAM bytes per launch of the dominant kernel from an ncu capture, if known")
     a = ap.parse_args()
     a.warmup = max(a.warmup, 3)
+    if a.stack:
+        run_stack(a)
+        return
     if a.kernel_case == "expert_forward":
         run_expert_forward_case(a)
         return

@@ -137,7 +137,11 @@ def report_pair(rep, name, a, b, ha=None, hb=None):
         rep[name + "_hidden_l2_by_layer"] = [round(v, 4) for v in l2]
 
 
-def assert_bars(rep, targets, peaked):
+# logits distance of the reference from the oracle, measured on a B200 with the reference built, for runs without it
+RECORDED_FLOOR = {"0.5b iid": 2.7e-2, "1.5b": 4.5e-2, "3b": 3.7e-2}
+
+
+def assert_bars(rep, targets, peaked, recorded_floor=0.0):
     """The stated bars on the pairs in `targets` (each "ours_vs_..."), against the noise floor measured in the
     same test where it exceeds them: the distance between the reference and its rounding-exact restatement,
     the oracle ("oracle_vs_reference_*"), which is bf16 rounding noise and nothing else.
@@ -157,8 +161,9 @@ def assert_bars(rep, targets, peaked):
     layer 24, 1.8-2.0 % in relative L2; more for wider and deeper shapes). Every layer is held to
     max(1.5 x floor of that layer, 2 x that drift model) for the max-abs-normalised error and to three
     quarters of it for the relative L2 error; for the first layers that is below the stated 2e-2, and a
-    defect in a layer shows as tens of percent from that layer on."""
-    floor_logits = rep.get("oracle_vs_reference_logits", 0.0)
+    defect in a layer shows as tens of percent from that layer on.
+    recorded_floor: the logits floor where the reference was not built and cannot be measured in the test."""
+    floor_logits = rep.get("oracle_vs_reference_logits", recorded_floor)
     for t in targets:
         assert rep[t + "_logits"] <= max(TOL, 1.5 * floor_logits), (t, rep)
         rows = rep[t + "_rows"]
@@ -236,6 +241,10 @@ def test_config1_batched_decode(variant, tmp_path):
     s.capture_hidden(0)
     ours = {c: [lg[c].copy()] for c in check}
     forced_all = {c: (ref_picks[j, :N] if have_ref else rand[j]) for j, c in enumerate(check)}
+    if not have_ref:  # the one the oracle sees follows the oracle's own greedy stream
+        o0 = oracle.Oracle(d, P + N + 8, ep, 0.1)
+        forced_all[56] = o0.generate(prompts[56], N)
+        o0.close()
     tok = np.array(nxt, dtype=np.int32)
     for k in range(N):
         for c in check:
@@ -259,7 +268,8 @@ def test_config1_batched_decode(variant, tmp_path):
     if have_ref:
         report_pair(rep, "oracle_vs_reference", orc, ref_logits[0], oh, rh)
     print("PARITY config1", variant or "iid", rep)
-    assert_bars(rep, ["ours_vs_oracle"] + (["ours_vs_reference"] if have_ref else []), variant == "peaked")
+    assert_bars(rep, ["ours_vs_oracle"] + (["ours_vs_reference"] if have_ref else []), variant == "peaked",
+                0.0 if variant == "peaked" else RECORDED_FLOOR["0.5b iid"])
     s.free()
 
 
@@ -363,7 +373,7 @@ def _large_shape_case(shape, P_long, P_short, N_long, batch, ref_layers, tmp_pat
         e.free()
         m.free()
         print("PARITY", shape, f"first {ref_layers} layers" if ref_layers < L else "all layers", rep)
-        assert_bars(rep, targets, False)  # random teacher stream: near-ties excused, raw within 3 sigma of the floor
+        assert_bars(rep, targets, False, RECORDED_FLOOR[shape])  # random teacher stream: near-ties excused, raw within 3 sigma of the floor
         if ref_layers < L:  # (3)
             rep3 = {}
             m = tffn.qwen_load(d)
@@ -376,7 +386,7 @@ def _large_shape_case(shape, P_long, P_short, N_long, batch, ref_layers, tmp_pat
                 if k in rep:
                     rep3[k] = rep[k]
             print("PARITY", shape, "all layers", rep3)
-            assert_bars(rep3, ["ours_vs_oracle"], False)
+            assert_bars(rep3, ["ours_vs_oracle"], False, RECORDED_FLOOR[shape])
             e.free()
             m.free()
     finally:

@@ -664,7 +664,7 @@ const char* kclass_name(int c) {
     static const char* names[KC_COUNT] = {"embed_rows", "rmsnorm_rows", "gemm_tc:qkv", "attn_decode",
                                           "gemm_tc:o_proj", "gemm_tc:gate_up_swiglu", "gemm_tc:down", "gemm_tc:lm_head",
                                           "argmax_rows", "decode_advance", "bs1_qkv", "bs1_oproj", "bs1_ffn", "bs1_lmhead", "tp_all_reduce",
-                                          "residual_rows", "gemm:mixer_in", "qk_norm_rope", "gemm:low_rank", "delta_prep", "delta_scan",
+                                          "residual_rows", "gemm:mixer_in", "qk_norm_rope", "gemm:low_rank", "delta_prep", "delta_scan", "delta_out",
                                           "gemm:router", "moe_route", "moe_gather", "gemm:expert_up", "gemm:expert_down"};
     return (c >= 0 && c < KC_COUNT) ? names[c] : "?";
 }

@@ -126,7 +126,7 @@ struct Expert {
 enum KClass : int {
     KC_EMBED = 0, KC_RMSNORM, KC_GEMM_QKV, KC_ATTENTION, KC_GEMM_OPROJ, KC_GEMM_GATEUP, KC_GEMM_DOWN,
     KC_GEMM_LMHEAD, KC_ARGMAX, KC_ADVANCE, KC_BS1_QKV, KC_BS1_OPROJ, KC_BS1_FFN, KC_BS1_LMHEAD, KC_ALLREDUCE,
-    KC_ROWS, KC_GEMM_IN, KC_QK_ROPE, KC_GEMM_LOWRANK, KC_DELTA_PREP, KC_DELTA_SCAN, KC_GEMM_ROUTER, KC_ROUTE, KC_GATHER,
+    KC_ROWS, KC_GEMM_IN, KC_QK_ROPE, KC_GEMM_LOWRANK, KC_DELTA_PREP, KC_DELTA_SCAN, KC_DELTA_OUT, KC_GEMM_ROUTER, KC_ROUTE, KC_GATHER,
     KC_GEMM_UP, KC_GEMM_EXPERT_DOWN, KC_COUNT
 };
 const char* kclass_name(int c);
@@ -151,7 +151,7 @@ struct StackState {
     std::vector<RopeSpec> rope_specs;
     int64_t h_ld = 0, proj_ld = 0, ctx_ld = 0, decay_ld = 0, gate_ld = 0, delta_ld = 0, router_ld = 0, act_ld = 0;
     int max_top = 0, max_experts = 0, moe_layers = 0, max_tiles = 0;
-    DeviceBuffer proj, delta, qn, kn, v, g, bk, decay, gate;
+    DeviceBuffer proj, delta, qn, kn, v, g, bk, o, decay, gate;
     DeviceBuffer router, counts, pair, pair_w, pair_row, xg, act_e, y, tiles;
     DeviceBuffer seg_first, seg_count, ones;
 };

@@ -83,6 +83,7 @@ void Model::load_stack(const std::string& dir) {
             l.v_off = l.k_off + (int)pad8(nq);
             l.in_rows = l.v_off + (int)pad8((int64_t)s.kv_heads * s.vdim);
         } else {
+            if (s.conv > 32) throw Error(kErrUnsupported, "short convolutions of more than 32 taps are not supported");
             if (!delta_supported(s.dim, s.vdim)) throw Error(kErrUnsupported, "delta-rule heads wider than 256 are not supported");
             auto rank = [&](const char* t) {  // rows of a [rank, width] tensor
                 const TensorInfo& ti = st.get(p + t);
@@ -98,6 +99,7 @@ void Model::load_stack(const std::string& dir) {
             l.g1_off = l.a1_off + (int)pad8(l.a_rank);
             l.in_rows = l.g1_off + (int)pad8(l.g_rank);
         }
+        if (s.top > 64) throw Error(kErrUnsupported, "more than 64 experts per token");
         if (s.experts + s.identity > 1024) throw Error(kErrUnsupported, "more than 1024 experts in a layer");
         layout_layer(l, H, [&](DeviceBuffer&, size_t bytes) { total += Slab::padded(bytes); });
     }
@@ -260,6 +262,7 @@ void Session::alloc_stack(bool f32) {
         s.kn.alloc(T * qn * 4);
         s.g.alloc(T * gn * 4);
         s.v.alloc(T * vn * 4);
+        s.o.alloc(T * vn * 4);
         s.bk.alloc(T * heads * 8);
         s.decay.alloc(T * s.decay_ld * 4);
         s.gate.alloc(T * s.gate_ld * 4);
@@ -458,6 +461,7 @@ void Session::run_stack(int T, int n_logit_rows, bool logit_rows_are_all, bool d
             d.v = s.v.as<float>();
             d.g = s.g.as<float>();
             d.bk = s.bk.as<float>();
+            d.o = s.o.as<float>();
             d.out = ctx_.p;
             d.out_ld = ctx_ld;
             d.tok_seq = tok_seq;
@@ -466,8 +470,10 @@ void Session::run_stack(int T, int n_logit_rows, bool logit_rows_are_all, bool d
             d.seg_count = seg_count;
             d.max_slots = max_batch_;
             d.status = status;
+            const bool fuse_out = decode && cache.dimP <= 128;
             step(KC_DELTA_PREP, [&](unsigned long long* tl) { launch_delta_prep(d, f32, T, stream_, pdl, tl); });
-            step(KC_DELTA_SCAN, [&](unsigned long long* tl) { launch_delta_scan(d, f32, n_segs, stream_, pdl, tl); });
+            step(KC_DELTA_SCAN, [&](unsigned long long* tl) { launch_delta_scan(d, f32, n_segs, fuse_out, m_->num_sms, stream_, pdl, tl); });
+            if (!fuse_out) step(KC_DELTA_OUT, [&](unsigned long long* tl) { launch_delta_out(d, f32, T, stream_, pdl, tl); });
         }
         run_product(KC_GEMM_OPROJ, l.wo.as<bf16>(), ctx_ld, ctx_.p, ctx_ld, (int)nv, H, GEMM_STORE_F32, s.delta.p, s.delta_ld);
         rows.source = ROWS_DELTA;
@@ -475,24 +481,35 @@ void Session::run_stack(int T, int n_logit_rows, bool logit_rows_are_all, bool d
         rows.delta_ld = s.delta_ld;
         rows.post_w = l.norm1b.as<float>();
         rows.next_w = sp.experts > 0 ? l.norm2.as<float>() : after;
+        const int outs = sp.experts + sp.identity;
+        MoeRoute r;
+        r.logits = s.router.as<float>();
+        r.ld = s.router_ld;
+        r.correction = l.correction.as<float>();
+        r.experts = sp.experts;
+        r.identity = sp.identity;
+        r.top = sp.top;
+        r.counts = s.counts.as<int>() + (size_t)std::max(cache.moe, 0) * s.max_experts;
+        r.pair = s.pair.as<int2>();
+        r.pair_w = s.pair_w.as<float>();
+        // few rows: the row kernel routes as well
+        const bool routed = sp.experts > 0 && rows_can_route(T, H, outs);
+        if (routed) {
+            rows.router_w = l.router.as<bf16>();
+            rows.router_ld = s.h_ld;
+            rows.route = r;
+        }
         step(KC_ROWS, [&](unsigned long long* tl) { launch_residual_rows(rows, f32, T, stream_, pdl, tl); });
+        rows.router_w = nullptr;
 
         if (sp.experts > 0) {
-            const int outs = sp.experts + sp.identity, pairs = T * sp.top;
+            const int pairs = T * sp.top;
             const int tile = f32 ? kGemmF32Tile : gemm_group_tile((pairs + outs - 1) / outs);
             const int tiles = std::min(sp.experts, pairs) + pairs / tile;
-            run_product(KC_GEMM_ROUTER, l.router.as<bf16>(), s.h_ld, xn, s.h_ld, H, outs, GEMM_STORE_F32, s.router.p, s.router_ld);
-            MoeRoute r;
-            r.logits = s.router.as<float>();
-            r.ld = s.router_ld;
-            r.correction = l.correction.as<float>();
-            r.experts = sp.experts;
-            r.identity = sp.identity;
-            r.top = sp.top;
-            r.counts = s.counts.as<int>() + (size_t)cache.moe * s.max_experts;
-            r.pair = s.pair.as<int2>();
-            r.pair_w = s.pair_w.as<float>();
-            step(KC_ROUTE, [&](unsigned long long* tl) { launch_moe_route(r, T, stream_, pdl, tl); });
+            if (!routed) {
+                run_product(KC_GEMM_ROUTER, l.router.as<bf16>(), s.h_ld, xn, s.h_ld, H, outs, GEMM_STORE_F32, s.router.p, s.router_ld);
+                step(KC_ROUTE, [&](unsigned long long* tl) { launch_moe_route(r, T, stream_, pdl, tl); });
+            }
             MoeGather g;
             g.x = xn_.p;
             g.x_ld = s.h_ld;
@@ -515,6 +532,7 @@ void Session::run_stack(int T, int n_logit_rows, bool logit_rows_are_all, bool d
                 e.grp_tiles = tiles;
                 e.grp_bn = tile;
                 e.grp_count = sp.experts;
+                e.grp_rows_hint = std::min(tiles, std::max(std::min(sp.experts, pairs), pairs / tile));
                 gemm(e, cls, pdl);
             };
             const int64_t ffp = pad8(sp.ff);

@@ -743,7 +743,8 @@ int launch_bn(const GemmCall& c, const GemmWorkspace& ws, cudaStream_t stream, i
         return (int)cudaErrorInvalidValue;
     p.grp = c.grp;
     const int total_kb = p.kblocks[0] + p.kblocks[1];
-    const int tiles = n_tiles * t_tiles * nprob;
+    // grouped: the grid has room for the worst case, the split policy goes by one tile per group that can have rows
+    const int tiles = c.grp && c.grp_rows_hint > 0 ? n_tiles * c.grp_rows_hint : n_tiles * t_tiles * nprob;
     p.t_tiles = t_tiles;
     // K splits = cluster size (1, 2, 4, 8 or 16). Inside a decode step one CTA takes in roughly one
     // stage (a 16 KB weight box and its activation box) per 0.5 us whatever the ring depth, about 50 GB/s
@@ -877,6 +878,9 @@ int launch_gemm(const GemmCall& c, const GemmWorkspace& ws, cudaStream_t stream,
             n_tiles * 8 <= ws.num_sms)
             return launch_bn<32>(c, ws, stream, kMaxSplits);
     }
+    // One row tile (a router): with wide token tiles a handful of CTAs would carry the whole launch and split it along
+    // K, exchanging planes that are mostly padding; narrow token tiles spread it over the SMs instead.
+    if (c.N <= BM && c.T > 64 && c.mode == GEMM_STORE_F32 && !c.out2 && c.op[1].K <= 0) return launch_bn<64>(c, ws, stream, force_splits);
     if (c.T <= 16) return launch_bn<16>(c, ws, stream, force_splits);
     if (c.T <= 32) return launch_bn<32>(c, ws, stream, force_splits);
     if (c.T <= 64) return launch_bn<64>(c, ws, stream, force_splits);

@@ -84,6 +84,7 @@ struct GemmCall {
     // (written by an earlier kernel, see GroupTile). op[1], op2 and GEMM_QKV are not available with it.
     const struct GroupTile* grp;
     int grp_tiles, grp_bn, grp_count;  // grp_count: groups in W
+    int grp_rows_hint;                 // tiles that will be in use, about (0: all)
 };
 struct GroupTile {
     int group;           // -1: this tile and all later ones are unused
@@ -212,6 +213,17 @@ void launch_attention_prefill(const float* q, KvView kv, int layer, const int* t
 
 // ------------------------------------------------------------------ layers with an fp32 residual stream
 // "f32" below selects the storage type of activations and cache: fp32 in a session that computes in fp32, else bf16.
+// A router's scores: softmax of fp32 logits over experts and identity outputs; the `top` largest of score + correction
+// are chosen, lowest index first among equals
+struct MoeRoute {
+    const float* logits;      // [T][ld], experts + identity columns
+    int64_t ld;
+    const float* correction;  // [experts + identity]
+    int experts, identity, top;
+    int* counts;              // [experts], zero before the launch
+    int2* pair;               // [T][top]: expert (-1: identity) and the pair's place within it
+    float* pair_w;            // [T][top] softmax score (without the correction)
+};
 enum RowSource : int { ROWS_KEEP = 0, ROWS_EMBED, ROWS_DELTA, ROWS_MOE };
 // One pass over the residual stream per sublayer: x = table[token] | x + norm(delta) * post_w | x + norm(sum of the
 // chosen experts' outputs) * post_w, then out = norm(x) * next_w. Norm: v / sqrt(mean(v^2) + eps). All in fp32.
@@ -237,8 +249,14 @@ struct ResidualRows {
     void* out;                // [.][out_ld]
     int64_t out_ld;
     const int* row_idx;       // with ROWS_KEEP: out row r = norm of x row row_idx[r]
+    // Optional (rows_can_route): the router of the mixture that reads `out`, in the same pass. route.logits is not used.
+    const bf16* router_w;     // [experts + identity][router_ld]
+    int64_t router_ld;
+    MoeRoute route;
 };
 int stack_rows_prepare();
+// few rows and a router small enough to be read once per row
+inline bool rows_can_route(int rows, int H, int outs) { return rows <= 128 && H % 8 == 0 && (size_t)H * outs * 2 <= (256u << 10); }
 void launch_residual_rows(const ResidualRows& a, bool f32, int rows, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
 
 // q|k|v rows of one projection -> per-head norm of q and k (weights shared by the heads), rotation of neighbouring
@@ -285,6 +303,7 @@ struct DeltaRule {
     float *v;                 // [T][heads][vdimP]
     float *g;                 // [T][heads][dimP] decays
     float *bk;                // [T][heads][2]: beta, k . q
+    float* o;                 // [T][heads][vdimP] raw output rows
     void* out;                // [T][out_ld]
     int64_t out_ld;
     const int *tok_seq, *tok_pos;
@@ -293,22 +312,17 @@ struct DeltaRule {
     int* status;
 };
 void launch_delta_prep(const DeltaRule& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
-void launch_delta_scan(const DeltaRule& a, bool f32, int n_segs, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
+// fused (decode; heads of up to 128 key channels): the scan writes the normed and gated rows; otherwise raw rows to
+// `o`, then launch_delta_out
+void launch_delta_scan(const DeltaRule& a, bool f32, int n_segs, bool fused, int num_sms, cudaStream_t s, bool pdl,
+                       unsigned long long* tl = nullptr);
+void launch_delta_out(const DeltaRule& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
 int delta_prepare();
 int delta_padded_dim(int dim);  // dimP
 inline bool delta_supported(int dim, int vdim) { return dim <= 256 && vdim <= 256; }
 
 // ------------------------------------------------------------------ mixture of experts
 int moe_prepare();
-struct MoeRoute {
-    const float* logits;      // [T][ld], experts + identity columns
-    int64_t ld;
-    const float* correction;  // [experts + identity]
-    int experts, identity, top;
-    int* counts;              // [experts], zero before the launch
-    int2* pair;               // [T][top]: expert (-1: identity) and the pair's place within it
-    float* pair_w;            // [T][top] softmax score (without the correction)
-};
 void launch_moe_route(const MoeRoute& a, int T, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
 struct MoeGather {
     const void* x;            // [T][x_ld]

@@ -5,6 +5,7 @@
 #include "act.cuh"
 #include "launch.h"
 #include "ptx.cuh"
+#include "route.cuh"
 
 namespace tffn {
 
@@ -22,49 +23,10 @@ __global__ void __launch_bounds__(kRouteWarps * 32) k_moe_route(const MoeRoute a
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = a.experts + a.identity;
     const int t = blockIdx.x * kRouteWarps + warp;
     if (t < T) {
-        float* s = route_smem + (size_t)warp * 2 * n;  // softmax scores, then what the choice is made by
-        float* choice = s + n;
+        float* s = route_smem + (size_t)warp * 2 * n;
         const float* z = a.logits + (size_t)t * a.ld;
-        float mx = -INFINITY;
-        for (int i = lane; i < n; i += 32) {
-            const float v = __ldcg(z + i);
-            s[i] = v;
-            mx = fmaxf(mx, v);
-        }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-        float sum = 0.f;
-        for (int i = lane; i < n; i += 32) {
-            const float e = expf(s[i] - mx);
-            s[i] = e;
-            sum += e;
-        }
-        const float inv = 1.f / warp_sum(sum);
-        for (int i = lane; i < n; i += 32) {
-            s[i] *= inv;
-            choice[i] = s[i] + __ldg(a.correction + i);
-        }
-        for (int j = 0; j < a.top; ++j) {  // lanes own strided entries: no exchange through shared memory is needed
-            float best = -INFINITY;
-            int bi = 0x7fffffff;
-            for (int i = lane; i < n; i += 32)
-                if (choice[i] > best) { best = choice[i]; bi = i; }
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
-                const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-                const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-                if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
-            }
-            if (bi >= n) bi = j;  // no finite score is left (NaN inputs): stay in range
-            if ((bi & 31) == lane) {
-                const float w = s[bi];
-                choice[bi] = -INFINITY;
-                int2 p = make_int2(-1, 0);
-                if (bi < a.experts) p = make_int2(bi, atomicAdd(a.counts + bi, 1));
-                a.pair[(size_t)t * a.top + j] = p;
-                a.pair_w[(size_t)t * a.top + j] = w;
-            }
-        }
+        for (int i = lane; i < n; i += 32) s[i] = __ldcg(z + i);
+        route_token(a, t, s, s + n, lane);
     }
     if (threadIdx.x == 0) tl_mark(tl, 2);
 }
@@ -83,6 +45,9 @@ __global__ void __launch_bounds__(kGatherThreads) k_moe_gather(const MoeGather a
     if (threadIdx.x == 0) tl_mark(tl, 1);
     const int tid = threadIdx.x, lane = tid & 31;
     const bool table = (int)blockIdx.x == T;
+    int2 mine = make_int2(-1, 0);  // threads from 32 on: the token's pairs, requested before the prefix sums are formed
+    const int jj = tid - 32;
+    if (!table && jj >= 0 && jj < a.top) mine = __ldcg(a.pair + (size_t)blockIdx.x * a.top + jj);
     if (tid < 32) {
         int rows = 0, tiles = 0;
         for (int e0 = 0; e0 < a.experts; e0 += 32) {
@@ -113,15 +78,19 @@ __global__ void __launch_bounds__(kGatherThreads) k_moe_gather(const MoeGather a
         for (int i = tile0[a.experts] + tid; i < a.max_tiles; i += kGatherThreads) a.tiles[i] = GroupTile{-1, 0, 0, 0};
     } else {
         const int t = blockIdx.x;
+        int* dest = tile0;  // [top], at most as many as threads 32 .. 127 (top <= 96)
+        if (jj >= 0 && jj < a.top) {
+            const int row = mine.x < 0 ? -1 : first[mine.x] + mine.y;
+            a.pair_row[(size_t)t * a.top + jj] = row;
+            dest[jj] = row;
+        }
         const uint4* src = (const uint4*)((const A*)a.x + (size_t)t * a.x_ld);
         const int n16 = (int)(a.x_ld * sizeof(A) / 16);  // rows are padded to 16 bytes
-        for (int j = 0; j < a.top; ++j) {
-            const int2 p = __ldcg(a.pair + (size_t)t * a.top + j);
-            const int row = p.x < 0 ? -1 : first[p.x] + p.y;
-            if (tid == 0) a.pair_row[(size_t)t * a.top + j] = row;
-            if (row < 0) continue;
-            uint4* dst = (uint4*)((A*)a.xg + (size_t)row * a.x_ld);
-            for (int i = tid; i < n16; i += kGatherThreads) dst[i] = __ldcg(src + i);
+        __syncthreads();
+        for (int i = tid; i < n16; i += kGatherThreads) {
+            const uint4 v = __ldcg(src + i);
+            for (int j = 0; j < a.top; ++j)
+                if (dest[j] >= 0) ((uint4*)((A*)a.xg + (size_t)dest[j] * a.x_ld))[i] = v;
         }
     }
     if (tid == 0) tl_mark(tl, 2);
@@ -142,7 +111,7 @@ void launch_moe_route(const MoeRoute& a, int T, cudaStream_t s, bool pdl, unsign
 }
 
 void launch_moe_gather(const MoeGather& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl) {
-    const size_t smem = (size_t)(2 * a.experts + 1) * 4;
+    const size_t smem = (size_t)(a.experts + (a.experts + 1 > a.top ? a.experts + 1 : a.top)) * 4;
     if (f32) launch_k(k_moe_gather<float>, dim3(T + 1), dim3(kGatherThreads), smem, s, pdl, a, T, tl);
     else launch_k(k_moe_gather<bf16>, dim3(T + 1), dim3(kGatherThreads), smem, s, pdl, a, T, tl);
 }

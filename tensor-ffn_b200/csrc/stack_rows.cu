@@ -5,11 +5,169 @@
 #include "act.cuh"
 #include "launch.h"
 #include "ptx.cuh"
+#include "route.cuh"
 
 namespace tffn {
 
 namespace {
 
+__device__ __forceinline__ void load4(const float* p, float (&v)[4]) {
+    const float4 q = __ldcg((const float4*)p);
+    v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+}
+__device__ __forceinline__ void load4(const bf16* p, float (&v)[4]) {
+    const uint2 q = __ldcg((const uint2*)p);
+    v[0] = bf16_lo(q.x); v[1] = bf16_hi(q.x); v[2] = bf16_lo(q.y); v[3] = bf16_hi(q.y);
+}
+__device__ __forceinline__ void store4(float* p, const float (&v)[4]) { *(float4*)p = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(bf16* p, const float (&v)[4]) {
+    *(uint2*)p = make_uint2((uint32_t)bf16_bits(v[0]) | ((uint32_t)bf16_bits(v[1]) << 16),
+                            (uint32_t)bf16_bits(v[2]) | ((uint32_t)bf16_bits(v[3]) << 16));
+}
+__device__ __forceinline__ float as_stored(float v, const float*) { return v; }
+__device__ __forceinline__ float as_stored(float v, const bf16*) { return bf16_round(v); }
+
+// The pass over rows whose width is a multiple of 4: a thread keeps its IT groups of four columns in registers from the
+// first load to the last store, all loads of a phase in flight together.
+template <typename A, int IT>
+__global__ void __launch_bounds__(512) k_residual_rows4(const ResidualRows a, unsigned long long* tl) {
+    extern __shared__ float rows4_smem[];  // with a router: the row as stored [H], logits [n], scratch [n]
+    __shared__ float red[32];
+    if (threadIdx.x == 0) tl_mark(tl, 0);
+    pdl_launch_dependents();
+    const int H = a.H, r = blockIdx.x, n = blockDim.x, tid = threadIdx.x;
+    // norm weights do not depend on earlier kernels
+    float pw[IT][4], nw[IT][4];
+#pragma unroll
+    for (int k = 0; k < IT; ++k) {
+        const int i = (tid + k * n) * 4;
+        if (i < H && a.source >= ROWS_DELTA) load4(a.post_w + i, pw[k]);
+        if (i < H && a.next_w) load4(a.next_w + i, nw[k]);
+    }
+    pdl_wait();
+    if (tid == 0) tl_mark(tl, 1);
+    const int src = (a.source == ROWS_KEEP && a.row_idx) ? __ldcg(a.row_idx + r) : r;
+    float* xr = a.x + (size_t)src * H;
+    A* out = (A*)a.out + (size_t)r * a.out_ld;
+    float x[IT][4], ss = 0.f;
+    if (a.source == ROWS_EMBED) {
+        int tok = __ldcg(a.tokens + r);
+        if (tok < 0 || tok >= a.V) {
+            if (tid == 0) dev_fail(a.status, DEV_ERR_BOUNDS);
+            tok = 0;
+        }
+        const bf16* e = a.table + (size_t)tok * a.table_ld;
+#pragma unroll
+        for (int k = 0; k < IT; ++k) {
+            const int i = (tid + k * n) * 4;
+            if (i < H) load4(e + i, x[k]);
+        }
+    } else {
+#pragma unroll
+        for (int k = 0; k < IT; ++k) {
+            const int i = (tid + k * n) * 4;
+            if (i < H) load4(xr + i, x[k]);
+        }
+    }
+    if (a.source >= ROWS_DELTA) {
+        float d[IT][4], sd = 0.f;
+        if (a.source == ROWS_DELTA) {
+#pragma unroll
+            for (int k = 0; k < IT; ++k) {
+                const int i = (tid + k * n) * 4;
+                if (i < H) load4(a.delta + (size_t)r * a.delta_ld + i, d[k]);
+            }
+        } else {
+#pragma unroll
+            for (int k = 0; k < IT; ++k) d[k][0] = d[k][1] = d[k][2] = d[k][3] = 0.f;
+            for (int j0 = 0; j0 < a.top; j0 += 4) {
+                const A* from[4];
+                float w[4];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const bool on = j0 + j < a.top;
+                    const int row = on ? __ldcg(a.pair_row + (size_t)r * a.top + j0 + j) : -1;
+                    w[j] = on ? __ldcg(a.pair_w + (size_t)r * a.top + j0 + j) : 0.f;
+                    from[j] = row < 0 ? out : (const A*)a.y + (size_t)row * a.y_ld;
+                }
+#pragma unroll
+                for (int k = 0; k < IT; ++k) {
+                    const int i = (tid + k * n) * 4;
+                    if (i < H) {
+                        float v[4][4];
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) load4(from[j] + i, v[j]);
+#pragma unroll
+                        for (int j = 0; j < 4; ++j)
+#pragma unroll
+                            for (int c = 0; c < 4; ++c) d[k][c] += w[j] * v[j][c];
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < IT; ++k)
+            if ((tid + k * n) * 4 < H) sd += d[k][0] * d[k][0] + d[k][1] * d[k][1] + d[k][2] * d[k][2] + d[k][3] * d[k][3];
+        sd = block_sum(sd, red);
+        const float dinv = 1.f / sqrtf(sd / (float)H + a.eps);
+#pragma unroll
+        for (int k = 0; k < IT; ++k)
+            if ((tid + k * n) * 4 < H) {
+#pragma unroll
+                for (int c = 0; c < 4; ++c) x[k][c] += d[k][c] * dinv * pw[k][c];
+            }
+    }
+#pragma unroll
+    for (int k = 0; k < IT; ++k) {
+        const int i = (tid + k * n) * 4;
+        if (i < H) {
+            if (a.source != ROWS_KEEP) store4(xr + i, x[k]);
+            ss += x[k][0] * x[k][0] + x[k][1] * x[k][1] + x[k][2] * x[k][2] + x[k][3] * x[k][3];
+        }
+    }
+    if (a.next_w) {
+        ss = block_sum(ss, red);
+        const float inv = 1.f / sqrtf(ss / (float)H + a.eps);
+#pragma unroll
+        for (int k = 0; k < IT; ++k) {
+            const int i = (tid + k * n) * 4;
+            if (i < H) {
+                float v[4];
+#pragma unroll
+                for (int c = 0; c < 4; ++c) v[c] = x[k][c] * inv * nw[k][c];
+                store4(out + i, v);
+                if (a.router_w) {
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) rows4_smem[i + c] = as_stored(v[c], out);
+                }
+            }
+        }
+    }
+    if (a.router_w) {
+        // logits: one warp per output, the row from shared memory, 16 bytes of weights per lane and step (H % 8 == 0)
+        const int warp = tid >> 5, lane = tid & 31, outs = a.route.experts + a.route.identity;
+        float* z = rows4_smem + H;
+        __syncthreads();
+        for (int e = warp; e < outs; e += n >> 5) {
+            const bf16* w = a.router_w + (size_t)e * a.router_ld;
+            float acc = 0.f;
+#pragma unroll 4
+            for (int i = lane * 8; i < H; i += 256) {
+                const uint4 q = __ldg((const uint4*)(w + i));
+                const float4 x0 = *(const float4*)(rows4_smem + i), x1 = *(const float4*)(rows4_smem + i + 4);
+                acc += bf16_lo(q.x) * x0.x + bf16_hi(q.x) * x0.y + bf16_lo(q.y) * x0.z + bf16_hi(q.y) * x0.w;
+                acc += bf16_lo(q.z) * x1.x + bf16_hi(q.z) * x1.y + bf16_lo(q.w) * x1.z + bf16_hi(q.w) * x1.w;
+            }
+            acc = warp_sum(acc);
+            if (lane == 0) z[e] = acc;
+        }
+        __syncthreads();
+        if (warp == 0) route_token(a.route, r, z, z + outs, lane);
+    }
+    if (tid == 0) tl_mark(tl, 2);
+}
+
+// the same for any width, one column at a time through shared memory (no router)
 template <typename A>
 __global__ void __launch_bounds__(512) k_residual_rows(const ResidualRows a, unsigned long long* tl) {
     extern __shared__ float rows_smem[];
@@ -92,6 +250,21 @@ __global__ void __launch_bounds__(512) k_residual_rows(const ResidualRows a, uns
     if (tid == 0) tl_mark(tl, 2);
 }
 
+__device__ __forceinline__ void load_pair(const float* p, float& x, float& y) {
+    const float2 v = __ldcg((const float2*)p);
+    x = v.x;
+    y = v.y;
+}
+__device__ __forceinline__ void load_pair(const bf16* p, float& x, float& y) {
+    const uint32_t v = __ldcg((const unsigned int*)p);
+    x = bf16_lo(v);
+    y = bf16_hi(v);
+}
+__device__ __forceinline__ void store_pair(float* p, float x, float y) { *(float2*)p = make_float2(x, y); }
+__device__ __forceinline__ void store_pair(bf16* p, float x, float y) {
+    *(uint32_t*)p = (uint32_t)bf16_bits(x) | ((uint32_t)bf16_bits(y) << 16);
+}
+
 // one warp per (token, head): heads 0 .. nh-1 are queries, then the keys, then the values
 constexpr int kQkWarps = 4;
 template <typename A>
@@ -116,16 +289,30 @@ __global__ void __launch_bounds__(kQkWarps * 32) k_qk_norm_rope(const QkNormRope
             if (lane == 0) dev_fail(a.status, DEV_ERR_BOUNDS);
         } else if (kind == 2) {
             A* dst = (A*)a.kv.v_pool + (((size_t)pg * nkv + head) * kPageTokens + pos % kPageTokens) * a.kv.vd;
-            for (int i = lane; i < dim; i += 32) act_store(dst + i, act_load(src + i));
+            if ((dim & 1) == 0) {
+                for (int i = lane * 2; i < dim; i += 64) {
+                    float x, y;
+                    load_pair(src + i, x, y);
+                    store_pair(dst + i, x, y);
+                }
+            } else {
+                for (int i = lane; i < dim; i += 32) act_store(dst + i, act_load(src + i));
+            }
         } else {
             // lane = pair (2i, 2i + 1)
             constexpr int MP = 8;  // heads of up to 512
+            const bool even = (dim & 1) == 0;
             float u0[MP], u1[MP], ss = 0.f;
 #pragma unroll
             for (int j = 0; j < MP; ++j) {
                 const int i = 2 * (lane + 32 * j);
-                u0[j] = i < dim ? act_load(src + i) : 0.f;
-                u1[j] = i + 1 < dim ? act_load(src + i + 1) : 0.f;
+                u0[j] = u1[j] = 0.f;
+                if (i + 1 < dim && even) {
+                    load_pair(src + i, u0[j], u1[j]);
+                } else {
+                    if (i < dim) u0[j] = act_load(src + i);
+                    if (i + 1 < dim) u1[j] = act_load(src + i + 1);
+                }
                 ss += u0[j] * u0[j] + u1[j] * u1[j];
             }
             const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dim + a.eps);
@@ -146,8 +333,7 @@ __global__ void __launch_bounds__(kQkWarps * 32) k_qk_norm_rope(const QkNormRope
                     if (kind == 0) {
                         *(float2*)(qd + i) = make_float2(x, y);
                     } else {
-                        act_store(kdst + i, x);
-                        act_store(kdst + i + 1, y);
+                        store_pair(kdst + i, x, y);
                     }
                 }
             }
@@ -158,11 +344,27 @@ __global__ void __launch_bounds__(kQkWarps * 32) k_qk_norm_rope(const QkNormRope
 
 constexpr int kRowsMaxSmem = 128 * 1024;
 
+template <typename A, int IT>
+cudaError_t rows4_attrs() {
+    cudaError_t e = cudaFuncSetAttribute(k_residual_rows4<A, IT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kRowsMaxSmem);
+    return e == cudaSuccess ? prefer_max_shared(k_residual_rows4<A, IT>) : e;
+}
+template <typename A>
+cudaError_t rows4_attrs_all() {
+    cudaError_t e = rows4_attrs<A, 1>();
+    if (e == cudaSuccess) e = rows4_attrs<A, 2>();
+    if (e == cudaSuccess) e = rows4_attrs<A, 4>();
+    if (e == cudaSuccess) e = rows4_attrs<A, 8>();
+    return e;
+}
+
 }  // namespace
 
 int stack_rows_prepare() {
     cudaError_t e = cudaFuncSetAttribute(k_residual_rows<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, kRowsMaxSmem);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(k_residual_rows<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, kRowsMaxSmem);
+    if (e == cudaSuccess) e = rows4_attrs_all<bf16>();
+    if (e == cudaSuccess) e = rows4_attrs_all<float>();
     if (e == cudaSuccess) e = prefer_max_shared(k_residual_rows<bf16>);
     if (e == cudaSuccess) e = prefer_max_shared(k_residual_rows<float>);
     if (e == cudaSuccess) e = prefer_max_shared(k_qk_norm_rope<bf16>);
@@ -170,11 +372,25 @@ int stack_rows_prepare() {
     return (int)e;
 }
 
+template <typename A>
+static void launch_rows(const ResidualRows& a, int rows, cudaStream_t s, bool pdl, unsigned long long* tl) {
+    if (a.H % 4) {
+        const int threads = a.H <= 512 ? 128 : (a.H <= 2048 ? 256 : 512);
+        launch_k(k_residual_rows<A>, dim3(rows), dim3(threads), (size_t)a.H * 8, s, pdl, a, tl);
+        return;
+    }
+    const int groups = a.H / 4;
+    const size_t smem = a.router_w ? (size_t)(a.H + 2 * (a.route.experts + a.route.identity)) * 4 : 0;
+    const int per = groups <= 256 ? 1 : groups <= 1024 ? 2 : groups <= 2048 ? 4 : 8;
+    const dim3 grid(rows), block(((groups + per - 1) / per + 31) / 32 * 32);
+    if (per == 1) launch_k(k_residual_rows4<A, 1>, grid, block, smem, s, pdl, a, tl);
+    else if (per == 2) launch_k(k_residual_rows4<A, 2>, grid, block, smem, s, pdl, a, tl);
+    else if (per == 4) launch_k(k_residual_rows4<A, 4>, grid, block, smem, s, pdl, a, tl);
+    else launch_k(k_residual_rows4<A, 8>, grid, block, smem, s, pdl, a, tl);
+}
 void launch_residual_rows(const ResidualRows& a, bool f32, int rows, cudaStream_t s, bool pdl, unsigned long long* tl) {
-    const int threads = a.H <= 512 ? 128 : (a.H <= 2048 ? 256 : 512);
-    const size_t smem = (size_t)a.H * 8;
-    if (f32) launch_k(k_residual_rows<float>, dim3(rows), dim3(threads), smem, s, pdl, a, tl);
-    else launch_k(k_residual_rows<bf16>, dim3(rows), dim3(threads), smem, s, pdl, a, tl);
+    if (f32) launch_rows<float>(a, rows, s, pdl, tl);
+    else launch_rows<bf16>(a, rows, s, pdl, tl);
 }
 
 void launch_qk_norm_rope(const QkNormRope& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl) {

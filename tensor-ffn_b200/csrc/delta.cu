@@ -47,6 +47,8 @@ __device__ __forceinline__ void load_v(const bf16* p, float (&x)[V]) {
 // nowhere (before the sequence). Bit lag of the masks; every lane of the warp calls it.
 struct ConvSource {
     uint32_t rows, ring;
+    bool inside;  // all of them rows
+    int place;    // this lane's lag: its place in the ring
 };
 __device__ __forceinline__ ConvSource conv_source(const DeltaRule& a, int t, int seq, int pos, int lane) {
     const int lag = lane;
@@ -55,6 +57,8 @@ __device__ __forceinline__ ConvSource conv_source(const DeltaRule& a, int t, int
     ConvSource s;
     s.rows = __ballot_sync(0xffffffffu, row);
     s.ring = __ballot_sync(0xffffffffu, in_seq && !row);
+    s.inside = __popc(s.rows) == a.taps;
+    s.place = in_seq && !row ? (pos - lag) % (a.taps - 1) : 0;  // lag 0 is always a row, so taps > 1 here
     return s;
 }
 
@@ -68,33 +72,63 @@ __device__ __forceinline__ void conv_silu(const DeltaRule& a, const ConvSource& 
     for (int i = 0; i < NI; ++i)
 #pragma unroll
         for (int v = 0; v < V; ++v) y[i][v] = 0.f;
-    for (int l0 = R; l0 >= 0; l0 -= 4) {  // oldest tap first
-        float x[4][NI][V], w[4][NI][V];
+    const A* row0 = (const A*)a.proj + (size_t)t * a.proj_ld + col;
+    const float* w0 = a.conv + chan;
+    if (cs.inside) {  // every input is a row of this launch
+        for (int l0 = R; l0 >= 0; l0 -= 4) {  // oldest tap first
+            float x[4][NI][V], w[4][NI][V];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const int lag = l0 - j;
-            const bool row = lag >= 0 && ((cs.rows >> lag) & 1u), ring = lag >= 0 && ((cs.ring >> lag) & 1u);
-            const A* src = (const A*)a.proj + (size_t)(row ? t - lag : 0) * a.proj_ld + col;
-            const float* old = a.ring + (size_t)seq * a.ring_stride + (size_t)(ring ? (pos - lag) % R : 0) * C + chan;
-            const float* wt = a.conv + (size_t)(lag >= 0 ? R - lag : 0) * C + chan;
+            for (int j = 0; j < 4; ++j) {
+                const int lag = l0 - j;
+                const A* src = row0 - (ptrdiff_t)lag * a.proj_ld;
+                const float* wt = w0 + (ptrdiff_t)(R - lag) * C;
 #pragma unroll
-            for (int i = 0; i < NI; ++i) {
-                const int d = (lane + 32 * i) * V;
+                for (int i = 0; i < NI; ++i) {
+                    const int d = (lane + 32 * i) * V;
 #pragma unroll
-                for (int v = 0; v < V; ++v) x[j][i][v] = w[j][i][v] = 0.f;
-                if (d < dim) {
-                    if (row) load_v<V>(src + d, x[j][i]);
-                    else if (ring) load_v<V>(old + d, x[j][i]);
-                    if (row || ring) load_v<V>(wt + d, w[j][i]);
+                    for (int v = 0; v < V; ++v) x[j][i][v] = w[j][i][v] = 0.f;
+                    if (lag >= 0 && d < dim) {
+                        load_v<V>(src + d, x[j][i]);
+                        load_v<V>(wt + d, w[j][i]);
+                    }
                 }
             }
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int i = 0; i < NI; ++i)
+#pragma unroll
+                    for (int v = 0; v < V; ++v) y[i][v] += w[j][i][v] * x[j][i][v];
         }
+    } else {
+        for (int l0 = R; l0 >= 0; l0 -= 4) {
+            float x[4][NI][V], w[4][NI][V];
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
+            for (int j = 0; j < 4; ++j) {
+                const int lag = l0 - j;
+                const bool row = lag >= 0 && ((cs.rows >> lag) & 1u), ring = lag >= 0 && ((cs.ring >> lag) & 1u);
+                const A* src = row0 - (ptrdiff_t)(row ? lag : 0) * a.proj_ld;
+                const float* old = a.ring + (size_t)seq * a.ring_stride + (size_t)__shfl_sync(0xffffffffu, cs.place, lag & 31) * C + chan;
+                const float* wt = w0 + (ptrdiff_t)(lag >= 0 ? R - lag : 0) * C;
 #pragma unroll
-            for (int i = 0; i < NI; ++i)
+                for (int i = 0; i < NI; ++i) {
+                    const int d = (lane + 32 * i) * V;
 #pragma unroll
-                for (int v = 0; v < V; ++v) y[i][v] += w[j][i][v] * x[j][i][v];
+                    for (int v = 0; v < V; ++v) x[j][i][v] = w[j][i][v] = 0.f;
+                    if (d < dim) {
+                        if (row) load_v<V>(src + d, x[j][i]);
+                        else if (ring) load_v<V>(old + d, x[j][i]);
+                        if (row || ring) load_v<V>(wt + d, w[j][i]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int i = 0; i < NI; ++i)
+#pragma unroll
+                    for (int v = 0; v < V; ++v) y[i][v] += w[j][i][v] * x[j][i][v];
+        }
     }
 #pragma unroll
     for (int i = 0; i < NI; ++i)
@@ -108,14 +142,13 @@ __device__ __forceinline__ void store_v(float* p, const float (&x)[V]) {
 }
 
 template <typename A, int V, int NI>
-__global__ void __launch_bounds__(kPrepWarps * 32) k_delta_prep(const DeltaRule a, int T, unsigned long long* tl) {
+__global__ void __launch_bounds__(kPrepWarps * 32) k_delta_prep(const DeltaRule a, unsigned long long* tl) {
     if (threadIdx.x == 0) tl_mark(tl, 0);
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31;
-    const long long unit = (long long)blockIdx.x * kPrepWarps + (threadIdx.x >> 5);
-    const int G = a.kv_heads, H = a.heads, per_tok = G + H;
-    const bool on = unit < (long long)T * per_tok;
-    const int t = on ? (int)(unit / per_tok) : 0, u = (int)(unit % per_tok);
+    const int G = a.kv_heads, H = a.heads;
+    const int t = blockIdx.y, u = blockIdx.x * kPrepWarps + (threadIdx.x >> 5);
+    const bool on = u < G + H;
     // slots and positions are older than the step's first kernel
     const int seq = __ldcg(a.tok_seq + t), pos = __ldcg(a.tok_pos + t);
     const ConvSource cs = conv_source(a, t, seq, pos, lane);
@@ -317,26 +350,44 @@ __global__ void __launch_bounds__(NT) k_delta_scan(const DeltaRule a, int cols, 
         __syncthreads();
         const float* buf = scan_buf + (size_t)(tile & 1) * kScanTokens * tokf;
         const int n = min(kScanTokens, count - tile * kScanTokens);
+        // The token's vectors in registers; with room for them, the next token's are requested before this token's sums
+        // are exchanged, so that the exchange hides the shared-memory latency.
+        constexpr bool AHEAD = !FUSED && J <= 2;
+        ulonglong2 q4[J], k4[J], g4[J];
+        auto vectors = [&](int k) {
+            const float* tok = buf + (size_t)k * tokf;
+#pragma unroll
+            for (int j = 0; j < J; ++j) {
+                const int d = 4 * (r + 8 * j);
+                q4[j] = *(const ulonglong2*)(tok + d);
+                k4[j] = *(const ulonglong2*)(tok + dimP + d);
+                g4[j] = *(const ulonglong2*)(tok + 2 * dimP + d);
+            }
+        };
+        if (AHEAD) vectors(0);
         for (int k = 0; k < n; ++k) {
             const float* tok = buf + (size_t)k * tokf;
+            if (!AHEAD) vectors(k);
             f32x2 t2[C], w2[C];
 #pragma unroll
             for (int c = 0; c < C; ++c) t2[c] = w2[c] = 0ull;
 #pragma unroll
             for (int j = 0; j < J; ++j) {
-                const int d = 4 * (r + 8 * j);
-                const ulonglong2 q4 = *(const ulonglong2*)(tok + d);
-                const ulonglong2 k4 = *(const ulonglong2*)(tok + dimP + d);
-                const ulonglong2 g4 = *(const ulonglong2*)(tok + 2 * dimP + d);
 #pragma unroll
                 for (int c = 0; c < C; ++c) {
-                    S[c][j][0] = mul2(S[c][j][0], g4.x);
-                    S[c][j][1] = mul2(S[c][j][1], g4.y);
-                    t2[c] = fma2(S[c][j][0], k4.x, t2[c]);
-                    w2[c] = fma2(S[c][j][0], q4.x, w2[c]);
-                    t2[c] = fma2(S[c][j][1], k4.y, t2[c]);
-                    w2[c] = fma2(S[c][j][1], q4.y, w2[c]);
+                    S[c][j][0] = mul2(S[c][j][0], g4[j].x);
+                    S[c][j][1] = mul2(S[c][j][1], g4[j].y);
+                    t2[c] = fma2(S[c][j][0], k4[j].x, t2[c]);
+                    w2[c] = fma2(S[c][j][0], q4[j].x, w2[c]);
+                    t2[c] = fma2(S[c][j][1], k4[j].y, t2[c]);
+                    w2[c] = fma2(S[c][j][1], q4[j].y, w2[c]);
                 }
+            }
+            ulonglong2 kk[J];  // this token's key for the update
+            if (AHEAD) {
+#pragma unroll
+                for (int j = 0; j < J; ++j) kk[j] = k4[j];
+                vectors(min(k + 1, n - 1));
             }
             const float2 bk = *(const float2*)(tok + 3 * dimP + cols);
             // Sums over the eight lanes by halving exchange (partners 4, 2, 1 lanes away): lane r ends with S^T k and
@@ -392,12 +443,12 @@ __global__ void __launch_bounds__(NT) k_delta_scan(const DeltaRule a, int cols, 
             }
 #pragma unroll
             for (int j = 0; j < J; ++j) {
-                const ulonglong2 k4 = *(const ulonglong2*)(tok + dimP + 4 * (r + 8 * j));
+                if (!AHEAD) kk[j] = *(const ulonglong2*)(tok + dimP + 4 * (r + 8 * j));
 #pragma unroll
                 for (int c = 0; c < C; ++c) {
                     const f32x2 uu = pack2(uc[c], uc[c]);
-                    S[c][j][0] = fma2(k4.x, uu, S[c][j][0]);
-                    S[c][j][1] = fma2(k4.y, uu, S[c][j][1]);
+                    S[c][j][0] = fma2(kk[j].x, uu, S[c][j][0]);
+                    S[c][j][1] = fma2(kk[j].y, uu, S[c][j][1]);
                 }
             }
         }
@@ -437,15 +488,14 @@ __global__ void __launch_bounds__(NT) k_delta_scan(const DeltaRule a, int cols, 
 
 // prompts: norm and gate of the raw output rows, one warp per (token, head)
 template <typename A>
-__global__ void __launch_bounds__(kPrepWarps * 32) k_delta_out(const DeltaRule a, int T, unsigned long long* tl) {
+__global__ void __launch_bounds__(kPrepWarps * 32) k_delta_out(const DeltaRule a, unsigned long long* tl) {
     if (threadIdx.x == 0) tl_mark(tl, 0);
     pdl_launch_dependents();
     pdl_wait();
     if (threadIdx.x == 0) tl_mark(tl, 1);
-    const long long unit = (long long)blockIdx.x * kPrepWarps + (threadIdx.x >> 5);
-    if (unit < (long long)T * a.heads) {
-        const size_t t = (size_t)(unit / a.heads);
-        const int h = (int)(unit % a.heads);
+    const int h = blockIdx.x * kPrepWarps + (threadIdx.x >> 5);
+    if (h < a.heads) {
+        const size_t t = blockIdx.y;
         const float* o = a.o + (t * a.heads + h) * a.vdimP;
         delta_out_row<A>(a, t, h, threadIdx.x & 31, [&](int d) { return __ldcg(o + d); });
     }
@@ -465,6 +515,7 @@ cudaError_t scan_attrs() {
     cudaError_t e = cudaSuccess;
     if constexpr (J <= 4) {
         e = scan_attr<A, J, 8, true, 256>();
+        if (e == cudaSuccess) e = scan_attr<A, J, 4, true, 256>();
         if (e == cudaSuccess) e = scan_attr<A, J, 8, false, 128>();
     }
     if (e == cudaSuccess) e = scan_attr<A, J, 4, false, 128>();
@@ -493,10 +544,12 @@ void launch_scan(const DeltaRule& a, int n_segs, bool fused, int num_sms, cudaSt
     };
     const int whole = (a.vdimP + 7) / 8 * 8;
     if constexpr (J <= 4) {
+        if (fused && a.heads * n_segs < num_sms && whole <= 128) return go(k_delta_scan<A, J, 4, true, 256>, 4, whole, true);
         if (fused) return go(k_delta_scan<A, J, 8, true, 256>, 8, whole, true);
-        // few sequences: half as many columns per lane and block, so that a token's chain of steps is shorter
-        const int units = a.heads * n_segs * ((a.vdimP + 63) / 64);
-        if (units > num_sms) return go(k_delta_scan<A, J, 8, false, 128>, 8, whole < 128 ? whole : 128, false);
+        // eight columns per lane need the fewest shared-memory reads; with few sequences half as many columns per lane
+        // and twice the warps make a token's chain of steps shorter
+        const long long warps = (long long)a.heads * n_segs * ((a.vdimP + 31) / 32);
+        if (warps >= 3ll * num_sms) return go(k_delta_scan<A, J, 8, false, 128>, 8, whole < 128 ? whole : 128, false);
     }
     go(k_delta_scan<A, J, 4, false, 128>, 4, whole < 64 ? whole : 64, false);
 }
@@ -512,13 +565,12 @@ void launch_scan_j(const DeltaRule& a, int n_segs, bool fused, int num_sms, cuda
 }
 template <typename A>
 void launch_prep(const DeltaRule& a, int T, cudaStream_t s, bool pdl, unsigned long long* tl) {
-    const long long units = (long long)T * (a.kv_heads + a.heads);
-    const dim3 grid((unsigned)((units + kPrepWarps - 1) / kPrepWarps)), block(kPrepWarps * 32);
+    const dim3 grid((a.kv_heads + a.heads + kPrepWarps - 1) / kPrepWarps, T), block(kPrepWarps * 32);
     const int wide = a.dimP > a.vdimP ? a.dimP : a.vdimP;
-    if (a.dim % 2 || a.vdim % 2) launch_k(k_delta_prep<A, 1, 8>, grid, block, 0, s, pdl, a, T, tl);
-    else if (wide <= 64) launch_k(k_delta_prep<A, 2, 1>, grid, block, 0, s, pdl, a, T, tl);
-    else if (wide <= 128) launch_k(k_delta_prep<A, 2, 2>, grid, block, 0, s, pdl, a, T, tl);
-    else launch_k(k_delta_prep<A, 2, 4>, grid, block, 0, s, pdl, a, T, tl);
+    if (a.dim % 2 || a.vdim % 2) launch_k(k_delta_prep<A, 1, 8>, grid, block, 0, s, pdl, a, tl);
+    else if (wide <= 64) launch_k(k_delta_prep<A, 2, 1>, grid, block, 0, s, pdl, a, tl);
+    else if (wide <= 128) launch_k(k_delta_prep<A, 2, 2>, grid, block, 0, s, pdl, a, tl);
+    else launch_k(k_delta_prep<A, 2, 4>, grid, block, 0, s, pdl, a, tl);
 }
 
 }  // namespace
@@ -539,10 +591,9 @@ void launch_delta_scan(const DeltaRule& a, bool f32, int n_segs, bool fused, int
     else launch_scan_j<bf16>(a, n_segs, fused, num_sms, s, pdl, tl);
 }
 void launch_delta_out(const DeltaRule& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl) {
-    const long long units = (long long)T * a.heads;
-    const dim3 grid((unsigned)((units + kPrepWarps - 1) / kPrepWarps)), block(kPrepWarps * 32);
-    if (f32) launch_k(k_delta_out<float>, grid, block, 0, s, pdl, a, T, tl);
-    else launch_k(k_delta_out<bf16>, grid, block, 0, s, pdl, a, T, tl);
+    const dim3 grid((a.heads + kPrepWarps - 1) / kPrepWarps, T), block(kPrepWarps * 32);
+    if (f32) launch_k(k_delta_out<float>, grid, block, 0, s, pdl, a, tl);
+    else launch_k(k_delta_out<bf16>, grid, block, 0, s, pdl, a, tl);
 }
 
 }  // namespace tffn

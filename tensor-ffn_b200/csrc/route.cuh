@@ -25,6 +25,7 @@ __device__ __forceinline__ void route_token(const MoeRoute& a, int t, float* s, 
         s[i] *= inv;
         choice[i] = s[i] + __ldg(a.correction + i);
     }
+    int mine[2] = {-1, -1};  // lane j keeps choices j and 32 + j (top <= 64)
     for (int j = 0; j < a.top; ++j) {
         float best = -INFINITY;
         int bi = 0x7fffffff;
@@ -37,8 +38,16 @@ __device__ __forceinline__ void route_token(const MoeRoute& a, int t, float* s, 
             if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
         }
         if (bi >= n) bi = j;  // no finite score is left (NaN inputs): stay in range
-        if ((bi & 31) == lane) {
-            choice[bi] = -INFINITY;
+        if ((bi & 31) == lane) choice[bi] = -INFINITY;
+        if ((j & 31) == lane) mine[j >> 5] = bi;
+    }
+    __syncwarp();  // every lane's scores are visible
+    // places within the experts: the choices' atomics in flight together
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int j = k * 32 + lane;
+        if (j < a.top) {
+            const int bi = mine[k];
             int2 p = make_int2(-1, 0);
             if (bi < a.experts) p = make_int2(bi, atomicAdd(a.counts + bi, 1));
             a.pair[(size_t)t * a.top + j] = p;

@@ -148,18 +148,26 @@ __global__ void __launch_bounds__(512) k_residual_rows4(const ResidualRows a, un
         const int warp = tid >> 5, lane = tid & 31, outs = a.route.experts + a.route.identity;
         float* z = rows4_smem + H;
         __syncthreads();
-        for (int e = warp; e < outs; e += n >> 5) {
-            const bf16* w = a.router_w + (size_t)e * a.router_ld;
-            float acc = 0.f;
+        const int warps = n >> 5;
+        for (int e0 = warp; e0 < outs; e0 += 2 * warps) {  // two outputs at a time: their loads in flight together
+            const int e1 = e0 + warps;
+            const bf16 *w0 = a.router_w + (size_t)e0 * a.router_ld, *w1 = a.router_w + (size_t)(e1 < outs ? e1 : e0) * a.router_ld;
+            float acc0 = 0.f, acc1 = 0.f;
 #pragma unroll 4
             for (int i = lane * 8; i < H; i += 256) {
-                const uint4 q = __ldg((const uint4*)(w + i));
+                const uint4 p = __ldg((const uint4*)(w0 + i)), q = __ldg((const uint4*)(w1 + i));
                 const float4 x0 = *(const float4*)(rows4_smem + i), x1 = *(const float4*)(rows4_smem + i + 4);
-                acc += bf16_lo(q.x) * x0.x + bf16_hi(q.x) * x0.y + bf16_lo(q.y) * x0.z + bf16_hi(q.y) * x0.w;
-                acc += bf16_lo(q.z) * x1.x + bf16_hi(q.z) * x1.y + bf16_lo(q.w) * x1.z + bf16_hi(q.w) * x1.w;
+                acc0 += bf16_lo(p.x) * x0.x + bf16_hi(p.x) * x0.y + bf16_lo(p.y) * x0.z + bf16_hi(p.y) * x0.w;
+                acc0 += bf16_lo(p.z) * x1.x + bf16_hi(p.z) * x1.y + bf16_lo(p.w) * x1.z + bf16_hi(p.w) * x1.w;
+                acc1 += bf16_lo(q.x) * x0.x + bf16_hi(q.x) * x0.y + bf16_lo(q.y) * x0.z + bf16_hi(q.y) * x0.w;
+                acc1 += bf16_lo(q.z) * x1.x + bf16_hi(q.z) * x1.y + bf16_lo(q.w) * x1.z + bf16_hi(q.w) * x1.w;
             }
-            acc = warp_sum(acc);
-            if (lane == 0) z[e] = acc;
+            acc0 = warp_sum(acc0);
+            acc1 = warp_sum(acc1);
+            if (lane == 0) {
+                z[e0] = acc0;
+                if (e1 < outs) z[e1] = acc1;
+            }
         }
         __syncthreads();
         if (warp == 0) route_token(a.route, r, z, z + outs, lane);
@@ -267,20 +275,20 @@ __device__ __forceinline__ void store_pair(bf16* p, float x, float y) {
 
 // one warp per (token, head): heads 0 .. nh-1 are queries, then the keys, then the values
 constexpr int kQkWarps = 4;
-template <typename A>
-__global__ void __launch_bounds__(kQkWarps * 32) k_qk_norm_rope(const QkNormRope a, int T, unsigned long long* tl) {
+template <typename A, int MP>  // MP pairs per lane: heads of up to 64 MP
+__global__ void __launch_bounds__(kQkWarps * 32) k_qk_norm_rope(const QkNormRope a, unsigned long long* tl) {
     if (threadIdx.x == 0) tl_mark(tl, 0);
     pdl_launch_dependents();
     pdl_wait();
     if (threadIdx.x == 0) tl_mark(tl, 1);
     const int lane = threadIdx.x & 31;
-    const long long unit = (long long)blockIdx.x * kQkWarps + (threadIdx.x >> 5);
+    const int t = blockIdx.y, u = blockIdx.x * kQkWarps + (threadIdx.x >> 5);
     const int nkv = a.kv.nkv, per_tok = a.nh + 2 * nkv;
-    if (unit < (long long)T * per_tok) {
-        const int t = (int)(unit / per_tok), u = (int)(unit % per_tok);
+    if (u < per_tok) {
         const int kind = u < a.nh ? 0 : (u < a.nh + nkv ? 1 : 2);
         const int head = kind == 0 ? u : (kind == 1 ? u - a.nh : u - a.nh - nkv);
         const int dim = kind == 2 ? a.vdim : a.dim;
+        const float* norm_w = kind == 0 ? a.q_norm : a.k_norm;
         const A* src = (const A*)a.qkv + (size_t)t * a.ld + (kind == 0 ? 0 : (kind == 1 ? a.k_off : a.v_off)) + (size_t)head * dim;
         const int pos = __ldcg(a.tok_pos + t), seq = __ldcg(a.tok_seq + t);
         const bool pos_ok = pos >= 0 && pos < a.max_pos;
@@ -300,7 +308,6 @@ __global__ void __launch_bounds__(kQkWarps * 32) k_qk_norm_rope(const QkNormRope
             }
         } else {
             // lane = pair (2i, 2i + 1)
-            constexpr int MP = 8;  // heads of up to 512
             const bool even = (dim & 1) == 0;
             float u0[MP], u1[MP], ss = 0.f;
 #pragma unroll
@@ -316,7 +323,7 @@ __global__ void __launch_bounds__(kQkWarps * 32) k_qk_norm_rope(const QkNormRope
                 ss += u0[j] * u0[j] + u1[j] * u1[j];
             }
             const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dim + a.eps);
-            const float* w = kind == 0 ? a.q_norm : a.k_norm;
+            const float* w = norm_w;
             float* qd = a.q_out + ((size_t)t * a.nh + head) * a.kv.hd;
             A* kdst = (A*)a.kv.k_pool + (((size_t)pg * nkv + head) * kPageTokens + pos % kPageTokens) * a.kv.hd;
 #pragma unroll
@@ -367,8 +374,10 @@ int stack_rows_prepare() {
     if (e == cudaSuccess) e = rows4_attrs_all<float>();
     if (e == cudaSuccess) e = prefer_max_shared(k_residual_rows<bf16>);
     if (e == cudaSuccess) e = prefer_max_shared(k_residual_rows<float>);
-    if (e == cudaSuccess) e = prefer_max_shared(k_qk_norm_rope<bf16>);
-    if (e == cudaSuccess) e = prefer_max_shared(k_qk_norm_rope<float>);
+    if (e == cudaSuccess) e = prefer_max_shared(k_qk_norm_rope<bf16, 2>);
+    if (e == cudaSuccess) e = prefer_max_shared(k_qk_norm_rope<bf16, 8>);
+    if (e == cudaSuccess) e = prefer_max_shared(k_qk_norm_rope<float, 2>);
+    if (e == cudaSuccess) e = prefer_max_shared(k_qk_norm_rope<float, 8>);
     return (int)e;
 }
 
@@ -382,7 +391,8 @@ static void launch_rows(const ResidualRows& a, int rows, cudaStream_t s, bool pd
     const int groups = a.H / 4;
     const size_t smem = a.router_w ? (size_t)(a.H + 2 * (a.route.experts + a.route.identity)) * 4 : 0;
     const int per = groups <= 256 ? 1 : groups <= 1024 ? 2 : groups <= 2048 ? 4 : 8;
-    const dim3 grid(rows), block(((groups + per - 1) / per + 31) / 32 * 32);
+    const int threads = ((groups + per - 1) / per + 31) / 32 * 32;
+    const dim3 grid(rows), block(a.router_w ? 512 : threads);  // routing: as many warps for the router's outputs as fit
     if (per == 1) launch_k(k_residual_rows4<A, 1>, grid, block, smem, s, pdl, a, tl);
     else if (per == 2) launch_k(k_residual_rows4<A, 2>, grid, block, smem, s, pdl, a, tl);
     else if (per == 4) launch_k(k_residual_rows4<A, 4>, grid, block, smem, s, pdl, a, tl);
@@ -394,10 +404,10 @@ void launch_residual_rows(const ResidualRows& a, bool f32, int rows, cudaStream_
 }
 
 void launch_qk_norm_rope(const QkNormRope& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl) {
-    const long long units = (long long)T * (a.nh + 2 * a.kv.nkv);
-    const dim3 grid((unsigned)((units + kQkWarps - 1) / kQkWarps)), block(kQkWarps * 32);
-    if (f32) launch_k(k_qk_norm_rope<float>, grid, block, 0, s, pdl, a, T, tl);
-    else launch_k(k_qk_norm_rope<bf16>, grid, block, 0, s, pdl, a, T, tl);
+    const dim3 grid((a.nh + 2 * a.kv.nkv + kQkWarps - 1) / kQkWarps, T), block(kQkWarps * 32);
+    const bool narrow = a.dim <= 128 && a.vdim <= 128;
+    if (f32) launch_k(narrow ? k_qk_norm_rope<float, 2> : k_qk_norm_rope<float, 8>, grid, block, 0, s, pdl, a, tl);
+    else launch_k(narrow ? k_qk_norm_rope<bf16, 2> : k_qk_norm_rope<bf16, 8>, grid, block, 0, s, pdl, a, tl);
 }
 
 }  // namespace tffn

@@ -144,7 +144,9 @@ __device__ __forceinline__ void attn_block16(uint32_t kbuf, uint32_t vbuf, int r
     }
 }
 
-template <int HD>
+// EXACT: the uniform layers' case (rows of exactly HD columns, at most 8 query heads per kv head, every earlier key
+// visible) with everything that AttnOptions and KvView leave open folded into constants.
+template <int HD, bool EXACT>
 __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __restrict__ q, KvView kv, int layer,
                                                               const int* __restrict__ tok_seq,
                                                               const int* __restrict__ tok_pos, bf16* __restrict__ ctx,
@@ -181,16 +183,17 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
     // unit = (t * nkv + kvh) * parts + part: the query heads of a kv head come in parts of at most 8
     const int unit = blockIdx.x;
     const int nkv = kv.nkv;
-    const int parts_per_kv = (G_all + 7) / 8;
-    const int part = unit % parts_per_kv;
+    const int parts_per_kv = EXACT ? 1 : (G_all + 7) / 8;
+    const int part = EXACT ? 0 : unit % parts_per_kv;
     const int t = unit / parts_per_kv / nkv, kvh = unit / parts_per_kv % nkv;
-    const int G = min(8, G_all - part * 8);
+    const int G = EXACT ? G_all : min(8, G_all - part * 8);
     const int head0 = kvh * G_all + part * 8;
-    const int kd = kv.hd, vd = kv.vd;  // widths of the cached rows: multiples of 8, at most HD
+    const int kd = EXACT ? HD : kv.hd, vd = EXACT ? HD : kv.vd;  // widths of the cached rows: multiples of 8, at most HD
+    const int vdim = EXACT ? HD : opt.vdim;
     const int split = blockIdx.y;
     const int seq = __ldcg(tok_seq + t);
     const int ctx_len = __ldcg(tok_pos + t) + 1;
-    const int lo = opt.chunk > 0 ? (ctx_len - 1) / opt.chunk * opt.chunk : 0;  // first visible key
+    const int lo = !EXACT && opt.chunk > 0 ? (ctx_len - 1) / opt.chunk * opt.chunk : 0;  // first visible key
     const int lo16 = lo & ~15;  // a warp's 16 rows start at a multiple of 16, so that they lie in one page
     int chunk = (ctx_len - lo16 + splits - 1) / splits;
     chunk = (chunk + kPageTokens - 1) / kPageTokens * kPageTokens;
@@ -334,9 +337,9 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
         }
     }
     __syncthreads();
-    const int G_part = min(8, G_all);  // heads of a full part: the stride of the partial results
+    const int G_part = EXACT ? G_all : min(8, G_all);  // heads of a full part: the stride of the partial results
     float* partial = ws + ((size_t)unit * splits + split) * (size_t)(G_part * (HD + 2));
-    bf16* ctx_tok = ctx + (size_t)t * opt.ctx_ld + (size_t)head0 * opt.vdim;
+    bf16* ctx_tok = ctx + (size_t)t * (EXACT ? (int64_t)nh * HD : opt.ctx_ld) + (size_t)head0 * vdim;
     for (int idx = tid; idx < G * HD; idx += kAttnCtaThreads) {
         const int g = idx / HD, d = idx % HD;
         float M = kNegBig;
@@ -351,7 +354,7 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
             A += mw[2 + d] * wgt;
         }
         if (splits == 1) {
-            if (d < opt.vdim) ctx_tok[(size_t)g * opt.vdim + d] = __float2bfloat16_rn(A / L);
+            if (d < vdim) ctx_tok[(size_t)g * vdim + d] = __float2bfloat16_rn(A / L);
         } else {
             partial[g * (HD + 2) + 2 + d] = A;
             if (d == 0) { partial[g * (HD + 2)] = M; partial[g * (HD + 2) + 1] = L; }
@@ -426,12 +429,12 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
 #pragma unroll
         for (int it = 0; it < ITERS; ++it) {
             const int idx = tid + it * kAttnCtaThreads;
-            if (idx < G * HD && idx % HD < opt.vdim) ctx_tok[(size_t)(idx / HD) * opt.vdim + idx % HD] = __float2bfloat16_rn(res[it]);
+            if (idx < G * HD && idx % HD < vdim) ctx_tok[(size_t)(idx / HD) * vdim + idx % HD] = __float2bfloat16_rn(res[it]);
         }
     } else {
         for (int idx = tid; idx < G * HD; idx += kAttnCtaThreads) {
             const int g = idx / HD, d = idx % HD;
-            if (d < opt.vdim) ctx_tok[(size_t)g * opt.vdim + d] = __float2bfloat16_rn(attn_merge_splits(parts, splits, G_part, HD, g, d));
+            if (d < vdim) ctx_tok[(size_t)g * vdim + d] = __float2bfloat16_rn(attn_merge_splits(parts, splits, G_part, HD, g, d));
         }
     }
     ATTN_TRACE(8);
@@ -444,7 +447,7 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_decode(const float* __
 // them, so the cache is read once per 8 tokens instead of once per token; warp w runs the same 16-key
 // blocks as the decode kernel over keys 0 .. pos_w (causal), owns its token's whole context and writes
 // its output rows itself: no merge.
-template <int HD>
+template <int HD, bool EXACT>
 __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_prefill(const float* __restrict__ q, KvView kv, int layer,
                                                                const int* __restrict__ tok_seq,
                                                                const int* __restrict__ tok_pos,
@@ -459,10 +462,11 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_prefill(const float* _
     pdl_wait();  // the previous kernel wrote q and the K/V rows of these very tokens
     if (threadIdx.x == 0) tl_mark(tl, 1);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int nkv = kv.nkv, parts_per_kv = (G_all + 7) / 8;  // query heads of a kv head in parts of at most 8
+    const int nkv = kv.nkv, parts_per_kv = EXACT ? 1 : (G_all + 7) / 8;  // query heads of a kv head in parts of at most 8
     const int kvh = blockIdx.y / parts_per_kv, part = blockIdx.y % parts_per_kv;
-    const int G = min(8, G_all - part * 8), head0 = kvh * G_all + part * 8;
-    const int kd = kv.hd, vd = kv.vd;
+    const int G = EXACT ? G_all : min(8, G_all - part * 8), head0 = kvh * G_all + part * 8;
+    const int kd = EXACT ? HD : kv.hd, vd = EXACT ? HD : kv.vd;
+    const int chunk = EXACT ? 0 : opt.chunk, vdim = EXACT ? HD : opt.vdim;
     const int first = __ldcg(grp_first + blockIdx.x), count = __ldcg(grp_count + blockIdx.x);
     const int seq = __ldcg(tok_seq + first);
     const int last_len = __ldcg(tok_pos + first + count - 1) + 1;  // positions ascend within a group
@@ -470,8 +474,8 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_prefill(const float* _
     const int t = first + (active ? warp : 0);
     const int my_len = active ? __ldcg(tok_pos + t) + 1 : 0;
     // first key visible to this warp's token, and the group's first key (page-aligned): a group may cross a chunk's edge
-    const int my_lo = (opt.chunk > 0 && active) ? (my_len - 1) / opt.chunk * opt.chunk : 0;
-    const int grp_lo = opt.chunk > 0 ? (__ldcg(tok_pos + first) / opt.chunk * opt.chunk) / kPageTokens * kPageTokens : 0;
+    const int my_lo = (chunk > 0 && active) ? (my_len - 1) / chunk * chunk : 0;
+    const int grp_lo = chunk > 0 ? (__ldcg(tok_pos + first) / chunk * chunk) / kPageTokens * kPageTokens : 0;
     const int* bt = kv.block_table + (size_t)seq * kv.max_pages_per_seq;
     const bf16* kpool = kv.k_pool + (size_t)layer * kv.layer_stride;
     const bf16* vpool = kv.v_pool + (size_t)layer * kv.layer_stride;
@@ -553,8 +557,7 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_prefill(const float* _
     l_run += __shfl_xor_sync(0xffffffffu, l_run, 2);
     if (active && hrow < G) {
         const float inv = 1.f / l_run;  // my_len >= 1: at least one key
-        const int vdim = opt.vdim;
-        bf16* dst = ctx + (size_t)t * opt.ctx_ld + (size_t)(head0 + hrow) * vdim + quad * 2;
+        bf16* dst = ctx + (size_t)t * (EXACT ? (int64_t)nh * HD : opt.ctx_ld) + (size_t)(head0 + hrow) * vdim + quad * 2;
 #pragma unroll
         for (int d = 0; d < C::DT; ++d) {
             const float a = (o[d][0] + o[d][2]) * inv, b = (o[d][1] + o[d][3]) * inv;  // P_hi V + P_lo V
@@ -640,11 +643,15 @@ __global__ void __launch_bounds__(kSimtWarps * 32) k_attn_simt(const float* __re
     if (tid == 0) tl_mark(tl, 2);
 }
 
+bool exact(const AttnOptions& o, const KvView& kv, int nh, int hd) {
+    return kv.hd == hd && kv.vd == hd && o.vdim == hd && o.ctx_ld == (int64_t)nh * hd && o.chunk == 0 && nh / kv.nkv <= 8;
+}
+
 template <int HD>
 void launch_hd(dim3 grid, cudaStream_t s, bool pdl, const float* q, const KvView& kv, int layer, const int* tok_seq,
                const int* tok_pos, bf16* ctx, int nh, int G, int splits, int early, const AttnOptions& opt, float* ws,
                int* counters, int* status, unsigned long long* tl, unsigned long long* trace) {
-    launch_k(k_attn_decode<HD>, grid, dim3(kAttnCtaThreads), (size_t)AttnCfg<HD>::SMEM, s, pdl, q, kv, layer, tok_seq, tok_pos, ctx,
+    launch_k(exact(opt, kv, nh, HD) ? k_attn_decode<HD, true> : k_attn_decode<HD, false>, grid, dim3(kAttnCtaThreads), (size_t)AttnCfg<HD>::SMEM, s, pdl, q, kv, layer, tok_seq, tok_pos, ctx,
              nh, G, splits, early, opt, ws, counters, status, tl, trace);
 }
 
@@ -652,7 +659,7 @@ template <int HD>
 void launch_prefill_hd(dim3 grid, cudaStream_t s, bool pdl, const float* q, const KvView& kv, int layer, const int* tok_seq,
                        const int* tok_pos, const int* grp_first, const int* grp_count, bf16* ctx, int nh, int G,
                        const AttnOptions& opt, int* status, unsigned long long* tl) {
-    launch_k(k_attn_prefill<HD>, grid, dim3(kAttnCtaThreads), (size_t)AttnCfg<HD>::SMEM, s, pdl, q, kv, layer, tok_seq, tok_pos,
+    launch_k(exact(opt, kv, nh, HD) ? k_attn_prefill<HD, true> : k_attn_prefill<HD, false>, grid, dim3(kAttnCtaThreads), (size_t)AttnCfg<HD>::SMEM, s, pdl, q, kv, layer, tok_seq, tok_pos,
              grp_first, grp_count, ctx, nh, G, opt, status, tl);
 }
 
@@ -666,17 +673,25 @@ AttnOptions resolve(AttnOptions o, const KvView& kv, int nh) {
 
 }  // namespace
 
+template <typename Kern>
+static cudaError_t attn_attrs(Kern k, int smem) {
+    const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    return e == cudaSuccess ? prefer_max_shared(k) : e;
+}
+template <int HD>
+static cudaError_t attn_attrs_hd() {
+    cudaError_t e = attn_attrs(k_attn_decode<HD, true>, AttnCfg<HD>::SMEM);
+    if (e == cudaSuccess) e = attn_attrs(k_attn_decode<HD, false>, AttnCfg<HD>::SMEM);
+    if (e == cudaSuccess) e = attn_attrs(k_attn_prefill<HD, true>, AttnCfg<HD>::SMEM);
+    if (e == cudaSuccess) e = attn_attrs(k_attn_prefill<HD, false>, AttnCfg<HD>::SMEM);
+    return e;
+}
+
 // The dynamic shared-memory opt-in is a per-device attribute of a kernel: every session makes it for
 // its own device (with that device current), outside of stream capture.
 int attn_prepare() {
-    cudaError_t e = cudaFuncSetAttribute(k_attn_decode<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, AttnCfg<64>::SMEM);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(k_attn_decode<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, AttnCfg<128>::SMEM);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(k_attn_prefill<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, AttnCfg<64>::SMEM);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(k_attn_prefill<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, AttnCfg<128>::SMEM);
-    if (e == cudaSuccess) e = prefer_max_shared(k_attn_decode<64>);
-    if (e == cudaSuccess) e = prefer_max_shared(k_attn_decode<128>);
-    if (e == cudaSuccess) e = prefer_max_shared(k_attn_prefill<64>);
-    if (e == cudaSuccess) e = prefer_max_shared(k_attn_prefill<128>);
+    cudaError_t e = attn_attrs_hd<64>();
+    if (e == cudaSuccess) e = attn_attrs_hd<128>();
     if (e == cudaSuccess) e = prefer_max_shared(k_attn_simt<float>);
     if (e == cudaSuccess) e = prefer_max_shared(k_attn_simt<bf16>);
     return (int)e;

@@ -578,13 +578,13 @@ __global__ void __launch_bounds__(kAttnCtaThreads) k_attn_prefill(const float* _
 // caches (a session that computes in fp32) and heads wider than 128. Every warp walks the visible keys with a stride
 // of kSimtWarps; the lanes share the dimensions of a key; exact exponentials; the warps merge at the end.
 constexpr int kSimtWarps = 8;
-constexpr int kSimtMaxLanes = 16;  // value columns per lane: heads of up to 512 columns
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(bf16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ void store_as(float* p, float v) { *p = v; }
 __device__ __forceinline__ void store_as(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
 
-template <typename C>
+// ML: value columns per lane, for heads of up to 32 ML value columns
+template <typename C, int ML>
 __global__ void __launch_bounds__(kSimtWarps * 32) k_attn_simt(const float* __restrict__ q, KvView kv, const int* __restrict__ tok_seq,
                                                                const int* __restrict__ tok_pos, C* __restrict__ ctx, int nh,
                                                                AttnOptions opt, int* status, unsigned long long* tl) {
@@ -605,9 +605,9 @@ __global__ void __launch_bounds__(kSimtWarps * 32) k_attn_simt(const float* __re
     const int* bt = kv.block_table + (size_t)seq * kv.max_pages_per_seq;
     const C* kpool = (const C*)kv.k_pool;
     const C* vpool = (const C*)kv.v_pool;
-    float m = kNegBig, l = 0.f, acc[kSimtMaxLanes];
+    float m = kNegBig, l = 0.f, acc[ML];
 #pragma unroll
-    for (int j = 0; j < kSimtMaxLanes; ++j) acc[j] = 0.f;
+    for (int j = 0; j < ML; ++j) acc[j] = 0.f;
     bool bad = false;
     for (int key = lo + warp; key <= last; key += kSimtWarps) {
         const int pg = __ldcg(bt + key / kPageTokens);
@@ -620,7 +620,7 @@ __global__ void __launch_bounds__(kSimtWarps * 32) k_attn_simt(const float* __re
         m = mn;
         l = l * corr + p;
 #pragma unroll
-        for (int j = 0; j < kSimtMaxLanes; ++j) {
+        for (int j = 0; j < ML; ++j) {
             const int d = j * 32 + lane;
             if (d < vdim) acc[j] = acc[j] * corr + p * to_f32(vpool[row * vd + d]);
         }
@@ -628,23 +628,28 @@ __global__ void __launch_bounds__(kSimtWarps * 32) k_attn_simt(const float* __re
     float* mw = merge + warp * (vdim + 2);
     if (lane == 0) { mw[0] = m; mw[1] = l; }
 #pragma unroll
-    for (int j = 0; j < kSimtMaxLanes; ++j)
+    for (int j = 0; j < ML; ++j)
         if (j * 32 + lane < vdim) mw[2 + j * 32 + lane] = acc[j];
     __syncthreads();
     float M = kNegBig, L = 0.f;
+    float gate = 1.f;
+    if (opt.gate) {
+        const float z = to_f32(((const C*)opt.gate)[(size_t)t * opt.gate_ld + head]);
+        gate = 1.f / (1.f + expf(-z));
+    }
     for (int w = 0; w < kSimtWarps; ++w) M = fmaxf(M, merge[w * (vdim + 2)]);
     for (int w = 0; w < kSimtWarps; ++w) L += merge[w * (vdim + 2) + 1] * expf(merge[w * (vdim + 2)] - M);
     for (int d = tid; d < vdim; d += kSimtWarps * 32) {
         float A = 0.f;
         for (int w = 0; w < kSimtWarps; ++w) A += merge[w * (vdim + 2) + 2 + d] * expf(merge[w * (vdim + 2)] - M);
-        store_as(ctx + (size_t)t * opt.ctx_ld + (size_t)head * vdim + d, A / L);
+        store_as(ctx + (size_t)t * opt.ctx_ld + (size_t)head * opt.head_ld + d, A / L * gate);
     }
     if (bad && lane == 0) dev_fail(status, DEV_ERR_BOUNDS);
     if (tid == 0) tl_mark(tl, 2);
 }
 
 bool exact(const AttnOptions& o, const KvView& kv, int nh, int hd) {
-    return kv.hd == hd && kv.vd == hd && o.vdim == hd && o.ctx_ld == (int64_t)nh * hd && o.chunk == 0 && nh / kv.nkv <= 8;
+    return kv.hd == hd && kv.vd == hd && o.vdim == hd && o.ctx_ld == (int64_t)nh * hd && o.chunk == 0 && !o.gate && nh / kv.nkv <= 8;
 }
 
 template <int HD>
@@ -667,7 +672,8 @@ void launch_prefill_hd(dim3 grid, cudaStream_t s, bool pdl, const float* q, cons
 AttnOptions resolve(AttnOptions o, const KvView& kv, int nh) {
     if (o.scale == 0.f) o.scale = 1.f / sqrtf((float)kv.hd);
     if (o.vdim == 0) o.vdim = kv.vd;
-    if (o.ctx_ld == 0) o.ctx_ld = (int64_t)nh * o.vdim;
+    if (o.head_ld == 0) o.head_ld = o.vdim;
+    if (o.ctx_ld == 0) o.ctx_ld = (int64_t)nh * o.head_ld;
     return o;
 }
 
@@ -692,8 +698,10 @@ static cudaError_t attn_attrs_hd() {
 int attn_prepare() {
     cudaError_t e = attn_attrs_hd<64>();
     if (e == cudaSuccess) e = attn_attrs_hd<128>();
-    if (e == cudaSuccess) e = prefer_max_shared(k_attn_simt<float>);
-    if (e == cudaSuccess) e = prefer_max_shared(k_attn_simt<bf16>);
+    if (e == cudaSuccess) e = prefer_max_shared(k_attn_simt<float, 16>);
+    if (e == cudaSuccess) e = prefer_max_shared(k_attn_simt<bf16, 16>);
+    if (e == cudaSuccess) e = prefer_max_shared(k_attn_simt<float, 32>);
+    if (e == cudaSuccess) e = prefer_max_shared(k_attn_simt<bf16, 32>);
     return (int)e;
 }
 
@@ -755,8 +763,9 @@ void launch_attention_simt(const float* q, KvView kv, bool f32, const int* tok_s
     const AttnOptions opt = resolve(options, kv, nh);
     const dim3 grid(nh, T), block(kSimtWarps * 32);
     const size_t smem = (size_t)(kv.hd + kSimtWarps * (opt.vdim + 2)) * 4;
-    if (f32) launch_k(k_attn_simt<float>, grid, block, smem, s, pdl, q, kv, tok_seq, tok_pos, (float*)ctx, nh, opt, status, tl);
-    else launch_k(k_attn_simt<bf16>, grid, block, smem, s, pdl, q, kv, tok_seq, tok_pos, (bf16*)ctx, nh, opt, status, tl);
+    const bool wide = opt.vdim > 512;
+    if (f32) launch_k(wide ? k_attn_simt<float, 32> : k_attn_simt<float, 16>, grid, block, smem, s, pdl, q, kv, tok_seq, tok_pos, (float*)ctx, nh, opt, status, tl);
+    else launch_k(wide ? k_attn_simt<bf16, 32> : k_attn_simt<bf16, 16>, grid, block, smem, s, pdl, q, kv, tok_seq, tok_pos, (bf16*)ctx, nh, opt, status, tl);
 }
 
 }  // namespace tffn

@@ -1,5 +1,5 @@
-// Gated delta rule with one decay per head and key channel, a recurrent mixer: per head a matrix S (key channels x
-// value columns) with, per token,
+// Gated delta rule with one decay per head and key channel or (HEAD_DECAY) per head, a recurrent mixer: per head a matrix
+// S (key channels x value columns) with, per token,
 //     S = g * S (rows), u = beta * (v - S^T k), S = S + k u^T, o = S^T q.
 // Two kernels per layer, for prompts and decoding alike:
 //   k_delta_prep  one warp per (token, head): the short causal convolutions with SiLU, the unit vectors q and k, beta and
@@ -190,7 +190,7 @@ __global__ void __launch_bounds__(kPrepWarps * 32) k_delta_prep(const DeltaRule 
                 }
             }
             const int rep = H / G;
-            for (int h = u * rep + lane; h < (u + 1) * rep; h += 32) a.bk[((size_t)t * H + h) * 2 + 1] = qk * qs * ks;
+            for (int h = u * rep + lane; h < (u + 1) * rep; h += 32) a.bk[((size_t)t * H + h) * (a.head_decay ? 4 : 2) + 1] = qk * qs * ks;
         } else {
             const int h = u - G;
             const float rate = -expf(__ldg(a.a_log + h));
@@ -201,7 +201,7 @@ __global__ void __launch_bounds__(kPrepWarps * 32) k_delta_prep(const DeltaRule 
                 const int d = (lane + 32 * i) * V;
 #pragma unroll
                 for (int v = 0; v < V; ++v) zz[i][v] = dt[i][v] = 0.f;
-                if (d < a.dim) {
+                if (d < a.dim && !a.head_decay) {
                     load_v<V>(z + d, zz[i]);
                     load_v<V>(a.dt_bias + h * a.dim + d, dt[i]);
                 }
@@ -214,15 +214,19 @@ __global__ void __launch_bounds__(kPrepWarps * 32) k_delta_prep(const DeltaRule 
             for (int i = 0; i < NI; ++i) {
                 const int d = (lane + 32 * i) * V;
                 if (d < a.vdimP) store_v<V>(vo + d, v[i]);
-                if (d < a.dimP) {
+                if (d < a.dimP && !a.head_decay) {
                     float g[V];
 #pragma unroll
                     for (int c = 0; c < V; ++c) g[c] = d < a.dim ? expf(rate * softplus_f32(zz[i][c] + dt[i][c])) : 0.f;
                     store_v<V>(go + d, g);
                 }
             }
-            if (lane == 0)
-                a.bk[((size_t)t * H + h) * 2] = sigmoid_f32(act_load((const A*)a.proj + (size_t)t * a.proj_ld + a.b_off + h));
+            if (lane == 0) {
+                const A* row = (const A*)a.proj + (size_t)t * a.proj_ld;
+                float* bk = a.bk + ((size_t)t * H + h) * (a.head_decay ? 4 : 2);
+                bk[0] = sigmoid_f32(act_load(row + a.b_off + h));
+                if (a.head_decay) bk[2] = expf(rate * softplus_f32(act_load(row + a.a_off + h) + __ldg(a.dt_bias + h)));
+            }
         }
     }
     if (threadIdx.x == 0) tl_mark(tl, 2);
@@ -257,17 +261,18 @@ __device__ __forceinline__ void cp_async8(void* dst, const void* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
-// one output row of a head: o / rms(o) * weight * sigmoid(gate). One warp; `at(d)` gives the raw value.
+// one output row of a head: o / rms(o) * weight * sigmoid(gate) or silu(gate). One warp; `at(d)` gives the raw value.
 template <typename A, typename At>
 __device__ __forceinline__ void delta_out_row(const DeltaRule& a, size_t t, int h, int lane, At at) {
     constexpr int NI = 8;  // vdim <= 256
     float o[NI], gate[NI], ss = 0.f;
-    const float* g = a.gate_in + t * a.gate_ld + (size_t)h * a.vdim;
+    const float* g = a.gate_in ? a.gate_in + t * a.gate_ld + (size_t)h * a.vdim : nullptr;
+    const A* gp = (const A*)a.proj + t * a.proj_ld + a.gate_off + (size_t)h * a.vdim;
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
         const int d = lane + 32 * i;
         o[i] = d < a.vdim ? at(d) : 0.f;
-        gate[i] = d < a.vdim ? __ldcg(g + d) : 0.f;
+        gate[i] = d < a.vdim ? (g ? __ldcg(g + d) : act_load(gp + d)) : 0.f;
         ss += o[i] * o[i];
     }
     const float inv = 1.f / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
@@ -275,21 +280,22 @@ __device__ __forceinline__ void delta_out_row(const DeltaRule& a, size_t t, int 
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
         const int d = lane + 32 * i;
-        if (d < a.vdim) act_store(out + d, o[i] * inv * __ldg(a.out_norm + d) * sigmoid_f32(gate[i]));
+        if (d < a.vdim) act_store(out + d, o[i] * inv * __ldg(a.out_norm + d) * sigmoid_f32(gate[i]) * (a.gate_silu ? gate[i] : 1.f));
     }
 }
 
 constexpr int kScanTokens = 8;  // tokens per stage
-__host__ __device__ inline int scan_token_floats(int dimP, int cols) { return 3 * dimP + cols + 4; }
-inline size_t scan_smem(int dimP, int cols, bool fused) {
-    return (size_t)kScanTokens * 2 * scan_token_floats(dimP, cols) * 4 + (fused ? (size_t)kScanTokens * cols * 4 : 0);
+// of a token: q | k | decays (one per key channel) | v | beta, k . q (and the head's decay)
+__host__ __device__ inline int scan_token_floats(int dimP, int cols, bool head_decay) { return (head_decay ? 2 : 3) * dimP + cols + 4; }
+inline size_t scan_smem(int dimP, int cols, bool fused, bool head_decay) {
+    return (size_t)kScanTokens * 2 * scan_token_floats(dimP, cols, head_decay) * 4 + (fused ? (size_t)kScanTokens * cols * 4 : 0);
 }
 
 // J = dimP / 32, C = value columns per lane: lane r of the eight that share C columns holds the key channels
 // 4 (r + 8 j) + {0..3} of each. Blocks take `cols` columns of a head (grid z covers the head). Whatever C and cols
 // are, a column's sums are formed in the same order. FUSED (one block per head): norm and gate of the output row here,
 // else the raw row goes to `o` for k_delta_out.
-template <typename A, int J, int C, bool FUSED, int NT>
+template <typename A, int J, int C, bool FUSED, int NT, bool HEAD_DECAY>
 __global__ void __launch_bounds__(NT) k_delta_scan(const DeltaRule a, int cols, unsigned long long* tl) {
     extern __shared__ __align__(16) float scan_buf[];
     if (threadIdx.x == 0) tl_mark(tl, 0);
@@ -298,7 +304,8 @@ __global__ void __launch_bounds__(NT) k_delta_scan(const DeltaRule a, int cols, 
     const int h = blockIdx.x, H = a.heads, G = a.kv_heads, kvh = h / (H / G);
     const int r = tid & 7, cb = blockIdx.z * cols, c0 = cb + (tid >> 3) * C;  // the block's and this lane's first column
     constexpr int dimP = 32 * J;
-    const int vdimP = a.vdimP, tokf = scan_token_floats(dimP, cols);
+    const int vdimP = a.vdimP, tokf = scan_token_floats(dimP, cols, HEAD_DECAY);
+    constexpr int vOff = (HEAD_DECAY ? 2 : 3) * dimP;  // within a token's floats
     const int ncols = min(cols, vdimP - cb);  // columns of this block that exist (a multiple of 4)
     float* o_s = scan_buf + (size_t)2 * kScanTokens * tokf;  // FUSED: [kScanTokens][cols]
     // The token lists and the state are older than this step's first kernel (a full dependency of the stream), so
@@ -329,15 +336,18 @@ __global__ void __launch_bounds__(NT) k_delta_scan(const DeltaRule a, int cols, 
         for (int k = warp; k < n; k += nwarps) {
             const size_t t = (size_t)first + tile * kScanTokens + k;
             float* dst = buf + (size_t)k * tokf;
-            const float *q = a.qn + (t * G + kvh) * dimP, *kk = a.kn + (t * G + kvh) * dimP, *g = a.g + (t * H + h) * dimP;
+            const float *q = a.qn + (t * G + kvh) * dimP, *kk = a.kn + (t * G + kvh) * dimP, *g = HEAD_DECAY ? nullptr : a.g + (t * H + h) * dimP;
             const float* v = a.v + (t * H + h) * vdimP + cb;
             for (int p = lane * 4; p < dimP; p += 128) {
                 cp_async16(dst + p, q + p);
                 cp_async16(dst + dimP + p, kk + p);
-                cp_async16(dst + 2 * dimP + p, g + p);
+                if constexpr (!HEAD_DECAY) cp_async16(dst + 2 * dimP + p, g + p);
             }
-            for (int p = lane * 4; p < ncols; p += 128) cp_async16(dst + 3 * dimP + p, v + p);
-            if (lane == 0) cp_async8(dst + 3 * dimP + cols, a.bk + (t * H + h) * 2);
+            for (int p = lane * 4; p < ncols; p += 128) cp_async16(dst + vOff + p, v + p);
+            if (lane == 0) {
+                if constexpr (HEAD_DECAY) cp_async16(dst + vOff + cols, a.bk + (t * H + h) * 4);
+                else cp_async8(dst + vOff + cols, a.bk + (t * H + h) * 2);
+            }
         }
     };
     const int tiles = (count + kScanTokens - 1) / kScanTokens;
@@ -361,7 +371,7 @@ __global__ void __launch_bounds__(NT) k_delta_scan(const DeltaRule a, int cols, 
                 const int d = 4 * (r + 8 * j);
                 q4[j] = *(const ulonglong2*)(tok + d);
                 k4[j] = *(const ulonglong2*)(tok + dimP + d);
-                g4[j] = *(const ulonglong2*)(tok + 2 * dimP + d);
+                if constexpr (!HEAD_DECAY) g4[j] = *(const ulonglong2*)(tok + 2 * dimP + d);
             }
         };
         if (AHEAD) vectors(0);
@@ -371,12 +381,17 @@ __global__ void __launch_bounds__(NT) k_delta_scan(const DeltaRule a, int cols, 
             f32x2 t2[C], w2[C];
 #pragma unroll
             for (int c = 0; c < C; ++c) t2[c] = w2[c] = 0ull;
+            f32x2 gh = 0ull;
+            if constexpr (HEAD_DECAY) {
+                const float g = tok[vOff + cols + 2];
+                gh = pack2(g, g);
+            }
 #pragma unroll
             for (int j = 0; j < J; ++j) {
 #pragma unroll
                 for (int c = 0; c < C; ++c) {
-                    S[c][j][0] = mul2(S[c][j][0], g4[j].x);
-                    S[c][j][1] = mul2(S[c][j][1], g4[j].y);
+                    S[c][j][0] = mul2(S[c][j][0], HEAD_DECAY ? gh : g4[j].x);
+                    S[c][j][1] = mul2(S[c][j][1], HEAD_DECAY ? gh : g4[j].y);
                     t2[c] = fma2(S[c][j][0], k4[j].x, t2[c]);
                     w2[c] = fma2(S[c][j][0], q4[j].x, w2[c]);
                     t2[c] = fma2(S[c][j][1], k4[j].y, t2[c]);
@@ -389,7 +404,7 @@ __global__ void __launch_bounds__(NT) k_delta_scan(const DeltaRule a, int cols, 
                 for (int j = 0; j < J; ++j) kk[j] = k4[j];
                 vectors(min(k + 1, n - 1));
             }
-            const float2 bk = *(const float2*)(tok + 3 * dimP + cols);
+            const float2 bk = *(const float2*)(tok + vOff + cols);
             // Sums over the eight lanes by halving exchange (partners 4, 2, 1 lanes away): lane r ends with S^T k and
             // S^T q of column r (C = 8), or of column r & 3 with S^T k in lanes 0-3 and S^T q in lanes 4-7 (C = 4).
             float uc[C];
@@ -409,7 +424,7 @@ __global__ void __launch_bounds__(NT) k_delta_scan(const DeltaRule a, int cols, 
                 const float ts = ((r & 1) ? ty[1] : ty[0]) + __shfl_xor_sync(0xffffffffu, (r & 1) ? ty[0] : ty[1], 1);
                 const float ws = ((r & 1) ? wy[1] : wy[0]) + __shfl_xor_sync(0xffffffffu, (r & 1) ? wy[0] : wy[1], 1);
                 const int col = c0 + r;
-                const float v = col - cb < ncols ? tok[3 * dimP + (col - cb)] : 0.f;
+                const float v = col - cb < ncols ? tok[vOff + (col - cb)] : 0.f;
                 const float u = bk.x * (v - ts);
 #pragma unroll
                 for (int c = 0; c < 8; ++c) uc[c] = __shfl_sync(0xffffffffu, u, (lane & ~7) | c);
@@ -430,7 +445,7 @@ __global__ void __launch_bounds__(NT) k_delta_scan(const DeltaRule a, int cols, 
                 for (int c = 0; c < 2; ++c) x2[c] = ((r & 2) ? x4[c + 2] : x4[c]) + __shfl_xor_sync(0xffffffffu, (r & 2) ? x4[c] : x4[c + 2], 2);
                 const float x = ((r & 1) ? x2[1] : x2[0]) + __shfl_xor_sync(0xffffffffu, (r & 1) ? x2[0] : x2[1], 1);
                 const int col = c0 + (r & 3);
-                const float v = col - cb < ncols ? tok[3 * dimP + (col - cb)] : 0.f;
+                const float v = col - cb < ncols ? tok[vOff + (col - cb)] : 0.f;
                 const float u = bk.x * (v - x);  // meaningful in lanes r < 4
 #pragma unroll
                 for (int c = 0; c < 4; ++c) uc[c] = __shfl_sync(0xffffffffu, u, (lane & ~7) | c);
@@ -502,24 +517,29 @@ __global__ void __launch_bounds__(kPrepWarps * 32) k_delta_out(const DeltaRule a
     if (threadIdx.x == 0) tl_mark(tl, 2);
 }
 
-template <typename A, int J, int C, bool FUSED, int NT>
+template <typename A, int J, int C, bool FUSED, int NT, bool HD>
 cudaError_t scan_attr() {
-    cudaError_t e = cudaFuncSetAttribute(k_delta_scan<A, J, C, FUSED, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         (int)scan_smem(32 * J, 256, true));
-    return e == cudaSuccess ? prefer_max_shared(k_delta_scan<A, J, C, FUSED, NT>) : e;
+    cudaError_t e = cudaFuncSetAttribute(k_delta_scan<A, J, C, FUSED, NT, HD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         (int)scan_smem(32 * J, 256, true, HD));
+    return e == cudaSuccess ? prefer_max_shared(k_delta_scan<A, J, C, FUSED, NT, HD>) : e;
 }
 // FUSED blocks hold a whole head of up to 256 columns; the others 128 threads, 128 columns (C = 8) or 64 (C = 4). Eight
 // columns of more than 128 key channels do not fit a lane's registers, and heads that wide are not fused.
-template <typename A, int J>
-cudaError_t scan_attrs() {
+template <typename A, int J, bool HD>
+cudaError_t scan_attrs_hd() {
     cudaError_t e = cudaSuccess;
     if constexpr (J <= 4) {
-        e = scan_attr<A, J, 8, true, 256>();
-        if (e == cudaSuccess) e = scan_attr<A, J, 4, true, 256>();
-        if (e == cudaSuccess) e = scan_attr<A, J, 8, false, 128>();
+        e = scan_attr<A, J, 8, true, 256, HD>();
+        if (e == cudaSuccess) e = scan_attr<A, J, 4, true, 256, HD>();
+        if (e == cudaSuccess) e = scan_attr<A, J, 8, false, 128, HD>();
     }
-    if (e == cudaSuccess) e = scan_attr<A, J, 4, false, 128>();
+    if (e == cudaSuccess) e = scan_attr<A, J, 4, false, 128, HD>();
     return e;
+}
+template <typename A, int J>
+cudaError_t scan_attrs() {
+    const cudaError_t e = scan_attrs_hd<A, J, false>();
+    return e == cudaSuccess ? scan_attrs_hd<A, J, true>() : e;
 }
 template <typename A>
 cudaError_t delta_attrs() {
@@ -536,22 +556,27 @@ cudaError_t delta_attrs() {
     return e;
 }
 
-template <typename A, int J>
-void launch_scan(const DeltaRule& a, int n_segs, bool fused, int num_sms, cudaStream_t s, bool pdl, unsigned long long* tl) {
+template <typename A, int J, bool HD>
+void launch_scan_hd(const DeltaRule& a, int n_segs, bool fused, int num_sms, cudaStream_t s, bool pdl, unsigned long long* tl) {
     auto go = [&](auto kernel, int C, int cols, bool f) {
         const int threads = (cols / C * 8 + 31) / 32 * 32;
-        launch_k(kernel, dim3(a.heads, n_segs, (a.vdimP + cols - 1) / cols), dim3(threads), scan_smem(32 * J, cols, f), s, pdl, a, cols, tl);
+        launch_k(kernel, dim3(a.heads, n_segs, (a.vdimP + cols - 1) / cols), dim3(threads), scan_smem(32 * J, cols, f, HD), s, pdl, a, cols, tl);
     };
     const int whole = (a.vdimP + 7) / 8 * 8;
     if constexpr (J <= 4) {
-        if (fused && a.heads * n_segs < num_sms && whole <= 128) return go(k_delta_scan<A, J, 4, true, 256>, 4, whole, true);
-        if (fused) return go(k_delta_scan<A, J, 8, true, 256>, 8, whole, true);
+        if (fused && a.heads * n_segs < num_sms && whole <= 128) return go(k_delta_scan<A, J, 4, true, 256, HD>, 4, whole, true);
+        if (fused) return go(k_delta_scan<A, J, 8, true, 256, HD>, 8, whole, true);
         // eight columns per lane need the fewest shared-memory reads; with few sequences half as many columns per lane
         // and twice the warps make a token's chain of steps shorter
         const long long warps = (long long)a.heads * n_segs * ((a.vdimP + 31) / 32);
-        if (warps >= 3ll * num_sms) return go(k_delta_scan<A, J, 8, false, 128>, 8, whole < 128 ? whole : 128, false);
+        if (warps >= 3ll * num_sms) return go(k_delta_scan<A, J, 8, false, 128, HD>, 8, whole < 128 ? whole : 128, false);
     }
-    go(k_delta_scan<A, J, 4, false, 128>, 4, whole < 64 ? whole : 64, false);
+    go(k_delta_scan<A, J, 4, false, 128, HD>, 4, whole < 64 ? whole : 64, false);
+}
+template <typename A, int J>
+void launch_scan(const DeltaRule& a, int n_segs, bool fused, int num_sms, cudaStream_t s, bool pdl, unsigned long long* tl) {
+    if (a.head_decay) launch_scan_hd<A, J, true>(a, n_segs, fused, num_sms, s, pdl, tl);
+    else launch_scan_hd<A, J, false>(a, n_segs, fused, num_sms, s, pdl, tl);
 }
 template <typename A>
 void launch_scan_j(const DeltaRule& a, int n_segs, bool fused, int num_sms, cudaStream_t s, bool pdl, unsigned long long* tl) {

@@ -131,7 +131,7 @@ Model* Model::load(const std::string& dir, int device, int tp_rank, int tp_size)
     static const struct {
         const char* family;
         void (Model::*load)(const std::string&);
-    } loaders[] = {{"Qwen2", &Model::load_qwen2}, {"Rafilix", &Model::load_stack}};
+    } loaders[] = {{"Qwen2", &Model::load_qwen2}, {"Rafilix", &Model::load_stack}, {"Razesun", &Model::load_stack}};
     for (const auto& l : loaders)
         if (m->cfg.family == l.family) {
             (m.get()->*l.load)(dir);
@@ -665,7 +665,8 @@ const char* kclass_name(int c) {
                                           "gemm_tc:o_proj", "gemm_tc:gate_up_swiglu", "gemm_tc:down", "gemm_tc:lm_head",
                                           "argmax_rows", "decode_advance", "bs1_qkv", "bs1_oproj", "bs1_ffn", "bs1_lmhead", "tp_all_reduce",
                                           "residual_rows", "gemm:mixer_in", "qk_norm_rope", "gemm:low_rank", "delta_prep", "delta_scan", "delta_out",
-                                          "gemm:router", "moe_route", "moe_gather", "gemm:expert_up", "gemm:expert_down"};
+                                          "gemm:router", "moe_route", "moe_gather", "gemm:expert_up", "gemm:expert_down",
+                                          "latent_prep", "gemm:query_up", "gemm:key_fold", "latent_rope", "gemm:value_up", "lru_prep", "gemm:lru_gates", "lru_scan", "gemm:out_down"};
     return (c >= 0 && c < KC_COUNT) ? names[c] : "?";
 }
 void Session::set_profile(bool on) {
@@ -740,7 +741,7 @@ int Session::build_groups(const int* seq, const int* pos, int T, int limit, int3
 
 // one GEMM of a step: tensor cores, or true fp32 in a session that computes in fp32
 void Session::gemm(GemmCall& call, int cls, bool pdl) {
-    if ((ablate_mask_ >> cls) & 1u) return;  // timing-only ablation: results are then meaningless
+    if (ablated(cls)) return;  // timing-only ablation: results are then meaningless
     call.pdl = pdl;
     call.tl = tl_next(cls);
     call.trace = (tl_on_ && (int)tl_cls_.size() - 1 == tl_trace_launch_) ? tl_trace_buf_.as<unsigned long long>() : nullptr;
@@ -776,7 +777,7 @@ Session::Staged Session::stage_rows(const int32_t* tsp, int T) {
 void Session::lm_head(const void* x, int64_t ldx, int n_rows, bool decode, bool pdl) {
     const int V = m_->cfg.vocab_size, Vl = m_->V;
     const bool tp = tp_ != nullptr;
-    auto live = [&](int cls) { return ((ablate_mask_ >> cls) & 1u) == 0; };
+    auto live = [&](int cls) { return !ablated(cls); };
     GemmCall g;
     memset(&g, 0, sizeof g);
     g.x_rows_alloc = cap_tokens_;
@@ -791,12 +792,13 @@ void Session::lm_head(const void* x, int64_t ldx, int n_rows, bool decode, bool 
     // idle by now and serves as scratch.
     const AttnWorkspace aw = attn_ws();
     const int v_tiles = (Vl + 127) / 128;
-    const bool fused_pick = !sampling() && !(st_ && st_->f32) && (size_t)n_rows * v_tiles * 2 <= aw.partial_floats;
+    const bool fused_pick = !sampling() && m_->cfg.logit_scale > 0.f /* the tiles' maxima are taken before the scale */ && !(st_ && st_->f32) && (size_t)n_rows * v_tiles * 2 <= aw.partial_floats;
     if (tp && !fused_pick) throw Error(kErrUnsupported, "tensor parallel: sampling and very large logit batches are not split across ranks");
     if (fused_pick) {
         g.amax_val = aw.partials;
         g.amax_idx = (int*)(aw.partials + (size_t)n_rows * v_tiles);
     }
+    g.out_scale = m_->cfg.logit_scale;
     g.out = (store_logits_ || !fused_pick) ? logits_.p : nullptr;
     gemm(g, KC_GEMM_LMHEAD, pdl);
     prof_begin(KC_ARGMAX);
@@ -869,7 +871,7 @@ void Session::run_batched(int T, int n_logit_rows, bool logit_rows_are_all, bool
     const int* tok_pos = decode ? seq_len_dev_.as<int>() : tok_pos_.as<int>();
     int* status = status_.as<int>();
     // timing-only ablation: a class in the mask is not launched (results are then meaningless)
-    auto live = [&](int cls) { return ((ablate_mask_ >> cls) & 1u) == 0; };
+    auto live = [&](int cls) { return !ablated(cls); };
     prof_begin(KC_EMBED);
     launch_embed(tokens, m_->embed.as<bf16>(), h_.as<bf16>(), T, H, V, status, stream_, false, tl_next(KC_EMBED));
     prof_end();

@@ -61,7 +61,9 @@ struct LayerWeights {
 
 // One entry of a layer list (Config::layers): weights as the kernels read them. Matrices bf16 with rows padded to 8
 // elements, vectors widened to fp32. w_in stacks every projection of the mixer's input (each block of rows padded to
-// 8), so that one GEMM makes them all: q | k | v (attention) or q | k | v | b | a1 | g1 (delta rule).
+// 8), so that one GEMM makes them all: q | k | v (attention), q | k | v | b | a1 | g1 (delta rule, decay and gate of low
+// rank), q | k | v | b | a | g (delta rule, one decay per head), dq | dkv | g (latent attention; dkv in a1_off, g in
+// g1_off) or y | x (real-gated recurrence; x in a1_off).
 struct StackLayer {
     LayerSpec spec;
     int in_rows = 0, k_off = 0, v_off = 0, b_off = 0, a1_off = 0, g1_off = 0;
@@ -70,7 +72,15 @@ struct StackLayer {
     DeviceBuffer norm1, norm1b, norm2, norm2b;  // in front of and behind the mixer and the feed-forward
     DeviceBuffer q_norm, k_norm;
     DeviceBuffer conv, a_log, dt_bias, out_norm;  // conv: [taps][channels]
-    DeviceBuffer router, correction, up, down;    // up [experts * ff][width], down [experts * width][ff]
+    // Latent attention. uq: the heads' unrotated rows (each head padded to 8), then the rotated rows of all heads
+    // [q_rows][q_rank]; uk: per head the transposed matrix [kv_rank][dim], which folds the key projection into the
+    // query; uv [heads * vdim][kv_rank].
+    DeviceBuffer uq, uk, uv, dq_norm, dkv_norm;
+    int q_rows = 0;
+    // Real-gated recurrence: gates of a part as 2 n rows [r | i][n], n = channels of a part; biases alike.
+    DeviceBuffer lru_gates, lru_gate_bias, lru_lam, conv_bias, x_bias, y_bias;
+    // feed-forward: up [experts * ff][width], down [experts * width][ff]; dense: gate and up [ff][width], down [width][ff]
+    DeviceBuffer router, correction, gate, up, down;
 };
 inline int64_t pad8(int64_t n) { return (n + 7) & ~(int64_t)7; }
 
@@ -98,8 +108,8 @@ struct Model {
     const bf16* lm_head = nullptr;
     std::vector<LayerWeights> layers;
     std::vector<StackLayer> stack;  // instead of `layers` when the configuration lists its layers
-    int64_t embed_ld = 0;           // row stride of embed (and of the LM head)
-    DeviceBuffer final_norm_f32;
+    int64_t embed_ld = 0;           // row stride of embed and of the LM head
+    DeviceBuffer final_norm_f32, embed_norm_f32;
     bool bs1_ok = false;
     uint64_t weight_bytes_base = 0;  // bytes one decode step streams (every matrix once, LM head included)
     static Model* load(const std::string& dir, int device, int tp_rank, int tp_size);
@@ -127,7 +137,8 @@ enum KClass : int {
     KC_EMBED = 0, KC_RMSNORM, KC_GEMM_QKV, KC_ATTENTION, KC_GEMM_OPROJ, KC_GEMM_GATEUP, KC_GEMM_DOWN,
     KC_GEMM_LMHEAD, KC_ARGMAX, KC_ADVANCE, KC_BS1_QKV, KC_BS1_OPROJ, KC_BS1_FFN, KC_BS1_LMHEAD, KC_ALLREDUCE,
     KC_ROWS, KC_GEMM_IN, KC_QK_ROPE, KC_GEMM_LOWRANK, KC_DELTA_PREP, KC_DELTA_SCAN, KC_DELTA_OUT, KC_GEMM_ROUTER, KC_ROUTE, KC_GATHER,
-    KC_GEMM_UP, KC_GEMM_EXPERT_DOWN, KC_COUNT
+    KC_GEMM_UP, KC_GEMM_EXPERT_DOWN, KC_LATENT_PREP, KC_GEMM_UQ, KC_GEMM_UK, KC_LATENT_ROPE, KC_GEMM_UV, KC_LRU_PREP, KC_GEMM_LRU, KC_LRU_SCAN,
+    KC_GEMM_OUT_DOWN, KC_COUNT
 };
 const char* kclass_name(int c);
 
@@ -138,10 +149,10 @@ struct StackState {
     bool f32 = false;
     size_t act = 2;  // bytes of an activation
     struct LayerCache {
-        DeviceBuffer k, v;         // attention: pages of this layer
-        KvView kv;
+        DeviceBuffer k, v;         // attention: pages of this layer (latent attention: one pool for both)
+        KvView kv;                 // latent attention with kv_from: the other layer's
         int rope = -1;             // index into rope
-        DeviceBuffer state, ring;  // delta rule: see DeltaRule
+        DeviceBuffer state, ring;  // recurrent mixers: see DeltaRule and RgLru
         size_t state_stride = 0, ring_stride = 0;
         int dimP = 0, vdimP = 0;
         int moe = -1;              // index of the layer among those with experts
@@ -152,6 +163,10 @@ struct StackState {
     int64_t h_ld = 0, proj_ld = 0, ctx_ld = 0, decay_ld = 0, gate_ld = 0, delta_ld = 0, router_ld = 0, act_ld = 0;
     int max_top = 0, max_experts = 0, moe_layers = 0, max_tiles = 0;
     DeviceBuffer proj, delta, qn, kn, v, g, bk, o, decay, gate;
+    DeviceBuffer xn2, ff_act;                 // dense feed-forward beside the mixer: its input, gated activations
+    DeviceBuffer cq, q_up, o_lat, u, lru_gate;  // latent attention; real-gated recurrence
+    int64_t cq_ld = 0, q_up_ld = 0, u_ld = 0, lru_gate_ld = 0;
+    size_t o_lat_cols = 0;
     DeviceBuffer router, counts, pair, pair_w, pair_row, xg, act_e, y, tiles;
     DeviceBuffer seg_first, seg_count, ones;
 };
@@ -220,6 +235,7 @@ private:
     bool own_stream_ = false;
     int launch_mode_ = 1;
     unsigned ablate_mask_ = 0;
+    bool ablated(int cls) const { return cls < 32 && ((ablate_mask_ >> cls) & 1u); }
     float sample_temp_ = 0.f;
     std::mt19937 sample_rng_{42};
     DeviceBuffer sample_u_;
@@ -291,6 +307,7 @@ private:
     void alloc_stack(bool f32);
     void run_stack(int T, int n_logit_rows, bool logit_rows_are_all, bool decode, int max_ctx, int n_groups, int n_segs);
     int attn_ctx(const LayerSpec& l, int max_ctx) const { return l.chunk > 0 && l.chunk < max_ctx ? l.chunk : max_ctx; }
+    int rope_table(const RopeSpec& spec);
     AttnOptions attn_options(const LayerSpec& l) const;
     // everything in a captured decode step's grids that depends on the context
     int decode_graph_key(int n_seqs, int max_ctx) const;

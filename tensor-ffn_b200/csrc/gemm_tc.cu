@@ -49,6 +49,7 @@ struct GemmDev {
     GemmQkvEpilogue qkv;  // GEMM_QKV only
     unsigned long long* trace;  // optional: 64 timestamps (ns) per CTA, see GemmCall::trace
     unsigned long long* tl;     // optional: step timeline of this launch
+    int batch, out_batch;       // batched launch (GemmCall::batch): X is a 3-D map (column, problem, row)
     const GroupTile* grp;       // grouped launch: one entry per token tile (blockIdx.y), see GemmCall::grp
     float* amax_val;            // GEMM_STORE_F32: per (token, tile) maximum and its index, or nullptr
     int* amax_idx;
@@ -168,7 +169,7 @@ __device__ __forceinline__ void finalize_qkv(const GemmDev& p, int n, int t, flo
     *(uint2*)dst = pack_bf16x4(o[0], o[1], o[2], o[3]);
 }
 
-__device__ __forceinline__ bool plain_is_vector(const GemmDev& p, int n) { return (n + 3 < p.N) && ((p.ldo & 3) == 0); }
+__device__ __forceinline__ bool plain_is_vector(const GemmDev& p, int n) { return (n + 3 < p.N) && (((p.ldo | p.out_batch) & 3) == 0); }
 
 // GEMM_RESIDUAL: the old values of rows n .. n+3 of token t (read through L2)
 __device__ __forceinline__ void prefetch_residual(const GemmDev& p, const void* out, int n, int t, FinalizePre& f) {
@@ -281,7 +282,7 @@ __global__ void __launch_bounds__(kGemmThreads, (BN <= 64) ? 2 : 1) k_gemm_tc(co
     uint32_t* tmem_slot = (uint32_t*)(acc_full + 1);
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int prob = blockIdx.y / p.t_tiles;  // independent problems (base / expert gate-up) share a launch
+    int prob = blockIdx.y / p.t_tiles;  // independent problems (base / expert gate-up) share a launch
     const int n0 = blockIdx.x * p.tile_n;
     int t0 = (blockIdx.y % p.t_tiles) * BN, t_end = p.T, w_row0 = n0;
     if (p.grp) {
@@ -295,8 +296,18 @@ __global__ void __launch_bounds__(kGemmThreads, (BN <= 64) ? 2 : 1) k_gemm_tc(co
         t_end = min(g.z, g.y + BN);
         w_row0 = g.x * p.N + n0;
     }
+    const bool batched = p.batch > 1;
+    const int prob_b = prob;
+    if (batched) {  // the problems share operand maps and output
+        w_row0 = prob_b * p.N + n0;
+        prob = 0;
+    }
     const bool halves = p.mode == GEMM_SWIGLU;  // A tile = 64 gate rows over 64 up rows, one accumulator
-    void* const out = p.out[prob];
+    void* out = p.out[prob];
+    if (batched) {
+        if (p.mode == GEMM_STORE_F32) out = (float*)out + (size_t)prob_b * p.out_batch;
+        else out = (bf16*)out + (size_t)prob_b * p.out_batch;
+    }
     const int total_kb = p.kblocks[0] + p.kblocks[1];
     const int kb_begin = (int)(((long long)blockIdx.z * total_kb) / p.splits);
     const int kb_end = (int)(((long long)(blockIdx.z + 1) * total_kb) / p.splits);
@@ -354,7 +365,9 @@ __global__ void __launch_bounds__(kGemmThreads, (BN <= 64) ? 2 : 1) k_gemm_tc(co
                 const int i = kb_begin + it;
                 const int seg = i >= p.kblocks[0] ? 1 : 0;
                 const int kb = seg ? i - p.kblocks[0] : i;
-                tma_load_2d(smem + it * Cfg::STAGE_BYTES + Cfg::A_BYTES, &p.tmX[prob * 2 + seg], kb * BK, t0, &full[it]);
+                uint8_t* b = smem + it * Cfg::STAGE_BYTES + Cfg::A_BYTES;
+                if (batched) tma_load_3d(b, &p.tmX[0], kb * BK, prob_b, t0, &full[it]);
+                else tma_load_2d(b, &p.tmX[prob * 2 + seg], kb * BK, t0, &full[it]);
             }
             for (int it = pre; it < n_iters; ++it) {
                 const int s = it % STAGES;
@@ -372,7 +385,8 @@ __global__ void __launch_bounds__(kGemmThreads, (BN <= 64) ? 2 : 1) k_gemm_tc(co
                 } else {
                     tma_load_2d(a, &p.tmW[prob * 2 + seg], kb * BK, w_row0, &full[s]);
                 }
-                tma_load_2d(b, &p.tmX[prob * 2 + seg], kb * BK, t0, &full[s]);
+                if (batched) tma_load_3d(b, &p.tmX[0], kb * BK, prob_b, t0, &full[s]);
+                else tma_load_2d(b, &p.tmX[prob * 2 + seg], kb * BK, t0, &full[s]);
             }
         }
     } else if (warp == 1) {
@@ -619,29 +633,29 @@ struct TmapKey {
     const void* ptr;
     uint64_t rows, cols, ld;
     uint32_t box_rows;
+    uint32_t batch, batch_ld;
     bool operator==(const TmapKey& o) const {
-        return ptr == o.ptr && rows == o.rows && cols == o.cols && ld == o.ld && box_rows == o.box_rows;
+        return ptr == o.ptr && rows == o.rows && cols == o.cols && ld == o.ld && box_rows == o.box_rows && batch == o.batch && batch_ld == o.batch_ld;
     }
 };
 struct TmapKeyHash {
     size_t operator()(const TmapKey& k) const {
-        return std::hash<const void*>()(k.ptr) ^ (k.rows * 1000003u) ^ (k.cols * 7919u) ^ (k.ld << 20) ^ k.box_rows;
+        return std::hash<const void*>()(k.ptr) ^ (k.rows * 1000003u) ^ (k.cols * 7919u) ^ (k.ld << 20) ^ k.box_rows ^ ((size_t)k.batch * 104729u);
     }
 };
 
-bool encode_tmap(CUtensorMap* tm, const bf16* ptr, uint64_t rows, uint64_t cols, uint64_t ld_elems, uint32_t box_rows);
-
-bool make_tmap(TmapCache* cache, CUtensorMap* tm, const bf16* ptr, uint64_t rows, uint64_t cols, uint64_t ld_elems, uint32_t box_rows);
-
-// 2-D bf16 tensor [rows, cols] with a row stride, box = box_rows x 64 columns, 128-byte swizzle
-bool encode_tmap(CUtensorMap* tm, const bf16* ptr, uint64_t rows, uint64_t cols, uint64_t ld_elems, uint32_t box_rows) {
+// bf16 tensor [rows, cols] with a row stride, box = box_rows x 64 columns, 128-byte swizzle. batch > 1: `batch` such
+// tensors interleaved in a row, batch_ld elements apart; 3-D (column, problem, row), a box of one problem
+bool encode_tmap(CUtensorMap* tm, const bf16* ptr, uint64_t rows, uint64_t cols, uint64_t ld_elems, uint32_t box_rows, uint32_t batch,
+                 uint32_t batch_ld) {
     EncodeTiledFn enc = get_encode();
     if (!enc) return false;
-    cuuint64_t dims[2] = {cols, rows};
-    cuuint64_t strides[1] = {ld_elems * 2};
-    cuuint32_t box[2] = {(cuuint32_t)BK, box_rows};
-    cuuint32_t estr[2] = {1, 1};
-    CUresult r = enc(tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (void*)ptr, dims, strides, box, estr,
+    const bool b = batch > 1;
+    cuuint64_t dims[3] = {cols, b ? batch : rows, rows};
+    cuuint64_t strides[2] = {(b ? batch_ld : ld_elems) * 2, ld_elems * 2};
+    cuuint32_t box[3] = {(cuuint32_t)BK, b ? 1u : box_rows, box_rows};
+    cuuint32_t estr[3] = {1, 1, 1};
+    CUresult r = enc(tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, b ? 3 : 2, (void*)ptr, dims, strides, box, estr,
                      CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                      CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     return r == CUDA_SUCCESS;
@@ -657,15 +671,16 @@ void tmap_cache_free(TmapCache* c) { delete c; }
 
 namespace {
 
-bool make_tmap(TmapCache* cache, CUtensorMap* tm, const bf16* ptr, uint64_t rows, uint64_t cols, uint64_t ld_elems, uint32_t box_rows) {
-    if (!cache) return encode_tmap(tm, ptr, rows, cols, ld_elems, box_rows);
-    TmapKey key{ptr, rows, cols, ld_elems, box_rows};
+bool make_tmap(TmapCache* cache, CUtensorMap* tm, const bf16* ptr, uint64_t rows, uint64_t cols, uint64_t ld_elems, uint32_t box_rows,
+               uint32_t batch = 1, uint32_t batch_ld = 0) {
+    if (!cache) return encode_tmap(tm, ptr, rows, cols, ld_elems, box_rows, batch, batch_ld);
+    TmapKey key{ptr, rows, cols, ld_elems, box_rows, batch, batch_ld};
     auto it = cache->maps.find(key);
     if (it != cache->maps.end()) {
         *tm = it->second;
         return true;
     }
-    if (!encode_tmap(tm, ptr, rows, cols, ld_elems, box_rows)) return false;
+    if (!encode_tmap(tm, ptr, rows, cols, ld_elems, box_rows, batch, batch_ld)) return false;
     cache->maps.emplace(key, *tm);
     return true;
 }
@@ -698,28 +713,33 @@ int launch_bn(const GemmCall& c, const GemmWorkspace& ws, cudaStream_t stream, i
     using Cfg = GemmCfg<BN>;
     GemmDev p;
     memset(&p, 0, sizeof p);
-    const int nprob = c.out2 ? 2 : 1;
+    const bool batched = c.batch > 1;
+    const int maps = c.out2 ? 2 : 1, nprob = batched ? c.batch : maps;
     const bool halves = c.mode == GEMM_SWIGLU;
     p.tile_n = halves ? BM / 2 : BM;
     if (halves && (c.op[0].K != c.op[1].K || c.op[0].X != c.op[1].X)) return (int)cudaErrorInvalidValue;
-    for (int pr = 0; pr < nprob; ++pr)
+    if (batched && (c.out2 || c.grp || c.op[1].K > 0 || c.x_batch % 8 || (c.mode != GEMM_STORE_F32 && c.mode != GEMM_STORE_BF16) || c.amax_val))
+        return (int)cudaErrorInvalidValue;
+    for (int pr = 0; pr < maps; ++pr)
         for (int i = 0; i < 2; ++i) {
             const GemmOperand& o = pr ? c.op2[i] : c.op[i];
             if (pr == 0) p.kblocks[i] = o.K > 0 ? (o.K + BK - 1) / BK : 0;
             if (o.K <= 0) continue;
             if (pr == 1 && (o.K + BK - 1) / BK != p.kblocks[i]) return (int)cudaErrorInvalidValue;
-            const uint64_t w_rows = (uint64_t)c.N * (c.grp ? c.grp_count : 1);
+            const uint64_t w_rows = (uint64_t)c.N * (c.grp ? c.grp_count : batched ? c.batch : 1);
             if (!make_tmap(ws.tmaps, &p.tmW[pr * 2 + i], o.W, w_rows, (uint64_t)o.K, (uint64_t)o.ldw, halves ? BM / 2 : BM)) return -1000;
             if (!make_tmap(ws.tmaps, &p.tmX[pr * 2 + i], o.X, (uint64_t)(c.x_rows_alloc > c.T ? c.x_rows_alloc : c.T), (uint64_t)o.K,
-                           (uint64_t)o.ldx, BN))
+                           (uint64_t)o.ldx, BN, batched ? (uint32_t)c.batch : 1u, (uint32_t)c.x_batch))
                 return -1000;
         }
     if (halves) p.kblocks[1] = 0;  // gate and up rows share one accumulator and one pass over K
     for (int i = 1; i < 4; ++i)  // keep unused maps valid
-        if (i >= nprob * 2 || (p.kblocks[i & 1] == 0 && !halves)) {
+        if (i >= maps * 2 || (p.kblocks[i & 1] == 0 && !halves)) {
             p.tmW[i] = p.tmW[0];
             p.tmX[i] = p.tmX[0];
         }
+    p.batch = batched ? c.batch : 1;
+    p.out_batch = batched ? c.out_batch : 0;
     p.N = c.N;
     p.T = c.T;
     p.mode = c.mode;

@@ -56,7 +56,7 @@ static Config read_qwen2(const JsonValue& j) {
     return c;
 }
 
-// ---------------------------------------------------------------- layer lists (Rafilix)
+// ---------------------------------------------------------------- layer lists (Rafilix, Razesun)
 // Every size and constant is stated by the file; nothing has a default.
 static const JsonValue& need_key(const JsonValue& j, const char* key, const std::string& where) {
     const JsonValue* v = j.find(key);
@@ -106,65 +106,128 @@ double rope_frequency(const RopeSpec& r, int i) {
     return (1.0 - s) * f / r.factor + s * f;
 }
 
-static LayerSpec read_layer(const JsonValue& j, const std::string& where) {
-    LayerSpec l;
-    const JsonValue& type = need_key(j, "type", where);
-    const JsonValue& m = need_key(j, "mixer", where);
-    const std::string mw = where + ".mixer";
+// ---- mixers: `m` is the layer's 'mixer' entry
+static void read_heads(const JsonValue& m, const std::string& mw, LayerSpec& l) {
     l.heads = need_size(m, "heads", mw);
     l.kv_heads = need_size(m, "kv_heads", mw);
     l.dim = need_size(m, "dim", mw);
     l.vdim = need_size(m, "vdim", mw);
     if (l.heads % l.kv_heads != 0) throw Error(kErrFormat, "config.json: " + mw + ": kv_heads do not divide heads");
-    if (type.is_string() && type.str == "attention") {
-        l.mixer = Mixer::Attention;
-        l.scale = (float)need_number(m, "scale", mw);
-        if (has_value(m, "rot")) l.rope = read_rope(need_key(m, "rot", mw), l.dim, mw + ".rot");
-        if (has_value(m, "mask")) l.chunk = need_size(need_key(m, "mask", mw), "size", mw + ".mask");
-    } else if (type.is_string() && type.str == "channel_delta") {
-        l.mixer = Mixer::ChannelDelta;
-        l.conv = need_size(m, "conv", mw);
-    } else {
-        throw Error(kErrUnsupported, "config.json: " + where + ": unknown layer type '" + type.str + "'");
-    }
+}
+static void read_attention(const JsonValue& m, const std::string& mw, LayerSpec& l) {
+    l.mixer = Mixer::Attention;
+    read_heads(m, mw, l);
+    l.scale = (float)need_number(m, "scale", mw);
+    if (has_value(m, "rot")) l.rope = read_rope(need_key(m, "rot", mw), l.dim, mw + ".rot");
+    if (has_value(m, "mask")) l.chunk = need_size(need_key(m, "mask", mw), "size", mw + ".mask");
+}
+static void read_channel_delta(const JsonValue& m, const std::string& mw, LayerSpec& l) {
+    l.mixer = Mixer::ChannelDelta;
+    read_heads(m, mw, l);
+    l.conv = need_size(m, "conv", mw);
+}
+static void read_delta(const JsonValue& m, const std::string& mw, LayerSpec& l) {
+    read_channel_delta(m, mw, l);
+    l.mixer = Mixer::Delta;
+}
+static void read_latent_attention(const JsonValue& m, const std::string& mw, LayerSpec& l) {
+    l.mixer = Mixer::LatentAttention;
+    l.heads = need_size(m, "heads", mw);
+    l.kv_heads = 1;  // one cached row per token, whatever the heads
+    l.dim = need_size(m, "dim", mw);
+    l.vdim = need_size(m, "vdim", mw);
+    l.rot_dim = need_size(m, "rot_dim", mw);
+    l.kv_rank = need_size(m, "kv_rank", mw);
+    l.q_rank = has_value(m, "q_rank") ? need_size(m, "q_rank", mw) : 0;  // 0: as many as the tensor has rows
+    l.scale = (float)need_number(m, "scale", mw);
+    l.rope = read_rope(need_key(m, "rot", mw), l.rot_dim, mw + ".rot");
+    l.rope.halves = true;
+    if (l.rope.dims != l.rot_dim) throw Error(kErrFormat, "config.json: " + mw + ": rot.dims differs from rot_dim");
+    if (has_value(m, "kv_from")) l.kv_from = need_size(m, "kv_from", mw, 0);
+}
+static void read_rglru(const JsonValue& m, const std::string& mw, LayerSpec& l) {
+    l.mixer = Mixer::Rglru;
+    l.lru_width = need_size(m, "width", mw);
+    l.lru_blocks = need_size(m, "blocks", mw);
+    l.conv = need_size(m, "conv", mw);
+    if (l.lru_width % l.lru_blocks != 0) throw Error(kErrFormat, "config.json: " + mw + ": blocks do not divide width");
+}
+
+// ---- feed-forwards: `f` is the layer's 'mlp' entry
+static void read_moe(const JsonValue& f, const std::string& fw, LayerSpec& l) {
+    l.ff = need_size(need_key(f, "expert", fw), "ff", fw + ".expert");
+    const JsonValue& r = need_key(f, "router", fw);
+    l.experts = need_size(r, "experts", fw + ".router");
+    l.identity = has_value(r, "identity") ? need_size(r, "identity", fw + ".router", 0) : 0;
+    l.top = need_size(r, "top", fw + ".router");
+    if (l.top > l.experts + l.identity) throw Error(kErrFormat, "config.json: " + fw + ".router: top exceeds the number of experts");
+}
+static void read_dense(const JsonValue& f, const std::string& fw, LayerSpec& l) { l.ff = need_size(f, "ff", fw); }
+
+// what a family's layers may be made of: the names in its config.json and their readers
+struct LayerPart {
+    const char* name;
+    void (*read)(const JsonValue& entry, const std::string& where, LayerSpec& l);
+};
+static void read_part(const std::vector<LayerPart>& parts, const JsonValue& name, const char* what, const JsonValue& entry, const std::string& where,
+                      const std::string& entry_where, LayerSpec& l) {
+    for (const LayerPart& p : parts)
+        if (name.is_string() && name.str == p.name) return p.read(entry, entry_where, l);
+    throw Error(kErrUnsupported, "config.json: " + where + ": unknown " + what + " '" + name.str + "'");
+}
+static LayerSpec read_layer(const JsonValue& j, const std::string& where, const std::vector<LayerPart>& mixers, const std::vector<LayerPart>& mlps) {
+    LayerSpec l;
+    read_part(mixers, need_key(j, "type", where), "layer type", need_key(j, "mixer", where), where, where + ".mixer", l);
     if (has_value(j, "mlp")) {
-        const std::string fw = where + ".mlp";
         const JsonValue& f = need_key(j, "mlp", where);
-        const JsonValue& kind = need_key(f, "kind", fw);
-        if (kind.str != "moe") throw Error(kErrUnsupported, "config.json: " + fw + ": unknown kind '" + kind.str + "'");
-        l.ff = need_size(need_key(f, "expert", fw), "ff", fw + ".expert");
-        const JsonValue& r = need_key(f, "router", fw);
-        l.experts = need_size(r, "experts", fw + ".router");
-        l.identity = has_value(r, "identity") ? need_size(r, "identity", fw + ".router", 0) : 0;
-        l.top = need_size(r, "top", fw + ".router");
-        if (l.top > l.experts + l.identity) throw Error(kErrFormat, "config.json: " + fw + ".router: top exceeds the number of experts");
+        read_part(mlps, need_key(f, "kind", where + ".mlp"), "kind", f, where + ".mlp", where + ".mlp", l);
     }
     return l;
 }
 
-static Config read_rafilix(const JsonValue& j) {
+static Config read_layer_list(const JsonValue& j, const std::vector<LayerPart>& mixers, const std::vector<LayerPart>& mlps) {
     Config c;
     c.hidden_size = need_size(j, "width", "the model");
     c.vocab_size = need_size(j, "vocab", "the model");
     c.rms_norm_eps = (float)need_number(need_key(j, "norm", "the model"), "eps", "norm");
     const JsonValue& ls = need_key(j, "layers", "the model");
     if (!ls.is_array() || ls.arr.empty()) throw Error(kErrFormat, "config.json: 'layers' is not a list of layers");
-    for (size_t i = 0; i < ls.arr.size(); ++i) c.layers.push_back(read_layer(ls.arr[i], "layer " + std::to_string(i)));
+    for (size_t i = 0; i < ls.arr.size(); ++i) c.layers.push_back(read_layer(ls.arr[i], "layer " + std::to_string(i), mixers, mlps));
+    for (size_t i = 0; i < c.layers.size(); ++i) {
+        const LayerSpec& l = c.layers[i];
+        if (l.kv_from < 0) continue;
+        const LayerSpec* from = l.kv_from < (int)i ? &c.layers[l.kv_from] : nullptr;
+        if (!from || from->mixer != Mixer::LatentAttention || from->kv_from >= 0 || from->kv_rank != l.kv_rank || from->rot_dim != l.rot_dim ||
+            !(from->rope == l.rope))
+            throw Error(kErrFormat, "config.json: layer " + std::to_string(i) + ".mixer.kv_from names no earlier layer with rows of this kind");
+    }
     c.num_layers = (int)c.layers.size();
     const LayerSpec& l0 = c.layers[0];
-    c.num_heads = l0.heads;
-    c.num_kv_heads = l0.kv_heads;
-    c.head_dim = l0.dim;
+    c.num_heads = std::max(1, l0.heads);  // a recurrence without heads counts as one
+    c.num_kv_heads = std::max(1, l0.kv_heads);
+    c.head_dim = l0.mixer == Mixer::Rglru ? l0.lru_width : l0.dim + l0.rot_dim;
     c.intermediate_size = 0;
     c.rope_theta = 0.f;
     for (const LayerSpec& l : c.layers) {
         c.intermediate_size = std::max(c.intermediate_size, l.ff);
-        if (l.mixer == Mixer::Attention && c.rope_theta == 0.f) c.rope_theta = (float)l.rope.base;
+        if (l.rope.dims > 0 && c.rope_theta == 0.f) c.rope_theta = (float)l.rope.base;
     }
     c.max_seq_len = 1 << 30;  // no table of positions is stored
     c.eos_token_id = first_int(j, "eos_token_id", -1);
     c.bos_token_id = first_int(j, "bos_token_id", -1);
     c.tie_embeddings = true;
+    return c;
+}
+static Config read_rafilix(const JsonValue& j) {
+    return read_layer_list(j, {{"attention", read_attention}, {"channel_delta", read_channel_delta}}, {{"moe", read_moe}});
+}
+static Config read_razesun(const JsonValue& j) {
+    Config c = read_layer_list(j, {{"latent_attention", read_latent_attention}, {"delta", read_delta}, {"rglru", read_rglru}}, {{"dense", read_dense}});
+    c.block = Block::Parallel;
+    c.residual_mult = (float)need_number(j, "residual_mult", "the model");
+    c.logit_scale = (float)need_number(j, "logit_scale", "the model");
+    c.embed_norm = true;
+    c.tie_embeddings = false;
     return c;
 }
 
@@ -177,6 +240,7 @@ static bool names_itself(const JsonValue& j, const char* name) {
 const std::vector<ModelFamily>& model_families() {
     static const std::vector<ModelFamily> families = {
         {"Rafilix", [](const JsonValue& j) { return names_itself(j, "Rafilix"); }, read_rafilix},
+        {"Razesun", [](const JsonValue& j) { return names_itself(j, "Razesun"); }, read_razesun},
         {"Qwen2", [](const JsonValue& j) { return j.find("architecture") == nullptr; }, read_qwen2},
     };
     return families;

@@ -28,19 +28,24 @@ enum { kOk = 0, kErrInvalid = -1, kErrIO = -2, kErrFormat = -3, kErrShape = -4, 
 // the uniform Qwen2 fields; the uniform fields then hold what is common (width, vocabulary, layer count, eps) or
 // the first layer's value.
 struct RopeSpec {
-    int dims = 0;         // rotated leading dimensions of a head (0: none), neighbours (2i, 2i + 1) form a pair
+    int dims = 0;         // rotated leading dimensions of a head (0: none)
+    bool halves = false;  // pairs are (i, i + dims / 2) instead of the neighbours (2i, 2i + 1)
     double base = 10000.0;
     bool scaled = false;  // wavelength-dependent frequency scaling: long waves / factor, short ones kept, a ramp between
     double factor = 1.0, low = 1.0, high = 1.0, original = 1.0;
     bool operator==(const RopeSpec& o) const {
-        return dims == o.dims && base == o.base && scaled == o.scaled && factor == o.factor && low == o.low && high == o.high &&
+        return dims == o.dims && halves == o.halves && base == o.base && scaled == o.scaled && factor == o.factor && low == o.low && high == o.high &&
                original == o.original;
     }
 };
 // frequency of pair i (radians per position)
 double rope_frequency(const RopeSpec& r, int i);
 
-enum class Mixer { Attention, ChannelDelta };
+// ChannelDelta and Delta: gated delta rule with one decay per head and key channel, or per head.
+// LatentAttention: keys and values of all heads are projections of one cached latent per token, and one rotated key part
+// is shared by the heads. Rglru: a recurrence with one real decay per channel behind a short convolution.
+enum class Mixer { Attention, ChannelDelta, Delta, LatentAttention, Rglru };
+inline bool is_delta(Mixer m) { return m == Mixer::ChannelDelta || m == Mixer::Delta; }
 struct LayerSpec {
     Mixer mixer = Mixer::Attention;
     int heads = 0, kv_heads = 0;  // query (value) heads; key/value (query/key) heads they share
@@ -49,10 +54,22 @@ struct LayerSpec {
     int chunk = 0;                // a position sees the keys of its own chunk of this many positions (0: every earlier key)
     float scale = 0.f;            // factor of the scores
     RopeSpec rope;
-    // gated delta rule with one decay per key channel
+    // latent attention (dim: the unrotated part of a head's query and key)
+    int rot_dim = 0, kv_rank = 0, q_rank = 0;
+    int kv_from = -1;             // >= 0: reads what that earlier layer cached instead of caching rows of its own
+    // recurrent mixers
     int conv = 0;                 // taps of the short causal convolution
-    // feed-forward: a mixture of squared-ReLU experts (experts == 0: none)
+    // real-gated linear recurrence
+    int lru_width = 0, lru_blocks = 0;  // channels; equal parts of them that share a gate matrix
+    // feed-forward of `ff` columns (0: none): dense and SiLU-gated, or (experts > 0) a mixture of squared-ReLU experts
     int experts = 0, identity = 0, top = 0, ff = 0;
+    // channels that go into the mixer's output projection
+    int out_cols() const { return mixer == Mixer::Rglru ? lru_width : heads * vdim; }
+};
+// How a layer puts its sublayers on the residual stream.
+enum class Block {
+    PostNorm,  // x += norm(mixer(norm(x))), then x += norm(ff(norm(x)))
+    Parallel,  // x += residual_mult * (mixer(norm1(x)) + ff(norm2(x))), both of the same x
 };
 
 struct Config {
@@ -63,6 +80,10 @@ struct Config {
     float rms_norm_eps = 1e-6f, rope_theta = 1e6f;
     int eos_token_id = 151645, bos_token_id = 151643;
     bool tie_embeddings = true;
+    // layer lists
+    Block block = Block::PostNorm;
+    float residual_mult = 1.f, logit_scale = 1.f;
+    bool embed_norm = false;        // the residual stream starts with the normed embedding
 };
 Config read_config(const std::string& model_dir);
 

@@ -85,6 +85,10 @@ struct GemmCall {
     const struct GroupTile* grp;
     int grp_tiles, grp_bn, grp_count;  // grp_count: groups in W
     int grp_rows_hint;                 // tiles that will be in use, about (0: all)
+    // Batched launch (the heads of a per-head projection, the parts of a block-diagonal matrix): `batch` > 1 products of
+    // N rows of W each (back to back in W), problem b reading columns [b * x_batch, b * x_batch + K) of X and writing
+    // columns [b * out_batch, b * out_batch + N) of out. Modes STORE_F32 and STORE_BF16, op[0] only; x_batch a multiple of 8.
+    int batch, x_batch, out_batch;
 };
 struct GroupTile {
     int group;           // -1: this tile and all later ones are unused
@@ -93,8 +97,8 @@ struct GroupTile {
 };
 // token tile (16 .. 256) of a grouped launch whose groups hold `rows` rows on average
 int gemm_group_tile(int rows);
-// The same products in true fp32 (fp32 X and out, fp32 FMA, weights still bf16): modes STORE_F32, STORE_BF16 and
-// RELU2 (which then store fp32), one operand pair per problem, grouped launches included. The operands' X pointers
+// The same products in true fp32 (fp32 X and out, fp32 FMA, weights still bf16): modes STORE_F32, STORE_BF16, RELU2 and
+// SWIGLU (which then store fp32), grouped and batched launches included; two operand pairs only in a plain launch. The operands' X pointers
 // are fp32 arrays behind the bf16 type.
 int launch_gemm_f32(const GemmCall& c, cudaStream_t stream);
 constexpr int kGemmF32Tile = 64;  // its token tile (grp_bn)
@@ -184,6 +188,9 @@ struct AttnOptions {
     int chunk = 0;      // > 0: only the keys of the query's own chunk of `chunk` positions, counted from position 0
     int vdim = 0;       // > 0: columns of an output head (kv.vd is the padded row); 0: kv.vd
     int64_t ctx_ld = 0; // row stride of ctx (0: nh * vdim)
+    int head_ld = 0;    // (launch_attention_simt) columns between the heads of a ctx row (0: vdim)
+    const void* gate = nullptr;  // (launch_attention_simt) optional [T][gate_ld], stored like activations: head h's output times sigmoid(gate[t][h])
+    int64_t gate_ld = 0;
 };
 // opt the attention kernels into their dynamic shared memory (once per device, outside stream capture)
 int attn_prepare();
@@ -191,7 +198,7 @@ int attn_prepare();
 int attention_splits(int T, int nh, int nkv, int hd, int max_ctx, const AttnWorkspace& ws, int num_sms);
 // whether the tensor-core kernels take this head geometry (else launch_attention_simt)
 inline bool attention_tc_supported(int hd, int vd) { return hd <= 128 && vd <= 128; }
-// One warp-per-key-group attention without tensor cores: any head size up to 512, bf16 or (f32) fp32 cache and
+// One warp-per-key-group attention without tensor cores: any key size up to 2048 and value size up to 1024, bf16 or (f32) fp32 cache and
 // output, prompt and decode rows alike.
 void launch_attention_simt(const float* q, KvView kv, bool f32, const int* tok_seq, const int* tok_pos, void* ctx, int T, int nh,
                            const AttnOptions& opt, int* status, cudaStream_t s, bool pdl = false, unsigned long long* tl = nullptr);
@@ -225,8 +232,9 @@ struct MoeRoute {
     float* pair_w;            // [T][top] softmax score (without the correction)
 };
 enum RowSource : int { ROWS_KEEP = 0, ROWS_EMBED, ROWS_DELTA, ROWS_MOE };
-// One pass over the residual stream per sublayer: x = table[token] | x + norm(delta) * post_w | x + norm(sum of the
-// chosen experts' outputs) * post_w, then out = norm(x) * next_w. Norm: v / sqrt(mean(v^2) + eps). All in fp32.
+// One pass over the residual stream per sublayer: x = table[token] (or its norm * embed_w) | x + norm(delta) * post_w, or
+// x + delta_mult * delta without post_w | x + norm(sum of the chosen experts' outputs) * post_w; then out = norm(x) * next_w
+// and, for a second sublayer that reads the same x, out2 = norm(x) * next2_w. Norm: v / sqrt(mean(v^2) + eps). All in fp32.
 struct ResidualRows {
     float* x;                 // [T][H]
     int H;
@@ -244,9 +252,13 @@ struct ResidualRows {
     const int* pair_row;      // [T][top] row of y, or -1: the pair's output is the sublayer's input itself (`out` before this call)
     const float* pair_w;      // [T][top]
     int top;
+    const float* embed_w;     // ROWS_EMBED, optional
     const float* post_w;      // norm of the sublayer's output
+    float delta_mult;         // ROWS_DELTA without post_w
     const float* next_w;      // nullptr: no `out`
     void* out;                // [.][out_ld]
+    const float* next2_w;     // nullptr: no `out2`; only with next_w and without a router
+    void* out2;               // [.][out_ld]
     int64_t out_ld;
     const int* row_idx;       // with ROWS_KEEP: out row r = norm of x row row_idx[r]
     // Optional (rows_can_route): the router of the mixture that reads `out`, in the same pass. route.logits is not used.
@@ -258,6 +270,36 @@ int stack_rows_prepare();
 // few rows and a router small enough to be read once per row
 inline bool rows_can_route(int rows, int H, int outs) { return rows <= 128 && H % 8 == 0 && (size_t)H * outs * 2 <= (256u << 10); }
 void launch_residual_rows(const ResidualRows& a, bool f32, int rows, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
+
+// ------------------------------------------------------------------ latent attention
+// A cached row holds the normed latent at [0, rank), zeros up to a multiple of 64, then the rotated key part; it is the key
+// of every head (whose key projection is folded into the query) and its first `rank` columns are the value.
+constexpr int kLatentMaxRank = 1024;
+inline int latent_rot_col(int rank) { return (rank + 63) / 64 * 64; }
+inline int latent_row_cols(int rank, int rot) { return latent_rot_col(rank) + (rot + 7) / 8 * 8; }
+// Rows of the input projection -> normed query latent and, for a layer with rows of its own, the cached row.
+struct LatentPrep {
+    const void* proj;         // [T][ld]: query latent at 0, latent and unrotated key part at kv_off
+    int64_t ld;
+    int kv_off, q_rank, rank, rot;
+    bool own_rows;
+    const float *q_norm, *kv_norm;
+    float eps;
+    const float2* rope;       // [max_pos][rot / 2] (cos, sin); pairs (i, i + rot / 2)
+    int max_pos;
+    const int *tok_seq, *tok_pos;
+    void* cq;                 // [T][cq_ld]
+    int64_t cq_ld;
+    KvView kv;
+    int* status;
+};
+void launch_latent_prep(const LatentPrep& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
+// the heads' rotated query parts [T][ld] at column `off`, `rot` columns each -> fp32 columns [rot_col, rot_col + rot) of
+// q [T][heads][q_cols]
+void launch_latent_rope(const void* q_up, int64_t ld, int off, int heads, int rot, const float2* rope, int max_pos, const int* tok_pos,
+                        float* q, int q_cols, int rot_col, bool f32, int T, int* status, cudaStream_t s, bool pdl,
+                        unsigned long long* tl = nullptr);
+int latent_prepare();
 
 // q|k|v rows of one projection -> per-head norm of q and k (weights shared by the heads), rotation of neighbouring
 // pairs, q in fp32 for the attention kernels, k and v into the sequence's page.
@@ -277,7 +319,7 @@ struct QkNormRope {
 };
 void launch_qk_norm_rope(const QkNormRope& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
 
-// ------------------------------------------------------------------ gated delta rule, one decay per key channel
+// ------------------------------------------------------------------ gated delta rule, one decay per key channel or per head
 // Recurrent state of a slot: S [heads][vdimP][dimP] fp32 (transposed: a value column's keys are contiguous; dimP a
 // multiple of 32, vdimP of 4, the padding stays zero) and the last taps - 1 inputs of the convolution as a ring
 // [taps - 1][channels] fp32 addressed by position. A sequence that starts at position 0 starts from zeros whatever
@@ -290,19 +332,23 @@ struct DeltaRule {
     int q_off, k_off, v_off, b_off;
     const float* conv;        // [taps][channels], channels = q | k | v
     const float* a_log;       // [heads]
-    const float* dt_bias;     // [heads * dim]
-    const float* decay_in;    // [T][decay_ld]: W_a2 (W_a1 h)
+    bool head_decay;          // one decay per head instead of one per key channel
+    const float* dt_bias;     // [heads * dim], head_decay: [heads]
+    const float* decay_in;    // [T][decay_ld] decay logits; head_decay: in proj at a_off
     int64_t decay_ld;
-    const float* gate_in;     // [T][gate_ld]: W_g2 (W_g1 h)
+    int a_off;
+    const float* gate_in;     // [T][gate_ld] gate logits, or nullptr: in proj at gate_off
     int64_t gate_ld;
+    int gate_off;
+    bool gate_silu;           // the output gate is silu(logit), otherwise sigmoid(logit)
     const float* out_norm;    // [vdim]
     float *state, *ring;      // of slot 0
     size_t state_stride, ring_stride;  // floats between slots
     // per token, from the preparation to the scan
     float *qn, *kn;           // [T][kv_heads][dimP] unit vectors, q scaled
     float *v;                 // [T][heads][vdimP]
-    float *g;                 // [T][heads][dimP] decays
-    float *bk;                // [T][heads][2]: beta, k . q
+    float *g;                 // [T][heads][dimP] decays (not with head_decay)
+    float *bk;                // [T][heads][2]: beta, k . q; head_decay: [T][heads][4]: beta, k . q, decay, unused
     float* o;                 // [T][heads][vdimP] raw output rows
     void* out;                // [T][out_ld]
     int64_t out_ld;
@@ -320,6 +366,37 @@ void launch_delta_out(const DeltaRule& a, bool f32, int T, cudaStream_t s, bool 
 int delta_prepare();
 int delta_padded_dim(int dim);  // dimP
 inline bool delta_supported(int dim, int vdim) { return dim <= 256 && vdim <= 256; }
+
+// ------------------------------------------------------------------ real-gated linear recurrence
+// Per channel, behind a short causal convolution u: S = a S + sqrt(1 - a^2) i u with log a = -8 r softplus(lam), the gates
+// r and i sigmoids of block-diagonal products of u; the mixer's row is S * gelu(y). State of a slot: S [width] and the
+// convolution's last inputs as a ring [taps - 1][width] addressed by position, fp32; a sequence starts from zeros.
+struct RgLru {
+    int width, blocks, taps;
+    const void* proj;         // [T][proj_ld]: y at 0, the convolution's input at x_off, both without their biases
+    int64_t proj_ld;
+    int x_off;
+    const float *x_bias, *y_bias, *conv_bias, *lam;  // [width]
+    const float* conv;        // [taps][width]
+    const float* gate_bias;   // [blocks][2][width / blocks]: r, i
+    void* u;                  // [T][u_ld], each part's channels padded to u_part, from the preparation to the gates' product and the scan
+    int64_t u_ld;
+    int u_part;
+    const float* gate_in;     // [T][gate_ld]: products, laid out like gate_bias
+    int64_t gate_ld;
+    float *state, *ring;      // of slot 0
+    size_t state_stride, ring_stride;  // floats between slots
+    void* out;                // [T][out_ld]
+    int64_t out_ld;
+    const int *tok_seq, *tok_pos;
+    const int *seg_first, *seg_count;  // runs of consecutive positions of one sequence among the T rows
+    int max_slots;
+    int* status;
+};
+void launch_lru_prep(const RgLru& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
+// one_each: every run is a single token (decode)
+void launch_lru_scan(const RgLru& a, bool f32, int n_segs, bool one_each, cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
+int lru_prepare();
 
 // ------------------------------------------------------------------ mixture of experts
 int moe_prepare();

@@ -41,7 +41,7 @@ __global__ void __launch_bounds__(512) k_residual_rows4(const ResidualRows a, un
 #pragma unroll
     for (int k = 0; k < IT; ++k) {
         const int i = (tid + k * n) * 4;
-        if (i < H && a.source >= ROWS_DELTA) load4(a.post_w + i, pw[k]);
+        if (i < H && a.post_w) load4(a.post_w + i, pw[k]);
         if (i < H && a.next_w) load4(a.next_w + i, nw[k]);
     }
     pdl_wait();
@@ -62,6 +62,23 @@ __global__ void __launch_bounds__(512) k_residual_rows4(const ResidualRows a, un
             const int i = (tid + k * n) * 4;
             if (i < H) load4(e + i, x[k]);
         }
+        if (a.embed_w) {
+            float se = 0.f;
+#pragma unroll
+            for (int k = 0; k < IT; ++k)
+                if ((tid + k * n) * 4 < H) se += x[k][0] * x[k][0] + x[k][1] * x[k][1] + x[k][2] * x[k][2] + x[k][3] * x[k][3];
+            const float einv = 1.f / sqrtf(block_sum(se, red) / (float)H + a.eps);
+#pragma unroll
+            for (int k = 0; k < IT; ++k) {
+                const int i = (tid + k * n) * 4;
+                if (i < H) {
+                    float w[4];
+                    load4(a.embed_w + i, w);
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) x[k][c] *= einv * w[c];
+                }
+            }
+        }
     } else {
 #pragma unroll
         for (int k = 0; k < IT; ++k) {
@@ -69,7 +86,20 @@ __global__ void __launch_bounds__(512) k_residual_rows4(const ResidualRows a, un
             if (i < H) load4(xr + i, x[k]);
         }
     }
-    if (a.source >= ROWS_DELTA) {
+    if (a.source == ROWS_DELTA && !a.post_w) {
+        float d[IT][4];
+#pragma unroll
+        for (int k = 0; k < IT; ++k) {
+            const int i = (tid + k * n) * 4;
+            if (i < H) load4(a.delta + (size_t)r * a.delta_ld + i, d[k]);
+        }
+#pragma unroll
+        for (int k = 0; k < IT; ++k)
+            if ((tid + k * n) * 4 < H) {
+#pragma unroll
+                for (int c = 0; c < 4; ++c) x[k][c] += a.delta_mult * d[k][c];
+            }
+    } else if (a.source >= ROWS_DELTA) {
         float d[IT][4], sd = 0.f;
         if (a.source == ROWS_DELTA) {
 #pragma unroll
@@ -136,6 +166,13 @@ __global__ void __launch_bounds__(512) k_residual_rows4(const ResidualRows a, un
 #pragma unroll
                 for (int c = 0; c < 4; ++c) v[c] = x[k][c] * inv * nw[k][c];
                 store4(out + i, v);
+                if (a.next2_w) {
+                    float w2[4], v2[4];
+                    load4(a.next2_w + i, w2);
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) v2[c] = x[k][c] * inv * w2[c];
+                    store4((A*)a.out2 + (size_t)r * a.out_ld + i, v2);
+                }
                 if (a.router_w) {
 #pragma unroll
                     for (int c = 0; c < 4; ++c) rows4_smem[i + c] = as_stored(v[c], out);
@@ -202,6 +239,25 @@ __global__ void __launch_bounds__(512) k_residual_rows(const ResidualRows a, uns
         for (int i = tid; i < H; i += n) {
             const float v = __bfloat162float(e[i]);
             xs[i] = v;
+            if (!a.embed_w) xr[i] = v;
+            ss += v * v;
+        }
+        if (a.embed_w) {
+            const float einv = 1.f / sqrtf(block_sum(ss, red) / (float)H + a.eps);
+            ss = 0.f;
+            for (int i = tid; i < H; i += n) {
+                const float v = xs[i] * einv * __ldg(a.embed_w + i);
+                xs[i] = v;
+                xr[i] = v;
+                ss += v * v;
+            }
+        }
+    } else if (a.source == ROWS_DELTA && !a.post_w) {
+        const float* d = a.delta + (size_t)r * a.delta_ld;
+#pragma unroll 4
+        for (int i = tid; i < H; i += n) {
+            const float v = __ldcg(xr + i) + a.delta_mult * __ldcg(d + i);
+            xs[i] = v;
             xr[i] = v;
             ss += v * v;
         }
@@ -254,6 +310,8 @@ __global__ void __launch_bounds__(512) k_residual_rows(const ResidualRows a, uns
         const float inv = 1.f / sqrtf(ss / (float)H + a.eps);
 #pragma unroll 4
         for (int i = tid; i < H; i += n) act_store(out + i, xs[i] * inv * __ldg(a.next_w + i));
+        if (a.next2_w)
+            for (int i = tid; i < H; i += n) act_store((A*)a.out2 + (size_t)r * a.out_ld + i, xs[i] * inv * __ldg(a.next2_w + i));
     }
     if (tid == 0) tl_mark(tl, 2);
 }

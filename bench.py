@@ -666,6 +666,80 @@ STACK_SIZES = {
     "w2048": dict(width=2048, vocab=32768, depth=8, heads=16, kv=2, dim=128, d_heads=16, d_kv=8, d_dim=128, experts=32, top=4, ff=1536,
                   identity=2, chunk=2048, rank=128, qwen_ff=4096),
 }
+# Razesun models beside the two stacks of the same width, depth and head sizes (a dense feed-forward as wide as the Qwen2
+# stack's; every fourth layer the same mixer: latent attention, real-gated recurrence, delta rule, latent attention on the
+# first one's rows)
+RAZESUN_SIZES = {
+    "z896": dict(beside="w896", rot=32, kv_rank=256, q_rank=384, lru=896, blocks=14),
+    "z2048": dict(beside="w2048", rot=64, kv_rank=512, q_rank=768, lru=2048, blocks=16),
+}
+
+
+def razesun_model(name: str) -> tuple[str, dict]:
+    import synth
+    y = RAZESUN_SIZES[name]
+    z = STACK_SIZES[y["beside"]]
+    mlp = synth.dense_mlp(z["qwen_ff"])
+    layers = []
+    for i in range(0, z["depth"], 4):
+        lat = lambda **kw: synth.latent_layer(z["heads"], z["dim"], y["rot"], z["dim"], y["kv_rank"], y["q_rank"], mlp=mlp, **kw)
+        layers += [lat(), synth.rglru_layer(y["lru"], y["blocks"], mlp=mlp),
+                   synth.delta_layer(z["d_heads"], z["d_kv"], z["d_dim"], z["d_dim"], mlp=mlp), lat(kv_from=i)]
+    cfg = synth.razesun_config(z["width"], z["vocab"], layers)
+    d = model_dir("razesun_" + name)
+    if not os.path.exists(os.path.join(d, ".complete")):
+        shutil.rmtree(d, ignore_errors=True)
+        synth.write_razesun(d, cfg, seed=7, fast=True)
+        open(os.path.join(d, ".complete"), "w").close()
+    return d, cfg
+
+
+def razesun_work(cfg: dict, rows: int, ctx: float, seqs: int) -> dict:
+    """stack_work for a Razesun model. Attention: cached rows once; FLOPs of the form with expanded keys and values (decode:
+    of the folded form, which reads the cache as it is)."""
+    H, out = cfg["width"], {}
+
+    def add(k, b, f=0.0):
+        x = out.setdefault(k, [0.0, 0.0])
+        x[0] += b
+        x[1] += f
+
+    def product(k, n, m, reps=1, out_bytes=2):  # rows x m -> rows x n, `reps` of them
+        add(k, reps * (n * m * 2 + rows * (m * 2 + n * out_bytes)), 2.0 * reps * rows * n * m)
+    for l in cfg["layers"]:
+        m = l["mixer"]
+        if l["type"] == "latent_attention":
+            h, d, rd, v, r, q = (m[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank"))
+            own = 0 if "kv_from" in m else r + rd
+            n_in, n_out = q + own + h, h * v
+            add("latent_prep", rows * 4 * (q + own))
+            product("gemm:query_up", h * (d + rd), q)
+            product("gemm:key_fold", r, d, h)
+            product("gemm:value_up", v, r, h)
+            per = (2 * r + rd) if rows == seqs else (d + rd + v) / 2
+            add("attn_decode", seqs * ctx * (r + rd) * 2 + rows * h * (4 * r + 2 * rd), 2.0 * rows * ctx * h * per)
+        elif l["type"] == "delta":
+            h, g, d, v = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            n_in, n_out = g * 2 * d + 2 * h * v + 2 * h, h * v
+            tok = 4 * (2 * g * d + h * v + 3 * h)
+            add("delta_prep", rows * (2 * (2 * g * d + h * v) + tok))
+            add("delta_scan", seqs * 2 * 4 * h * d * v + rows * (tok + (2 * 4 * h * v if rows > seqs else 2 * h * v)), 8.0 * rows * h * d * v)
+            if rows > seqs:
+                add("delta_out", rows * h * v * (4 + 2 + 2))
+        else:
+            w, b = m["width"], m["blocks"]
+            n_in, n_out = 2 * w, w
+            add("lru_prep", rows * w * 4)
+            product("gemm:lru_gates", 2 * w // b, w // b, b, 4)
+            add("lru_scan", rows * w * (8 + 2 + 2 + 2) + seqs * w * 8)
+        product("gemm:mixer_in", n_in, H)
+        ff = l["mlp"]["ff"]
+        add("gemm_tc:gate_up_swiglu", 2 * ff * H * 2 + rows * (H + ff) * 2, 4.0 * rows * ff * H)
+        add("gemm:out_down", (n_out + ff) * H * 2 + rows * ((n_out + ff) * 2 + H * 4), 2.0 * rows * (n_out + ff) * H)
+        add("residual_rows", rows * H * (4 + 4 + 4 + 2 + 2))
+    add("embed_rows", rows * H * (2 + 4 + 2 + 2))
+    add("gemm_tc:lm_head", cfg["vocab"] * H * 2 + seqs * H * 2, 2.0 * seqs * cfg["vocab"] * H)
+    return out
 
 
 def stack_models(name: str) -> tuple[str, dict, str, dict]:
@@ -753,7 +827,7 @@ def qwen_work(cfg: dict, rows: int, ctx: float, seqs: int) -> dict:
 
 
 def run_stack(a):
-    """--stack SIZE: prefill and decode throughput of a layer-list (Rafilix) model and of the Qwen2 stack beside it, with
+    """--stack SIZE: prefill and decode throughput of a layer-list model and of the stacks beside it, with
     the time every kernel class adds to a decode step (in-kernel stamps) and to a prefill launch (CUDA events), against
     the measured roofline (the larger of bytes / HBM peak and FLOPs / bf16 GEMM peak; the recurrence's FLOPs are fp32
     work of the CUDA cores and are listed, not converted). One JSON line. L2 is not flushed: weights of a decode step
@@ -768,17 +842,23 @@ def run_stack(a):
     if os.path.exists(pk):
         with open(pk) as f:
             tflops = float(json.load(f)["bf16_tflops"])
-    d, cfg, q, qcfg = stack_models(a.stack)
-    rank = STACK_SIZES[a.stack]["rank"]
+    stack = RAZESUN_SIZES[a.stack]["beside"] if a.stack in RAZESUN_SIZES else a.stack
+    d, cfg, q, qcfg = stack_models(stack)
+    sizes = STACK_SIZES[stack]
+    rank = sizes["rank"]
+    works = {"rafilix": (d, lambda rows, ctx, seqs: stack_work(cfg, rows, ctx, rank, seqs)), "qwen2": (q, lambda rows, ctx, seqs: qwen_work(qcfg, rows, ctx, seqs))}
+    first = "rafilix"
+    if a.stack in RAZESUN_SIZES:
+        zd, zcfg = razesun_model(a.stack)
+        works = {"razesun": (zd, lambda rows, ctx, seqs: razesun_work(zcfg, rows, ctx, seqs)), **works}
+        first = "razesun"
     sampler = ClockSampler(None)
-    line = {"metric": f"layer-list model {a.stack}: decode tok/s and prefill tok/s beside a Qwen2 stack of equal size", "unit": "tok/s",
+    line = {"metric": f"layer-list model {a.stack}: decode tok/s and prefill tok/s beside {' and '.join(k for k in works if k != first)} stacks of equal size", "unit": "tok/s",
             "data": "synthetic", "dtype": "bf16", "steps": a.steps, "warmup": a.warmup, "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "kind": kind},
-            "sizes": STACK_SIZES[a.stack]}
+            "sizes": {**sizes, **RAZESUN_SIZES.get(a.stack, {})}}
     K = min(a.steps, 64)
-    for which, path in (("rafilix", d), ("qwen2", q)):
+    for which, (path, work) in works.items():
         model = tffn.load_model(path)
-        work = (lambda rows, ctx, seqs: stack_work(cfg, rows, ctx, rank, seqs)) if which == "rafilix" else \
-            (lambda rows, ctx, seqs: qwen_work(qcfg, rows, ctx, seqs))
         res = {"weight_bytes": model.weight_bytes(False)}
 
         def table(times, w):  # times: class -> (us per step, launches per step)
@@ -809,7 +889,7 @@ def run_stack(a):
         n, P = a.seqs, a.prompt
         sess = tffn.Session(model, max_batch=n, max_seq=P + K * 5 + a.warmup + 64, stream=stream.cuda_stream)
         sess.set_launch_mode(a.launch_mode)
-        prompts = np.random.default_rng(3).integers(2, STACK_SIZES[a.stack]["vocab"], (n, P)).astype(np.int32)
+        prompts = np.random.default_rng(3).integers(2, sizes["vocab"], (n, P)).astype(np.int32)
         e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
         times = []
         for rep in range(max(a.warmup, 3) + 5):
@@ -839,7 +919,7 @@ def run_stack(a):
         s1.prefill([prompts[0]])
         res["decode_bs1"] = decode(s1, 1, P + K * 2.5)
         s1.free()
-        long_p = np.random.default_rng(4).integers(2, STACK_SIZES[a.stack]["vocab"], 4096).astype(np.int32)
+        long_p = np.random.default_rng(4).integers(2, sizes["vocab"], 4096).astype(np.int32)
         s2 = tffn.Session(model, max_batch=1, max_seq=4200, stream=stream.cuda_stream)
         s2.set_launch_mode(a.launch_mode)
         times = []
@@ -864,7 +944,7 @@ def run_stack(a):
         s2.free()
         model.free()
         line[which] = res
-    line["value"] = line["rafilix"]["decode"]["tok_s"]
+    line["value"] = line[first]["decode"]["tok_s"]
     line["clocks"] = sampler.stop()
     print(json.dumps(line), flush=True)
 
@@ -892,8 +972,8 @@ def main():
     ap.add_argument("--kernel-case", default="", choices=["", "gemm", "expert_forward"],
                     help="run only the tensor-core GEMM on the decode step's two largest shapes (gate|up rows, LM head) "
                          "through the op-level entry point and exit: the small program that ncu captures are taken from")
-    ap.add_argument("--stack", default="", choices=[""] + sorted(STACK_SIZES),
-                    help="measure a layer-list (Rafilix) model of this size beside a Qwen2 stack of equal size and exit")
+    ap.add_argument("--stack", default="", choices=[""] + sorted(STACK_SIZES) + sorted(RAZESUN_SIZES),
+                    help="measure a layer-list model of this size (w: Rafilix, z: Razesun) beside stacks of equal size and exit")
     ap.add_argument("--traffic", type=float, default=None,
                     help="DRAM bytes per launch of the dominant kernel from an ncu capture, if known")
     a = ap.parse_args()

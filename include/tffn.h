@@ -60,7 +60,8 @@ int tffn_device_count(void);
 int tffn_config_read(const char* model_dir, tffn_config* out);
 /* Name of the model family config.json belongs to: "Qwen2" (the reference's), or the value of its "architecture"
  * key for the families that list their layers ("Rafilix": chunked attention and gated-delta-rule layers, mixtures
- * of squared-ReLU experts, fp32 residual stream). Unknown names give TFFN_ERR_UNSUPPORTED. For such a family
+ * of squared-ReLU experts; "Razesun": latent attention, delta-rule and real-gated recurrent layers beside a dense
+ * feed-forward; both with an fp32 residual stream). Unknown names give TFFN_ERR_UNSUPPORTED. For such a family
  * tffn_config_read reports the width, the layer count, the vocabulary and eps; its per-head fields are the first
  * layer's, eos / bos are -1 when the file has none, and max_position_embeddings is unbounded. Returns the length
  * of the name (at most cap - 1 characters and a NUL are written). */

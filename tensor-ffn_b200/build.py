@@ -17,7 +17,7 @@ OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libtffn.so")
 CLI = os.path.join(HERE, "tensor-ffn-inference")
 LIB_SOURCES = ["host_io.cpp", "c_api.cpp", "tp_comm.cpp", "engine.cu", "engine_stack.cu", "gemm_tc.cu", "gemm_f32.cu",
-               "rows.cu", "stack_rows.cu", "attn.cu", "latent.cu", "delta.cu", "rglru.cu", "moe.cu", "decode_bs1.cu", "noalloc.cu"]
+               "rows.cu", "stack_rows.cu", "attn.cu", "attn_latent.cu", "latent.cu", "delta.cu", "rglru.cu", "moe.cu", "decode_bs1.cu", "noalloc.cu"]
 CLI_SOURCES = ["cli_main.cpp"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC,-Wall,-Wno-unused-function", "--expt-relaxed-constexpr"]

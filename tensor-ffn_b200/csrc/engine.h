@@ -152,6 +152,7 @@ struct StackState {
         DeviceBuffer k, v;         // attention: pages of this layer (latent attention: one pool for both)
         KvView kv;                 // latent attention with kv_from: the other layer's
         int rope = -1;             // index into rope
+        bool tc = false;           // latent attention: on the tensor cores
         DeviceBuffer state, ring;  // recurrent mixers: see DeltaRule and RgLru
         size_t state_stride = 0, ring_stride = 0;
         int dimP = 0, vdimP = 0;
@@ -164,7 +165,7 @@ struct StackState {
     int max_top = 0, max_experts = 0, moe_layers = 0, max_tiles = 0;
     DeviceBuffer proj, delta, qn, kn, v, g, bk, o, decay, gate;
     DeviceBuffer xn2, ff_act;                 // dense feed-forward beside the mixer: its input, gated activations
-    DeviceBuffer cq, q_up, o_lat, u, lru_gate;  // latent attention; real-gated recurrence
+    DeviceBuffer cq, q_up, q_lat, o_lat, u, lru_gate;  // latent attention; real-gated recurrence
     int64_t cq_ld = 0, q_up_ld = 0, u_ld = 0, lru_gate_ld = 0;
     size_t o_lat_cols = 0;
     DeviceBuffer router, counts, pair, pair_w, pair_row, xg, act_e, y, tiles;

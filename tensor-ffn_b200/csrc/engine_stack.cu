@@ -309,6 +309,7 @@ void Session::alloc_stack(bool f32) {
     s.layers.resize(m->stack.size());
     size_t q_cols = 0, qn = 0, vn = 0, gn = 0, heads = 0, pairs = 0;
     bool dense = false;
+    size_t q_lat_cols = 0;
     for (size_t i = 0; i < m->stack.size(); ++i) {
         const StackLayer& l = m->stack[i];
         const LayerSpec& sp = l.spec;
@@ -346,7 +347,9 @@ void Session::alloc_stack(bool f32) {
             }
             s.cq_ld = std::max<int64_t>(s.cq_ld, pad8(sp.q_rank));
             s.q_up_ld = std::max<int64_t>(s.q_up_ld, pad8(l.q_rows));
-            q_cols = std::max<size_t>(q_cols, (size_t)sp.heads * kv.hd);
+            c.tc = !f32 && attention_latent_supported(sp.kv_rank, sp.rot_dim, sp.heads);
+            if (c.tc) q_lat_cols = std::max<size_t>(q_lat_cols, (size_t)sp.heads * pad8(sp.kv_rank));
+            else q_cols = std::max<size_t>(q_cols, (size_t)sp.heads * kv.hd);
             s.o_lat_cols = std::max<size_t>(s.o_lat_cols, (size_t)sp.heads * pad8(sp.kv_rank));
         } else if (sp.mixer == Mixer::Rglru) {
             c.state_stride = (size_t)sp.lru_width;
@@ -399,6 +402,7 @@ void Session::alloc_stack(bool f32) {
         s.cq.alloc(T * s.cq_ld * s.act);
         s.q_up.alloc(T * s.q_up_ld * s.act);
         s.o_lat.alloc(T * s.o_lat_cols * s.act);
+        if (q_lat_cols) s.q_lat.alloc(T * q_lat_cols * s.act);
     }
     if (s.u_ld) {
         s.u.alloc(T * s.u_ld * s.act);
@@ -433,6 +437,7 @@ void Session::alloc_stack(bool f32) {
     cuda_check((cudaError_t)delta_prepare(), "delta_prepare", __FILE__, __LINE__);
     cuda_check((cudaError_t)moe_prepare(), "moe_prepare", __FILE__, __LINE__);
     cuda_check((cudaError_t)latent_prepare(), "latent_prepare", __FILE__, __LINE__);
+    cuda_check((cudaError_t)attention_latent_prepare(), "attention_latent_prepare", __FILE__, __LINE__);
     cuda_check((cudaError_t)lru_prepare(), "lru_prepare", __FILE__, __LINE__);
 }
 
@@ -472,11 +477,12 @@ int Session::decode_graph_key(int n_seqs, int max_ctx) const {
     }
     int key = 0;  // at most 64 splits per layer; layers that see the same context agree, so one digit per distinct choice
     std::vector<int> seen;
-    for (const StackLayer& l : m_->stack) {
-        if (l.spec.mixer != Mixer::Attention) continue;
-        const int wide = (int)pad8(std::max(l.spec.dim, l.spec.vdim));
-        const int sp = attention_splits(n_seqs, l.spec.heads, l.spec.kv_heads, wide, attn_ctx(l.spec, max_ctx), attn_ws(), m_->num_sms);
-        seen.push_back(sp);
+    for (size_t i = 0; i < m_->stack.size(); ++i) {
+        const LayerSpec& l = m_->stack[i].spec;
+        if (l.mixer == Mixer::Attention)
+            seen.push_back(attention_splits(n_seqs, l.heads, l.kv_heads, (int)pad8(std::max(l.dim, l.vdim)), attn_ctx(l, max_ctx), attn_ws(), m_->num_sms));
+        else if (l.mixer == Mixer::LatentAttention && st_->layers[i].tc)
+            seen.push_back(attention_latent_splits(n_seqs, l.kv_rank, l.rot_dim, l.heads, max_ctx, attn_ws(), m_->num_sms));
     }
     for (int sp : seen) key = (int)(((uint32_t)key * 257u + (uint32_t)sp) & 0x3fffffffu);
     return key;
@@ -644,22 +650,56 @@ void Session::run_stack(int T, int n_logit_rows, bool logit_rows_are_all, bool d
             step(KC_LATENT_PREP, [&](unsigned long long* tl) { launch_latent_prep(p, f32, T, stream_, pdl, tl); });
             run_product(KC_GEMM_UQ, l.uq.as<bf16>(), pad8(sp.q_rank), s.cq.p, s.cq_ld, sp.q_rank, l.q_rows, GEMM_STORE_BF16, s.q_up.p, s.q_up_ld);
             // a head's key projection folded into its query: q . (W_uk c) = (W_uk^T q) . c
-            batched(KC_GEMM_UK, sp.heads, l.uk.as<bf16>(), dim8, s.q_up.p, s.q_up_ld, dim8, sp.dim, sp.kv_rank, GEMM_STORE_F32, q_.p,
-                    (int64_t)sp.heads * kd, kd);
-            step(KC_LATENT_ROPE, [&](unsigned long long* tl) {
-                launch_latent_rope(s.q_up.p, s.q_up_ld, sp.heads * dim8, sp.heads, sp.rot_dim, p.rope, max_seq_, tok_pos, q_.as<float>(), kd, rot_col,
-                                   f32, T, status, stream_, pdl, tl);
-            });
-            AttnOptions opt;
-            opt.scale = sp.scale;
-            opt.vdim = sp.kv_rank;
-            opt.ctx_ld = (int64_t)sp.heads * rank8;
-            opt.head_ld = rank8;
-            opt.gate = act_at(s.proj, l.g1_off);
-            opt.gate_ld = l.in_rows;
-            step(KC_ATTENTION, [&](unsigned long long* tl) {
-                launch_attention_simt(q_.as<float>(), cache.kv, f32, tok_seq, tok_pos, s.o_lat.p, T, sp.heads, opt, status, stream_, pdl, tl);
-            });
+            if (cache.tc) {
+                batched(KC_GEMM_UK, sp.heads, l.uk.as<bf16>(), dim8, s.q_up.p, s.q_up_ld, dim8, sp.dim, sp.kv_rank, GEMM_STORE_BF16, s.q_lat.p,
+                        (int64_t)sp.heads * rank8, rank8);
+                LatentAttn at;
+                memset(&at, 0, sizeof at);
+                at.q_lat = s.q_lat.as<bf16>();
+                at.rows_alloc = cap_tokens_;
+                at.q_up = s.q_up.as<bf16>();
+                at.q_up_ld = s.q_up_ld;
+                at.rot_off = sp.heads * dim8;
+                at.rot = sp.rot_dim;
+                at.rank = sp.kv_rank;
+                at.heads = sp.heads;
+                at.rope = p.rope;
+                at.max_pos = max_seq_;
+                at.scale = sp.scale;
+                at.kv = cache.kv;
+                at.tok_seq = tok_seq;
+                at.tok_pos = tok_pos;
+                at.grp_first = grp_first_.as<int>();
+                at.grp_count = grp_count_.as<int>();
+                at.gate = (const bf16*)act_at(s.proj, l.g1_off);
+                at.gate_ld = l.in_rows;
+                at.out = s.o_lat.as<bf16>();
+                at.head_ld = rank8;
+                at.only_newest_row_fresh = decode;
+                at.status = status;
+                step(KC_ATTENTION, [&](unsigned long long* tl) {
+                    const int rc = launch_attention_latent(at, T, n_groups, max_ctx, attn_ws(), m_->num_sms, tmaps_, stream_, pdl, tl);
+                    if (rc == -1000) throw Error(kErrCuda, "cuTensorMapEncodeTiled failed or is unavailable");
+                    if (rc != 0) cuda_check((cudaError_t)rc, "latent attention launch", __FILE__, __LINE__);
+                });
+            } else {
+                batched(KC_GEMM_UK, sp.heads, l.uk.as<bf16>(), dim8, s.q_up.p, s.q_up_ld, dim8, sp.dim, sp.kv_rank, GEMM_STORE_F32, q_.p,
+                        (int64_t)sp.heads * kd, kd);
+                step(KC_LATENT_ROPE, [&](unsigned long long* tl) {
+                    launch_latent_rope(s.q_up.p, s.q_up_ld, sp.heads * dim8, sp.heads, sp.rot_dim, p.rope, max_seq_, tok_pos, q_.as<float>(), kd, rot_col,
+                                       f32, T, status, stream_, pdl, tl);
+                });
+                AttnOptions opt;
+                opt.scale = sp.scale;
+                opt.vdim = sp.kv_rank;
+                opt.ctx_ld = (int64_t)sp.heads * rank8;
+                opt.head_ld = rank8;
+                opt.gate = act_at(s.proj, l.g1_off);
+                opt.gate_ld = l.in_rows;
+                step(KC_ATTENTION, [&](unsigned long long* tl) {
+                    launch_attention_simt(q_.as<float>(), cache.kv, f32, tok_seq, tok_pos, s.o_lat.p, T, sp.heads, opt, status, stream_, pdl, tl);
+                });
+            }
             batched(KC_GEMM_UV, sp.heads, l.uv.as<bf16>(), rank8, s.o_lat.p, (int64_t)sp.heads * rank8, rank8, sp.kv_rank, sp.vdim, GEMM_STORE_BF16,
                     ctx_.p, ctx_ld, sp.vdim);
         } else if (sp.mixer == Mixer::Rglru) {

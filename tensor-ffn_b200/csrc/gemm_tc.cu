@@ -848,6 +848,10 @@ int launch_bn(const GemmCall& c, const GemmWorkspace& ws, cudaStream_t stream, i
 
 }  // namespace
 
+bool make_tmap_2d(TmapCache* cache, CUtensorMap* tm, const bf16* ptr, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows) {
+    return make_tmap(cache, tm, ptr, rows, cols, ld, box_rows);
+}
+
 int gemm_prepare() {
     cudaError_t e;
 #define TFFN_PREP(BN)                                                                                                 \

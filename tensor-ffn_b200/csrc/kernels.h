@@ -108,6 +108,8 @@ constexpr int kGemmF32Tile = 64;  // its token tile (grp_bn)
 struct TmapCache;
 TmapCache* tmap_cache_create();
 void tmap_cache_free(TmapCache* c);
+// bf16 tensor [rows, cols] with a row stride of ld elements, boxes of box_rows x 64 columns with the 128-byte swizzle
+bool make_tmap_2d(TmapCache* cache, CUtensorMap* tm, const bf16* ptr, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows);
 
 struct GemmWorkspace {
     int* status;  // device status word
@@ -300,6 +302,34 @@ void launch_latent_rope(const void* q_up, int64_t ld, int off, int heads, int ro
                         float* q, int q_cols, int rot_col, bool f32, int T, int* status, cudaStream_t s, bool pdl,
                         unsigned long long* tl = nullptr);
 int latent_prepare();
+// The attention itself on the tensor cores (bf16 sessions): the unrotated queries come with the key projections folded in,
+// the rotated parts as projected. Groups as in launch_attention_prefill; n_groups = 0: every row is a token of its own
+// (decode), its context possibly in splits (see launch_attention for only_newest_row_fresh).
+struct LatentAttn {
+    const bf16* q_lat;        // [rows_alloc][heads][head_ld]
+    int rows_alloc;
+    const bf16* q_up;         // rotated parts, before the rotation: [T][q_up_ld], `rot` columns per head from rot_off
+    int64_t q_up_ld;
+    int rot_off, rot, rank, heads;
+    const float2* rope;
+    int max_pos;
+    float scale;
+    KvView kv;
+    const int *tok_seq, *tok_pos, *grp_first, *grp_count;
+    const bf16* gate;         // [T][gate_ld]: head h's output times sigmoid(gate[t][h])
+    int64_t gate_ld;
+    bf16* out;                // [T][heads][head_ld] weighted latents
+    int head_ld;              // rank padded to 8
+    bool only_newest_row_fresh;
+    int* status;
+};
+constexpr int kLatentSplitKeys = 512;  // fewest keys of a context split
+bool attention_latent_supported(int rank, int rot, int heads);  // otherwise launch_attention_simt
+int attention_latent_splits(int rows, int rank, int rot, int heads, int max_ctx, const AttnWorkspace& ws, int num_sms);
+// returns cudaError (launch) or -1000 if the tensor maps could not be encoded
+int launch_attention_latent(const LatentAttn& a, int T, int n_groups, int max_ctx, const AttnWorkspace& ws, int num_sms, TmapCache* tmaps,
+                            cudaStream_t s, bool pdl, unsigned long long* tl = nullptr);
+int attention_latent_prepare();
 
 // q|k|v rows of one projection -> per-head norm of q and k (weights shared by the heads), rotation of neighbouring
 // pairs, q in fp32 for the attention kernels, k and v into the sequence's page.

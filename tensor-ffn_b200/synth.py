@@ -290,14 +290,87 @@ def rafilix_specs(cfg: dict, rank: int = 16, qk_norm: float = 1.0):
     return specs
 
 
+# Razesun: mixers 'latent_attention', 'delta', 'rglru' beside a dense feed-forward
+def latent_layer(heads, dim, rot_dim, vdim, kv_rank, q_rank, base=10000.0, scale=None, kv_from=None, mlp=None) -> dict:
+    m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "q_rank": q_rank,
+         "scale": scale if scale is not None else (dim + rot_dim) ** -0.5, "rot": {"base": base, "dims": rot_dim}}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "latent_attention", "mixer": m, "mlp": mlp}
+
+
+def delta_layer(heads, kv_heads, dim, vdim, conv=4, mlp=None) -> dict:
+    return dict(channel_delta_layer(heads, kv_heads, dim, vdim, conv, mlp), type="delta")
+
+
+def rglru_layer(width, blocks, conv=4, mlp=None) -> dict:
+    return {"type": "rglru", "mixer": {"width": width, "blocks": blocks, "conv": conv}, "mlp": mlp}
+
+
+def dense_mlp(ff) -> dict:
+    return {"kind": "dense", "ff": ff}
+
+
+def razesun_config(width, vocab, layers, eps=1e-5, residual_mult=0.5, logit_scale=0.7) -> dict:
+    return {"architecture": "Razesun", "width": width, "vocab": vocab, "norm": {"eps": eps}, "residual_mult": residual_mult,
+            "logit_scale": logit_scale, "layers": layers}
+
+
+def razesun_specs(cfg: dict, sharp: float = 1.0):
+    """(name, shape, kind, parameter) of every tensor, kinds as in rafilix_specs. sharp: weight of the query latent's norm
+    (large values let single keys decide a score's softmax)."""
+    H = cfg["width"]
+    lin = lambda name, out, inp, gain=1.0: (name, (out, inp), "w", gain * inp ** -0.5)
+    specs = [("embed", (cfg["vocab"], H), "w", 0.5), ("embed.norm", (H,), "n", 1.0)]
+    for i, layer in enumerate(cfg["layers"]):
+        m, n = layer["mixer"], f"l{i}."
+        p, f = n + "mix.", n + "mlp."
+        specs.append((n + "norm1", (H,), "n", 1.0))
+        if layer["type"] == "latent_attention":
+            h, d, rd, v, r, q = (m[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank"))
+            specs += [lin(p + "dq", q, H), (p + "dq.norm", (q,), "n", sharp), lin(p + "uq", h * (d + rd), q)]
+            if "kv_from" not in m:
+                specs += [lin(p + "dkv", r + rd, H), (p + "dkv.norm", (r,), "n", 1.0)]
+            specs += [lin(p + "uk", h * d, r), lin(p + "uv", h * v, r), lin(p + "g", h, H)]
+            out = h * v
+        elif layer["type"] == "delta":
+            h, g, d, v = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            specs += [lin(p + "q", g * d, H), lin(p + "k", g * d, H), lin(p + "v", h * v, H)]
+            specs += [(p + t + ".conv", (c, m["conv"]), "w", 0.6) for t, c in (("q", g * d), ("k", g * d), ("v", h * v))]
+            specs += [lin(p + "b", h, H), (p + "A_log", (h,), "u", (-3.0, 1.0)), (p + "norm", (v,), "n", 1.0), lin(p + "a", h, H),
+                      (p + "dt_bias", (h,), "u", (-4.0, 1.0)), lin(p + "g", h * v, H)]
+            out = h * v
+        else:
+            w, b = m["width"], m["blocks"]
+            specs += [lin(p + "y", w, H), (p + "y.b", (w,), "w", 0.3), lin(p + "x", w, H), (p + "x.b", (w,), "w", 0.3),
+                      (p + "conv", (w, m["conv"]), "w", 0.6), (p + "conv.b", (w,), "w", 0.3)]
+            for t in ("ra", "ri"):
+                specs += [(p + t, (b, w // b, w // b), "w", (w // b) ** -0.5), (p + t + ".b", (b, w // b), "w", 0.5)]
+            specs.append((p + "lam", (w,), "u", (-6.0, 1.0)))
+            out = w
+        specs.append(lin(p + "o", H, out))
+        if layer.get("mlp"):
+            ff = layer["mlp"]["ff"]
+            specs += [(n + "norm2", (H,), "n", 1.0), lin(f + "gate", ff, H), lin(f + "up", ff, H), lin(f + "down", H, ff)]
+    return specs + [("final.norm", (H,), "n", 1.0), lin("head", cfg["vocab"], H)]
+
+
 def write_rafilix(dirpath: str, cfg: dict, seed: int = 1, rank: int = 16, qk_norm: float = 1.0, fast: bool = False, edit=None) -> dict:
+    return write_layer_list(dirpath, cfg, rafilix_specs(cfg, rank, qk_norm), seed, fast, edit)
+
+
+def write_razesun(dirpath: str, cfg: dict, seed: int = 1, sharp: float = 1.0, fast: bool = False, edit=None) -> dict:
+    return write_layer_list(dirpath, cfg, razesun_specs(cfg, sharp), seed, fast, edit)
+
+
+def write_layer_list(dirpath: str, cfg: dict, specs: list, seed: int, fast: bool, edit) -> dict:
     """config.json and model.safetensors with seeded random weights. edit(name, float array) -> array or None may replace
     a tensor before it is rounded to bf16. fast: matrices cut out of one random block (throughput runs)."""
     os.makedirs(dirpath, exist_ok=True)
     with open(os.path.join(dirpath, "config.json"), "w") as f:
         json.dump(cfg, f, indent=1)
     out = []
-    for i, (name, shape, kind, par) in enumerate(rafilix_specs(cfg, rank, qk_norm)):
+    for i, (name, shape, kind, par) in enumerate(specs):
         n = int(np.prod(shape))
         if fast and kind == "w" and n > 1 << 16:
             out.append((name, shape, _tiled_bf16([seed, i], n, float(np.float16(par)))))

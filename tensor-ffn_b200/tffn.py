@@ -139,7 +139,7 @@ def qwen_config_from_json(model_dir: str) -> Config:
 
 
 def model_family(model_dir: str) -> str:
-    """name of the model family a config.json belongs to ("Qwen2", "Rafilix")"""
+    """name of the model family a config.json belongs to ("Qwen2", "Rafilix", "Razesun")"""
     buf = ctypes.create_string_buffer(64)
     _check(_L.tffn_config_family(model_dir.encode(), buf, 64))
     return buf.value.decode()

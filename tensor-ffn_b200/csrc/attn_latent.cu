@@ -1,15 +1,22 @@
-// Latent attention on the tensor cores, prompts and decoding alike. A cached row is the key of every head (the heads' key
-// projections are folded into the queries) and its first `rank` columns are the value, so the heads of up to eight tokens of
-// a sequence are the 128 rows of one tile:
+// Latent attention on the tensor cores. A cached row is the key of every head (the heads' key projections are folded into
+// the queries) and its first `rank` columns are the value.
+//
+// Prompts (k_attn_latent): the heads of up to eight tokens of a sequence are the 128 rows of one tile:
 //   S[row, key] = Q[row, :] . K[key, :]      tcgen05.mma, Q and K in shared memory (both K-major)
 //   O[row, :]  += P[row, :] . K[:, columns]  tcgen05.mma, P in tensor memory, K read the other way round (N-major)
-// One CTA = the rows of one tile x at most 256 value columns x one context split, 6 warps:
+// One CTA = the rows of one tile x at most 256 value columns, 6 warps:
 //   warps 0-3  thread = row: S out of tensor memory, online softmax in fp32, P back as a bf16 pair (hi + lo, 16 mantissa
 //              bits), the rotated part of Q at the start, and the output rows at the end
 //   warp 4     TMA producer: Q, then 64 keys (two pages) per stage, 64 columns per box with the 128-byte swizzle
 //   warp 5     tensor memory, MMA issue
-// The reference maximum of a row moves only when it would be exceeded by more than 2^8, so O is rarely rescaled. Splits
-// leave partial rows and the last one to finish (a ticket, no waiting) adds them up in split order.
+// The reference maximum of a row moves only when it would be exceeded by more than 2^8, so O is rarely rescaled.
+//
+// Decoding (k_attn_latent_decode): one token's heads would leave most of those rows empty, so keys and value columns take
+// the long side instead, S^T[key, head] = K . Q^T and O^T[column, head] += K^T . P^T: all value columns in one CTA. P^T is
+// written to shared memory next to its lo part (twice the columns of one product). One CTA = 16 or 32 heads of a token x
+// one context split, the same six warps (thread = key). Splits leave partial rows and the last one to finish (a ticket, no
+// waiting) adds them up in split order.
+//
 // Rows of a page past the end of a sequence are finite (zeros or an earlier request's normed latents) and weigh zero.
 #include "act.cuh"
 #include "launch.h"
@@ -47,7 +54,8 @@ struct LatentDev {
     int tile_tokens, subs;             // tokens of a tile; tiles a group may need
     int q_rows;                        // rows of the Q box
     int rank, slices, slice_cols;
-    int stages, splits, early;
+    int stages;
+    int splits, early;                 // decoding only
     float scale_log2;
     const bf16* gate;                  // [T][gate_ld]
     long long gate_ld;
@@ -87,26 +95,103 @@ __device__ __forceinline__ float exp2_fast(float x) {
     return y;
 }
 
+// 64 keys of a sequence (its `tile`-th) into the stage of the ring that is theirs; tile0: the CTA's first tile. A page past
+// the end is replaced by the last one, its keys are masked.
+__device__ __forceinline__ void load_tile(const LatentDev& p, int seq, int len, int tile, int blocks, int stage_bytes, uint8_t* ring, uint64_t* full,
+                                          int tile0 = 0) {
+    const int* bt = p.block_table + (size_t)seq * p.max_pages_per_seq;
+    const int st = (tile - tile0) % p.stages, last_page = (len - 1) / kPageTokens;
+    uint8_t* dst = ring + st * stage_bytes;
+    mbar_arrive_expect_tx(&full[st], stage_bytes);
+    for (int h = 0; h < TK / kPageTokens; ++h) {
+        int pg = __ldg(bt + min(tile * (TK / kPageTokens) + h, last_page));
+        if (pg < 0 || pg >= p.num_pages) {
+            dev_fail(p.status, DEV_ERR_BOUNDS);
+            pg = 0;
+        }
+        for (int b = 0; b < blocks; ++b) tma_load_2d(dst + b * kBlockBytes + h * kPageTokens * 128, &p.tmK, b * 64, pg * kPageTokens, &full[st]);
+    }
+}
+
+// The rotated parts of Q, rows 0 .. rows - 1 of the tile (row = token * part_heads + head), into the blocks behind the latent
+// ones; columns past `rot` are zero, and so are rows of heads that do not exist. The 128 softmax threads call it.
+__device__ __forceinline__ void rotate_q(const LatentDev& p, int t0, int head0, int nheads, int rows, uint8_t* q_rot, int q_block) {
+    const int half = p.rot / 2, tid = threadIdx.x, zero_to = (p.rot + 15) / 16 * 16;
+    auto at = [&](int r, int col) {  // address of the 8 columns from `col` (a multiple of 8) of row r
+        const int c = (col & 63) >> 3;
+        return q_rot + (col >> 6) * q_block + r * 128 + ((c ^ (r & 7)) << 4);
+    };
+    if (half % 8 == 0) {
+        constexpr int B = 4;  // pieces of 8 pairs with their loads in flight together
+        const int pieces = half / 8, n = rows * pieces;
+        for (int i0 = tid; i0 < n; i0 += B * kRowsMax) {
+            uint4 u[B], v[B];
+            float4 cs[B][4];
+#pragma unroll
+            for (int k = 0; k < B; ++k) {
+                const int i = i0 + k * kRowsMax, r = i / pieces, c = i % pieces * 8, h = r % p.part_heads, t = t0 + r / p.part_heads;
+                u[k] = v[k] = make_uint4(0u, 0u, 0u, 0u);
+                if (i < n) {
+                    const int pos = min(max(__ldcg(p.tok_pos + t), 0), p.max_pos - 1);
+                    const float4* f = (const float4*)(p.rope + (size_t)pos * half + c);
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) cs[k][q] = __ldg(f + q);
+                    if (h < nheads) {
+                        const bf16* src = p.q_up + (size_t)t * p.q_up_ld + p.rot_off + (size_t)(head0 + h) * p.rot + c;
+                        u[k] = __ldcg((const uint4*)src);
+                        v[k] = __ldcg((const uint4*)(src + half));
+                    }
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < B; ++k) {
+                const int i = i0 + k * kRowsMax, r = i / pieces, c = i % pieces * 8;
+                if (i >= n) break;
+                const uint32_t uu[4] = {u[k].x, u[k].y, u[k].z, u[k].w}, vv[4] = {v[k].x, v[k].y, v[k].z, v[k].w};
+                uint32_t a[4], b[4];
+#pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                    const float4 f = cs[k][q];
+                    const float u0 = bf16_lo(uu[q]), u1 = bf16_hi(uu[q]), v0 = bf16_lo(vv[q]), v1 = bf16_hi(vv[q]);
+                    a[q] = (uint32_t)bf16_bits(u0 * f.x - v0 * f.y) | ((uint32_t)bf16_bits(u1 * f.z - v1 * f.w) << 16);
+                    b[q] = (uint32_t)bf16_bits(v0 * f.x + u0 * f.y) | ((uint32_t)bf16_bits(v1 * f.z + u1 * f.w) << 16);
+                }
+                *(uint4*)at(r, c) = make_uint4(a[0], a[1], a[2], a[3]);
+                *(uint4*)at(r, half + c) = make_uint4(b[0], b[1], b[2], b[3]);
+            }
+        }
+        return;  // rot is a multiple of 16
+    }
+    auto put = [&](int r, int col, float x) { *(bf16*)(at(r, col & ~7) + (col & 7) * 2) = __float2bfloat16_rn(x); };
+    for (int i = tid; i < rows * half; i += kRowsMax) {
+        const int r = i / half, c = i % half, h = r % p.part_heads, t = t0 + r / p.part_heads;
+        const int pos = min(max(__ldcg(p.tok_pos + t), 0), p.max_pos - 1);
+        const float2 cs = __ldg(p.rope + (size_t)pos * half + c);
+        const bf16* src = p.q_up + (size_t)t * p.q_up_ld + p.rot_off + (size_t)(head0 + h) * p.rot + c;
+        const float u = h < nheads ? act_load(src) : 0.f, v = h < nheads ? act_load(src + half) : 0.f;
+        put(r, c, u * cs.x - v * cs.y);
+        put(r, half + c, v * cs.x + u * cs.y);
+    }
+    for (int i = tid; i < rows * (zero_to - p.rot); i += kRowsMax) put(i / (zero_to - p.rot), p.rot + i % (zero_to - p.rot), 0.f);
+}
+
 __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_constant__ LatentDev p) {
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[2], q_full, p_full, pv_done;
     __shared__ uint32_t tmem_slot;
-    __shared__ int s_last;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
     // unit = ((group * subs + sub) * parts + part) * slices + slice
     const int unit = blockIdx.x, slice = unit % p.slices, part = unit / p.slices % p.parts;
-    const int sub = unit / p.slices / p.parts % p.subs, group = unit / p.slices / p.parts / p.subs;
+    const int sub = unit / p.slices / p.parts % p.subs;
+    const int group = gridDim.x / (p.slices * p.parts * p.subs) - 1 - unit / p.slices / p.parts / p.subs;  // later groups see more keys: first
     const int g_first = p.grp_first ? __ldcg(p.grp_first + group) : group, g_count = p.grp_first ? __ldcg(p.grp_count + group) : 1;
     const int t0 = g_first + sub * p.tile_tokens, ntok = min(p.tile_tokens, g_count - sub * p.tile_tokens);
     const int head0 = part * p.part_heads, nheads = min(p.part_heads, p.heads - head0);
     const int seq = __ldcg(p.tok_seq + (ntok > 0 ? t0 : g_first));
     const int len = ntok > 0 ? __ldcg(p.tok_pos + t0 + ntok - 1) + 1 : 0;  // positions ascend within a group
-    int per_split = (len + p.splits - 1) / p.splits;
-    per_split = (per_split + TK - 1) / TK * TK;
-    const int k_begin = blockIdx.y * per_split, k_end = min(len, k_begin + per_split);
-    const int n_tiles = k_end > k_begin ? (k_end - k_begin + TK - 1) / TK : 0;
+    const int n_tiles = (len + TK - 1) / TK;
     const bool len_ok = len <= p.max_pos && (len + kPageTokens - 1) / kPageTokens <= p.max_pages_per_seq;
 
     const int rank_blocks = (p.rank + 63) / 64, rot_blocks = (p.rot + 63) / 64, blocks = rank_blocks + rot_blocks;
@@ -149,34 +234,13 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_consta
         if (lane == 0) {
             prefetch_tmap(&p.tmQ);
             prefetch_tmap(&p.tmK);
-            const int* bt = p.block_table + (size_t)seq * p.max_pages_per_seq;
-            const int last_page = (len - 1) / kPageTokens;
-            auto load_tile = [&](int j) {
-                const int st = j % p.stages;
-                uint8_t* dst = k_s + st * stage_bytes;
-                mbar_arrive_expect_tx(&k_full[st], stage_bytes);
-                for (int h = 0; h < TK / kPageTokens; ++h) {
-                    // a page past the end is replaced by the last one; its keys are masked
-                    int pg = __ldg(bt + min((k_begin + j * TK) / kPageTokens + h, last_page));
-                    if (pg < 0 || pg >= p.num_pages) {
-                        dev_fail(p.status, DEV_ERR_BOUNDS);
-                        pg = 0;
-                    }
-                    for (int b = 0; b < blocks; ++b)
-                        tma_load_2d(dst + b * kBlockBytes + h * kPageTokens * 128, &p.tmK, b * 64, pg * kPageTokens, &k_full[st]);
-                }
-            };
-            // In decode everything but the newest row is older than the step's first kernel
-            int next = 0;
-            if (p.early)
-                while (next < min(p.stages, tiles) && k_begin + (next + 1) * TK <= last_page * kPageTokens) load_tile(next++);
             pdl_wait();
             tl_mark(p.tl, 1);
             if (tiles > 0) mbar_arrive_expect_tx(&q_full, rank_blocks * q_block);  // no copy that nobody waits for
             for (int b = 0; b < rank_blocks && tiles > 0; ++b) tma_load_2d(q_s + b * q_block, &p.tmQ, b * 64, t0 * p.heads + head0, &q_full);
-            for (; next < tiles; ++next) {
+            for (int next = 0; next < tiles; ++next) {
                 if (next >= p.stages && !mbar_wait(&k_empty[next % p.stages], (uint32_t)(next / p.stages - 1) & 1u, p.status, DEV_ERR_EMPTY_WAIT)) break;
-                load_tile(next);
+                load_tile(p, seq, len, next, blocks, stage_bytes, k_s, k_full);
             }
         }
     } else if (warp == 5) {
@@ -218,30 +282,10 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_consta
         }
     } else {
         pdl_wait();
-        // the rotated part of Q: block rank_blocks and on, columns past `rot` zero
-        {
-            const int half = p.rot / 2, zero_to = (p.rot + 15) / 16 * 16;
-            auto put = [&](int r, int col, float v) {
-                uint8_t* blk = q_s + (rank_blocks + col / 64) * q_block;
-                const int c = col % 64;
-                *(bf16*)(blk + r * 128 + (((c >> 3) ^ (r & 7)) << 4) + (c & 7) * 2) = __float2bfloat16_rn(v);
-            };
-            const int rows = ntok * p.part_heads;
-            for (int i = tid; i < rows * half; i += kRowsMax) {
-                const int r = i / half, c = i % half, h = r % p.part_heads, t = t0 + r / p.part_heads;
-                if (h >= nheads) continue;
-                const bf16* src = p.q_up + (size_t)t * p.q_up_ld + p.rot_off + (size_t)(head0 + h) * p.rot;
-                const float u = act_load(src + c), v = act_load(src + half + c);
-                const int pos = __ldcg(p.tok_pos + t);
-                const float2 cs = __ldg(p.rope + (size_t)(pos >= 0 && pos < p.max_pos ? pos : 0) * half + c);
-                put(r, c, u * cs.x - v * cs.y);
-                put(r, half + c, v * cs.x + u * cs.y);
-            }
-            for (int i = tid; i < rows * (zero_to - p.rot); i += kRowsMax) put(i / (zero_to - p.rot), p.rot + i % (zero_to - p.rot), 0.f);
-            fence_proxy_async_smem();
-            mbar_arrive(&q_full);
-        }
-        const int my_end = active ? min(k_end, __ldcg(p.tok_pos + row_t) + 1) : 0;
+        rotate_q(p, t0, head0, nheads, ntok * p.part_heads, q_s + rank_blocks * q_block, q_block);
+        fence_proxy_async_smem();
+        mbar_arrive(&q_full);
+        const int my_end = active ? __ldcg(p.tok_pos + row_t) + 1 : 0;
         const uint32_t lane_addr = tmem + ((uint32_t)(warp * 32) << 16);
         const int ncols16 = (min(p.slice_cols, p.rank - slice * p.slice_cols) + 15) / 16;
         bool ok = true;
@@ -253,7 +297,7 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_consta
 #pragma unroll
             for (int c = 0; c < TK / 16; ++c) tmem_ld16(lane_addr + kColS + (j & 1) * TK + c * 16, s[c]);
             tc_wait_ld();
-            const int live = my_end - (k_begin + j * TK);  // visible keys of this tile
+            const int live = my_end - j * TK;  // visible keys of this tile
             float mx = kNeg;
 #pragma unroll
             for (int i = 0; i < TK; ++i) {
@@ -312,19 +356,14 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_consta
         // ---- this slice's columns of the row
         const int col0 = slice * p.slice_cols;
         float mult = 0.f;
-        if (active && l_sum > 0.f && p.splits == 1) {
-            const float z = act_load(p.gate + (size_t)row_t * p.gate_ld + head0 + row_head);
-            mult = sigmoid_f32(z) / l_sum;
-        }
+        if (active && l_sum > 0.f) mult = sigmoid_f32(act_load(p.gate + (size_t)row_t * p.gate_ld + head0 + row_head)) / l_sum;
         bf16* dst = p.out + ((size_t)row_t * p.heads + head0 + row_head) * p.head_ld + col0;
-        // partial rows: [unit][split][row][slice_cols + 2], the last two: maximum, sum
-        float* part_row = p.ws + (((size_t)unit * p.splits + blockIdx.y) * p.part_heads + row_head) * (p.slice_cols + 2);
         if (tiles > 0 && ok) {
             for (int c = 0; c < ncols16; ++c) {
                 uint32_t o[16];
                 tmem_ld16(lane_addr + kColO + c * 16, o);
                 tc_wait_ld();
-                if (active && p.splits == 1) {
+                if (active) {
 #pragma unroll
                     for (int i = 0; i < 16; i += 8) {
                         uint32_t w[4];
@@ -333,51 +372,371 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_consta
                             w[k] = (uint32_t)bf16_bits(__uint_as_float(o[i + 2 * k]) * mult) | ((uint32_t)bf16_bits(__uint_as_float(o[i + 2 * k + 1]) * mult) << 16);
                         if (col0 + c * 16 + i < p.rank) *(uint4*)(dst + c * 16 + i) = make_uint4(w[0], w[1], w[2], w[3]);
                     }
-                } else if (active) {
-#pragma unroll
-                    for (int i = 0; i < 16; i += 2) *(uint2*)(part_row + c * 16 + i) = make_uint2(o[i], o[i + 1]);
                 }
                 __syncwarp();
             }
         }
-        if (p.splits > 1 && active) {
-            part_row[p.slice_cols] = m_ref;
-            part_row[p.slice_cols + 1] = l_sum;
-        }
     }
     tc_fence_before();
-    if (p.splits > 1) __threadfence();
     __syncthreads();
     if (warp == 5) tmem_dealloc(tmem, kTmemCols);
+    if (tid == 0) tl_mark(p.tl, 2);
+}
+
+// ---------------------------------------------------------------------------------------------- decoding
+constexpr int kDecSoftmax = 128;           // threads of the softmax warps
+constexpr int kDecP = TK * 128;            // one P^T buffer: 64 keys x (hi | lo) heads, rows of 128 bytes
+constexpr int kDecMaxSplits = 64;
+__host__ __device__ inline int partial_ld(int rank) { return (rank + 3) / 4 * 4 + 4; }  // floats of a split's partial row
+__device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ bool softmax_any(bool x) {
+    int r;
+    asm volatile(
+        "{\n\t.reg .pred p, q;\n\t"
+        "setp.ne.b32 p, %1, 0;\n\t"
+        "bar.red.or.pred q, 1, 128, p;\n\t"
+        "selp.b32 %0, 1, 0, q;\n\t}"
+        : "=r"(r)
+        : "r"((int)x)
+        : "memory");
+    return r != 0;
+}
+
+// HP: heads of a tile (16 or 32)
+template <int HP>
+__global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid_constant__ LatentDev p, uint32_t tmem_cols) {
+    extern __shared__ uint8_t smem_raw[];
+    uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+    __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[2], p_full[2], pv_done[2], q_full;
+    __shared__ uint32_t tmem_slot;
+    __shared__ int s_last;
+    __shared__ float s_max[4][HP], s_sum[4][HP], s_mult[HP];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+
+    const int unit = blockIdx.x, t = unit / p.parts, part = unit % p.parts;
+    const int head0 = part * p.part_heads, nheads = min(p.part_heads, p.heads - head0);
+    const int seq = __ldcg(p.tok_seq + t), len = __ldcg(p.tok_pos + t) + 1;
+    int per_split = (len + p.splits - 1) / p.splits;
+    per_split = (per_split + TK - 1) / TK * TK;
+    const int k_begin = blockIdx.y * per_split, k_end = min(len, k_begin + per_split);
+    const bool len_ok = len <= p.max_pos && (len + kPageTokens - 1) / kPageTokens <= p.max_pages_per_seq;
+    const int tiles = len_ok && k_end > k_begin ? (k_end - k_begin + TK - 1) / TK : 0;
+
+    const int rank_blocks = (p.rank + 63) / 64, rot_blocks = (p.rot + 63) / 64, blocks = rank_blocks + rot_blocks;
+    const int mblocks = (p.rank + 127) / 128;
+    constexpr int q_block = HP * 128;
+    const int stage_bytes = blocks * kBlockBytes;
+    uint8_t* const q_s = smem;
+    uint8_t* const p_s = smem + blocks * q_block;
+    uint8_t* const k_s = p_s + 2 * kDecP;
+    constexpr uint32_t colO = 2 * HP;
+
+    if (tid == 0) {
+        tl_mark(p.tl, 0);
+        for (int i = 0; i < p.stages; ++i) {
+            mbar_init(&k_full[i], 1);
+            mbar_init(&k_empty[i], 1);
+        }
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(&s_full[i], 1);
+            mbar_init(&p_full[i], kDecSoftmax);  // two: the softmax may be a tile ahead of the product
+            mbar_init(&pv_done[i], 1);
+        }
+        mbar_init(&q_full, 1 + kDecSoftmax);
+        fence_mbar_init();
+    }
+    if (warp == 5) {
+        tmem_alloc(&tmem_slot, tmem_cols);
+        tmem_relinquish();
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = tmem_slot;
+    pdl_launch_dependents();
+    if (!len_ok && tid == 0) dev_fail(p.status, DEV_ERR_BOUNDS);
+
+    if (warp == 4) {
+        if (lane == 0) {
+            prefetch_tmap(&p.tmQ);
+            prefetch_tmap(&p.tmK);
+            // everything but the newest row is older than the step's first kernel
+            const int first_tile = k_begin / TK, old_keys = (len - 1) / kPageTokens * kPageTokens;
+            int next = 0;
+            if (p.early)
+                while (next < min(p.stages, tiles) && k_begin + (next + 1) * TK <= old_keys) {
+                    load_tile(p, seq, len, first_tile + next, blocks, stage_bytes, k_s, k_full, first_tile);
+                    ++next;
+                }
+            pdl_wait();
+            tl_mark(p.tl, 1);
+            if (tiles > 0) mbar_arrive_expect_tx(&q_full, rank_blocks * q_block);  // no copy that nobody waits for
+            for (int b = 0; b < rank_blocks && tiles > 0; ++b) tma_load_2d(q_s + b * q_block, &p.tmQ, b * 64, t * p.heads + head0, &q_full);
+            for (; next < tiles; ++next) {
+                if (next >= p.stages && !mbar_wait(&k_empty[next % p.stages], (uint32_t)(next / p.stages - 1) & 1u, p.status, DEV_ERR_EMPTY_WAIT)) break;
+                load_tile(p, seq, len, first_tile + next, blocks, stage_bytes, k_s, k_full, first_tile);
+            }
+        }
+    } else if (warp == 5) {
+        if (lane == 0 && tiles > 0) {
+            constexpr uint32_t idesc_s = umma_idesc_bf16(TK, HP);
+            constexpr uint32_t idesc_o = umma_idesc_bf16(128, 2 * HP) | (1u << 15) | (1u << 16);  // A and B with their K extent in rows
+            const uint32_t q_a = smem_u32(q_s), k_a = smem_u32(k_s), p_a = smem_u32(p_s);
+            const int rank_steps = (p.rank + 15) / 16, rot_steps = (p.rot + 15) / 16;
+            auto scores = [&](int j) {
+                const int st = j % p.stages;
+                if (!mbar_wait(&k_full[st], (uint32_t)(j / p.stages) & 1u, p.status, DEV_ERR_FULL_WAIT)) return false;
+                tc_fence_after();
+                const uint32_t kb = k_a + st * stage_bytes, d = tmem + (j & 1) * HP;
+                for (int i = 0; i < rank_steps + rot_steps; ++i) {
+                    const int i2 = i < rank_steps ? i : rank_blocks * 4 + (i - rank_steps);
+                    const uint32_t in = (uint32_t)(i2 & 3) * 32;
+                    umma_bf16(d, umma_desc_k128(kb + (i2 >> 2) * kBlockBytes + in), umma_desc_k128(q_a + (i2 >> 2) * q_block + in), idesc_s, i > 0);
+                }
+                umma_commit(&s_full[j & 1]);
+                return true;
+            };
+            const bool ahead = p.stages > 1;  // the scores of the next tile run while this tile's softmax does
+            bool ok = mbar_wait(&q_full, 0, p.status, DEV_ERR_FULL_WAIT) && scores(0);
+            for (int j = 0; j < tiles && ok; ++j) {
+                if (ahead && j + 1 < tiles) ok = scores(j + 1);
+                if (!ok || !mbar_wait(&p_full[j & 1], (uint32_t)(j >> 1) & 1u, p.status, DEV_ERR_ACC_WAIT)) break;
+                tc_fence_after();
+                const uint32_t v = k_a + (j % p.stages) * stage_bytes, pb = p_a + (j & 1) * kDecP;
+                for (int mb = 0; mb < mblocks; ++mb)
+#pragma unroll
+                    for (int kk = 0; kk < TK / 16; ++kk)
+                        umma_bf16(tmem + colO + mb * 2 * HP, desc_n128(v + mb * 2 * kBlockBytes + kk * 2048), desc_n128(pb + kk * 2048), idesc_o,
+                                  j > 0 || kk > 0);
+                umma_commit(&k_empty[j % p.stages]);
+                umma_commit(&pv_done[j & 1]);
+                if (!ahead && j + 1 < tiles) ok = scores(j + 1);
+            }
+        }
+    } else {
+        pdl_wait();
+        rotate_q(p, t, head0, nheads, p.part_heads, q_s + rank_blocks * q_block, q_block);
+        for (int i = tid; i < (HP - p.part_heads) * rot_blocks * 8; i += kDecSoftmax)  // rows without a head
+            *(uint4*)(q_s + (rank_blocks + i / 8 % rot_blocks) * q_block + (p.part_heads + i / 8 / rot_blocks) * 128 + i % 8 * 16) = make_uint4(0u, 0u, 0u, 0u);
+        fence_proxy_async_smem();
+        mbar_arrive(&q_full);
+        // rows of S^T: key 16 w + l of the tile is lane l < 16 of warp w
+        const uint32_t lane_addr = tmem + ((uint32_t)(warp * 32) << 16);
+        const int row = warp * 16 + (lane & 15);
+        float m_ref[HP], l_sum[HP];
+#pragma unroll
+        for (int h = 0; h < HP; ++h) {
+            m_ref[h] = kNeg;
+            l_sum[h] = 0.f;
+        }
+        bool ok = true;  // after a wait has run out the warp goes through the motions, so that the others' barriers complete
+        auto wait = [&](uint64_t* bar, uint32_t parity) {
+            if (ok) ok = __all_sync(0xffffffffu, mbar_wait(bar, parity, p.status, DEV_ERR_ACC_WAIT));
+        };
+        for (int j = 0; j < tiles; ++j) {
+            wait(&s_full[j & 1], (uint32_t)(j >> 1) & 1u);
+            tc_fence_after();
+            float s[HP];
+#pragma unroll
+            for (int c = 0; c < HP / 16; ++c) {
+                uint32_t v[16];
+                tmem_ld16(lane_addr + (j & 1) * HP + c * 16, v);
+                tc_wait_ld();
+#pragma unroll
+                for (int i = 0; i < 16; ++i) s[c * 16 + i] = __uint_as_float(v[i]) * p.scale_log2;
+            }
+            const bool live = lane < 16 && k_begin + j * TK + row < k_end;
+            bool up = j == 0;
+#pragma unroll
+            for (int h = 0; h < HP; ++h) {
+                if (!live) s[h] = kNeg;
+                up = up || (h < nheads && s[h] > m_ref[h] + 8.f);
+            }
+            if (softmax_any(up)) {  // the reference maxima move to the running maxima
+#pragma unroll
+                for (int h = 0; h < HP; ++h) {
+                    float m = s[h];
+#pragma unroll
+                    for (int o = 8; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+                    if (lane == 0) s_max[warp][h] = m;
+                }
+                softmax_sync();
+                if (j > 0) {
+                    wait(&pv_done[(j - 1) & 1], (uint32_t)((j - 1) >> 1) & 1u);
+                    tc_fence_after();
+                }
+                float corr[HP];
+#pragma unroll
+                for (int h = 0; h < HP; ++h) {
+                    const float m = fmaxf(fmaxf(fmaxf(s_max[0][h], s_max[1][h]), fmaxf(s_max[2][h], s_max[3][h])), m_ref[h]);
+                    corr[h] = exp2_fast(m_ref[h] - m);
+                    m_ref[h] = m;
+                    l_sum[h] *= corr[h];
+                }
+                if (j > 0) {
+                    for (int c = 0; c < mblocks * 2; ++c) {
+#pragma unroll
+                        for (int q = 0; q < HP / 16; ++q) {
+                            uint32_t o[16];
+                            tmem_ld16(lane_addr + colO + c * HP + q * 16, o);
+                            tc_wait_ld();
+#pragma unroll
+                            for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * corr[q * 16 + i]);
+                            tmem_st16(lane_addr + colO + c * HP + q * 16, o);
+                        }
+                    }
+                    tc_wait_st();
+                }
+                softmax_sync();  // s_max may be written again
+            }
+            uint32_t hi[HP / 2], lo[HP / 2];
+#pragma unroll
+            for (int h = 0; h < HP; h += 2) {
+                const float a = live ? exp2_fast(s[h] - m_ref[h]) : 0.f, b = live ? exp2_fast(s[h + 1] - m_ref[h + 1]) : 0.f;
+                l_sum[h] += a;
+                l_sum[h + 1] += b;
+                const __nv_bfloat162 h2 = __floats2bfloat162_rn(a, b);
+                hi[h / 2] = *(const uint32_t*)&h2;
+                const __nv_bfloat162 l2 = __floats2bfloat162_rn(a - bf16_lo(hi[h / 2]), b - bf16_hi(hi[h / 2]));
+                lo[h / 2] = *(const uint32_t*)&l2;
+            }
+            if (j > 1) wait(&pv_done[j & 1], (uint32_t)((j - 2) >> 1) & 1u);  // the buffer's last product is done
+            if (lane < 16) {
+                uint8_t* dst = p_s + (j & 1) * kDecP + row * 128;
+#pragma unroll
+                for (int c = 0; c < HP / 8; ++c) {
+                    *(uint4*)(dst + ((c ^ (row & 7)) << 4)) = make_uint4(hi[4 * c], hi[4 * c + 1], hi[4 * c + 2], hi[4 * c + 3]);
+                    *(uint4*)(dst + (((c + HP / 8) ^ (row & 7)) << 4)) = make_uint4(lo[4 * c], lo[4 * c + 1], lo[4 * c + 2], lo[4 * c + 3]);
+                }
+            }
+            fence_proxy_async_smem();
+            tc_fence_before();
+            mbar_arrive(&p_full[j & 1]);
+        }
+        if (tiles > 0) wait(&pv_done[(tiles - 1) & 1], (uint32_t)((tiles - 1) >> 1) & 1u);
+        tc_fence_after();
+        // ---- sums over the keys, then this thread's value columns (lane = column of a group of 128)
+#pragma unroll
+        for (int h = 0; h < HP; ++h) {
+            const float l = warp_sum(l_sum[h]);
+            if (lane == 0) s_sum[warp][h] = l;
+        }
+        softmax_sync();
+        const size_t row_ld = partial_ld(p.rank), ml_at = row_ld - 4;  // partial rows: [unit][split][part_heads][row_ld], at its end: maximum, sum
+        float* parts = p.ws + ((size_t)unit * p.splits + blockIdx.y) * p.part_heads * row_ld;
+        if (tid < nheads) {
+            const float l = s_sum[0][tid] + s_sum[1][tid] + s_sum[2][tid] + s_sum[3][tid];
+            if (p.splits == 1) {
+                s_mult[tid] = sigmoid_f32(act_load(p.gate + (size_t)t * p.gate_ld + head0 + tid)) / l;
+            } else {
+                float m = kNeg;
+#pragma unroll
+                for (int h = 0; h < HP; ++h) m = h == tid ? m_ref[h] : m;
+                parts[tid * row_ld + ml_at] = m;
+                parts[tid * row_ld + ml_at + 1] = l;
+            }
+        }
+        softmax_sync();
+        if (tiles > 0) {
+            for (int mb = 0; mb < mblocks; ++mb) {
+                const int col = mb * 128 + warp * 32 + lane;
+#pragma unroll
+                for (int q = 0; q < HP / 16; ++q) {
+                    uint32_t a[16], b[16];
+                    tmem_ld16(lane_addr + colO + mb * 2 * HP + q * 16, a);
+                    tmem_ld16(lane_addr + colO + mb * 2 * HP + HP + q * 16, b);
+                    tc_wait_ld();
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) {
+                        const int h = q * 16 + i;
+                        const float o = __uint_as_float(a[i]) + __uint_as_float(b[i]);  // P_hi V + P_lo V
+                        if (col < p.rank && h < nheads) {
+                            if (p.splits == 1) p.out[((size_t)t * p.heads + head0 + h) * p.head_ld + col] = __float2bfloat16_rn(o * s_mult[h]);
+                            else parts[h * row_ld + col] = o;
+                        }
+                    }
+                    __syncwarp();
+                }
+            }
+        }
+        if (p.splits > 1) __threadfence();
+    }
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 5) tmem_dealloc(tmem, tmem_cols);
     if (p.splits > 1) {
         if (tid == 0) {
+            __threadfence();
             const int old = atomicAdd(&p.counters[unit], 1);
             s_last = old == p.splits - 1;
             if (s_last) p.counters[unit] = 0;
         }
         __syncthreads();
-        if (s_last && ntok > 0) {
+        if (s_last) {
             __threadfence();
-            const int cols = min(p.slice_cols, p.rank - slice * p.slice_cols), ld = p.slice_cols + 2, pad_cols = (cols + 7) / 8 * 8;
-            const float* parts = p.ws + (size_t)unit * p.splits * p.part_heads * ld;
+            // weight of split z for head h: 2^(m_z - M) gate / sum; in the idle buffers of P
+            const size_t row_ld = partial_ld(p.rank), step = p.part_heads * row_ld;
+            const float* parts = p.ws + (size_t)unit * p.splits * step;
+            float* wgt = (float*)p_s;  // [HP][splits]
+            static_assert(HP * kDecMaxSplits * 4 <= 2 * kDecP, "");
             for (int h = warp; h < nheads; h += kThreads / 32) {
-                const float* row = parts + (size_t)h * ld;
-                const size_t step = (size_t)p.part_heads * ld;
-                float M = kNeg, L = 0.f;
-                for (int z = 0; z < p.splits; ++z) M = fmaxf(M, __ldcg(row + z * step + p.slice_cols));
-                for (int z = 0; z < p.splits; ++z) L += __ldcg(row + z * step + p.slice_cols + 1) * exp2_fast(__ldcg(row + z * step + p.slice_cols) - M);
-                const float mult = sigmoid_f32(act_load(p.gate + (size_t)t0 * p.gate_ld + head0 + h)) / L;
-                bf16* dst = p.out + ((size_t)t0 * p.heads + head0 + h) * p.head_ld + slice * p.slice_cols;
-                for (int c = lane * 4; c < pad_cols; c += 128) {
-                    float a[4] = {0.f, 0.f, 0.f, 0.f};
-                    for (int z = 0; z < p.splits; ++z) {
-                        const float w = exp2_fast(__ldcg(row + z * step + p.slice_cols) - M);
-                        if (__ldcg(row + z * step + p.slice_cols + 1) <= 0.f) continue;  // a split without keys wrote no columns
-                        const float2 x = __ldcg((const float2*)(row + z * step + c)), y = __ldcg((const float2*)(row + z * step + c + 2));
-                        a[0] += w * x.x; a[1] += w * x.y; a[2] += w * y.x; a[3] += w * y.y;
-                    }
-                    *(uint2*)(dst + c) = make_uint2((uint32_t)bf16_bits(a[0] * mult) | ((uint32_t)bf16_bits(a[1] * mult) << 16),
-                                                    (uint32_t)bf16_bits(a[2] * mult) | ((uint32_t)bf16_bits(a[3] * mult) << 16));
+                const float* ml = parts + h * row_ld + row_ld - 4;
+                float m[2], l[2], M = kNeg, L = 0.f;
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const int z = lane + 32 * i;
+                    m[i] = z < p.splits ? __ldcg(ml + z * step) : kNeg;
+                    l[i] = z < p.splits ? __ldcg(ml + z * step + 1) : 0.f;
+                    M = fmaxf(M, m[i]);
+                }
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+#pragma unroll
+                for (int i = 0; i < 2; ++i) L += l[i] * exp2_fast(m[i] - M);
+                L = warp_sum(L);
+                const float mult = sigmoid_f32(act_load(p.gate + (size_t)t * p.gate_ld + head0 + h)) / L;
+#pragma unroll
+                for (int i = 0; i < 2; ++i)
+                    if (lane + 32 * i < p.splits) wgt[h * p.splits + lane + 32 * i] = l[i] > 0.f ? exp2_fast(m[i] - M) * mult : 0.f;
+            }
+            __syncthreads();
+            // a piece = four columns of a head; the loads of four pieces and two splits in flight together
+            const int per_head = (p.rank + 3) / 4, n = nheads * per_head;
+            for (int i0 = tid; i0 < n; i0 += 4 * kThreads) {
+                float o[4][4];
+#pragma unroll
+                for (int k = 0; k < 4; ++k) o[k][0] = o[k][1] = o[k][2] = o[k][3] = 0.f;
+                for (int z0 = 0; z0 < p.splits; z0 += 2) {
+                    float4 x[4][2];
+                    float w[4][2];
+#pragma unroll
+                    for (int k = 0; k < 4; ++k)
+#pragma unroll
+                        for (int q = 0; q < 2; ++q) {
+                            const int i = min(i0 + k * kThreads, n - 1), h = i / per_head, z = z0 + q;
+                            w[k][q] = z < p.splits ? wgt[h * p.splits + z] : 0.f;
+                            x[k][q] = make_float4(0.f, 0.f, 0.f, 0.f);
+                            if (w[k][q] > 0.f) x[k][q] = __ldcg((const float4*)(parts + z * step + h * row_ld) + i % per_head);
+                        }
+#pragma unroll
+                    for (int k = 0; k < 4; ++k)
+#pragma unroll
+                        for (int q = 0; q < 2; ++q) {
+                            o[k][0] += w[k][q] * x[k][q].x;
+                            o[k][1] += w[k][q] * x[k][q].y;
+                            o[k][2] += w[k][q] * x[k][q].z;
+                            o[k][3] += w[k][q] * x[k][q].w;
+                        }
+                }
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    const int i = i0 + k * kThreads, h = i / per_head, c = i % per_head * 4;
+                    if (i >= n) break;
+                    bf16* dst = p.out + ((size_t)t * p.heads + head0 + h) * p.head_ld + c;  // rows padded to 8 columns
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) o[k][q] = c + q < p.rank ? o[k][q] : 0.f;
+                    *(uint2*)dst = make_uint2((uint32_t)bf16_bits(o[k][0]) | ((uint32_t)bf16_bits(o[k][1]) << 16),
+                                              (uint32_t)bf16_bits(o[k][2]) | ((uint32_t)bf16_bits(o[k][3]) << 16));
                 }
             }
         }
@@ -387,44 +746,65 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_consta
 
 // how a launch is cut into tiles; stages == 0: does not fit
 struct LatentPlan {
-    int part_heads, parts, tile_tokens, q_rows, slices, slice_cols, stages, smem;
+    int part_heads, parts, tile_tokens, q_rows, slices, slice_cols, stages, smem, tmem_cols;
 };
-LatentPlan plan(int rank, int rot, int heads, bool prompt) {
+constexpr int kStaticSmem = 2048;  // room for the kernels' static shared memory
+
+LatentPlan plan_prompt(int rank, int rot, int heads) {
     LatentPlan l;
     const int blocks = (rank + 63) / 64 + (rot + 63) / 64;
     l.parts = (heads + kRowsMax - 1) / kRowsMax;
     l.part_heads = (heads + l.parts - 1) / l.parts;
-    l.tile_tokens = prompt ? std::max(1, std::min(8, kRowsMax / l.part_heads)) : 1;
+    l.tile_tokens = std::max(1, std::min(8, kRowsMax / l.part_heads));
     l.slices = (rank + kSliceCols - 1) / kSliceCols;
     l.slice_cols = ((rank + l.slices - 1) / l.slices + 63) / 64 * 64;
     l.slices = (rank + l.slice_cols - 1) / l.slice_cols;
-    const int fixed = 1024 + 512;  // alignment, static shared memory
+    l.tmem_cols = kTmemCols;
     for (;; l.tile_tokens = (l.tile_tokens + 1) / 2) {
         l.q_rows = (l.tile_tokens * l.part_heads + 7) / 8 * 8;
         const int q = blocks * l.q_rows * 128;
-        l.stages = std::min(kMaxStages, (kSmemLimit - fixed - q) / (blocks * kBlockBytes));
+        l.stages = std::min(kMaxStages, (kSmemLimit - kStaticSmem - 1024 - q) / (blocks * kBlockBytes));
         // an operand tile is always read as 128 rows: what follows the last block of Q has to exist
         l.smem = 1024 + q + std::max(l.stages * blocks * kBlockBytes, (kRowsMax - l.q_rows) * 128);
-        if (l.stages >= 1 && l.smem <= kSmemLimit - 512) return l;
+        if (l.stages >= 1 && l.smem <= kSmemLimit - kStaticSmem) return l;
         l.stages = 0;
         if (l.tile_tokens == 1) return l;
     }
 }
 
+LatentPlan plan_decode(int rank, int rot, int heads) {
+    LatentPlan l;
+    memset(&l, 0, sizeof l);
+    const int blocks = (rank + 63) / 64 + (rot + 63) / 64, mblocks = (rank + 127) / 128;
+    for (int hp = heads > 16 ? 32 : 16; hp >= 16; hp /= 2) {
+        l.parts = (heads + hp - 1) / hp;
+        l.part_heads = (heads + l.parts - 1) / l.parts;
+        l.q_rows = hp;
+        const int cols = 2 * hp + mblocks * 2 * hp, fixed = 1024 + blocks * hp * 128 + 2 * kDecP;
+        l.tmem_cols = 32;
+        while (l.tmem_cols < cols) l.tmem_cols *= 2;
+        l.stages = std::min(kMaxStages, (kSmemLimit - kStaticSmem - fixed) / (blocks * kBlockBytes));
+        l.smem = fixed + l.stages * blocks * kBlockBytes;
+        if (l.stages >= 1 && l.tmem_cols <= 512) return l;
+    }
+    l.stages = 0;
+    return l;
+}
+
 }  // namespace
 
 bool attention_latent_supported(int rank, int rot, int heads) {
-    return heads >= 1 && plan(rank, rot, heads, false).stages >= 1 && plan(rank, rot, heads, true).stages >= 1;
+    return heads >= 1 && plan_decode(rank, rot, heads).stages >= 1 && plan_prompt(rank, rot, heads).stages >= 1;
 }
 
 int attention_latent_splits(int rows, int rank, int rot, int heads, int max_ctx, const AttnWorkspace& ws, int num_sms) {
-    const LatentPlan l = plan(rank, rot, heads, false);
-    const int units = rows * l.parts * l.slices;
+    const LatentPlan l = plan_decode(rank, rot, heads);
+    const int units = rows * l.parts;
     int splits = 1;
     if (units * 2 <= num_sms) {
-        splits = std::min(num_sms / units, (max_ctx + kLatentSplitKeys - 1) / kLatentSplitKeys);
-        splits = std::max(1, std::min(splits, 64));
-        while (splits > 1 && ((size_t)units * splits * l.part_heads * (l.slice_cols + 2) > ws.partial_floats || units > ws.num_counters)) --splits;
+        splits = std::min(num_sms / units, max_ctx / kLatentSplitKeys);
+        splits = std::max(1, std::min(splits, kDecMaxSplits));
+        while (splits > 1 && ((size_t)units * splits * l.part_heads * partial_ld(rank) > ws.partial_floats || units > ws.num_counters)) --splits;
     }
     return splits;
 }
@@ -432,7 +812,7 @@ int attention_latent_splits(int rows, int rank, int rot, int heads, int max_ctx,
 int launch_attention_latent(const LatentAttn& a, int T, int n_groups, int max_ctx, const AttnWorkspace& ws, int num_sms, TmapCache* tmaps,
                             cudaStream_t s, bool pdl, unsigned long long* tl) {
     const bool prompt = n_groups > 0;
-    const LatentPlan l = plan(a.rank, a.rot, a.heads, prompt);
+    const LatentPlan l = prompt ? plan_prompt(a.rank, a.rot, a.heads) : plan_decode(a.rank, a.rot, a.heads);
     if (l.stages < 1 || a.head_ld % 8 || a.kv.hd != latent_row_cols(a.rank, a.rot)) return (int)cudaErrorInvalidValue;
     LatentDev p;
     memset(&p, 0, sizeof p);
@@ -449,20 +829,17 @@ int launch_attention_latent(const LatentAttn& a, int T, int n_groups, int max_ct
     p.num_pages = a.kv.num_pages;
     p.tok_seq = a.tok_seq;
     p.tok_pos = a.tok_pos;
-    p.grp_first = prompt ? a.grp_first : nullptr;
+    p.grp_first = a.grp_first;
     p.grp_count = a.grp_count;
     p.heads = a.heads;
     p.part_heads = l.part_heads;
     p.parts = l.parts;
     p.tile_tokens = l.tile_tokens;
-    p.subs = prompt ? (8 + l.tile_tokens - 1) / l.tile_tokens : 1;
     p.q_rows = l.q_rows;
     p.rank = a.rank;
     p.slices = l.slices;
     p.slice_cols = l.slice_cols;
     p.stages = l.stages;
-    p.splits = prompt ? 1 : attention_latent_splits(T, a.rank, a.rot, a.heads, max_ctx, ws, num_sms);
-    p.early = pdl && a.only_newest_row_fresh;
     p.scale_log2 = a.scale * 1.4426950408889634f;
     p.gate = a.gate;
     p.gate_ld = a.gate_ld;
@@ -472,13 +849,27 @@ int launch_attention_latent(const LatentAttn& a, int T, int n_groups, int max_ct
     p.counters = ws.counters;
     p.status = a.status;
     p.tl = tl;
-    const int units = (prompt ? n_groups * p.subs : T) * l.parts * l.slices;
-    return (int)launch_k(k_attn_latent, dim3(units, p.splits), dim3(kThreads), (size_t)l.smem, s, pdl, p);
+    if (prompt) {
+        p.subs = (8 + l.tile_tokens - 1) / l.tile_tokens;
+        return (int)launch_k(k_attn_latent, dim3(n_groups * p.subs * l.parts * l.slices), dim3(kThreads), (size_t)l.smem, s, pdl, p);
+    }
+    p.splits = attention_latent_splits(T, a.rank, a.rot, a.heads, max_ctx, ws, num_sms);
+    p.early = pdl && a.only_newest_row_fresh;
+    const dim3 grid(T * l.parts, p.splits);
+    if (l.q_rows == 16) return (int)launch_k(k_attn_latent_decode<16>, grid, dim3(kThreads), (size_t)l.smem, s, pdl, p, (uint32_t)l.tmem_cols);
+    return (int)launch_k(k_attn_latent_decode<32>, grid, dim3(kThreads), (size_t)l.smem, s, pdl, p, (uint32_t)l.tmem_cols);
 }
 
+template <typename Kern>
+static cudaError_t latent_attr(Kern k) {
+    const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - kStaticSmem);
+    return e == cudaSuccess ? prefer_max_shared(k) : e;
+}
 int attention_latent_prepare() {
-    cudaError_t e = cudaFuncSetAttribute(k_attn_latent, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 512);
-    return (int)(e == cudaSuccess ? prefer_max_shared(k_attn_latent) : e);
+    cudaError_t e = latent_attr(k_attn_latent);
+    if (e == cudaSuccess) e = latent_attr(k_attn_latent_decode<16>);
+    if (e == cudaSuccess) e = latent_attr(k_attn_latent_decode<32>);
+    return (int)e;
 }
 
 }  // namespace tffn

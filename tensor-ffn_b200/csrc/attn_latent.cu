@@ -4,17 +4,18 @@
 // Prompts (k_attn_latent): the heads of up to eight tokens of a sequence are the 128 rows of one tile:
 //   S[row, key] = Q[row, :] . K[key, :]      tcgen05.mma, Q and K in shared memory (both K-major)
 //   O[row, :]  += P[row, :] . K[:, columns]  tcgen05.mma, P in tensor memory, K read the other way round (N-major)
-// One CTA = the rows of one tile x at most 256 value columns, 6 warps:
+// One CTA = the rows of one tile x at most 256 value columns, 7 warps:
 //   warps 0-3  thread = row: S out of tensor memory, online softmax in fp32, P back as a bf16 pair (hi + lo, 16 mantissa
 //              bits), the rotated part of Q at the start, and the output rows at the end
 //   warp 4     TMA producer: Q, then 64 keys (two pages) per stage, 64 columns per box with the 128-byte swizzle
-//   warp 5     tensor memory, MMA issue
+//   warp 5     tensor memory, issue of S (two tiles ahead of the softmax where the ring is deep enough)
+//   warp 6     issue of O
 // The reference maximum of a row moves only when it would be exceeded by more than 2^8, so O is rarely rescaled.
 //
 // Decoding (k_attn_latent_decode): one token's heads would leave most of those rows empty, so keys and value columns take
 // the long side instead, S^T[key, head] = K . Q^T and O^T[column, head] += K^T . P^T: all value columns in one CTA. P^T is
 // written to shared memory next to its lo part (twice the columns of one product). One CTA = 16 or 32 heads of a token x
-// one context split, the same six warps (thread = key). Splits leave partial rows and the last one to finish (a ticket, no
+// one context split, the same seven warps (thread = key). Splits leave partial rows and the last one to finish (a ticket, no
 // waiting) adds them up in split order.
 //
 // Rows of a page past the end of a sequence are finite (zeros or an earlier request's normed latents) and weigh zero.
@@ -31,8 +32,8 @@ namespace {
 constexpr int TK = 64;                     // keys per stage
 constexpr int kRowsMax = 128;              // rows of a tile
 constexpr int kSliceCols = 256;            // value columns of a CTA
-constexpr int kThreads = 192;
-constexpr int kMaxStages = 4;
+constexpr int kThreads = 224;
+constexpr int kMaxStages = 6;
 constexpr int kBlockBytes = TK * 128;      // 64 keys x 64 columns
 constexpr int kSmemLimit = 227 * 1024;
 constexpr uint32_t kTmemCols = 512, kColS = 0, kColP = 2 * TK, kColO = 3 * TK;  // S twice, P hi | lo, O
@@ -68,16 +69,17 @@ struct LatentDev {
 };
 
 // shared-memory descriptor of an operand whose rows are its K extent: 64 columns (128 swizzled bytes) per row, groups of 64
-// columns kBlockBytes apart (leading byte offset), groups of 8 rows 1024 bytes apart (stride byte offset)
-__device__ __forceinline__ uint64_t desc_n128(uint32_t smem_addr) {
-    return (uint64_t)((smem_addr & 0x3FFFFu) >> 4) | ((uint64_t)(kBlockBytes >> 4) << 16) | (64ull << 32) | (1ull << 46) | (2ull << 61);
+// columns block_bytes apart (leading byte offset), groups of 8 rows 1024 bytes apart (stride byte offset)
+__device__ __forceinline__ uint64_t desc_n128(uint32_t smem_addr, int block_bytes) {
+    return (uint64_t)((smem_addr & 0x3FFFFu) >> 4) | ((uint64_t)(block_bytes >> 4) << 16) | (64ull << 32) | (1ull << 46) | (2ull << 61);
 }
 // D[tmem] (+)= A[tmem] * B[smem]
 __device__ __forceinline__ void umma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
     asm volatile(
-        "{\n\t.reg .pred p;\n\t"
+        "{\n\t.reg .pred p, q;\n\t"
         "setp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}" ::"r"(d_tmem),
+        "elect.sync _|q, 0xffffffff;\n\t"
+        "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}" ::"r"(d_tmem),
         "r"(a_tmem), "l"(bdesc), "r"(idesc), "r"(accumulate)
         : "memory");
 }
@@ -95,92 +97,135 @@ __device__ __forceinline__ float exp2_fast(float x) {
     return y;
 }
 
-// 64 keys of a sequence (its `tile`-th) into the stage of the ring that is theirs; tile0: the CTA's first tile. A page past
-// the end is replaced by the last one, its keys are masked.
-__device__ __forceinline__ void load_tile(const LatentDev& p, int seq, int len, int tile, int blocks, int stage_bytes, uint8_t* ring, uint64_t* full,
-                                          int tile0 = 0) {
-    const int* bt = p.block_table + (size_t)seq * p.max_pages_per_seq;
-    const int st = (tile - tile0) % p.stages, last_page = (len - 1) / kPageTokens;
-    uint8_t* dst = ring + st * stage_bytes;
-    mbar_arrive_expect_tx(&full[st], stage_bytes);
-    for (int h = 0; h < TK / kPageTokens; ++h) {
-        int pg = __ldg(bt + min(tile * (TK / kPageTokens) + h, last_page));
-        if (pg < 0 || pg >= p.num_pages) {
-            dev_fail(p.status, DEV_ERR_BOUNDS);
-            pg = 0;
-        }
-        for (int b = 0; b < blocks; ++b) tma_load_2d(dst + b * kBlockBytes + h * kPageTokens * 128, &p.tmK, b * 64, pg * kPageTokens, &full[st]);
-    }
+// every lane of an issuing warp waits (acquire), the outcome is made uniform
+__device__ __forceinline__ bool mma_wait(uint64_t* bar, uint32_t parity, int* status, int code) {
+    return __all_sync(0xffffffffu, mbar_wait(bar, parity, status, code));
 }
 
+// The producer warp's view of a sequence's pages: KEYS keys (whole pages) per tile, page ids fetched 32 at a time (lane = page).
+template <int KEYS>
+struct PageLoader {
+    const LatentDev& p;
+    const int* bt;
+    int page0, last_page, blocks, lane;  // first page of tile 0; last page of the sequence
+    uint32_t ring, full;                 // shared memory: stages, their barriers
+    int ids;
+
+    __device__ __forceinline__ PageLoader(const LatentDev& p_, int seq, int len, int key0, int blocks_, void* ring_, uint64_t* full_, int lane_)
+        : p(p_), bt(p_.block_table + (size_t)seq * p_.max_pages_per_seq), page0(key0 / kPageTokens), last_page((len - 1) / kPageTokens),
+          blocks(blocks_), lane(lane_), ring(smem_u32(ring_)), full(smem_u32(full_)), ids(0) {}
+    // the whole warp. Pages past the end are replaced by the last one; their keys are masked.
+    __device__ __forceinline__ void load(int tile) {
+        constexpr int PAGES = KEYS / kPageTokens;
+        const int st = tile % p.stages;
+        const uint32_t bar = full + st * 8, dst = ring + st * (blocks * KEYS * 128);
+        if ((tile * PAGES) % 32 == 0) {
+            ids = __ldg(bt + min(page0 + tile * PAGES + lane, last_page));
+            if (ids < 0 || ids >= p.num_pages) {
+                dev_fail(p.status, DEV_ERR_BOUNDS);
+                ids = 0;
+            }
+        }
+        mbar_arrive_expect_tx_elect(bar, blocks * KEYS * 128);
+#pragma unroll
+        for (int h = 0; h < PAGES; ++h) {
+            const int row = __shfl_sync(0xffffffffu, ids, (tile * PAGES + h) % 32) * kPageTokens;
+            const uint32_t to = dst + h * kPageTokens * 128;
+#pragma unroll 4
+            for (int b = 0; b < blocks; ++b) tma_load_2d_elect(to + b * (KEYS * 128), &p.tmK, b * 64, row, bar);
+        }
+    }
+};
+
 // The rotated parts of Q, rows 0 .. rows - 1 of the tile (row = token * part_heads + head), into the blocks behind the latent
-// ones; columns past `rot` are zero, and so are rows of heads that do not exist. The 128 softmax threads call it.
-__device__ __forceinline__ void rotate_q(const LatentDev& p, int t0, int head0, int nheads, int rows, uint8_t* q_rot, int q_block) {
-    const int half = p.rot / 2, tid = threadIdx.x, zero_to = (p.rot + 15) / 16 * 16;
-    auto at = [&](int r, int col) {  // address of the 8 columns from `col` (a multiple of 8) of row r
-        const int c = (col & 63) >> 3;
-        return q_rot + (col >> 6) * q_block + r * 128 + ((c ^ (r & 7)) << 4);
-    };
-    if (half % 8 == 0) {
-        constexpr int B = 4;  // pieces of 8 pairs with their loads in flight together
-        const int pieces = half / 8, n = rows * pieces;
-        for (int i0 = tid; i0 < n; i0 += B * kRowsMax) {
-            uint4 u[B], v[B];
-            float4 cs[B][4];
+// ones; columns past `rot` are zero, and so are rows of heads that do not exist. The 128 softmax threads call it. Angles are
+// older than the previous kernel (they are read by the constructor), the parts themselves are not.
+struct QueryRotation {
+    static constexpr int B = 4;  // pieces of 8 pairs with their loads in flight together
+    const LatentDev& p;
+    int t0, head0, nheads, rows, half, q_block;
+    uint8_t* q_rot;
+    float4 cs[B][4];
+
+    // `i`-th piece of the first batch and of the ones that follow it: row, first pair
+    __device__ __forceinline__ void load_angles(int i0) {
+        const int pieces = half / 8;
 #pragma unroll
-            for (int k = 0; k < B; ++k) {
-                const int i = i0 + k * kRowsMax, r = i / pieces, c = i % pieces * 8, h = r % p.part_heads, t = t0 + r / p.part_heads;
-                u[k] = v[k] = make_uint4(0u, 0u, 0u, 0u);
-                if (i < n) {
-                    const int pos = min(max(__ldcg(p.tok_pos + t), 0), p.max_pos - 1);
-                    const float4* f = (const float4*)(p.rope + (size_t)pos * half + c);
+        for (int k = 0; k < B; ++k) {
+            const int i = i0 + k * kRowsMax;
+            if (i < rows * pieces) {
+                const int pos = min(max(__ldcg(p.tok_pos + t0 + i / pieces / p.part_heads), 0), p.max_pos - 1);
+                const float4* f = (const float4*)(p.rope + (size_t)pos * half + i % pieces * 8);
 #pragma unroll
-                    for (int q = 0; q < 4; ++q) cs[k][q] = __ldg(f + q);
-                    if (h < nheads) {
-                        const bf16* src = p.q_up + (size_t)t * p.q_up_ld + p.rot_off + (size_t)(head0 + h) * p.rot + c;
+                for (int q = 0; q < 4; ++q) cs[k][q] = __ldg(f + q);
+            }
+        }
+    }
+    __device__ __forceinline__ QueryRotation(const LatentDev& p_, int t0_, int head0_, int nheads_, int rows_, uint8_t* q_rot_, int q_block_)
+        : p(p_), t0(t0_), head0(head0_), nheads(nheads_), rows(rows_), half(p_.rot / 2), q_block(q_block_), q_rot(q_rot_) {
+        if (half % 8 == 0) load_angles(threadIdx.x);
+    }
+    __device__ __forceinline__ uint8_t* at(int r, int col) const {  // the 8 columns from `col` (a multiple of 8) of row r
+        return q_rot + (col >> 6) * q_block + r * 128 + ((((col & 63) >> 3) ^ (r & 7)) << 4);
+    }
+    __device__ __forceinline__ void put(int r, int col, float x) const { *(bf16*)(at(r, col & ~7) + (col & 7) * 2) = __float2bfloat16_rn(x); }
+
+    __device__ __forceinline__ void store() {
+        const int tid = threadIdx.x;
+        if (half % 8 == 0) {  // rot is a multiple of 16: no columns to clear
+            const int pieces = half / 8, n = rows * pieces;
+            for (int i0 = tid; i0 < n; i0 += B * kRowsMax) {
+                if (i0 != tid) load_angles(i0);
+                uint4 u[B], v[B];
+#pragma unroll
+                for (int k = 0; k < B; ++k) {
+                    const int i = i0 + k * kRowsMax, r = i / pieces, h = r % p.part_heads;
+                    u[k] = v[k] = make_uint4(0u, 0u, 0u, 0u);
+                    if (i < n && h < nheads) {
+                        const bf16* src = p.q_up + (size_t)(t0 + r / p.part_heads) * p.q_up_ld + p.rot_off + (size_t)(head0 + h) * p.rot + i % pieces * 8;
                         u[k] = __ldcg((const uint4*)src);
                         v[k] = __ldcg((const uint4*)(src + half));
                     }
                 }
-            }
 #pragma unroll
-            for (int k = 0; k < B; ++k) {
-                const int i = i0 + k * kRowsMax, r = i / pieces, c = i % pieces * 8;
-                if (i >= n) break;
-                const uint32_t uu[4] = {u[k].x, u[k].y, u[k].z, u[k].w}, vv[4] = {v[k].x, v[k].y, v[k].z, v[k].w};
-                uint32_t a[4], b[4];
+                for (int k = 0; k < B; ++k) {
+                    const int i = i0 + k * kRowsMax, r = i / pieces, c = i % pieces * 8;
+                    if (i >= n) break;
+                    const uint32_t uu[4] = {u[k].x, u[k].y, u[k].z, u[k].w}, vv[4] = {v[k].x, v[k].y, v[k].z, v[k].w};
+                    uint32_t a[4], b[4];
 #pragma unroll
-                for (int q = 0; q < 4; ++q) {
-                    const float4 f = cs[k][q];
-                    const float u0 = bf16_lo(uu[q]), u1 = bf16_hi(uu[q]), v0 = bf16_lo(vv[q]), v1 = bf16_hi(vv[q]);
-                    a[q] = (uint32_t)bf16_bits(u0 * f.x - v0 * f.y) | ((uint32_t)bf16_bits(u1 * f.z - v1 * f.w) << 16);
-                    b[q] = (uint32_t)bf16_bits(v0 * f.x + u0 * f.y) | ((uint32_t)bf16_bits(v1 * f.z + u1 * f.w) << 16);
+                    for (int q = 0; q < 4; ++q) {
+                        const float4 f = cs[k][q];
+                        const float u0 = bf16_lo(uu[q]), u1 = bf16_hi(uu[q]), v0 = bf16_lo(vv[q]), v1 = bf16_hi(vv[q]);
+                        a[q] = (uint32_t)bf16_bits(u0 * f.x - v0 * f.y) | ((uint32_t)bf16_bits(u1 * f.z - v1 * f.w) << 16);
+                        b[q] = (uint32_t)bf16_bits(v0 * f.x + u0 * f.y) | ((uint32_t)bf16_bits(v1 * f.z + u1 * f.w) << 16);
+                    }
+                    *(uint4*)at(r, c) = make_uint4(a[0], a[1], a[2], a[3]);
+                    *(uint4*)at(r, half + c) = make_uint4(b[0], b[1], b[2], b[3]);
                 }
-                *(uint4*)at(r, c) = make_uint4(a[0], a[1], a[2], a[3]);
-                *(uint4*)at(r, half + c) = make_uint4(b[0], b[1], b[2], b[3]);
             }
+            return;
         }
-        return;  // rot is a multiple of 16
+        const int zero_to = (p.rot + 15) / 16 * 16;
+        for (int i = tid; i < rows * half; i += kRowsMax) {
+            const int r = i / half, c = i % half, h = r % p.part_heads, t = t0 + r / p.part_heads;
+            const int pos = min(max(__ldcg(p.tok_pos + t), 0), p.max_pos - 1);
+            const float2 f = __ldg(p.rope + (size_t)pos * half + c);
+            const bf16* src = p.q_up + (size_t)t * p.q_up_ld + p.rot_off + (size_t)(head0 + h) * p.rot + c;
+            const float u = h < nheads ? act_load(src) : 0.f, v = h < nheads ? act_load(src + half) : 0.f;
+            put(r, c, u * f.x - v * f.y);
+            put(r, half + c, v * f.x + u * f.y);
+        }
+        for (int i = tid; i < rows * (zero_to - p.rot); i += kRowsMax) put(i / (zero_to - p.rot), p.rot + i % (zero_to - p.rot), 0.f);
     }
-    auto put = [&](int r, int col, float x) { *(bf16*)(at(r, col & ~7) + (col & 7) * 2) = __float2bfloat16_rn(x); };
-    for (int i = tid; i < rows * half; i += kRowsMax) {
-        const int r = i / half, c = i % half, h = r % p.part_heads, t = t0 + r / p.part_heads;
-        const int pos = min(max(__ldcg(p.tok_pos + t), 0), p.max_pos - 1);
-        const float2 cs = __ldg(p.rope + (size_t)pos * half + c);
-        const bf16* src = p.q_up + (size_t)t * p.q_up_ld + p.rot_off + (size_t)(head0 + h) * p.rot + c;
-        const float u = h < nheads ? act_load(src) : 0.f, v = h < nheads ? act_load(src + half) : 0.f;
-        put(r, c, u * cs.x - v * cs.y);
-        put(r, half + c, v * cs.x + u * cs.y);
-    }
-    for (int i = tid; i < rows * (zero_to - p.rot); i += kRowsMax) put(i / (zero_to - p.rot), p.rot + i % (zero_to - p.rot), 0.f);
-}
+};
 
 __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_constant__ LatentDev p) {
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
-    __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[2], q_full, p_full, pv_done;
+    __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[2], p_full[2], q_full, pv_done;
     __shared__ uint32_t tmem_slot;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;
 
     // unit = ((group * subs + sub) * parts + part) * slices + slice
     const int unit = blockIdx.x, slice = unit % p.slices, part = unit / p.slices % p.parts;
@@ -208,7 +253,8 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_consta
         mbar_init(&s_full[0], 1);
         mbar_init(&s_full[1], 1);
         mbar_init(&q_full, 1 + kRowsMax);
-        mbar_init(&p_full, kRowsMax);
+        mbar_init(&p_full[0], kRowsMax);
+        mbar_init(&p_full[1], kRowsMax);
         mbar_init(&pv_done, 1);
         fence_mbar_init();
     }
@@ -234,55 +280,71 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_consta
         if (lane == 0) {
             prefetch_tmap(&p.tmQ);
             prefetch_tmap(&p.tmK);
-            pdl_wait();
-            tl_mark(p.tl, 1);
-            if (tiles > 0) mbar_arrive_expect_tx(&q_full, rank_blocks * q_block);  // no copy that nobody waits for
-            for (int b = 0; b < rank_blocks && tiles > 0; ++b) tma_load_2d(q_s + b * q_block, &p.tmQ, b * 64, t0 * p.heads + head0, &q_full);
-            for (int next = 0; next < tiles; ++next) {
-                if (next >= p.stages && !mbar_wait(&k_empty[next % p.stages], (uint32_t)(next / p.stages - 1) & 1u, p.status, DEV_ERR_EMPTY_WAIT)) break;
-                load_tile(p, seq, len, next, blocks, stage_bytes, k_s, k_full);
+        }
+        __syncwarp();
+        pdl_wait();
+        if (lane == 0) tl_mark(p.tl, 1);
+        if (tiles > 0) {  // no copy that nobody waits for
+            PageLoader<TK> pages(p, seq, len, 0, blocks, k_s, k_full, lane);
+            mbar_arrive_expect_tx_elect(smem_u32(&q_full), rank_blocks * q_block);
+            for (int b = 0; b < rank_blocks; ++b) tma_load_2d_elect(smem_u32(q_s + b * q_block), &p.tmQ, b * 64, t0 * p.heads + head0, smem_u32(&q_full));
+            bool ok = true;
+            for (int j = 0; j < tiles && ok; ++j) {
+                if (j >= p.stages) ok = __all_sync(0xffffffffu, mbar_wait(&k_empty[j % p.stages], (uint32_t)(j / p.stages - 1) & 1u, p.status, DEV_ERR_EMPTY_WAIT));
+                if (ok) pages.load(j);
             }
         }
     } else if (warp == 5) {
-        if (lane == 0 && tiles > 0) {
+        if (tiles > 0) {
             constexpr uint32_t idesc_s = umma_idesc_bf16(kRowsMax, TK);
-            const int ncols = min(p.slice_cols, (p.rank - slice * p.slice_cols + 15) / 16 * 16);
-            const uint32_t idesc_o = umma_idesc_bf16(kRowsMax, ncols) | (1u << 16);  // B is N-major
             const uint32_t q_a = smem_u32(q_s), k_a = smem_u32(k_s);
-            const int rank_steps = (p.rank + 15) / 16, rot_steps = (p.rot + 15) / 16;
-            auto scores = [&](int j) {
-                const int st = j % p.stages;
-                if (!mbar_wait(&k_full[st], (uint32_t)(j / p.stages) & 1u, p.status, DEV_ERR_FULL_WAIT)) return false;
-                tc_fence_after();
-                const uint32_t kb = k_a + st * stage_bytes, d = tmem + kColS + (j & 1) * TK;
-                for (int i = 0; i < rank_steps + rot_steps; ++i) {
-                    const int i2 = i < rank_steps ? i : rank_blocks * 4 + (i - rank_steps);
-                    const uint32_t in = (uint32_t)(i2 & 3) * 32;
-                    umma_bf16(d, umma_desc_k128(q_a + (i2 >> 2) * q_block + in), umma_desc_k128(kb + (i2 >> 2) * kBlockBytes + in), idesc_s, i > 0);
-                }
-                umma_commit(&s_full[j & 1]);
-                return true;
-            };
-            const bool ahead = p.stages > 1;  // the scores of the next tile run while this tile's softmax does
-            bool ok = mbar_wait(&q_full, 0, p.status, DEV_ERR_FULL_WAIT) && scores(0);
+            const int last_steps = ((p.rot - 1) % 64 + 16) / 16;
+            bool ok = mma_wait(&q_full, 0, p.status, DEV_ERR_FULL_WAIT);
             for (int j = 0; j < tiles && ok; ++j) {
-                if (ahead && j + 1 < tiles) ok = scores(j + 1);
-                if (!ok || !mbar_wait(&p_full, (uint32_t)j & 1u, p.status, DEV_ERR_ACC_WAIT)) break;
+                const int st = j % p.stages;
+                // the softmax has read S of tile j - 2 (it says so with its P)
+                if (j > 1) ok = mma_wait(&p_full[j & 1], (uint32_t)((j - 2) >> 1) & 1u, p.status, DEV_ERR_ACC_WAIT);
+                ok = ok && mma_wait(&k_full[st], (uint32_t)(j / p.stages) & 1u, p.status, DEV_ERR_FULL_WAIT);
+                if (!ok) break;
                 tc_fence_after();
-                const uint32_t v = k_a + (j % p.stages) * stage_bytes + slice * (p.slice_cols / 64) * kBlockBytes;
+                const uint32_t d = tmem + kColS + (j & 1) * TK;
+                // descriptors advance by constants: address / 16
+                uint64_t qd = umma_desc_k128(q_a), kd = umma_desc_k128(k_a + st * stage_bytes);
 #pragma unroll
-                for (int half = 0; half < 2; ++half)  // P hi, P lo
+                for (int i = 0; i < 4; ++i) umma_bf16_elect(d, qd + 2 * i, kd + 2 * i, idesc_s, i > 0);  // the latent has a block at least
+#pragma unroll 2
+                for (int blk = 2; blk < blocks; ++blk) {
+                    qd += q_block >> 4;
+                    kd += kBlockBytes >> 4;
 #pragma unroll
-                    for (int kk = 0; kk < TK / 16; ++kk)
-                        umma_bf16_ts(tmem + kColO, tmem + kColP + half * (TK / 2) + kk * 8, desc_n128(v + kk * 2048), idesc_o, j > 0 || half > 0 || kk > 0);
-                umma_commit(&k_empty[j % p.stages]);
-                umma_commit(&pv_done);
-                if (!ahead && j + 1 < tiles) ok = scores(j + 1);
+                    for (int i = 0; i < 4; ++i) umma_bf16_elect(d, qd + 2 * i, kd + 2 * i, idesc_s, 1);
+                }
+                qd += q_block >> 4;
+                kd += kBlockBytes >> 4;
+                for (int i = 0; i < last_steps; ++i) umma_bf16_elect(d, qd + 2 * i, kd + 2 * i, idesc_s, 1);  // Q is not defined past these steps
+                umma_commit_elect(&s_full[j & 1]);
             }
         }
+    } else if (warp == 6) {
+        const int ncols = min(p.slice_cols, (p.rank - slice * p.slice_cols + 15) / 16 * 16);
+        const uint32_t idesc_o = umma_idesc_bf16(kRowsMax, ncols) | (1u << 16);  // B has its K extent in rows
+        const uint32_t v_a = smem_u32(k_s) + slice * (p.slice_cols / 64) * kBlockBytes;
+        for (int j = 0; j < tiles; ++j) {
+            if (!mma_wait(&p_full[j & 1], (uint32_t)(j >> 1) & 1u, p.status, DEV_ERR_ACC_WAIT)) break;
+            tc_fence_after();
+            const uint64_t vd = desc_n128(v_a + (j % p.stages) * stage_bytes, kBlockBytes);
+#pragma unroll
+            for (int half = 0; half < 2; ++half)  // P hi, P lo
+#pragma unroll
+                for (int kk = 0; kk < TK / 16; ++kk)
+                    umma_bf16_ts(tmem + kColO, tmem + kColP + half * (TK / 2) + kk * 8, vd + kk * 128, idesc_o, j > 0 || half > 0 || kk > 0);
+            umma_commit_elect(&k_empty[j % p.stages]);
+            umma_commit_elect(&pv_done);
+        }
     } else {
+        QueryRotation rotation(p, t0, head0, nheads, max(ntok, 0) * p.part_heads, q_s + rank_blocks * q_block, q_block);
         pdl_wait();
-        rotate_q(p, t0, head0, nheads, ntok * p.part_heads, q_s + rank_blocks * q_block, q_block);
+        rotation.store();
         fence_proxy_async_smem();
         mbar_arrive(&q_full);
         const int my_end = active ? __ldcg(p.tok_pos + row_t) + 1 : 0;
@@ -349,7 +411,7 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_consta
             }
             tc_wait_st();
             tc_fence_before();
-            mbar_arrive(&p_full);
+            mbar_arrive(&p_full[j & 1]);
         }
         if (tiles > 0 && ok) ok = __all_sync(0xffffffffu, mbar_wait(&pv_done, (uint32_t)(tiles - 1) & 1u, p.status, DEV_ERR_ACC_WAIT));
         tc_fence_after();
@@ -385,7 +447,6 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_consta
 
 // ---------------------------------------------------------------------------------------------- decoding
 constexpr int kDecSoftmax = 128;           // threads of the softmax warps
-constexpr int kDecP = TK * 128;            // one P^T buffer: 64 keys x (hi | lo) heads, rows of 128 bytes
 constexpr int kDecMaxSplits = 64;
 __host__ __device__ inline int partial_ld(int rank) { return (rank + 3) / 4 * 4 + 4; }  // floats of a split's partial row
 __device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
@@ -402,8 +463,9 @@ __device__ __forceinline__ bool softmax_any(bool x) {
     return r != 0;
 }
 
-// HP: heads of a tile (16 or 32)
-template <int HP>
+// HP: heads of a tile (16 or 32). KEYS: keys of a tile, 64, or 32 (one page; half of the rows of S^T are not used) where rows
+// are so wide that the ring would hold too few tiles of 64.
+template <int HP, int KEYS>
 __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid_constant__ LatentDev p, uint32_t tmem_cols) {
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -411,24 +473,24 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
     __shared__ uint32_t tmem_slot;
     __shared__ int s_last;
     __shared__ float s_max[4][HP], s_sum[4][HP], s_mult[HP];
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;
 
     const int unit = blockIdx.x, t = unit / p.parts, part = unit % p.parts;
     const int head0 = part * p.part_heads, nheads = min(p.part_heads, p.heads - head0);
     const int seq = __ldcg(p.tok_seq + t), len = __ldcg(p.tok_pos + t) + 1;
     int per_split = (len + p.splits - 1) / p.splits;
-    per_split = (per_split + TK - 1) / TK * TK;
+    per_split = (per_split + KEYS - 1) / KEYS * KEYS;
     const int k_begin = blockIdx.y * per_split, k_end = min(len, k_begin + per_split);
     const bool len_ok = len <= p.max_pos && (len + kPageTokens - 1) / kPageTokens <= p.max_pages_per_seq;
-    const int tiles = len_ok && k_end > k_begin ? (k_end - k_begin + TK - 1) / TK : 0;
+    const int tiles = len_ok && k_end > k_begin ? (k_end - k_begin + KEYS - 1) / KEYS : 0;
 
     const int rank_blocks = (p.rank + 63) / 64, rot_blocks = (p.rot + 63) / 64, blocks = rank_blocks + rot_blocks;
     const int mblocks = (p.rank + 127) / 128;
-    constexpr int q_block = HP * 128;
-    const int stage_bytes = blocks * kBlockBytes;
+    constexpr int q_block = HP * 128, k_block = KEYS * 128, p_buf = KEYS * 128;  // a P^T buffer: rows of 128 bytes, (hi | lo) heads of a key
+    const int stage_bytes = blocks * k_block;
     uint8_t* const q_s = smem;
     uint8_t* const p_s = smem + blocks * q_block;
-    uint8_t* const k_s = p_s + 2 * kDecP;
+    uint8_t* const k_s = p_s + 2 * p_buf;
     constexpr uint32_t colO = 2 * HP;
 
     if (tid == 0) {
@@ -460,62 +522,82 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
         if (lane == 0) {
             prefetch_tmap(&p.tmQ);
             prefetch_tmap(&p.tmK);
-            // everything but the newest row is older than the step's first kernel
-            const int first_tile = k_begin / TK, old_keys = (len - 1) / kPageTokens * kPageTokens;
-            int next = 0;
-            if (p.early)
-                while (next < min(p.stages, tiles) && k_begin + (next + 1) * TK <= old_keys) {
-                    load_tile(p, seq, len, first_tile + next, blocks, stage_bytes, k_s, k_full, first_tile);
-                    ++next;
-                }
-            pdl_wait();
-            tl_mark(p.tl, 1);
-            if (tiles > 0) mbar_arrive_expect_tx(&q_full, rank_blocks * q_block);  // no copy that nobody waits for
-            for (int b = 0; b < rank_blocks && tiles > 0; ++b) tma_load_2d(q_s + b * q_block, &p.tmQ, b * 64, t * p.heads + head0, &q_full);
-            for (; next < tiles; ++next) {
-                if (next >= p.stages && !mbar_wait(&k_empty[next % p.stages], (uint32_t)(next / p.stages - 1) & 1u, p.status, DEV_ERR_EMPTY_WAIT)) break;
-                load_tile(p, seq, len, first_tile + next, blocks, stage_bytes, k_s, k_full, first_tile);
-            }
+        }
+        __syncwarp();
+        PageLoader<KEYS> pages(p, seq, max(len, 1), k_begin, blocks, k_s, k_full, lane);
+        // everything but the newest row is older than the step's first kernel
+        const int old_keys = (len - 1) / kPageTokens * kPageTokens;
+        int next = 0;
+        if (p.early)
+            for (; next < min(p.stages, tiles) && k_begin + (next + 1) * KEYS <= old_keys; ++next) pages.load(next);
+        pdl_wait();
+        if (lane == 0) tl_mark(p.tl, 1);
+        if (tiles > 0) {  // no copy that nobody waits for
+            mbar_arrive_expect_tx_elect(smem_u32(&q_full), rank_blocks * q_block);
+            for (int b = 0; b < rank_blocks; ++b) tma_load_2d_elect(smem_u32(q_s + b * q_block), &p.tmQ, b * 64, t * p.heads + head0, smem_u32(&q_full));
+        }
+        bool ok = true;
+        for (; next < tiles && ok; ++next) {
+            if (next >= p.stages) ok = __all_sync(0xffffffffu, mbar_wait(&k_empty[next % p.stages], (uint32_t)(next / p.stages - 1) & 1u, p.status, DEV_ERR_EMPTY_WAIT));
+            if (ok) pages.load(next);
         }
     } else if (warp == 5) {
-        if (lane == 0 && tiles > 0) {
-            constexpr uint32_t idesc_s = umma_idesc_bf16(TK, HP);
-            constexpr uint32_t idesc_o = umma_idesc_bf16(128, 2 * HP) | (1u << 15) | (1u << 16);  // A and B with their K extent in rows
-            const uint32_t q_a = smem_u32(q_s), k_a = smem_u32(k_s), p_a = smem_u32(p_s);
-            const int rank_steps = (p.rank + 15) / 16, rot_steps = (p.rot + 15) / 16;
-            auto scores = [&](int j) {
-                const int st = j % p.stages;
-                if (!mbar_wait(&k_full[st], (uint32_t)(j / p.stages) & 1u, p.status, DEV_ERR_FULL_WAIT)) return false;
-                tc_fence_after();
-                const uint32_t kb = k_a + st * stage_bytes, d = tmem + (j & 1) * HP;
-                for (int i = 0; i < rank_steps + rot_steps; ++i) {
-                    const int i2 = i < rank_steps ? i : rank_blocks * 4 + (i - rank_steps);
-                    const uint32_t in = (uint32_t)(i2 & 3) * 32;
-                    umma_bf16(d, umma_desc_k128(kb + (i2 >> 2) * kBlockBytes + in), umma_desc_k128(q_a + (i2 >> 2) * q_block + in), idesc_s, i > 0);
-                }
-                umma_commit(&s_full[j & 1]);
-                return true;
-            };
-            const bool ahead = p.stages > 1;  // the scores of the next tile run while this tile's softmax does
-            bool ok = mbar_wait(&q_full, 0, p.status, DEV_ERR_FULL_WAIT) && scores(0);
+        if (tiles > 0) {
+            constexpr uint32_t idesc_s = umma_idesc_bf16(64, HP);
+            const uint32_t q_a = smem_u32(q_s), k_a = smem_u32(k_s);
+            const int last_steps = ((p.rot - 1) % 64 + 16) / 16;
+            bool ok = mma_wait(&q_full, 0, p.status, DEV_ERR_FULL_WAIT);
             for (int j = 0; j < tiles && ok; ++j) {
-                if (ahead && j + 1 < tiles) ok = scores(j + 1);
-                if (!ok || !mbar_wait(&p_full[j & 1], (uint32_t)(j >> 1) & 1u, p.status, DEV_ERR_ACC_WAIT)) break;
+                const int st = j % p.stages;
+                // the softmax has read S of tile j - 2 (it says so with its P)
+                if (j > 1) ok = mma_wait(&p_full[j & 1], (uint32_t)((j - 2) >> 1) & 1u, p.status, DEV_ERR_ACC_WAIT);
+                ok = ok && mma_wait(&k_full[st], (uint32_t)(j / p.stages) & 1u, p.status, DEV_ERR_FULL_WAIT);
+                if (!ok) break;
                 tc_fence_after();
-                const uint32_t v = k_a + (j % p.stages) * stage_bytes, pb = p_a + (j & 1) * kDecP;
-                for (int mb = 0; mb < mblocks; ++mb)
+                const uint32_t d = tmem + (j & 1) * HP;
+                // descriptors advance by constants: address / 16
+                uint64_t qd = umma_desc_k128(q_a), kd = umma_desc_k128(k_a + st * stage_bytes);
 #pragma unroll
-                    for (int kk = 0; kk < TK / 16; ++kk)
-                        umma_bf16(tmem + colO + mb * 2 * HP, desc_n128(v + mb * 2 * kBlockBytes + kk * 2048), desc_n128(pb + kk * 2048), idesc_o,
-                                  j > 0 || kk > 0);
-                umma_commit(&k_empty[j % p.stages]);
-                umma_commit(&pv_done[j & 1]);
-                if (!ahead && j + 1 < tiles) ok = scores(j + 1);
+                for (int i = 0; i < 4; ++i) umma_bf16_elect(d, kd + 2 * i, qd + 2 * i, idesc_s, i > 0);  // the latent has a block at least
+#pragma unroll 2
+                for (int blk = 2; blk < blocks; ++blk) {
+                    qd += q_block >> 4;
+                    kd += k_block >> 4;
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) umma_bf16_elect(d, kd + 2 * i, qd + 2 * i, idesc_s, 1);
+                }
+                qd += q_block >> 4;
+                kd += k_block >> 4;
+                for (int i = 0; i < last_steps; ++i) umma_bf16_elect(d, kd + 2 * i, qd + 2 * i, idesc_s, 1);  // Q is not defined past these steps
+                umma_commit_elect(&s_full[j & 1]);
             }
         }
+    } else if (warp == 6) {
+        constexpr uint32_t idesc_o = umma_idesc_bf16(128, 2 * HP) | (1u << 15) | (1u << 16);  // A and B with their K extent in rows
+        const uint32_t k_a = smem_u32(k_s), p_a = smem_u32(p_s);
+        for (int j = 0; j < tiles; ++j) {
+            if (!mma_wait(&p_full[j & 1], (uint32_t)(j >> 1) & 1u, p.status, DEV_ERR_ACC_WAIT)) break;
+            tc_fence_after();
+            uint64_t vd = desc_n128(k_a + (j % p.stages) * stage_bytes, k_block);
+            const uint64_t pd = desc_n128(p_a + (j & 1) * p_buf, p_buf);
+            const uint32_t again = j > 0;
+            uint32_t d = tmem + colO;
+#pragma unroll 2
+            for (int mb = 0; mb < mblocks; ++mb) {
+                umma_bf16_elect(d, vd, pd, idesc_o, again);
+#pragma unroll
+                for (int kk = 1; kk < KEYS / 16; ++kk) umma_bf16_elect(d, vd + kk * 128, pd + kk * 128, idesc_o, 1);
+                vd += 2 * k_block >> 4;
+                d += 2 * HP;
+            }
+            umma_commit_elect(&k_empty[j % p.stages]);
+            umma_commit_elect(&pv_done[j & 1]);
+        }
     } else {
+        QueryRotation rotation(p, t, head0, nheads, p.part_heads, q_s + rank_blocks * q_block, q_block);
         pdl_wait();
-        rotate_q(p, t, head0, nheads, p.part_heads, q_s + rank_blocks * q_block, q_block);
+        const float gate = tid < nheads ? act_load(p.gate + (size_t)t * p.gate_ld + head0 + tid) : 0.f;
+        rotation.store();
         for (int i = tid; i < (HP - p.part_heads) * rot_blocks * 8; i += kDecSoftmax)  // rows without a head
             *(uint4*)(q_s + (rank_blocks + i / 8 % rot_blocks) * q_block + (p.part_heads + i / 8 / rot_blocks) * 128 + i % 8 * 16) = make_uint4(0u, 0u, 0u, 0u);
         fence_proxy_async_smem();
@@ -545,14 +627,23 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
 #pragma unroll
                 for (int i = 0; i < 16; ++i) s[c * 16 + i] = __uint_as_float(v[i]) * p.scale_log2;
             }
-            const bool live = lane < 16 && k_begin + j * TK + row < k_end;
-            bool up = j == 0;
+            const bool live = lane < 16 && row < KEYS && k_begin + j * KEYS + row < k_end;
+            if (j == 0) {  // the first key's scores are the first reference
+                if (tid == 0) {
+#pragma unroll
+                    for (int h = 0; h < HP; ++h) s_max[0][h] = s[h];
+                }
+                softmax_sync();
+#pragma unroll
+                for (int h = 0; h < HP; ++h) m_ref[h] = s_max[0][h];
+            }
+            bool up = false;
 #pragma unroll
             for (int h = 0; h < HP; ++h) {
                 if (!live) s[h] = kNeg;
                 up = up || (h < nheads && s[h] > m_ref[h] + 8.f);
             }
-            if (softmax_any(up)) {  // the reference maxima move to the running maxima
+            if (softmax_any(up)) {  // rare: the reference maxima move to the running maxima
 #pragma unroll
                 for (int h = 0; h < HP; ++h) {
                     float m = s[h];
@@ -601,8 +692,8 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
                 lo[h / 2] = *(const uint32_t*)&l2;
             }
             if (j > 1) wait(&pv_done[j & 1], (uint32_t)((j - 2) >> 1) & 1u);  // the buffer's last product is done
-            if (lane < 16) {
-                uint8_t* dst = p_s + (j & 1) * kDecP + row * 128;
+            if (lane < 16 && row < KEYS) {
+                uint8_t* dst = p_s + (j & 1) * p_buf + row * 128;
 #pragma unroll
                 for (int c = 0; c < HP / 8; ++c) {
                     *(uint4*)(dst + ((c ^ (row & 7)) << 4)) = make_uint4(hi[4 * c], hi[4 * c + 1], hi[4 * c + 2], hi[4 * c + 3]);
@@ -615,47 +706,58 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
         }
         if (tiles > 0) wait(&pv_done[(tiles - 1) & 1], (uint32_t)((tiles - 1) >> 1) & 1u);
         tc_fence_after();
-        // ---- sums over the keys, then this thread's value columns (lane = column of a group of 128)
+        // ---- sums over the keys
 #pragma unroll
         for (int h = 0; h < HP; ++h) {
-            const float l = warp_sum(l_sum[h]);
+            float l = l_sum[h];
+#pragma unroll
+            for (int o = 8; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);  // lanes 16 and on hold nothing
             if (lane == 0) s_sum[warp][h] = l;
         }
         softmax_sync();
-        const size_t row_ld = partial_ld(p.rank), ml_at = row_ld - 4;  // partial rows: [unit][split][part_heads][row_ld], at its end: maximum, sum
+        const int row_ld = partial_ld(p.rank);  // partial rows: [unit][split][part_heads][row_ld], at their end: maximum, sum
         float* parts = p.ws + ((size_t)unit * p.splits + blockIdx.y) * p.part_heads * row_ld;
         if (tid < nheads) {
             const float l = s_sum[0][tid] + s_sum[1][tid] + s_sum[2][tid] + s_sum[3][tid];
-            if (p.splits == 1) {
-                s_mult[tid] = sigmoid_f32(act_load(p.gate + (size_t)t * p.gate_ld + head0 + tid)) / l;
-            } else {
+            s_mult[tid] = p.splits == 1 ? sigmoid_f32(gate) / l : 1.f;
+            if (p.splits > 1) {
                 float m = kNeg;
 #pragma unroll
                 for (int h = 0; h < HP; ++h) m = h == tid ? m_ref[h] : m;
-                parts[tid * row_ld + ml_at] = m;
-                parts[tid * row_ld + ml_at + 1] = l;
+                parts[tid * row_ld + row_ld - 4] = m;
+                parts[tid * row_ld + row_ld - 3] = l;
             }
         }
         softmax_sync();
+        // ---- O^T (lane = column of a group of 128) through the idle ring, rows of ld_s floats, then row by row
         if (tiles > 0) {
+            const int ld_s = (p.rank + 127) / 128 * 128 + 4;
+            float* const o_s = (float*)k_s;
             for (int mb = 0; mb < mblocks; ++mb) {
-                const int col = mb * 128 + warp * 32 + lane;
 #pragma unroll
-                for (int q = 0; q < HP / 16; ++q) {
+                for (int g = 0; g < HP / 16; ++g) {
                     uint32_t a[16], b[16];
-                    tmem_ld16(lane_addr + colO + mb * 2 * HP + q * 16, a);
-                    tmem_ld16(lane_addr + colO + mb * 2 * HP + HP + q * 16, b);
+                    tmem_ld16(lane_addr + colO + mb * 2 * HP + g * 16, a);
+                    tmem_ld16(lane_addr + colO + mb * 2 * HP + HP + g * 16, b);
                     tc_wait_ld();
 #pragma unroll
-                    for (int i = 0; i < 16; ++i) {
-                        const int h = q * 16 + i;
-                        const float o = __uint_as_float(a[i]) + __uint_as_float(b[i]);  // P_hi V + P_lo V
-                        if (col < p.rank && h < nheads) {
-                            if (p.splits == 1) p.out[((size_t)t * p.heads + head0 + h) * p.head_ld + col] = __float2bfloat16_rn(o * s_mult[h]);
-                            else parts[h * row_ld + col] = o;
-                        }
-                    }
-                    __syncwarp();
+                    for (int i = 0; i < 16; ++i)  // P_hi V + P_lo V
+                        o_s[(g * 16 + i) * ld_s + mb * 128 + warp * 32 + lane] = __uint_as_float(a[i]) + __uint_as_float(b[i]);
+                }
+            }
+            softmax_sync();
+            const int per_head = (p.rank + 3) / 4;
+            for (int h = warp; h < nheads; h += 4) {
+                const float mult = s_mult[h];
+                const float4* src = (const float4*)(o_s + h * ld_s);
+                bf16* dst = p.out + ((size_t)t * p.heads + head0 + h) * p.head_ld;
+#pragma unroll 4
+                for (int c = lane; c < per_head; c += 32) {
+                    const float4 o = src[c];
+                    if (p.splits == 1)  // columns of the padding are zero in the cache, so they are here
+                        *(uint2*)(dst + c * 4) = make_uint2((uint32_t)bf16_bits(o.x * mult) | ((uint32_t)bf16_bits(o.y * mult) << 16),
+                                                            (uint32_t)bf16_bits(o.z * mult) | ((uint32_t)bf16_bits(o.w * mult) << 16));
+                    else *(float4*)(parts + (size_t)h * row_ld + c * 4) = o;
                 }
             }
         }
@@ -678,7 +780,7 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
             const size_t row_ld = partial_ld(p.rank), step = p.part_heads * row_ld;
             const float* parts = p.ws + (size_t)unit * p.splits * step;
             float* wgt = (float*)p_s;  // [HP][splits]
-            static_assert(HP * kDecMaxSplits * 4 <= 2 * kDecP, "");
+            static_assert(HP * kDecMaxSplits * 4 <= 2 * p_buf, "");
             for (int h = warp; h < nheads; h += kThreads / 32) {
                 const float* ml = parts + h * row_ld + row_ld - 4;
                 float m[2], l[2], M = kNeg, L = 0.f;
@@ -746,7 +848,7 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
 
 // how a launch is cut into tiles; stages == 0: does not fit
 struct LatentPlan {
-    int part_heads, parts, tile_tokens, q_rows, slices, slice_cols, stages, smem, tmem_cols;
+    int part_heads, parts, tile_tokens, q_rows, slices, slice_cols, stages, smem, tmem_cols, keys;
 };
 constexpr int kStaticSmem = 2048;  // room for the kernels' static shared memory
 
@@ -756,6 +858,7 @@ LatentPlan plan_prompt(int rank, int rot, int heads) {
     l.parts = (heads + kRowsMax - 1) / kRowsMax;
     l.part_heads = (heads + l.parts - 1) / l.parts;
     l.tile_tokens = std::max(1, std::min(8, kRowsMax / l.part_heads));
+    l.keys = TK;
     l.slices = (rank + kSliceCols - 1) / kSliceCols;
     l.slice_cols = ((rank + l.slices - 1) / l.slices + 63) / 64 * 64;
     l.slices = (rank + l.slice_cols - 1) / l.slice_cols;
@@ -780,12 +883,18 @@ LatentPlan plan_decode(int rank, int rot, int heads) {
         l.parts = (heads + hp - 1) / hp;
         l.part_heads = (heads + l.parts - 1) / l.parts;
         l.q_rows = hp;
-        const int cols = 2 * hp + mblocks * 2 * hp, fixed = 1024 + blocks * hp * 128 + 2 * kDecP;
+        const int cols = 2 * hp + mblocks * 2 * hp;
         l.tmem_cols = 32;
         while (l.tmem_cols < cols) l.tmem_cols *= 2;
-        l.stages = std::min(kMaxStages, (kSmemLimit - kStaticSmem - fixed) / (blocks * kBlockBytes));
-        l.smem = fixed + l.stages * blocks * kBlockBytes;
-        if (l.stages >= 1 && l.tmem_cols <= 512) return l;
+        if (l.tmem_cols > 512) continue;
+        for (l.keys = TK; l.keys >= kPageTokens; l.keys /= 2) {
+            // S^T always has 64 rows: with 32 keys its operand reaches a block past its own
+            const int stage = blocks * l.keys * 128, fixed = 1024 + blocks * hp * 128 + 2 * l.keys * 128 + (TK - l.keys) * 128;
+            l.stages = std::min(kMaxStages, (kSmemLimit - kStaticSmem - fixed) / stage);
+            const int out = hp * ((rank + 127) / 128 * 128 + 4) * 4;  // O^T passes through the ring
+            l.smem = fixed + std::max(l.stages * stage, out);
+            if (l.stages >= (l.keys == TK ? 2 : 1) && l.smem <= kSmemLimit - kStaticSmem) return l;
+        }
     }
     l.stages = 0;
     return l;
@@ -856,8 +965,9 @@ int launch_attention_latent(const LatentAttn& a, int T, int n_groups, int max_ct
     p.splits = attention_latent_splits(T, a.rank, a.rot, a.heads, max_ctx, ws, num_sms);
     p.early = pdl && a.only_newest_row_fresh;
     const dim3 grid(T * l.parts, p.splits);
-    if (l.q_rows == 16) return (int)launch_k(k_attn_latent_decode<16>, grid, dim3(kThreads), (size_t)l.smem, s, pdl, p, (uint32_t)l.tmem_cols);
-    return (int)launch_k(k_attn_latent_decode<32>, grid, dim3(kThreads), (size_t)l.smem, s, pdl, p, (uint32_t)l.tmem_cols);
+    const auto kernel = l.q_rows == 16 ? (l.keys == TK ? k_attn_latent_decode<16, TK> : k_attn_latent_decode<16, kPageTokens>)
+                                       : (l.keys == TK ? k_attn_latent_decode<32, TK> : k_attn_latent_decode<32, kPageTokens>);
+    return (int)launch_k(kernel, grid, dim3(kThreads), (size_t)l.smem, s, pdl, p, (uint32_t)l.tmem_cols);
 }
 
 template <typename Kern>
@@ -867,8 +977,10 @@ static cudaError_t latent_attr(Kern k) {
 }
 int attention_latent_prepare() {
     cudaError_t e = latent_attr(k_attn_latent);
-    if (e == cudaSuccess) e = latent_attr(k_attn_latent_decode<16>);
-    if (e == cudaSuccess) e = latent_attr(k_attn_latent_decode<32>);
+    if (e == cudaSuccess) e = latent_attr(k_attn_latent_decode<16, TK>);
+    if (e == cudaSuccess) e = latent_attr(k_attn_latent_decode<16, kPageTokens>);
+    if (e == cudaSuccess) e = latent_attr(k_attn_latent_decode<32, TK>);
+    if (e == cudaSuccess) e = latent_attr(k_attn_latent_decode<32, kPageTokens>);
     return (int)e;
 }
 

@@ -15,8 +15,9 @@
 // Decoding (k_attn_latent_decode): one token's heads would leave most of those rows empty, so keys and value columns take
 // the long side instead, S^T[key, head] = K . Q^T and O^T[column, head] += K^T . P^T: all value columns in one CTA. P^T is
 // written to shared memory next to its lo part (twice the columns of one product). One CTA = 16 or 32 heads of a token x
-// one context split, the same seven warps (thread = key). Splits leave partial rows and the last one to finish (a ticket, no
-// waiting) adds them up in split order.
+// one context split, the same seven warps (thread = key). Up to eight splits are a thread-block cluster and add up their rows through
+// distributed shared memory; more leave partial rows and the last one to finish (a ticket, no waiting) adds them up. Both in
+// split order.
 //
 // Rows of a page past the end of a sequence are finite (zeros or an earlier request's normed latents) and weigh zero.
 #include "act.cuh"
@@ -56,7 +57,7 @@ struct LatentDev {
     int q_rows;                        // rows of the Q box
     int rank, slices, slice_cols;
     int stages;
-    int splits, early;                 // decoding only
+    int splits, cluster, early;        // decoding only; cluster: the splits are one thread-block cluster
     float scale_log2;
     const bf16* gate;                  // [T][gate_ld]
     long long gate_ld;
@@ -140,8 +141,9 @@ struct PageLoader {
 // The rotated parts of Q, rows 0 .. rows - 1 of the tile (row = token * part_heads + head), into the blocks behind the latent
 // ones; columns past `rot` are zero, and so are rows of heads that do not exist. The 128 softmax threads call it. Angles are
 // older than the previous kernel (they are read by the constructor), the parts themselves are not.
+// B: pieces of 8 pairs with their loads in flight together
+template <int B>
 struct QueryRotation {
-    static constexpr int B = 4;  // pieces of 8 pairs with their loads in flight together
     const LatentDev& p;
     int t0, head0, nheads, rows, half, q_block;
     uint8_t* q_rot;
@@ -342,7 +344,7 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_consta
             umma_commit_elect(&pv_done);
         }
     } else {
-        QueryRotation rotation(p, t0, head0, nheads, max(ntok, 0) * p.part_heads, q_s + rank_blocks * q_block, q_block);
+        QueryRotation<4> rotation(p, t0, head0, nheads, max(ntok, 0) * p.part_heads, q_s + rank_blocks * q_block, q_block);
         pdl_wait();
         rotation.store();
         fence_proxy_async_smem();
@@ -447,7 +449,7 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent(const __grid_consta
 
 // ---------------------------------------------------------------------------------------------- decoding
 constexpr int kDecSoftmax = 128;           // threads of the softmax warps
-constexpr int kDecMaxSplits = 64;
+constexpr int kDecMaxSplits = 64, kClusterSplits = 8;
 __host__ __device__ inline int partial_ld(int rank) { return (rank + 3) / 4 * 4 + 4; }  // floats of a split's partial row
 __device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 __device__ __forceinline__ bool softmax_any(bool x) {
@@ -472,7 +474,8 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
     __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[2], p_full[2], pv_done[2], q_full;
     __shared__ uint32_t tmem_slot;
     __shared__ int s_last;
-    __shared__ float s_max[4][HP], s_sum[4][HP], s_mult[HP];
+    __shared__ float s_max[4][HP], s_sum[4][HP], s_mult[HP], s_rehearsal[128];
+    __shared__ float2 s_ml[HP];  // cluster: this split's maximum and sum per head
     const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;
 
     const int unit = blockIdx.x, t = unit / p.parts, part = unit % p.parts;
@@ -492,6 +495,7 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
     uint8_t* const p_s = smem + blocks * q_block;
     uint8_t* const k_s = p_s + 2 * p_buf;
     constexpr uint32_t colO = 2 * HP;
+    const int o_ld = (p.rank + 127) / 128 * 128 + 4;  // floats of a row of O on its way out
 
     if (tid == 0) {
         tl_mark(p.tl, 0);
@@ -517,6 +521,11 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
     const uint32_t tmem = tmem_slot;
     pdl_launch_dependents();
     if (!len_ok && tid == 0) dev_fail(p.status, DEV_ERR_BOUNDS);
+    // Everything but the newest row is older than the step's first kernel, so the first tiles are requested before the
+    // wait for the previous kernel. With the first one there, the time until then goes into a rehearsal: one tile whose
+    // keys all weigh zero passes through every warp, so that their instructions are at hand when the queries arrive.
+    const int old_keys = (len - 1) / kPageTokens * kPageTokens;
+    const int warm = p.early && tiles > 0 && k_begin + KEYS <= old_keys ? 1 : 0;
 
     if (warp == 4) {
         if (lane == 0) {
@@ -525,8 +534,6 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
         }
         __syncwarp();
         PageLoader<KEYS> pages(p, seq, max(len, 1), k_begin, blocks, k_s, k_full, lane);
-        // everything but the newest row is older than the step's first kernel
-        const int old_keys = (len - 1) / kPageTokens * kPageTokens;
         int next = 0;
         if (p.early)
             for (; next < min(p.stages, tiles) && k_begin + (next + 1) * KEYS <= old_keys; ++next) pages.load(next);
@@ -546,15 +553,16 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
             constexpr uint32_t idesc_s = umma_idesc_bf16(64, HP);
             const uint32_t q_a = smem_u32(q_s), k_a = smem_u32(k_s);
             const int last_steps = ((p.rot - 1) % 64 + 16) / 16;
-            bool ok = mma_wait(&q_full, 0, p.status, DEV_ERR_FULL_WAIT);
-            for (int j = 0; j < tiles && ok; ++j) {
-                const int st = j % p.stages;
-                // the softmax has read S of tile j - 2 (it says so with its P)
-                if (j > 1) ok = mma_wait(&p_full[j & 1], (uint32_t)((j - 2) >> 1) & 1u, p.status, DEV_ERR_ACC_WAIT);
+            bool ok = true;
+            for (int it = 0; it < tiles + warm && ok; ++it) {
+                const int j = max(it - warm, 0), st = j % p.stages;
+                if (it == warm) ok = mma_wait(&q_full, 0, p.status, DEV_ERR_FULL_WAIT);
+                // the softmax has read S of the tile before the previous one (it says so with its P)
+                if (it > 1) ok = ok && mma_wait(&p_full[it & 1], (uint32_t)((it - 2) >> 1) & 1u, p.status, DEV_ERR_ACC_WAIT);
                 ok = ok && mma_wait(&k_full[st], (uint32_t)(j / p.stages) & 1u, p.status, DEV_ERR_FULL_WAIT);
                 if (!ok) break;
                 tc_fence_after();
-                const uint32_t d = tmem + (j & 1) * HP;
+                const uint32_t d = tmem + (it & 1) * HP;
                 // descriptors advance by constants: address / 16
                 uint64_t qd = umma_desc_k128(q_a), kd = umma_desc_k128(k_a + st * stage_bytes);
 #pragma unroll
@@ -569,18 +577,19 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
                 qd += q_block >> 4;
                 kd += k_block >> 4;
                 for (int i = 0; i < last_steps; ++i) umma_bf16_elect(d, kd + 2 * i, qd + 2 * i, idesc_s, 1);  // Q is not defined past these steps
-                umma_commit_elect(&s_full[j & 1]);
+                umma_commit_elect(&s_full[it & 1]);
             }
         }
     } else if (warp == 6) {
         constexpr uint32_t idesc_o = umma_idesc_bf16(128, 2 * HP) | (1u << 15) | (1u << 16);  // A and B with their K extent in rows
         const uint32_t k_a = smem_u32(k_s), p_a = smem_u32(p_s);
-        for (int j = 0; j < tiles; ++j) {
-            if (!mma_wait(&p_full[j & 1], (uint32_t)(j >> 1) & 1u, p.status, DEV_ERR_ACC_WAIT)) break;
+        for (int it = 0; it < tiles + warm; ++it) {
+            const int j = max(it - warm, 0);
+            if (!mma_wait(&p_full[it & 1], (uint32_t)(it >> 1) & 1u, p.status, DEV_ERR_ACC_WAIT)) break;
             tc_fence_after();
             uint64_t vd = desc_n128(k_a + (j % p.stages) * stage_bytes, k_block);
-            const uint64_t pd = desc_n128(p_a + (j & 1) * p_buf, p_buf);
-            const uint32_t again = j > 0;
+            const uint64_t pd = desc_n128(p_a + (it & 1) * p_buf, p_buf);
+            const uint32_t again = it > 0;
             uint32_t d = tmem + colO;
 #pragma unroll 2
             for (int mb = 0; mb < mblocks; ++mb) {
@@ -590,183 +599,228 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
                 vd += 2 * k_block >> 4;
                 d += 2 * HP;
             }
-            umma_commit_elect(&k_empty[j % p.stages]);
-            umma_commit_elect(&pv_done[j & 1]);
+            if (it >= warm) umma_commit_elect(&k_empty[j % p.stages]);
+            umma_commit_elect(&pv_done[it & 1]);
         }
     } else {
-        QueryRotation rotation(p, t, head0, nheads, p.part_heads, q_s + rank_blocks * q_block, q_block);
-        pdl_wait();
-        const float gate = tid < nheads ? act_load(p.gate + (size_t)t * p.gate_ld + head0 + tid) : 0.f;
-        rotation.store();
-        for (int i = tid; i < (HP - p.part_heads) * rot_blocks * 8; i += kDecSoftmax)  // rows without a head
-            *(uint4*)(q_s + (rank_blocks + i / 8 % rot_blocks) * q_block + (p.part_heads + i / 8 / rot_blocks) * 128 + i % 8 * 16) = make_uint4(0u, 0u, 0u, 0u);
-        fence_proxy_async_smem();
-        mbar_arrive(&q_full);
+        float gate = 0.f;
+        QueryRotation<1> rotation(p, t, head0, nheads, p.part_heads, q_s + rank_blocks * q_block, q_block);
         // rows of S^T: key 16 w + l of the tile is lane l < 16 of warp w
         const uint32_t lane_addr = tmem + ((uint32_t)(warp * 32) << 16);
         const int row = warp * 16 + (lane & 15);
-        float m_ref[HP], l_sum[HP];
-#pragma unroll
-        for (int h = 0; h < HP; ++h) {
-            m_ref[h] = kNeg;
-            l_sum[h] = 0.f;
-        }
         bool ok = true;  // after a wait has run out the warp goes through the motions, so that the others' barriers complete
         auto wait = [&](uint64_t* bar, uint32_t parity) {
             if (ok) ok = __all_sync(0xffffffffu, mbar_wait(bar, parity, p.status, DEV_ERR_ACC_WAIT));
         };
-        for (int j = 0; j < tiles; ++j) {
-            wait(&s_full[j & 1], (uint32_t)(j >> 1) & 1u);
-            tc_fence_after();
-            float s[HP];
-#pragma unroll
-            for (int c = 0; c < HP / 16; ++c) {
-                uint32_t v[16];
-                tmem_ld16(lane_addr + (j & 1) * HP + c * 16, v);
-                tc_wait_ld();
-#pragma unroll
-                for (int i = 0; i < 16; ++i) s[c * 16 + i] = __uint_as_float(v[i]) * p.scale_log2;
-            }
-            const bool live = lane < 16 && row < KEYS && k_begin + j * KEYS + row < k_end;
-            if (j == 0) {  // the first key's scores are the first reference
-                if (tid == 0) {
-#pragma unroll
-                    for (int h = 0; h < HP; ++h) s_max[0][h] = s[h];
-                }
-                softmax_sync();
-#pragma unroll
-                for (int h = 0; h < HP; ++h) m_ref[h] = s_max[0][h];
-            }
-            bool up = false;
+        int it = 0;  // tiles so far, the rehearsal's included
+        for (int pass = 1 - warm; pass < 2; ++pass) {
+            const bool real = pass == 1;
+            const int n = real ? tiles : 1;
+            float m_ref[HP], l_sum[HP];
 #pragma unroll
             for (int h = 0; h < HP; ++h) {
-                if (!live) s[h] = kNeg;
-                up = up || (h < nheads && s[h] > m_ref[h] + 8.f);
+                m_ref[h] = kNeg;
+                l_sum[h] = 0.f;
             }
-            if (softmax_any(up)) {  // rare: the reference maxima move to the running maxima
-#pragma unroll
-                for (int h = 0; h < HP; ++h) {
-                    float m = s[h];
-#pragma unroll
-                    for (int o = 8; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-                    if (lane == 0) s_max[warp][h] = m;
-                }
-                softmax_sync();
-                if (j > 0) {
-                    wait(&pv_done[(j - 1) & 1], (uint32_t)((j - 1) >> 1) & 1u);
-                    tc_fence_after();
-                }
-                float corr[HP];
-#pragma unroll
-                for (int h = 0; h < HP; ++h) {
-                    const float m = fmaxf(fmaxf(fmaxf(s_max[0][h], s_max[1][h]), fmaxf(s_max[2][h], s_max[3][h])), m_ref[h]);
-                    corr[h] = exp2_fast(m_ref[h] - m);
-                    m_ref[h] = m;
-                    l_sum[h] *= corr[h];
-                }
-                if (j > 0) {
-                    for (int c = 0; c < mblocks * 2; ++c) {
-#pragma unroll
-                        for (int q = 0; q < HP / 16; ++q) {
-                            uint32_t o[16];
-                            tmem_ld16(lane_addr + colO + c * HP + q * 16, o);
-                            tc_wait_ld();
-#pragma unroll
-                            for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * corr[q * 16 + i]);
-                            tmem_st16(lane_addr + colO + c * HP + q * 16, o);
-                        }
-                    }
-                    tc_wait_st();
-                }
-                softmax_sync();  // s_max may be written again
-            }
-            uint32_t hi[HP / 2], lo[HP / 2];
-#pragma unroll
-            for (int h = 0; h < HP; h += 2) {
-                const float a = live ? exp2_fast(s[h] - m_ref[h]) : 0.f, b = live ? exp2_fast(s[h + 1] - m_ref[h + 1]) : 0.f;
-                l_sum[h] += a;
-                l_sum[h + 1] += b;
-                const __nv_bfloat162 h2 = __floats2bfloat162_rn(a, b);
-                hi[h / 2] = *(const uint32_t*)&h2;
-                const __nv_bfloat162 l2 = __floats2bfloat162_rn(a - bf16_lo(hi[h / 2]), b - bf16_hi(hi[h / 2]));
-                lo[h / 2] = *(const uint32_t*)&l2;
-            }
-            if (j > 1) wait(&pv_done[j & 1], (uint32_t)((j - 2) >> 1) & 1u);  // the buffer's last product is done
-            if (lane < 16 && row < KEYS) {
-                uint8_t* dst = p_s + (j & 1) * p_buf + row * 128;
-#pragma unroll
-                for (int c = 0; c < HP / 8; ++c) {
-                    *(uint4*)(dst + ((c ^ (row & 7)) << 4)) = make_uint4(hi[4 * c], hi[4 * c + 1], hi[4 * c + 2], hi[4 * c + 3]);
-                    *(uint4*)(dst + (((c + HP / 8) ^ (row & 7)) << 4)) = make_uint4(lo[4 * c], lo[4 * c + 1], lo[4 * c + 2], lo[4 * c + 3]);
-                }
-            }
+            if (real) pdl_wait();
+            if (tid < nheads) gate = act_load(p.gate + (size_t)t * p.gate_ld + head0 + tid);
+            rotation.store();
+            for (int i = tid; i < (HP - p.part_heads) * rot_blocks * 8; i += kDecSoftmax)  // rows without a head
+                *(uint4*)(q_s + (rank_blocks + i / 8 % rot_blocks) * q_block + (p.part_heads + i / 8 / rot_blocks) * 128 + i % 8 * 16) = make_uint4(0u, 0u, 0u, 0u);
             fence_proxy_async_smem();
-            tc_fence_before();
-            mbar_arrive(&p_full[j & 1]);
-        }
-        if (tiles > 0) wait(&pv_done[(tiles - 1) & 1], (uint32_t)((tiles - 1) >> 1) & 1u);
-        tc_fence_after();
-        // ---- sums over the keys
+            if (real) mbar_arrive(&q_full);
+            for (int j = 0; j < n; ++j, ++it) {
+                wait(&s_full[it & 1], (uint32_t)(it >> 1) & 1u);
+                tc_fence_after();
+                float s[HP];
 #pragma unroll
-        for (int h = 0; h < HP; ++h) {
-            float l = l_sum[h];
-#pragma unroll
-            for (int o = 8; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);  // lanes 16 and on hold nothing
-            if (lane == 0) s_sum[warp][h] = l;
-        }
-        softmax_sync();
-        const int row_ld = partial_ld(p.rank);  // partial rows: [unit][split][part_heads][row_ld], at their end: maximum, sum
-        float* parts = p.ws + ((size_t)unit * p.splits + blockIdx.y) * p.part_heads * row_ld;
-        if (tid < nheads) {
-            const float l = s_sum[0][tid] + s_sum[1][tid] + s_sum[2][tid] + s_sum[3][tid];
-            s_mult[tid] = p.splits == 1 ? sigmoid_f32(gate) / l : 1.f;
-            if (p.splits > 1) {
-                float m = kNeg;
-#pragma unroll
-                for (int h = 0; h < HP; ++h) m = h == tid ? m_ref[h] : m;
-                parts[tid * row_ld + row_ld - 4] = m;
-                parts[tid * row_ld + row_ld - 3] = l;
-            }
-        }
-        softmax_sync();
-        // ---- O^T (lane = column of a group of 128) through the idle ring, rows of ld_s floats, then row by row
-        if (tiles > 0) {
-            const int ld_s = (p.rank + 127) / 128 * 128 + 4;
-            float* const o_s = (float*)k_s;
-            for (int mb = 0; mb < mblocks; ++mb) {
-#pragma unroll
-                for (int g = 0; g < HP / 16; ++g) {
-                    uint32_t a[16], b[16];
-                    tmem_ld16(lane_addr + colO + mb * 2 * HP + g * 16, a);
-                    tmem_ld16(lane_addr + colO + mb * 2 * HP + HP + g * 16, b);
+                for (int c = 0; c < HP / 16; ++c) {
+                    uint32_t v[16];
+                    tmem_ld16(lane_addr + (it & 1) * HP + c * 16, v);
                     tc_wait_ld();
 #pragma unroll
-                    for (int i = 0; i < 16; ++i)  // P_hi V + P_lo V
-                        o_s[(g * 16 + i) * ld_s + mb * 128 + warp * 32 + lane] = __uint_as_float(a[i]) + __uint_as_float(b[i]);
+                    for (int i = 0; i < 16; ++i) s[c * 16 + i] = __uint_as_float(v[i]) * p.scale_log2;
+                }
+                const bool live = real && lane < 16 && row < KEYS && k_begin + j * KEYS + row < k_end;
+                if (j == 0) {  // the first key's scores are the first reference
+                    if (tid == 0) {
+#pragma unroll
+                        for (int h = 0; h < HP; ++h) s_max[0][h] = s[h];
+                    }
+                    softmax_sync();
+#pragma unroll
+                    for (int h = 0; h < HP; ++h) m_ref[h] = s_max[0][h];
+                }
+                bool up = false;
+#pragma unroll
+                for (int h = 0; h < HP; ++h) {
+                    if (!live) s[h] = kNeg;
+                    up = up || (h < nheads && s[h] > m_ref[h] + 8.f);
+                }
+                if (softmax_any(up)) {  // rare: the reference maxima move to the running maxima
+#pragma unroll
+                    for (int h = 0; h < HP; ++h) {
+                        float m = s[h];
+#pragma unroll
+                        for (int o = 8; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+                        if (lane == 0) s_max[warp][h] = m;
+                    }
+                    softmax_sync();
+                    if (j > 0) {
+                        wait(&pv_done[(it - 1) & 1], (uint32_t)((it - 1) >> 1) & 1u);
+                        tc_fence_after();
+                    }
+                    float corr[HP];
+#pragma unroll
+                    for (int h = 0; h < HP; ++h) {
+                        const float m = fmaxf(fmaxf(fmaxf(s_max[0][h], s_max[1][h]), fmaxf(s_max[2][h], s_max[3][h])), m_ref[h]);
+                        corr[h] = exp2_fast(m_ref[h] - m);
+                        m_ref[h] = m;
+                        l_sum[h] *= corr[h];
+                    }
+                    if (j > 0) {
+                        for (int c = 0; c < mblocks * 2; ++c) {
+#pragma unroll
+                            for (int q = 0; q < HP / 16; ++q) {
+                                uint32_t o[16];
+                                tmem_ld16(lane_addr + colO + c * HP + q * 16, o);
+                                tc_wait_ld();
+#pragma unroll
+                                for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * corr[q * 16 + i]);
+                                tmem_st16(lane_addr + colO + c * HP + q * 16, o);
+                            }
+                        }
+                        tc_wait_st();
+                    }
+                    softmax_sync();  // s_max may be written again
+                }
+                uint32_t hi[HP / 2], lo[HP / 2];
+#pragma unroll
+                for (int h = 0; h < HP; h += 2) {
+                    const float a = live ? exp2_fast(s[h] - m_ref[h]) : 0.f, b = live ? exp2_fast(s[h + 1] - m_ref[h + 1]) : 0.f;
+                    l_sum[h] += a;
+                    l_sum[h + 1] += b;
+                    const __nv_bfloat162 h2 = __floats2bfloat162_rn(a, b);
+                    hi[h / 2] = *(const uint32_t*)&h2;
+                    const __nv_bfloat162 l2 = __floats2bfloat162_rn(a - bf16_lo(hi[h / 2]), b - bf16_hi(hi[h / 2]));
+                    lo[h / 2] = *(const uint32_t*)&l2;
+                }
+                if (it > 1) wait(&pv_done[it & 1], (uint32_t)((it - 2) >> 1) & 1u);  // the buffer's last product is done
+                if (lane < 16 && row < KEYS) {
+                    uint8_t* dst = p_s + (it & 1) * p_buf + row * 128;
+#pragma unroll
+                    for (int c = 0; c < HP / 8; ++c) {
+                        *(uint4*)(dst + ((c ^ (row & 7)) << 4)) = make_uint4(hi[4 * c], hi[4 * c + 1], hi[4 * c + 2], hi[4 * c + 3]);
+                        *(uint4*)(dst + (((c + HP / 8) ^ (row & 7)) << 4)) = make_uint4(lo[4 * c], lo[4 * c + 1], lo[4 * c + 2], lo[4 * c + 3]);
+                    }
+                }
+                fence_proxy_async_smem();
+                tc_fence_before();
+                mbar_arrive(&p_full[it & 1]);
+            }
+            if (n > 0) wait(&pv_done[(it - 1) & 1], (uint32_t)((it - 1) >> 1) & 1u);
+            tc_fence_after();
+            // ---- sums over the keys
+#pragma unroll
+            for (int h = 0; h < HP; ++h) {
+                float l = l_sum[h];
+#pragma unroll
+                for (int o = 8; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);  // lanes 16 and on hold nothing
+                if (lane == 0) s_sum[warp][h] = l;
+            }
+            softmax_sync();
+            const int row_ld = partial_ld(p.rank);  // partial rows: [unit][split][part_heads][row_ld], at their end: maximum, sum
+            float* parts = p.ws + ((size_t)unit * p.splits + blockIdx.y) * p.part_heads * row_ld;
+            if (tid < nheads) {
+                const float l = s_sum[0][tid] + s_sum[1][tid] + s_sum[2][tid] + s_sum[3][tid];
+                s_mult[tid] = p.splits == 1 ? sigmoid_f32(gate) / l : 1.f;
+                if (p.splits > 1) {
+                    float m = kNeg;
+#pragma unroll
+                    for (int h = 0; h < HP; ++h) m = h == tid ? m_ref[h] : m;
+                    s_ml[tid] = make_float2(m, l);
+                    if (real && !p.cluster) *(float2*)(parts + tid * row_ld + row_ld - 4) = make_float2(m, l);
                 }
             }
             softmax_sync();
-            const int per_head = (p.rank + 3) / 4;
-            for (int h = warp; h < nheads; h += 4) {
-                const float mult = s_mult[h];
-                const float4* src = (const float4*)(o_s + h * ld_s);
-                bf16* dst = p.out + ((size_t)t * p.heads + head0 + h) * p.head_ld;
+            // ---- O^T (lane = column of a group of 128) through the idle ring, rows of ld_s floats, then row by row
+            if (n > 0) {
+                const int ld_s = real ? o_ld : 0, mb_s = real ? 128 : 0;
+                float* const o_s = real ? (float*)k_s : s_rehearsal;
+                for (int mb = 0; mb < mblocks; ++mb) {
+#pragma unroll
+                    for (int g = 0; g < HP / 16; ++g) {
+                        uint32_t a[16], b[16];
+                        tmem_ld16(lane_addr + colO + mb * 2 * HP + g * 16, a);
+                        tmem_ld16(lane_addr + colO + mb * 2 * HP + HP + g * 16, b);
+                        tc_wait_ld();
+#pragma unroll
+                        for (int i = 0; i < 16; ++i)  // P_hi V + P_lo V
+                            o_s[(g * 16 + i) * ld_s + mb * mb_s + warp * 32 + lane] = __uint_as_float(a[i]) + __uint_as_float(b[i]);
+                    }
+                }
+                softmax_sync();
+                const int per_head = (p.rank + 3) / 4;
+                for (int h = warp; h < nheads && real && !p.cluster; h += 4) {
+                    const float mult = s_mult[h];
+                    const float4* src = (const float4*)(o_s + h * ld_s);
+                    bf16* dst = p.out + ((size_t)t * p.heads + head0 + h) * p.head_ld;
 #pragma unroll 4
-                for (int c = lane; c < per_head; c += 32) {
-                    const float4 o = src[c];
-                    if (p.splits == 1)  // columns of the padding are zero in the cache, so they are here
-                        *(uint2*)(dst + c * 4) = make_uint2((uint32_t)bf16_bits(o.x * mult) | ((uint32_t)bf16_bits(o.y * mult) << 16),
-                                                            (uint32_t)bf16_bits(o.z * mult) | ((uint32_t)bf16_bits(o.w * mult) << 16));
-                    else *(float4*)(parts + (size_t)h * row_ld + c * 4) = o;
+                    for (int c = lane; c < per_head; c += 32) {
+                        const float4 o = src[c];
+                        if (p.splits == 1)  // columns of the padding are zero in the cache, so they are here
+                            *(uint2*)(dst + c * 4) = make_uint2((uint32_t)bf16_bits(o.x * mult) | ((uint32_t)bf16_bits(o.y * mult) << 16),
+                                                                (uint32_t)bf16_bits(o.z * mult) | ((uint32_t)bf16_bits(o.w * mult) << 16));
+                        else *(float4*)(parts + (size_t)h * row_ld + c * 4) = o;
+                    }
                 }
             }
         }
-        if (p.splits > 1) __threadfence();
+        if (p.splits > 1 && !p.cluster) __threadfence();
     }
     tc_fence_before();
     __syncthreads();
     if (warp == 5) tmem_dealloc(tmem, tmem_cols);
-    if (p.splits > 1) {
+    if (p.cluster) {
+        // The splits are a thread-block cluster: each rank adds up the heads that are its own, in split order, out of the
+        // shared memory of all.
+        cluster_sync_all();
+        const int rank = (int)cluster_ctarank(), per_head = (p.rank + 3) / 4;
+        const uint32_t ml = smem_u32(s_ml), o_s = smem_u32(k_s);
+        for (int h = rank + p.splits * warp; h < nheads; h += p.splits * (kThreads / 32)) {
+            float w[kClusterSplits], M = kNeg, L = 0.f;
+#pragma unroll
+            for (int z = 0; z < kClusterSplits; ++z) {
+                w[z] = z < p.splits ? ld_shared_cluster_f32(map_shared_rank(ml + h * 8, z)) : kNeg;
+                M = fmaxf(M, w[z]);
+            }
+#pragma unroll
+            for (int z = 0; z < kClusterSplits; ++z) {
+                const float l = z < p.splits ? ld_shared_cluster_f32(map_shared_rank(ml + h * 8 + 4, z)) : 0.f;
+                w[z] = l > 0.f ? exp2_fast(w[z] - M) : 0.f;  // a split without keys has no rows
+                L += l * w[z];
+            }
+            const float mult = sigmoid_f32(act_load(p.gate + (size_t)t * p.gate_ld + head0 + h)) / L;
+            bf16* dst = p.out + ((size_t)t * p.heads + head0 + h) * p.head_ld;
+            for (int c = lane; c < per_head; c += 32) {
+                float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                for (int z = 0; z < kClusterSplits; ++z) {
+                    if (w[z] == 0.f) continue;
+                    float4 x;
+                    asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(x.x), "=f"(x.y), "=f"(x.z), "=f"(x.w)
+                                 : "r"(map_shared_rank(o_s + (uint32_t)(h * o_ld + c * 4) * 4, z)) : "memory");
+                    o.x += w[z] * x.x;
+                    o.y += w[z] * x.y;
+                    o.z += w[z] * x.z;
+                    o.w += w[z] * x.w;
+                }
+                *(uint2*)(dst + c * 4) = make_uint2((uint32_t)bf16_bits(o.x * mult) | ((uint32_t)bf16_bits(o.y * mult) << 16),
+                                                    (uint32_t)bf16_bits(o.z * mult) | ((uint32_t)bf16_bits(o.w * mult) << 16));
+            }
+        }
+        cluster_sync_all();  // no rank leaves while its rows are read
+    } else if (p.splits > 1) {
         if (tid == 0) {
             __threadfence();
             const int old = atomicAdd(&p.counters[unit], 1);
@@ -850,7 +904,7 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
 struct LatentPlan {
     int part_heads, parts, tile_tokens, q_rows, slices, slice_cols, stages, smem, tmem_cols, keys;
 };
-constexpr int kStaticSmem = 2048;  // room for the kernels' static shared memory
+constexpr int kStaticSmem = 3072;  // room for the kernels' static shared memory
 
 LatentPlan plan_prompt(int rank, int rot, int heads) {
     LatentPlan l;
@@ -911,9 +965,13 @@ int attention_latent_splits(int rows, int rank, int rot, int heads, int max_ctx,
     const int units = rows * l.parts;
     int splits = 1;
     if (units * 2 <= num_sms) {
-        splits = std::min(num_sms / units, max_ctx / kLatentSplitKeys);
-        splits = std::max(1, std::min(splits, kDecMaxSplits));
-        while (splits > 1 && ((size_t)units * splits * l.part_heads * partial_ld(rank) > ws.partial_floats || units > ws.num_counters)) --splits;
+        const int room = num_sms / units, many = std::min(std::min(room, max_ctx / kLatentSplitKeys), kDecMaxSplits);
+        if (many > kClusterSplits) {
+            splits = many;
+            while (splits > kClusterSplits && ((size_t)units * splits * l.part_heads * partial_ld(rank) > ws.partial_floats || units > ws.num_counters)) --splits;
+        } else {
+            while (splits < kClusterSplits && splits * 2 <= room && max_ctx / (splits * 2) >= kLatentClusterKeys) splits *= 2;
+        }
     }
     return splits;
 }
@@ -964,10 +1022,11 @@ int launch_attention_latent(const LatentAttn& a, int T, int n_groups, int max_ct
     }
     p.splits = attention_latent_splits(T, a.rank, a.rot, a.heads, max_ctx, ws, num_sms);
     p.early = pdl && a.only_newest_row_fresh;
+    p.cluster = p.splits > 1 && p.splits <= kClusterSplits;
     const dim3 grid(T * l.parts, p.splits);
     const auto kernel = l.q_rows == 16 ? (l.keys == TK ? k_attn_latent_decode<16, TK> : k_attn_latent_decode<16, kPageTokens>)
                                        : (l.keys == TK ? k_attn_latent_decode<32, TK> : k_attn_latent_decode<32, kPageTokens>);
-    return (int)launch_k(kernel, grid, dim3(kThreads), (size_t)l.smem, s, pdl, p, (uint32_t)l.tmem_cols);
+    return (int)launch_k_cluster(kernel, grid, dim3(kThreads), dim3(1, p.cluster ? p.splits : 1), (size_t)l.smem, s, pdl, p, (uint32_t)l.tmem_cols);
 }
 
 template <typename Kern>

@@ -323,7 +323,8 @@ struct LatentAttn {
     bool only_newest_row_fresh;
     int* status;
 };
-constexpr int kLatentSplitKeys = 512;  // fewest keys of a context split
+// fewest keys of a context split: of those that add up within a cluster, and of more than eight
+constexpr int kLatentClusterKeys = 128, kLatentSplitKeys = 512;
 bool attention_latent_supported(int rank, int rot, int heads);  // otherwise launch_attention_simt
 int attention_latent_splits(int rows, int rank, int rot, int heads, int max_ctx, const AttnWorkspace& ws, int num_sms);
 // returns cudaError (launch) or -1000 if the tensor maps could not be encoded

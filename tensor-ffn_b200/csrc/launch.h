@@ -21,6 +21,27 @@ inline cudaError_t launch_k(Kern k, dim3 grid, dim3 block, size_t smem, cudaStre
     return cudaLaunchKernelEx(&cfg, k, args...);
 }
 
+// the same with thread-block clusters
+template <typename Kern, typename... Args>
+inline cudaError_t launch_k_cluster(Kern k, dim3 grid, dim3 block, dim3 cluster, size_t smem, cudaStream_t s, bool pdl, Args... args) {
+    if (cluster.x * cluster.y * cluster.z <= 1) return launch_k(k, grid, block, smem, s, pdl, args...);
+    cudaLaunchConfig_t cfg = cudaLaunchConfig_t{};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = s;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = cluster.x;
+    attr[0].val.clusterDim.y = cluster.y;
+    attr[0].val.clusterDim.z = cluster.z;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = pdl ? 2 : 1;
+    return cudaLaunchKernelEx(&cfg, k, args...);
+}
+
 // Ask for the largest shared-memory carveout for a kernel, whatever it uses itself. The kernels of a
 // decode step are resident together (dependent launches let the next ones start early and fetch their
 // weights). An SM cannot change its L1 / shared-memory split while CTAs are resident on it: if the small

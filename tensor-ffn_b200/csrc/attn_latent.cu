@@ -733,7 +733,7 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
             float* parts = p.ws + ((size_t)unit * p.splits + blockIdx.y) * p.part_heads * row_ld;
             if (tid < nheads) {
                 const float l = s_sum[0][tid] + s_sum[1][tid] + s_sum[2][tid] + s_sum[3][tid];
-                s_mult[tid] = p.splits == 1 ? sigmoid_f32(gate) / l : 1.f;
+                s_mult[tid] = sigmoid_f32(gate) / (p.splits == 1 ? l : 1.f);
                 if (p.splits > 1) {
                     float m = kNeg;
 #pragma unroll
@@ -785,38 +785,61 @@ __global__ void __launch_bounds__(kThreads, 1) k_attn_latent_decode(const __grid
         // The splits are a thread-block cluster: each rank adds up the heads that are its own, in split order, out of the
         // shared memory of all.
         cluster_sync_all();
-        const int rank = (int)cluster_ctarank(), per_head = (p.rank + 3) / 4;
-        const uint32_t ml = smem_u32(s_ml), o_s = smem_u32(k_s);
-        for (int h = rank + p.splits * warp; h < nheads; h += p.splits * (kThreads / 32)) {
-            float w[kClusterSplits], M = kNeg, L = 0.f;
+        const int rank = (int)cluster_ctarank(), per_head = (p.rank + 3) / 4, own = (nheads - rank + p.splits - 1) / p.splits;
+        float* wgt = (float*)p_s;  // [own head][split], in the idle buffers of P
+        if (tid < own) {
+            const uint32_t ml = smem_u32(s_ml) + (rank + tid * p.splits) * 8;
+            float m[kClusterSplits], l[kClusterSplits], M = kNeg, L = 0.f;
 #pragma unroll
             for (int z = 0; z < kClusterSplits; ++z) {
-                w[z] = z < p.splits ? ld_shared_cluster_f32(map_shared_rank(ml + h * 8, z)) : kNeg;
-                M = fmaxf(M, w[z]);
+                const uint32_t from = map_shared_rank(ml, z < p.splits ? z : 0);
+                m[z] = ld_shared_cluster_f32(from);
+                l[z] = z < p.splits ? ld_shared_cluster_f32(from + 4) : 0.f;
             }
+#pragma unroll
+            for (int z = 0; z < kClusterSplits; ++z) M = fmaxf(M, m[z]);
 #pragma unroll
             for (int z = 0; z < kClusterSplits; ++z) {
-                const float l = z < p.splits ? ld_shared_cluster_f32(map_shared_rank(ml + h * 8 + 4, z)) : 0.f;
-                w[z] = l > 0.f ? exp2_fast(w[z] - M) : 0.f;  // a split without keys has no rows
-                L += l * w[z];
+                m[z] = l[z] > 0.f ? exp2_fast(m[z] - M) : 0.f;  // a split without keys has no rows
+                L += l[z] * m[z];
             }
-            const float mult = sigmoid_f32(act_load(p.gate + (size_t)t * p.gate_ld + head0 + h)) / L;
-            bf16* dst = p.out + ((size_t)t * p.heads + head0 + h) * p.head_ld;
-            for (int c = lane; c < per_head; c += 32) {
-                float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+            const float mult = s_mult[rank + tid * p.splits] / L;
 #pragma unroll
-                for (int z = 0; z < kClusterSplits; ++z) {
-                    if (w[z] == 0.f) continue;
-                    float4 x;
-                    asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(x.x), "=f"(x.y), "=f"(x.z), "=f"(x.w)
-                                 : "r"(map_shared_rank(o_s + (uint32_t)(h * o_ld + c * 4) * 4, z)) : "memory");
-                    o.x += w[z] * x.x;
-                    o.y += w[z] * x.y;
-                    o.z += w[z] * x.z;
-                    o.w += w[z] * x.w;
-                }
-                *(uint2*)(dst + c * 4) = make_uint2((uint32_t)bf16_bits(o.x * mult) | ((uint32_t)bf16_bits(o.y * mult) << 16),
-                                                    (uint32_t)bf16_bits(o.z * mult) | ((uint32_t)bf16_bits(o.w * mult) << 16));
+            for (int z = 0; z < kClusterSplits; ++z) wgt[tid * kClusterSplits + z] = m[z] * mult;
+        }
+        __syncthreads();
+        // a piece = four columns of a head; two pieces and two splits with their loads in flight together
+        const uint32_t o_s = smem_u32(k_s);
+        const int n = own * per_head;
+        for (int i0 = tid; i0 < n; i0 += 2 * kThreads) {
+            float o[2][4];
+#pragma unroll
+            for (int k = 0; k < 2; ++k) o[k][0] = o[k][1] = o[k][2] = o[k][3] = 0.f;
+            for (int z0 = 0; z0 < p.splits; z0 += 2) {
+                float x[2][2][4], w[2][2];
+#pragma unroll
+                for (int k = 0; k < 2; ++k)
+#pragma unroll
+                    for (int q = 0; q < 2; ++q) {
+                        const int i = min(i0 + k * kThreads, n - 1), h = i / per_head, c = i % per_head;
+                        w[k][q] = wgt[h * kClusterSplits + z0 + q];
+                        const uint32_t from = map_shared_rank(o_s + (uint32_t)((rank + h * p.splits) * o_ld + c * 4) * 4, z0 + q);
+                        asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(x[k][q][0]), "=f"(x[k][q][1]), "=f"(x[k][q][2]), "=f"(x[k][q][3])
+                                     : "r"(from) : "memory");
+                    }
+#pragma unroll
+                for (int k = 0; k < 2; ++k)
+#pragma unroll
+                    for (int q = 0; q < 2; ++q)
+#pragma unroll
+                        for (int c = 0; c < 4; ++c) o[k][c] += w[k][q] > 0.f ? w[k][q] * x[k][q][c] : 0.f;
+            }
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const int i = i0 + k * kThreads, h = rank + i / per_head * p.splits;
+                if (i < n)
+                    *(uint2*)(p.out + ((size_t)t * p.heads + head0 + h) * p.head_ld + i % per_head * 4) =
+                        make_uint2((uint32_t)bf16_bits(o[k][0]) | ((uint32_t)bf16_bits(o[k][1]) << 16), (uint32_t)bf16_bits(o[k][2]) | ((uint32_t)bf16_bits(o[k][3]) << 16));
             }
         }
         cluster_sync_all();  // no rank leaves while its rows are read
@@ -947,7 +970,7 @@ LatentPlan plan_decode(int rank, int rot, int heads) {
             l.stages = std::min(kMaxStages, (kSmemLimit - kStaticSmem - fixed) / stage);
             const int out = hp * ((rank + 127) / 128 * 128 + 4) * 4;  // O^T passes through the ring
             l.smem = fixed + std::max(l.stages * stage, out);
-            if (l.stages >= (l.keys == TK ? 2 : 1) && l.smem <= kSmemLimit - kStaticSmem) return l;
+            if (l.stages >= (l.keys == TK ? 3 : 1) && l.smem <= kSmemLimit - kStaticSmem) return l;
         }
     }
     l.stages = 0;

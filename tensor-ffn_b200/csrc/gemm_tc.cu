@@ -908,6 +908,13 @@ int launch_gemm(const GemmCall& c, const GemmWorkspace& ws, cudaStream_t stream,
     // One row tile (a router): with wide token tiles a handful of CTAs would carry the whole launch and split it along
     // K, exchanging planes that are mostly padding; narrow token tiles spread it over the SMs instead.
     if (c.N <= BM && c.T > 64 && c.mode == GEMM_STORE_F32 && !c.out2 && c.op[1].K <= 0) return launch_bn<64>(c, ws, stream, force_splits);
+    // Many tiles of a short K extent (prompts): the set-up and epilogue of a tile weigh as much as its products, and three
+    // CTAs of 64 tokens per SM cover them better than one of 256 (4 096 tokens, K 64 to 896: 5 to 30 % less time per launch).
+    {
+        const int total_kb = (c.op[0].K + BK - 1) / BK + (c.op[1].K > 0 && c.mode != GEMM_SWIGLU ? (c.op[1].K + BK - 1) / BK : 0);
+        const long long tiles = (long long)((c.N + BM - 1) / BM) * ((c.T + 63) / 64) * (c.batch > 1 ? c.batch : 1) * (c.mode == GEMM_SWIGLU ? 2 : 1);
+        if (force_splits == 0 && c.T > 64 && total_kb <= 14 && tiles >= 4ll * ws.num_sms) return launch_bn<64>(c, ws, stream, force_splits);
+    }
     if (c.T <= 16) return launch_bn<16>(c, ws, stream, force_splits);
     if (c.T <= 32) return launch_bn<32>(c, ws, stream, force_splits);
     if (c.T <= 64) return launch_bn<64>(c, ws, stream, force_splits);

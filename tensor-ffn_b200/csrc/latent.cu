@@ -9,7 +9,6 @@ namespace tffn {
 namespace {
 
 constexpr int kPrepThreads = 128;
-constexpr int kPrepGroups = 4;  // groups of four columns a thread keeps in registers
 
 __device__ __forceinline__ void load4(const float* p, float (&v)[4]) {
     const float4 q = __ldcg((const float4*)p);
@@ -25,76 +24,104 @@ __device__ __forceinline__ void store4(bf16* p, const float (&v)[4]) {
                             (uint32_t)bf16_bits(v[2]) | ((uint32_t)bf16_bits(v[3]) << 16));
 }
 
-// dst = src / sqrt(mean(src^2) + eps) * w over n columns; src and dst 16-byte aligned, columns past n are left alone
-template <typename A>
-__device__ __forceinline__ void norm_row(const A* src, const float* w, A* dst, int n, float eps, float* red) {
-    constexpr int kept = kPrepThreads * kPrepGroups * 4;
-    float v[kPrepGroups][4], ss = 0.f;
+// dst = src / sqrt(mean(src^2) + eps) * w over n columns; src and dst 16-byte aligned, columns past n are left alone. The
+// weights of the columns a thread keeps in registers (IT groups of four) are fetched by the constructor, ahead of the wait
+// for src.
+template <int IT>
+struct NormRow {
+    static constexpr int kept = kPrepThreads * IT * 4;
+    const float* w;
+    int n;
+    float g[IT][4];
+    __device__ __forceinline__ NormRow(const float* w_, int n_) : w(w_), n(n_) {
 #pragma unroll
-    for (int k = 0; k < kPrepGroups; ++k) {
-        const int i = (threadIdx.x + k * kPrepThreads) * 4;
+        for (int k = 0; k < IT; ++k) {
+            const int i = (threadIdx.x + k * kPrepThreads) * 4;
+            if (i + 3 < n) {
+                const float4 q = __ldg((const float4*)(w + i));
+                g[k][0] = q.x; g[k][1] = q.y; g[k][2] = q.z; g[k][3] = q.w;
+            } else {
 #pragma unroll
-        for (int c = 0; c < 4; ++c) v[k][c] = 0.f;
-        if (i + 3 < n) {
-            load4(src + i, v[k]);
-        } else {
-#pragma unroll
-            for (int c = 0; c < 4; ++c)
-                if (i + c < n) v[k][c] = act_load(src + i + c);
-        }
-#pragma unroll
-        for (int c = 0; c < 4; ++c) ss += v[k][c] * v[k][c];
-    }
-    for (int i = kept + threadIdx.x; i < n; i += kPrepThreads) {
-        const float x = act_load(src + i);
-        ss += x * x;
-    }
-    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
-#pragma unroll
-    for (int k = 0; k < kPrepGroups; ++k) {
-        const int i = (threadIdx.x + k * kPrepThreads) * 4;
-        if (i + 3 < n) {
-            const float4 g = __ldg((const float4*)(w + i));
-            const float o[4] = {v[k][0] * inv * g.x, v[k][1] * inv * g.y, v[k][2] * inv * g.z, v[k][3] * inv * g.w};
-            store4(dst + i, o);
-        } else {
-#pragma unroll
-            for (int c = 0; c < 4; ++c)
-                if (i + c < n) act_store(dst + i + c, v[k][c] * inv * __ldg(w + i + c));
+                for (int c = 0; c < 4; ++c) g[k][c] = i + c < n ? __ldg(w + i + c) : 0.f;
+            }
         }
     }
-    for (int i = kept + threadIdx.x; i < n; i += kPrepThreads) act_store(dst + i, act_load(src + i) * inv * __ldg(w + i));
-}
+    template <typename A>
+    __device__ __forceinline__ void run(const A* src, A* dst, float eps, float* red) const {
+        float v[IT][4], ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < IT; ++k) {
+            const int i = (threadIdx.x + k * kPrepThreads) * 4;
+#pragma unroll
+            for (int c = 0; c < 4; ++c) v[k][c] = 0.f;
+            if (i + 3 < n) {
+                load4(src + i, v[k]);
+            } else {
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+                    if (i + c < n) v[k][c] = act_load(src + i + c);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < IT; ++k)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) ss += v[k][c] * v[k][c];
+        for (int i = kept + threadIdx.x; i < n; i += kPrepThreads) {
+            const float x = act_load(src + i);
+            ss += x * x;
+        }
+        const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+#pragma unroll
+        for (int k = 0; k < IT; ++k) {
+            const int i = (threadIdx.x + k * kPrepThreads) * 4;
+            const float o[4] = {v[k][0] * inv * g[k][0], v[k][1] * inv * g[k][1], v[k][2] * inv * g[k][2], v[k][3] * inv * g[k][3]};
+            if (i + 3 < n) {
+                store4(dst + i, o);
+            } else {
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+                    if (i + c < n) act_store(dst + i + c, o[c]);
+            }
+        }
+        for (int i = kept + threadIdx.x; i < n; i += kPrepThreads) act_store(dst + i, act_load(src + i) * inv * __ldg(w + i));
+    }
+};
 
 // grid (1 or 2, T): x = 0 the query latent, x = 1 the cached row
-template <typename A>
+template <typename A, int IT>
 __global__ void __launch_bounds__(kPrepThreads) k_latent_prep(const LatentPrep a, unsigned long long* tl) {
     __shared__ float red[32];
     if (threadIdx.x == 0) tl_mark(tl, 0);
     pdl_launch_dependents();
-    pdl_wait();
-    if (threadIdx.x == 0) tl_mark(tl, 1);
     const int t = blockIdx.y;
     const A* row = (const A*)a.proj + (size_t)t * a.ld;
     if (blockIdx.x == 0) {
-        norm_row<A>(row, a.q_norm, (A*)a.cq + (size_t)t * a.cq_ld, a.q_rank, a.eps, red);
+        const NormRow<IT> norm(a.q_norm, a.q_rank);
+        pdl_wait();
+        if (threadIdx.x == 0) tl_mark(tl, 1);
+        norm.run(row, (A*)a.cq + (size_t)t * a.cq_ld, a.eps, red);
     } else {
-        const int pos = __ldcg(a.tok_pos + t), seq = __ldcg(a.tok_seq + t);
+        // slots, positions and the block table are older than the step's first kernel
+        const NormRow<IT> norm(a.kv_norm, a.rank);
+        const int pos = __ldcg(a.tok_pos + t), seq = __ldcg(a.tok_seq + t), half = a.rot / 2, rot_col = (a.rank + 63) / 64 * 64;
         const bool pos_ok = pos >= 0 && pos < a.max_pos;
         const int pg = pos_ok ? __ldcg(a.kv.block_table + (size_t)seq * a.kv.max_pages_per_seq + pos / kPageTokens) : -1;
+        float2 cs = make_float2(1.f, 0.f);
+        if (pos_ok && (int)threadIdx.x < half) cs = __ldg(a.rope + (size_t)pos * half + threadIdx.x);
+        pdl_wait();
+        if (threadIdx.x == 0) tl_mark(tl, 1);
         if (pg < 0 || pg >= a.kv.num_pages) {
             if (threadIdx.x == 0) dev_fail(a.status, DEV_ERR_BOUNDS);
         } else {
             A* dst = (A*)a.kv.k_pool + ((size_t)pg * kPageTokens + pos % kPageTokens) * a.kv.hd;
             const A* src = row + a.kv_off;
-            const int half = a.rot / 2, rot_col = (a.rank + 63) / 64 * 64;
             for (int i = threadIdx.x; i < half; i += kPrepThreads) {
+                if (i >= kPrepThreads) cs = __ldg(a.rope + (size_t)pos * half + i);
                 const float u = act_load(src + a.rank + i), v = act_load(src + a.rank + half + i);
-                const float2 cs = __ldg(a.rope + (size_t)pos * half + i);
                 act_store(dst + rot_col + i, u * cs.x - v * cs.y);
                 act_store(dst + rot_col + half + i, v * cs.x + u * cs.y);
             }
-            norm_row<A>(src, a.kv_norm, dst, a.rank, a.eps, red);
+            norm.run(src, dst, a.eps, red);
         }
     }
     if (threadIdx.x == 0) tl_mark(tl, 2);
@@ -130,20 +157,33 @@ __global__ void __launch_bounds__(kRopeWarps * 32) k_latent_rope(const A* __rest
     if (threadIdx.x == 0) tl_mark(tl, 2);
 }
 
+template <typename A>
+cudaError_t prep_attrs() {
+    cudaError_t e = prefer_max_shared(k_latent_prep<A, 1>);
+    if (e == cudaSuccess) e = prefer_max_shared(k_latent_prep<A, 2>);
+    if (e == cudaSuccess) e = prefer_max_shared(k_latent_prep<A, 4>);
+    return e;
+}
+template <typename A>
+void prep(const LatentPrep& a, int T, cudaStream_t s, bool pdl, unsigned long long* tl) {
+    const dim3 grid(a.own_rows ? 2 : 1, T), block(kPrepThreads);
+    const int n = a.q_rank > a.rank ? a.q_rank : a.rank;
+    launch_k(n <= 512 ? k_latent_prep<A, 1> : n <= 1024 ? k_latent_prep<A, 2> : k_latent_prep<A, 4>, grid, block, 0, s, pdl, a, tl);
+}
+
 }  // namespace
 
 int latent_prepare() {
-    cudaError_t e = prefer_max_shared(k_latent_prep<bf16>);
-    if (e == cudaSuccess) e = prefer_max_shared(k_latent_prep<float>);
+    cudaError_t e = prep_attrs<bf16>();
+    if (e == cudaSuccess) e = prep_attrs<float>();
     if (e == cudaSuccess) e = prefer_max_shared(k_latent_rope<bf16>);
     if (e == cudaSuccess) e = prefer_max_shared(k_latent_rope<float>);
     return (int)e;
 }
 
 void launch_latent_prep(const LatentPrep& a, bool f32, int T, cudaStream_t s, bool pdl, unsigned long long* tl) {
-    const dim3 grid(a.own_rows ? 2 : 1, T), block(kPrepThreads);
-    if (f32) launch_k(k_latent_prep<float>, grid, block, 0, s, pdl, a, tl);
-    else launch_k(k_latent_prep<bf16>, grid, block, 0, s, pdl, a, tl);
+    if (f32) prep<float>(a, T, s, pdl, tl);
+    else prep<bf16>(a, T, s, pdl, tl);
 }
 
 void launch_latent_rope(const void* q_up, int64_t ld, int off, int heads, int rot, const float2* rope, int max_pos, const int* tok_pos,

@@ -51,11 +51,22 @@ __global__ void __launch_bounds__(kConvThreads) k_lru_prep(const RgLru a, unsign
         rows = __ballot_sync(0xffffffffu, row);
         ring = __ballot_sync(0xffffffffu, in_seq && !row);
     }
-    float w_now[V], xb[V], y[V];
-    const bool on = ch < a.width;
+    // Taps, biases and the ring are older than the step's first kernel as well: only rows of this launch wait. The four
+    // youngest inputs have their loads in flight together.
+    constexpr int NEAR = 4;
+    float xb[V], y[V], w[NEAR][V], x[NEAR][V];
+    const bool on = ch < a.width && seq >= 0 && seq < a.max_slots && pos >= 0;
+    const float* old = a.ring + (size_t)(on ? seq : 0) * a.ring_stride + ch;
     if (on) {
         load_cols<V>(a.conv_bias + ch, y);
         load_cols<V>(a.x_bias + ch, xb);
+#pragma unroll
+        for (int lag = 0; lag < NEAR; ++lag) {
+#pragma unroll
+            for (int v = 0; v < V; ++v) w[lag][v] = x[lag][v] = 0.f;
+            if (lag <= R && ((rows | ring) >> lag & 1u)) load_cols<V>(a.conv + (size_t)(R - lag) * a.width + ch, w[lag]);
+            if (lag <= R && (ring >> lag & 1u)) load_cols<V>(old + (size_t)((pos - lag) % R) * a.width, x[lag]);
+        }
     }
     pdl_wait();
     if (threadIdx.x == 0) tl_mark(tl, 1);
@@ -65,23 +76,22 @@ __global__ void __launch_bounds__(kConvThreads) k_lru_prep(const RgLru a, unsign
     }
     if (on) {
         const A* x0 = (const A*)a.proj + (size_t)t * a.proj_ld + a.x_off + ch;
-        const float* old = a.ring + (size_t)seq * a.ring_stride + ch;
-#pragma unroll 4
-        for (int lag = R; lag >= 0; --lag) {
-            float x[V];
-            if ((rows >> lag) & 1u) {
-                load_cols<V>(x0 - (ptrdiff_t)lag * a.proj_ld, x);
 #pragma unroll
-                for (int v = 0; v < V; ++v) x[v] += xb[v];
-            } else if ((ring >> lag) & 1u) {
-                load_cols<V>(old + (size_t)((pos - lag) % R) * a.width, x);
-            } else {
-                continue;
-            }
-            load_cols<V>(a.conv + (size_t)(R - lag) * a.width + ch, w_now);
+        for (int lag = 0; lag < NEAR; ++lag)
+            if (rows >> lag & 1u) load_cols<V>(x0 - (ptrdiff_t)lag * a.proj_ld, x[lag]);
+        for (int lag = R; lag >= NEAR; --lag) {  // long convolutions: the older inputs
+            float xo[V], wo[V];
+            if (!((rows | ring) >> lag & 1u)) continue;
+            load_cols<V>(a.conv + (size_t)(R - lag) * a.width + ch, wo);
+            if (rows >> lag & 1u) load_cols<V>(x0 - (ptrdiff_t)lag * a.proj_ld, xo);
+            else load_cols<V>(old + (size_t)((pos - lag) % R) * a.width, xo);
 #pragma unroll
-            for (int v = 0; v < V; ++v) y[v] += w_now[v] * x[v];
+            for (int v = 0; v < V; ++v) y[v] += wo[v] * (xo[v] + (rows >> lag & 1u ? xb[v] : 0.f));
         }
+#pragma unroll
+        for (int lag = NEAR - 1; lag >= 0; --lag)  // oldest first; a projection still lacks its bias, the ring does not
+#pragma unroll
+            for (int v = 0; v < V; ++v) y[v] += w[lag][v] * (x[lag][v] + (rows >> lag & 1u ? xb[v] : 0.f));
         const int n = a.width / a.blocks;
         A* dst = (A*)a.u + (size_t)t * a.u_ld + (ch / n) * a.u_part + ch % n;
 #pragma unroll

@@ -132,8 +132,8 @@ def dense(h, w, p):
     return (silu(h @ w[p + "gate"].T) * (h @ w[p + "up"].T)) @ w[p + "down"].T
 
 
-def forward(cfg, w, tokens):
-    """-> (logits [T, vocab], residual stream after every layer [layers, T, width])"""
+def forward(cfg, w, tokens, last=None):
+    """-> (logits [T, vocab], residual stream after every layer [layers, T, width]); last: the logits of so many last tokens"""
     eps, mult = cfg["norm"]["eps"], cfg["residual_mult"]
     x = rms_norm(w["embed"][np.asarray(tokens)].astype(F), w["embed.norm"], eps)
     after, kept = [], {}
@@ -152,4 +152,5 @@ def forward(cfg, w, tokens):
             y = y + dense(rms_norm(x, w[n + "norm2"], eps), w, n + "mlp.")
         x = x + mult * y
         after.append(x.copy())
+    x = x if last is None else x[-last:]
     return rms_norm(x, w["final.norm"], eps) @ w["head"].T * cfg["logit_scale"], np.stack(after)

@@ -86,8 +86,9 @@ class Case:
         s.set_launch_mode(mode)
         return s
 
-    def expect(self, tokens):
-        return plain.forward(self.plain_cfg, self.w, tokens)
+    def expect(self, tokens, last=None):
+        """last: logits of that many positions at the end only"""
+        return plain.forward(self.plain_cfg, self.w, tokens, last)
 
     def tokens(self, n, seed=0):
         return np.random.default_rng([11, seed]).integers(0, self.cfg["vocab"], n).astype(np.int32)

@@ -141,7 +141,7 @@ def test_one_far_key(tmp_path, decoded, compute):
     filler = c.tokens(1300, seed=5)
     filler[np.isin(filler, [key, ask])] = other
     s = c.session(compute, max_seq=1400)
-    for kpos, apos in [(0, 1), (0, 63), (31, 64), (32, 65), (63, 64), (64, 127), (5, 511), (511, 512), (512, 640), (0, 1099), (383, 1099), (384, 1150),
+    for kpos, apos in [(0, 1), (0, 63), (31, 64), (32, 65), (63, 64), (64, 127), (10, 300), (5, 511), (511, 512), (512, 640), (0, 1099), (383, 1099), (384, 1150),
                        (575, 1151), (576, 1200), (1098, 1099), (1023, 1024)]:
         t = filler[:apos + 1].copy()
         t[kpos], t[apos] = key, ask
@@ -156,6 +156,25 @@ def test_one_far_key(tmp_path, decoded, compute):
         else:
             got = s.qwen_forward(t)[apos:]
         check(got, want[None], compute, (kpos, apos))
+    s.free()
+
+
+def test_one_key_among_thousands(tmp_path):
+    """a context of more splits than a cluster holds: their rows go through the workspace; a key in the first, in the middle
+    and in the last of them"""
+    c, key, ask, other = plant_key(tmp_path)
+    filler = c.tokens(4750, seed=6)
+    filler[np.isin(filler, [key, ask])] = other
+    s = c.session("bfloat16", max_seq=4800)
+    for kpos in (3, 2304, 4700):
+        t = filler.copy()
+        t[kpos], t[-1] = key, ask
+        want = c.expect(t, last=1)[0]
+        s.qwen_reset()
+        s.prefill([t[:-1]])
+        check(s.decode_step(t[-1:], want_logits=True)[1], want, "bfloat16", kpos)
+        t[kpos] = other
+        assert error(c.expect(t, last=1)[0], want)[0] > 3 * LIMIT["bfloat16"]  # the plant is seen
     s.free()
 
 

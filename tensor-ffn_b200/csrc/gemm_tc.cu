@@ -902,8 +902,12 @@ int launch_gemm(const GemmCall& c, const GemmWorkspace& ws, cudaStream_t stream,
         // not enough to fill the SMs with 64-token tiles; with 32-token tiles twice as many CTAs (two per SM)
         // stream half as many k-blocks each (measured: 12.6 -> 11.6 us per launch inside a step).
         if (force_splits == 0 && c.mode != GEMM_SWIGLU && !c.out2 && c.T > 32 && c.T <= 64 && total_kb >= 64 &&
-            n_tiles * 8 <= ws.num_sms)  // 16 splits as long as two CTAs per SM hold them all, else 8 (16 tiles: 28 -> 14 us)
-            return launch_bn<32>(c, ws, stream, n_tiles * 2 * kMaxSplits <= 2 * ws.num_sms ? kMaxSplits : kMaxSplits / 2);
+            n_tiles * 8 <= ws.num_sms) {
+            // 16 splits as long as two CTAs per SM hold them all, else 8 (16 tiles: 28 -> 14 us). The bf16 residual
+            // epilogue keeps its order of summation.
+            const bool second_wave = c.mode == GEMM_STORE_F32 && n_tiles * 2 * kMaxSplits > 2 * ws.num_sms;
+            return launch_bn<32>(c, ws, stream, second_wave ? kMaxSplits / 2 : kMaxSplits);
+        }
     }
     // One row tile (a router): with wide token tiles a handful of CTAs would carry the whole launch and split it along
     // K, exchanging planes that are mostly padding; narrow token tiles spread it over the SMs instead.
